@@ -33,7 +33,7 @@ class ExecutionProfile(str, Enum):
 @dataclass(frozen=True)
 class SchedulerConfig:
     """Mirrors ``EngineLoopConfig`` (``hipengine/generation/engine_loop.py:155-213``) with this engine's defaults."""
-    policy: str = "protect_decode"          # protect_decode | protect_ttft | fair | token_budget
+    policy: str = "protect_decode"          # protect_decode | protect_ttft | fair | token_budget | mixed
     max_prefill_chunk_tokens: int = 4096
     round_prefill_token_budget: int = 4096
     round_decode_row_budget: int = 64
@@ -93,6 +93,7 @@ class EngineConfig:
     speculative: SpeculativeConfig = field(default_factory=SpeculativeConfig)
     parallel: ParallelConfig = field(default_factory=ParallelConfig)
     use_cuda_graphs: bool = True
+    compute_dtype: str = "bfloat16"         # bfloat16 | float32 (families that declare it; ``models/registry.py``)
     command_timeout_seconds: float = 300.0
 
     @staticmethod

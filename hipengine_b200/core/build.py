@@ -93,24 +93,59 @@ def build_plan(extra_flags: Sequence[str] = ()) -> Dict[str, object]:
     return {"nvcc": nvcc, "flags": flags, "sources": [str(s) for s in sources()], "output": str(lib_path())}
 
 
+SUBSET = "subset"        # variant name of a library linked from some of the sources (same flags and objects as the product)
+
+
+def ensure(only: Sequence[str] = ()) -> Path:
+    """Make a usable product library available to this process: the full one when it is up to date, else one built from
+    the sources named in ``only`` (all of them when empty), e.g. what a single model family needs on a fresh checkout."""
+    if variant() not in ("", SUBSET):
+        return lib_path()                                    # an explicitly chosen variant is the caller's business
+    if nvcc_path() is None or not only:
+        if lib_path("").exists() and (nvcc_path() is None or _up_to_date()):
+            os.environ.pop("HE_NATIVE_VARIANT", None)
+            return lib_path("")
+        return build()
+    if _up_to_date():
+        os.environ.pop("HE_NATIVE_VARIANT", None)
+        return lib_path("")
+    p = build(name=SUBSET, only=only)
+    os.environ["HE_NATIVE_VARIANT"] = SUBSET
+    return p
+
+
+def _up_to_date() -> bool:
+    """Does the full product library correspond to the sources as they are?"""
+    try:
+        manifest = json.loads((OUT_DIR / "manifest.json").read_text())
+    except Exception:
+        return False
+    cver = _compiler_version(nvcc_path() or "")
+    keys = [_key(s, NVCC_FLAGS, cver) for s in sources()]
+    link = hashlib.sha256("".join(keys).encode()).hexdigest()
+    return lib_path("").exists() and manifest.get("__link__") == link
+
+
 def build(verbose: bool = False, force: bool = False, extra_flags: Sequence[str] = (), jobs: int = 0,
-          name: str = "") -> Path:
-    """Compile every source for sm_100a and link ``libhe_b200.so`` (or the variant ``libhe_b200_<name>.so`` with the
-    variant's flags plus ``extra_flags``).  Returns the library path."""
+          name: str = "", only: Sequence[str] = ()) -> Path:
+    """Compile every source (or the files named in ``only``) for sm_100a and link ``libhe_b200.so`` (or the variant
+    ``libhe_b200_<name>.so`` with the variant's flags plus ``extra_flags``).  Returns the library path."""
     nvcc = nvcc_path()
     if nvcc is None:
         raise RuntimeError("nvcc not found; set HE_NVCC or install the CUDA toolkit")
     OUT_DIR.mkdir(parents=True, exist_ok=True)
-    obj_dir = OUT_DIR / ("obj" if not name else f"obj_{name}")
+    own_flags = name not in ("", SUBSET)
+    obj_dir = OUT_DIR / (f"obj_{name}" if own_flags else "obj")
     obj_dir.mkdir(exist_ok=True)
     flags = list(NVCC_FLAGS) + list(VARIANT_FLAGS.get(name, [])) + list(extra_flags)
     cver = _compiler_version(nvcc)
-    manifest_path = OUT_DIR / ("manifest.json" if not name else f"manifest_{name}.json")
+    manifest_path = OUT_DIR / (f"manifest_{name}.json" if own_flags else "manifest.json")
+    link_entry = "__link__" if name != SUBSET else "__link_subset__"
     try:
         manifest = json.loads(manifest_path.read_text())
     except Exception:
         manifest = {}
-    srcs = sources()
+    srcs = [s for s in sources() if not only or s.name in only]
     todo = []
     objs = []
     for s in srcs:
@@ -136,14 +171,16 @@ def build(verbose: bool = False, force: bool = False, extra_flags: Sequence[str]
                 manifest[src_name] = k
     lib = lib_path(name)
     link_key = hashlib.sha256(("".join(manifest.get(s.name, "") for s in srcs)).encode()).hexdigest()
-    if todo or not lib.exists() or manifest.get("__link__") != link_key:
-        cmd = [nvcc, "-shared", "-o", str(lib)] + [str(o) for o in objs] + ["-Xcompiler", "-fPIC"]
+    if todo or not lib.exists() or manifest.get(link_entry) != link_key:
+        tmp = lib.with_suffix(f".{os.getpid()}.tmp")         # linked beside its place, then moved: never half a library
+        cmd = [nvcc, "-shared", "-o", str(tmp)] + [str(o) for o in objs] + ["-Xcompiler", "-fPIC"]
         if verbose:
             print(" ".join(cmd), flush=True)
         r = subprocess.run(cmd, capture_output=True, text=True)
         if r.returncode != 0:
             raise RuntimeError(f"link failed:\n{r.stdout}\n{r.stderr}")
-        manifest["__link__"] = link_key
+        os.replace(tmp, lib)
+        manifest[link_entry] = link_key
     manifest_path.write_text(json.dumps(manifest, indent=1, sort_keys=True))
     return lib
 

@@ -28,6 +28,7 @@ struct AttnDecArgs {
   int window;                 // > 0: only the last `window` keys are visible
   float scale;
   int* status;                // optional status word: a bounded wait that gave up records its code here
+  float softcap;              // > 0: score <- softcap * tanh(score / softcap), after the scale
 };
 
 namespace {
@@ -249,13 +250,24 @@ __device__ __forceinline__ void bulk_row(void* smem_dst, const void* gsrc, uint3
 }
 __device__ __forceinline__ void cons_sync() { asm volatile("bar.sync 1, %0;" ::"n"(NCONS * 32) : "memory"); }
 
-template <int D, int G>
+// GT > 0: compile-time group of GT query heads per KV head.  GT == 0: any group; a group of more than eight heads is
+// cut into equal chunks of at most eight, each its own CTA (grid.y = KV heads x chunks).
+template <int D, int GT>
 __global__ void __launch_bounds__(NTHREADS) attn_decode_mma_kernel(const AttnDecArgs a) {
-  static_assert(G <= 8 && D % 64 == 0, "group of <= 8 query heads, head_dim a multiple of 64");
+  static_assert(GT <= 8 && D % 64 == 0, "group of <= 8 query heads, head_dim a multiple of 64");
   extern __shared__ __align__(128) uint8_t smem_raw[];
   constexpr int PITCH = pitch<D>();
   constexpr int STAGE = TILE_KEYS * PITCH;
-  const int sp = blockIdx.x, hk = blockIdx.y, r = blockIdx.z;
+  const int sp = blockIdx.x, r = blockIdx.z;
+  int hk = blockIdx.y, h0 = hk * GT, gc = GT;          // KV head, first query head, query heads of this CTA
+  if constexpr (GT == 0) {
+    const int gt = a.H / a.Hkv, nchunk = (gt + 7) / 8, per = (gt + nchunk - 1) / nchunk, ch = blockIdx.y % nchunk;
+    hk = blockIdx.y / nchunk;
+    h0 = hk * gt + ch * per;
+    gc = min(per, gt - ch * per);
+    if (gc <= 0) return;
+  }
+  const int G = GT > 0 ? GT : gc;
   pdl_wait();
   pdl_launch();
   const int ctx = a.ctx_len[r];
@@ -318,7 +330,7 @@ __global__ void __launch_bounds__(NTHREADS) attn_decode_mma_kernel(const AttnDec
   for (int i = tid; i < 8 * (PITCH / 16); i += NCONS * 32) {
     const int g = i / (PITCH / 16), c = i % (PITCH / 16);
     uint4 v = make_uint4(0u, 0u, 0u, 0u);
-    if (g < G && c < D / 8) v = *reinterpret_cast<const uint4*>(a.q + ((size_t)r * a.H + hk * G + g) * D + c * 8);
+    if (g < G && c < D / 8) v = *reinterpret_cast<const uint4*>(a.q + ((size_t)r * a.H + h0 + g) * D + c * 8);
     *reinterpret_cast<uint4*>(q_s + (size_t)g * PITCH + c * 16) = v;
   }
   for (int i = tid; i < (8 - G) * (PP / 16); i += NCONS * 32) {
@@ -354,10 +366,16 @@ __global__ void __launch_bounds__(NTHREADS) attn_decode_mma_kernel(const AttnDec
         if (g < G) {
           float* row = sc + (size_t)g * a.split_len + key0;
           const float NEG = -INFINITY;
-          row[kc] = key0 + kc < n ? s0[0] * a.scale : NEG;
-          row[kc + 1] = key0 + kc + 1 < n ? s0[1] * a.scale : NEG;
-          row[8 + kc] = key0 + 8 + kc < n ? s1[0] * a.scale : NEG;
-          row[8 + kc + 1] = key0 + 8 + kc + 1 < n ? s1[1] * a.scale : NEG;
+          float sv[4] = {s0[0] * a.scale, s0[1] * a.scale, s1[0] * a.scale, s1[1] * a.scale};
+          if (a.softcap > 0.f) {
+            const float ic = 1.f / a.softcap;
+#pragma unroll
+            for (int e = 0; e < 4; ++e) sv[e] = a.softcap * tanh_f(sv[e] * ic);
+          }
+          row[kc] = key0 + kc < n ? sv[0] : NEG;
+          row[kc + 1] = key0 + kc + 1 < n ? sv[1] : NEG;
+          row[8 + kc] = key0 + 8 + kc < n ? sv[2] : NEG;
+          row[8 + kc + 1] = key0 + 8 + kc + 1 < n ? sv[3] : NEG;
         }
       }
       __syncwarp();
@@ -373,7 +391,7 @@ __global__ void __launch_bounds__(NTHREADS) attn_decode_mma_kernel(const AttnDec
 
   // ---- phase 2: per-head softmax statistics of the span, P as bf16 rows
   const int n16 = (n + 15) & ~15;                       // keys covered by the live pages
-  float* part_base = a.partial + (((size_t)r * a.H + hk * G) * a.max_splits + sp) * (D + 2);
+  float* part_base = a.partial + (((size_t)r * a.H + h0) * a.max_splits + sp) * (D + 2);
   for (int g = warp; g < G; g += NCONS) {
     const float* srow = sc + (size_t)g * a.split_len;
     __nv_bfloat16* prow = reinterpret_cast<__nv_bfloat16*>(p_s + (size_t)g * PP);
@@ -500,20 +518,22 @@ bool mma_decode_enabled() {
   return v != 0;
 }
 
-template <int D, int G>
+template <int D, int GT>
 int launch_split_mma(const AttnDecArgs& a, cudaStream_t stream) {
-  const size_t smem = mma_dec::smem_bytes<D>(G, a.split_len);
+  const int group = a.H / a.Hkv, chunks = GT > 0 ? 1 : (group + 7) / 8;
+  const size_t smem = mma_dec::smem_bytes<D>((group + chunks - 1) / chunks, a.split_len);
+  if (smem > 220 * 1024) return -HE_ERR_BAD_ARG;
   static size_t configured[64] = {};
   int dev = 0;
   if (cudaGetDevice(&dev) != cudaSuccess || dev < 0 || dev >= 64) dev = 0;
   if (smem > configured[dev]) {
-    cudaError_t e = cudaFuncSetAttribute(mma_dec::attn_decode_mma_kernel<D, G>,
+    cudaError_t e = cudaFuncSetAttribute(mma_dec::attn_decode_mma_kernel<D, GT>,
                                          cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (e != cudaSuccess) return (int)e;
     configured[dev] = smem;
   }
-  dim3 grid(a.max_splits, a.Hkv, a.R);
-  cudaError_t le = launch_pdl(mma_dec::attn_decode_mma_kernel<D, G>, grid, dim3(mma_dec::NTHREADS), smem, stream, a);
+  dim3 grid(a.max_splits, a.Hkv * chunks, a.R);
+  cudaError_t le = launch_pdl(mma_dec::attn_decode_mma_kernel<D, GT>, grid, dim3(mma_dec::NTHREADS), smem, stream, a);
   if (le != cudaSuccess) return (int)le;
   return 0;
 }
@@ -545,6 +565,12 @@ int launch_split(const AttnDecArgs& a, cudaStream_t stream) {
 
 template <int D>
 int dispatch_g(const AttnDecArgs& a, cudaStream_t stream) {
+  const int group = a.H / a.Hkv;
+  if (a.softcap > 0.f || group == 5 || group > 8 || group == 7) {
+    // soft-capped scores and the other group sizes exist on the tensor-core kernel only
+    if (a.page != 16 || a.split_len % 16 != 0) return -HE_ERR_BAD_ARG;
+    return launch_split_mma<D, 0>(a, stream);
+  }
   switch (a.H / a.Hkv) {
     case 1: return launch_split<D, 1>(a, stream);
     case 2: return launch_split<D, 2>(a, stream);

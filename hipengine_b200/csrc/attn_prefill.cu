@@ -27,6 +27,13 @@ struct PrefillArgs {
   __nv_bfloat16* out;          // [T][H*D]
   int T, H, Hkv, page, pos0, window;
   float scale_log2;            // scale * log2(e)
+  // several segments in one launch: rows [seg_start[s], seg_start[s+1]) belong to segment s, sit at consecutive
+  // positions from pos[seg_start[s]] and attend the pages of block-table row seg_slot[s].  Null: one segment (above).
+  const int* seg_start;
+  const int* seg_slot;
+  const int* pos;
+  int n_seg, max_pages;
+  float cap_in, cap_log2;      // soft cap: score * log2(e) = cap_log2 * tanh(q.k * cap_in)
 };
 
 __device__ __forceinline__ void cp_async16(void* smem, const void* gmem, bool valid) {
@@ -58,15 +65,32 @@ __device__ __forceinline__ uint32_t pack_bf16(float a, float b) {
   return *reinterpret_cast<uint32_t*>(&h);
 }
 
-template <int D>
-__global__ void __launch_bounds__(NTHR) flash_prefill_kernel(const PrefillArgs a) {
+template <int D, bool CAP>
+__global__ void __launch_bounds__(NTHR) flash_prefill_kernel(const PrefillArgs args) {
   constexpr int LDS = D + 8;                 // padded row stride (elements) -> conflict-free ldmatrix
   extern __shared__ __align__(16) __nv_bfloat16 sm[];
   __nv_bfloat16* sQ = sm;                    // [BM][LDS]
   __nv_bfloat16* sK = sQ + BM * LDS;         // [2][BN][LDS]
   __nv_bfloat16* sV = sK + 2 * BN * LDS;     // [2][BN][LDS]
 
-  const int qt = gridDim.x - 1 - blockIdx.x; // heavy (late) tiles first
+  PrefillArgs a = args;
+  int qt = gridDim.x - 1 - blockIdx.x;       // heavy (late) tiles first
+  if (a.seg_start != nullptr) {
+    int s = 0;
+    for (; s < a.n_seg; ++s) {
+      const int tiles = (a.seg_start[s + 1] - a.seg_start[s] + BM - 1) / BM;
+      if (qt < tiles) break;
+      qt -= tiles;
+    }
+    if (s == a.n_seg) return;
+    const int row0 = a.seg_start[s];
+    a.T = a.seg_start[s + 1] - row0;
+    a.pos0 = a.pos[row0];
+    a.block_table += (size_t)a.seg_slot[s] * a.max_pages;
+    a.q += (size_t)row0 * a.H * D;
+    a.out += (size_t)row0 * a.H * D;
+    if (a.gate != nullptr) a.gate += (size_t)row0 * a.H * D;
+  }
   const int h = blockIdx.y, hk = h / (a.H / a.Hkv);
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const int g = lane >> 2, c = lane & 3;
@@ -143,6 +167,29 @@ __global__ void __launch_bounds__(NTHR) flash_prefill_kernel(const PrefillArgs a
     // ---- mask + online softmax (rows g and g+8 of this warp's 16)
     const int k0 = kv_begin + tile * BN;
     float mx[2] = {-INFINITY, -INFINITY};
+    if constexpr (CAP) {
+      // soft cap: the power series when every score of the warp's tile is small against the cap, else the quotient form
+      float xm = 0.f;
+#pragma unroll
+      for (int j = 0; j < BN / 8; ++j)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          sacc[j][e] *= a.cap_in;
+          xm = fmaxf(xm, fabsf(sacc[j][e]));
+        }
+      if (__any_sync(0xffffffffu, xm >= TANH_SERIES_MAX)) {
+#pragma unroll
+        for (int j = 0; j < BN / 8; ++j)
+#pragma unroll
+          for (int e = 0; e < 4; ++e) sacc[j][e] = tanh_f(sacc[j][e]);
+      } else {
+#pragma unroll
+        for (int j = 0; j < BN / 8; ++j)
+#pragma unroll
+          for (int e = 0; e < 4; ++e) sacc[j][e] = tanh_series_f(sacc[j][e]);
+      }
+    }
+    const float sc_log2 = CAP ? a.cap_log2 : a.scale_log2;
 #pragma unroll
     for (int j = 0; j < BN / 8; ++j) {
 #pragma unroll
@@ -151,7 +198,7 @@ __global__ void __launch_bounds__(NTHR) flash_prefill_kernel(const PrefillArgs a
         const int qp = qrow0 + (e >> 1) * 8;
         bool ok = key <= qp && key < kv_end;
         if (a.window > 0) ok = ok && key > qp - a.window;
-        const float v = ok ? sacc[j][e] * a.scale_log2 : -INFINITY;
+        const float v = ok ? sacc[j][e] * sc_log2 : -INFINITY;
         sacc[j][e] = v;
         mx[e >> 1] = fmaxf(mx[e >> 1], v);
       }
@@ -229,14 +276,14 @@ __global__ void __launch_bounds__(NTHR) flash_prefill_kernel(const PrefillArgs a
   }
 }
 
-template <int D>
-int launch(const PrefillArgs& a, cudaStream_t stream) {
+template <int D, bool CAP>
+int launch(const PrefillArgs& a, int tiles, cudaStream_t stream) {
   const size_t smem = (size_t)(BM + 4 * BN) * (D + 8) * sizeof(__nv_bfloat16);
   // set per call (cheap): the attribute belongs to the (function, device) pair, not to the process
-  cudaError_t e = cudaFuncSetAttribute(flash_prefill_kernel<D>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+  cudaError_t e = cudaFuncSetAttribute(flash_prefill_kernel<D, CAP>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
   if (e != cudaSuccess) return (int)e;
-  dim3 grid((a.T + BM - 1) / BM, a.H);
-  flash_prefill_kernel<D><<<grid, NTHR, smem, stream>>>(a);
+  dim3 grid(tiles, a.H);
+  flash_prefill_kernel<D, CAP><<<grid, NTHR, smem, stream>>>(a);
   HE_LAUNCH_CHECK();
   return 0;
 }
@@ -249,15 +296,48 @@ HE_API int he_flash_prefill(const void* q, const void* gate, const void* kv_cach
                             cudaStream_t stream) {
   if (T <= 0) return 0;
   if (H % Hkv != 0) return -HE_ERR_BAD_ARG;
-  PrefillArgs a;
+  PrefillArgs a = {};
   a.q = (const __nv_bfloat16*)q; a.gate = (const __nv_bfloat16*)gate; a.kv = (const __nv_bfloat16*)kv_cache;
   a.block_table = (const int*)block_table_row; a.out = (__nv_bfloat16*)out;
   a.T = T; a.H = H; a.Hkv = Hkv; a.page = page; a.pos0 = pos0; a.window = window;
   a.scale_log2 = scale * 1.4426950408889634f;
+  const int tiles = (T + BM - 1) / BM;
   switch (D) {
-    case 64: return launch<64>(a, stream);
-    case 128: return launch<128>(a, stream);
-    case 256: return launch<256>(a, stream);
+    case 64: return launch<64, false>(a, tiles, stream);
+    case 128: return launch<128, false>(a, tiles, stream);
+    case 256: return launch<256, false>(a, tiles, stream);
+    default: return -HE_ERR_BAD_ARG;
+  }
+}
+
+// Several segments in one launch (see PrefillArgs); `seg_start` holds n_seg + 1 absolute row offsets into q / out and
+// `tiles` the total of 64-row tiles over the segments (each rounded up; more is allowed).  softcap 0: none.
+HE_API int he_flash_prefill_segs(const void* q, const void* gate, const void* kv_cache, const void* block_table,
+                                 int max_pages, const int* seg_start, const int* seg_slot, const int* pos, int n_seg,
+                                 int tiles, void* out, int H, int Hkv, int D, int page, float scale, int window,
+                                 float softcap, cudaStream_t stream) {
+  if (n_seg <= 0 || tiles <= 0) return 0;
+  if (H % Hkv != 0 || seg_start == nullptr || seg_slot == nullptr || pos == nullptr) return -HE_ERR_BAD_ARG;
+  PrefillArgs a = {};
+  a.q = (const __nv_bfloat16*)q; a.gate = (const __nv_bfloat16*)gate; a.kv = (const __nv_bfloat16*)kv_cache;
+  a.block_table = (const int*)block_table; a.out = (__nv_bfloat16*)out;
+  a.H = H; a.Hkv = Hkv; a.page = page; a.window = window;
+  a.seg_start = seg_start; a.seg_slot = seg_slot; a.pos = pos; a.n_seg = n_seg; a.max_pages = max_pages;
+  a.scale_log2 = scale * 1.4426950408889634f;
+  if (softcap > 0.f) {
+    a.cap_in = scale / softcap;
+    a.cap_log2 = softcap * 1.4426950408889634f;
+    switch (D) {
+      case 64: return launch<64, true>(a, tiles, stream);
+      case 128: return launch<128, true>(a, tiles, stream);
+      case 256: return launch<256, true>(a, tiles, stream);
+      default: return -HE_ERR_BAD_ARG;
+    }
+  }
+  switch (D) {
+    case 64: return launch<64, false>(a, tiles, stream);
+    case 128: return launch<128, false>(a, tiles, stream);
+    case 256: return launch<256, false>(a, tiles, stream);
     default: return -HE_ERR_BAD_ARG;
   }
 }

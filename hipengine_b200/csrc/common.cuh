@@ -134,6 +134,25 @@ __device__ __forceinline__ float gelu_tanh_f(float x) {
   const float k = 0.7978845608028654f;
   return 0.5f * x * (1.f + tanhf(k * (x + 0.044715f * x * x * x)));
 }
+// min(g, limit) * sigmoid(1.702 min(g, limit)) * (clamp(u, -limit, limit) + 1)
+__device__ __forceinline__ float clamped_glu_f(float g, float u, float limit) {
+  g = fminf(g, limit);
+  u = fminf(fmaxf(u, -limit), limit);
+  return g * sigmoid_f(1.702f * g) * (u + 1.f);
+}
+// tanh with ~1e-6 absolute error from fast instructions: the power series near zero (where the quotient form loses
+// its leading digits), 1 - 2 / (e^{2|x|} + 1) elsewhere
+constexpr float TANH_SERIES_MAX = 0.25f;
+__device__ __forceinline__ float tanh_series_f(float x) {
+  const float y = x * x;
+  return x * (1.f + y * (-1.f / 3.f + y * (2.f / 15.f + y * (-17.f / 315.f + y * (62.f / 2835.f)))));
+}
+__device__ __forceinline__ float tanh_exp_f(float x) {
+  return copysignf(1.f - __fdividef(2.f, __expf(2.f * fabsf(x)) + 1.f), x);
+}
+__device__ __forceinline__ float tanh_f(float x) {
+  return fabsf(x) < TANH_SERIES_MAX ? tanh_series_f(x) : tanh_exp_f(x);
+}
 __device__ __forceinline__ float softplus20_f(float x) { return x > 20.f ? x : log1pf(__expf(x)); }
 
 __device__ __forceinline__ uint4 ldg128(const void* p) { return __ldg(reinterpret_cast<const uint4*>(p)); }

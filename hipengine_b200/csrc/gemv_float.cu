@@ -1,0 +1,391 @@
+// Streaming matrix-vector products with bfloat16 weights for 1..16 activation rows (decode and short portions).
+//
+// One CTA of eight warps owns 16 weight rows (or 16 gate rows and the same 16 up rows); the warps split K in 64-column
+// units, so a unit of one row is a full 128-byte line.  The product runs on mma.sync m16n8k16 with the WEIGHTS as the
+// 16-row operand and the activation rows as the 8 (or 16) columns: a lane reads 16 consecutive bytes of a weight row
+// from global memory straight into fragment registers, because any permutation of the K order is allowed as long as both
+// operands use the same one.  Weights pass through no shared memory and are read exactly once; the first unit batch is
+// requested before the kernel waits for its predecessor.
+//   norm      : RMS norm needs no separate pass: sum over k of w[k] (x[k] g[k]) is scaled by 1/rms(x) at the end, and
+//               every warp accumulates the squares of the columns it reads anyway (fp32)
+//   epilogue  : fp32 / bf16 store, fp32 residual add, or act(gate) * up (SiLU, tanh-GELU, clamped GLU)
+// The expert forms add an indirection: grid.y is a (token, expert) pair or a token, the weight base comes from the
+// routed expert id, and the down projection walks the concatenated columns of all selected experts (and the shared
+// one), which adds the k expert outputs in a fixed order inside the accumulator.
+#include "common.cuh"
+
+using namespace he;
+
+struct FloatGemvSeg {
+  const __nv_bfloat16* w;
+  const __nv_bfloat16* w2;   // gate/up pair: the up rows
+  void* out;
+  long long out_stride;
+  int n_rows;
+  int epi;                   // 0 f32, 1 bf16, 2 f32 +=, 3 silu(g)*u, 4 gelu_tanh(g)*u, 5 clamped GLU (all bf16)
+};
+
+struct FloatGemvArgs {
+  FloatGemvSeg seg[4];
+  int n_seg;
+  int K;                     // columns, multiple of 8
+  long long ldw;             // elements between weight rows (all segments)
+  int R;
+  int x_dtype;               // 0 f32, 1 bf16
+  const void* x;
+  long long x_stride;
+  const float* norm_w;       // fp32 rows only
+  float eps;
+  int norm_n;                // columns the mean square is taken over (zero-padded rows are wider)
+  float limit;               // epi 5
+};
+
+struct FloatMoeArgs {
+  const void* x;             // gate/up: fp32 residual rows [T][ldx]
+  long long ldx;
+  const float* norm_w;
+  float eps;
+  int norm_n;
+  const int* ids;            // [T][k]
+  const float* wts;          // [T][k]
+  const float* sg;           // [T] (stride ld_sg) logit of the shared expert's gate, or null
+  long long ld_sg;
+  const __nv_bfloat16* w1;   // gate/up: [E][2F][K] (gate rows, then up rows); down: [E][N][F]
+  const __nv_bfloat16* w1s;  // shared expert, same form with Fs, or null
+  int E, T, k, K, F, Fs, N;
+  int act;                   // epilogue code 3..5
+  float limit;
+  __nv_bfloat16* rows;       // [T*k][F] activations of the selected experts, routing weight folded in
+  __nv_bfloat16* rows_s;     // [T][Fs] activations of the shared expert, gate folded in
+  float* h;                  // down: residual rows, added in place
+  long long ldh;
+};
+
+namespace {
+
+constexpr int NW = 8;         // warps per CTA
+constexpr int UK = 64;        // columns per unit
+
+__device__ __forceinline__ void mma_16816(float (&c)[4], uint32_t a0, uint32_t a1, uint32_t a2, uint32_t a3, uint32_t b0,
+                                          uint32_t b1) {
+  asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
+               : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
+               : "r"(a0), "r"(a1), "r"(a2), "r"(a3), "r"(b0), "r"(b1));
+}
+__device__ __forceinline__ uint32_t pack2(float a, float b) {
+  __nv_bfloat162 h = __floats2bfloat162_rn(a, b);
+  return *reinterpret_cast<uint32_t*>(&h);
+}
+
+__device__ __forceinline__ float glu_f(float g, float u, int epi, float limit) {
+  if (epi == 3) return silu_f(g) * u;
+  if (epi == 4) return gelu_tanh_f(g) * u;
+  return clamped_glu_f(g, u, limit);
+}
+
+// eight activation values of row `r` at column k as four bf16x2 words (zero outside); fp32 rows are scaled by the norm
+// weight and their squares go into ss
+template <bool XF32>
+__device__ __forceinline__ uint4 load_x(const void* x, size_t off, bool live, const float* norm_w, int k, float& ss) {
+  if (!live) return make_uint4(0u, 0u, 0u, 0u);
+  if constexpr (XF32) {
+    const float4* p = reinterpret_cast<const float4*>(reinterpret_cast<const float*>(x) + off);
+    float4 a = p[0], b = p[1];
+    if (norm_w != nullptr) {
+      ss += a.x * a.x + a.y * a.y + a.z * a.z + a.w * a.w + b.x * b.x + b.y * b.y + b.z * b.z + b.w * b.w;
+      const float4 u = __ldg(reinterpret_cast<const float4*>(norm_w + k));
+      const float4 v = __ldg(reinterpret_cast<const float4*>(norm_w + k + 4));
+      a.x *= u.x; a.y *= u.y; a.z *= u.z; a.w *= u.w;
+      b.x *= v.x; b.y *= v.y; b.z *= v.z; b.w *= v.w;
+    }
+    return make_uint4(pack2(a.x, a.y), pack2(a.z, a.w), pack2(b.x, b.y), pack2(b.z, b.w));
+  } else {
+    return *reinterpret_cast<const uint4*>(reinterpret_cast<const __nv_bfloat16*>(x) + off);
+  }
+}
+
+template <int MT, int NT>
+struct Tile {
+  float part[NW][MT * 16][NT * 8 + 1];
+  float ssq[NW][NT * 8];
+};
+
+template <int MT, int NT>
+__device__ __forceinline__ void store_partials(Tile<MT, NT>& sm, const float (&acc)[MT][NT][4], float (&ss)[NT]) {
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, g = lane >> 2, c = lane & 3;
+#pragma unroll
+  for (int m = 0; m < MT; ++m)
+#pragma unroll
+    for (int n = 0; n < NT; ++n) {
+      sm.part[warp][m * 16 + g][n * 8 + 2 * c] = acc[m][n][0];
+      sm.part[warp][m * 16 + g][n * 8 + 2 * c + 1] = acc[m][n][1];
+      sm.part[warp][m * 16 + g + 8][n * 8 + 2 * c] = acc[m][n][2];
+      sm.part[warp][m * 16 + g + 8][n * 8 + 2 * c + 1] = acc[m][n][3];
+    }
+#pragma unroll
+  for (int n = 0; n < NT; ++n) {
+    ss[n] += __shfl_xor_sync(0xffffffffu, ss[n], 1);
+    ss[n] += __shfl_xor_sync(0xffffffffu, ss[n], 2);
+    if (c == 0) sm.ssq[warp][n * 8 + g] = ss[n];
+  }
+}
+
+template <int MT, int NT>
+__device__ __forceinline__ float sum_partials(const Tile<MT, NT>& sm, int row, int col) {
+  float v = 0.f;
+#pragma unroll
+  for (int w = 0; w < NW; ++w) v += sm.part[w][row][col];
+  return v;
+}
+
+template <int MT, int NT>
+__device__ __forceinline__ float inv_rms_of(const Tile<MT, NT>& sm, int col, int n, float eps) {
+  float s = 0.f;
+#pragma unroll
+  for (int w = 0; w < NW; ++w) s += sm.ssq[w][col];
+  return rsqrtf(s / (float)n + eps);
+}
+
+// acc += W[16 MT rows][K] x[K][8 NT]: this warp's units.  wrow[m][half] points at column 8c of row (g + 8 half) of tile m.
+// EARLY: the weights do not depend on earlier kernels, so the first batch is requested before griddepcontrol.wait.
+template <int MT, int NT, bool XF32, bool EARLY>
+__device__ __forceinline__ void product(const __nv_bfloat16* const (&wrow)[MT][2], int K, const void* x,
+                                        long long x_stride, int R, const float* norm_w, float (&acc)[MT][NT][4],
+                                        float (&ss)[NT]) {
+  constexpr int UN = MT == 1 ? 4 : 2;                    // units in flight per warp: 16 x 16 bytes per lane
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, g = lane >> 2, c = lane & 3;
+  const int units = (K + UK - 1) / UK;
+  uint4 A[UN][2][MT][2];
+  auto load_a = [&](int u0) {
+#pragma unroll
+    for (int i = 0; i < UN; ++i)
+#pragma unroll
+      for (int s = 0; s < 2; ++s) {
+        const int k = (u0 + i * NW) * UK + s * 32;
+        const bool live = k + 8 * c < K;
+#pragma unroll
+        for (int m = 0; m < MT; ++m)
+#pragma unroll
+          for (int hf = 0; hf < 2; ++hf)
+            A[i][s][m][hf] = live ? ldg128_stream(wrow[m][hf] + k) : make_uint4(0u, 0u, 0u, 0u);
+      }
+  };
+  if (EARLY) {
+    load_a(warp);
+    pdl_wait();
+  }
+  for (int u0 = warp; u0 < units; u0 += UN * NW) {
+    if (!EARLY || u0 != warp) load_a(u0);
+#pragma unroll
+    for (int i = 0; i < UN; ++i)
+#pragma unroll
+      for (int s = 0; s < 2; ++s) {
+        const int k = (u0 + i * NW) * UK + s * 32 + 8 * c;
+#pragma unroll
+        for (int n = 0; n < NT; ++n) {
+          const int r = n * 8 + g;
+          const uint4 b = load_x<XF32>(x, (size_t)r * x_stride + k, r < R && k < K, norm_w, k, ss[n]);
+#pragma unroll
+          for (int m = 0; m < MT; ++m) {
+            mma_16816(acc[m][n], A[i][s][m][0].x, A[i][s][m][1].x, A[i][s][m][0].y, A[i][s][m][1].y, b.x, b.y);
+            mma_16816(acc[m][n], A[i][s][m][0].z, A[i][s][m][1].z, A[i][s][m][0].w, A[i][s][m][1].w, b.z, b.w);
+          }
+        }
+      }
+  }
+}
+
+// grid: items of all segments (16 rows, or 16 gate/up row pairs when MT == 2)
+template <int MT, int NT, bool XF32>
+__global__ void __launch_bounds__(NW * 32, 2) gemv_float_kernel(const __grid_constant__ FloatGemvArgs a) {
+  __shared__ Tile<MT, NT> sm;
+  pdl_launch();
+  const int lane = threadIdx.x & 31, g = lane >> 2, c = lane & 3;
+  int item = blockIdx.x, si = 0;
+  while (si < a.n_seg - 1 && item >= (a.seg[si].n_rows + 15) / 16) {
+    item -= (a.seg[si].n_rows + 15) / 16;
+    ++si;
+  }
+  const FloatGemvSeg& sg = a.seg[si];
+  const int row0 = item * 16;
+  const __nv_bfloat16* wrow[MT][2];
+#pragma unroll
+  for (int hf = 0; hf < 2; ++hf) {
+    const size_t off = (size_t)min(row0 + g + 8 * hf, sg.n_rows - 1) * a.ldw + 8 * c;
+    wrow[0][hf] = sg.w + off;
+    if constexpr (MT == 2) wrow[1][hf] = sg.w2 + off;
+  }
+  float acc[MT][NT][4] = {};
+  float ss[NT] = {};
+  product<MT, NT, XF32, true>(wrow, a.K, a.x, a.x_stride, a.R, a.norm_w, acc, ss);
+  store_partials<MT, NT>(sm, acc, ss);
+  __syncthreads();
+  for (int o = threadIdx.x; o < 16 * NT * 8; o += NW * 32) {
+    const int row = o & 15, col = o >> 4, n = row0 + row;
+    if (col >= a.R || n >= sg.n_rows) continue;
+    const float inv = a.norm_w != nullptr ? inv_rms_of<MT, NT>(sm, col, a.norm_n, a.eps) : 1.f;
+    const float v = sum_partials<MT, NT>(sm, row, col) * inv;
+    const size_t off = (size_t)col * sg.out_stride + n;
+    if constexpr (MT == 2) {
+      const float u = sum_partials<MT, NT>(sm, 16 + row, col) * inv;
+      reinterpret_cast<__nv_bfloat16*>(sg.out)[off] = f32_to_bf16(glu_f(v, u, sg.epi, a.limit));
+    } else if (sg.epi == 0) {
+      reinterpret_cast<float*>(sg.out)[off] = v;
+    } else if (sg.epi == 1) {
+      reinterpret_cast<__nv_bfloat16*>(sg.out)[off] = f32_to_bf16(v);
+    } else {
+      reinterpret_cast<float*>(sg.out)[off] += v;
+    }
+  }
+}
+
+// grid (ceil(max(F, Fs) / 16), T * k [+ T]): activation rows of the selected experts, then of the shared expert
+__global__ void __launch_bounds__(NW * 32, 2) moe_gateup_float_kernel(const __grid_constant__ FloatMoeArgs a) {
+  __shared__ Tile<2, 1> sm;
+  pdl_launch();
+  pdl_wait();
+  const int lane = threadIdx.x & 31, g = lane >> 2, c = lane & 3;
+  const int p = blockIdx.y;
+  const bool shared = p >= a.T * a.k;
+  const int t = shared ? p - a.T * a.k : p / a.k;
+  const int F = shared ? a.Fs : a.F;
+  const int row0 = blockIdx.x * 16;
+  if (row0 >= F) return;
+  int e = shared ? 0 : a.ids[p];
+  if (!shared && (!HE_INDEX_OK(e, a.E, HE_SITE_MOE_EXPERT_ID) || e < 0 || e >= a.E)) e = 0;
+  const __nv_bfloat16* base = shared ? a.w1s : a.w1 + (size_t)e * 2 * F * a.K;
+  const __nv_bfloat16* wrow[2][2];
+#pragma unroll
+  for (int hf = 0; hf < 2; ++hf) {
+    const int r = min(row0 + g + 8 * hf, F - 1);
+    wrow[0][hf] = base + (size_t)r * a.K + 8 * c;
+    wrow[1][hf] = base + (size_t)(F + r) * a.K + 8 * c;
+  }
+  float acc[2][1][4] = {};
+  float ss[1] = {};
+  product<2, 1, true, false>(wrow, a.K, reinterpret_cast<const float*>(a.x) + (size_t)t * a.ldx, a.ldx, 1, a.norm_w, acc,
+                             ss);
+  store_partials<2, 1>(sm, acc, ss);
+  __syncthreads();
+  const int row = threadIdx.x, n = row0 + row;
+  if (row < 16 && n < F) {
+    const float inv = a.norm_w != nullptr ? inv_rms_of<2, 1>(sm, 0, a.norm_n, a.eps) : 1.f;
+    const float gv = sum_partials<2, 1>(sm, row, 0) * inv, uv = sum_partials<2, 1>(sm, 16 + row, 0) * inv;
+    const float wt = shared ? (a.sg != nullptr ? sigmoid_f(a.sg[(size_t)t * a.ld_sg]) : 1.f) : a.wts[p];
+    const float v = glu_f(gv, uv, a.act, a.limit) * wt;
+    if (shared) a.rows_s[(size_t)t * F + n] = f32_to_bf16(v);
+    else a.rows[(size_t)p * F + n] = f32_to_bf16(v);
+  }
+}
+
+// grid (ceil(N / 16), T): h[t] += sum over the token's experts (and the shared one) of W_down row . activation row
+__global__ void __launch_bounds__(NW * 32, 2) moe_down_float_kernel(const __grid_constant__ FloatMoeArgs a) {
+  __shared__ Tile<1, 1> sm;
+  __shared__ int e_s[32];
+  pdl_launch();
+  pdl_wait();
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, g = lane >> 2, c = lane & 3;
+  const int t = blockIdx.y, row0 = blockIdx.x * 16;
+  if (threadIdx.x < a.k) {
+    int e = a.ids[(size_t)t * a.k + threadIdx.x];
+    if (!HE_INDEX_OK(e, a.E, HE_SITE_MOE_EXPERT_ID) || e < 0 || e >= a.E) e = 0;
+    e_s[threadIdx.x] = e;
+  }
+  __syncthreads();
+  const int upe = (a.F + UK - 1) / UK, ups = a.w1s != nullptr ? (a.Fs + UK - 1) / UK : 0;
+  const int units = a.k * upe + ups;
+  const int ra = min(row0 + g, a.N - 1), rb = min(row0 + g + 8, a.N - 1);
+  float acc[1][1][4] = {};
+  float ss[1] = {};
+  constexpr int UN = 4;
+  for (int u0 = warp; u0 < units; u0 += UN * NW) {
+    uint4 A[UN][2][2], B[UN][2];
+#pragma unroll
+    for (int i = 0; i < UN; ++i) {
+      const int u = u0 + i * NW;
+      const bool sh = u >= a.k * upe;
+      const int j = sh ? 0 : u / upe;
+      const int k0 = (sh ? u - a.k * upe : u - j * upe) * UK;
+      const int F = sh ? a.Fs : a.F;
+      const __nv_bfloat16* wb = sh ? a.w1s : a.w1 + (size_t)e_s[j] * a.N * F;
+      const __nv_bfloat16* xb = sh ? a.rows_s + (size_t)t * F : a.rows + ((size_t)t * a.k + j) * F;
+#pragma unroll
+      for (int s = 0; s < 2; ++s) {
+        const int k = k0 + s * 32 + 8 * c;
+        const bool live = u < units && k < F;
+        A[i][s][0] = live ? ldg128_stream(wb + (size_t)ra * F + k) : make_uint4(0u, 0u, 0u, 0u);
+        A[i][s][1] = live ? ldg128_stream(wb + (size_t)rb * F + k) : make_uint4(0u, 0u, 0u, 0u);
+        B[i][s] = live && g == 0 ? *reinterpret_cast<const uint4*>(xb + k) : make_uint4(0u, 0u, 0u, 0u);
+      }
+    }
+#pragma unroll
+    for (int i = 0; i < UN; ++i)
+#pragma unroll
+      for (int s = 0; s < 2; ++s) {
+        mma_16816(acc[0][0], A[i][s][0].x, A[i][s][1].x, A[i][s][0].y, A[i][s][1].y, B[i][s].x, B[i][s].y);
+        mma_16816(acc[0][0], A[i][s][0].z, A[i][s][1].z, A[i][s][0].w, A[i][s][1].w, B[i][s].z, B[i][s].w);
+      }
+  }
+  store_partials<1, 1>(sm, acc, ss);
+  __syncthreads();
+  const int n = row0 + (int)threadIdx.x;
+  if (threadIdx.x < 16 && n < a.N) a.h[(size_t)t * a.ldh + n] += sum_partials<1, 1>(sm, threadIdx.x, 0);
+}
+
+template <int MT>
+int launch_rows(const FloatGemvArgs& a, int items, cudaStream_t stream) {
+  cudaError_t e;
+  const dim3 grid(items), block(NW * 32);
+  if (a.x_dtype == 0) {
+    e = a.R <= 8 ? launch_pdl(gemv_float_kernel<MT, 1, true>, grid, block, 0, stream, a)
+                 : launch_pdl(gemv_float_kernel<MT, 2, true>, grid, block, 0, stream, a);
+  } else {
+    e = a.R <= 8 ? launch_pdl(gemv_float_kernel<MT, 1, false>, grid, block, 0, stream, a)
+                 : launch_pdl(gemv_float_kernel<MT, 2, false>, grid, block, 0, stream, a);
+  }
+  return (int)e;
+}
+
+}  // namespace
+
+// Rows of x (fp32 with an optional fused RMS norm, or bf16) times up to four bf16 weight segments of the same width.
+// All segments of a launch are plain (epi 0..2) or all are gate/up pairs (epi 3..5).
+HE_API int he_gemv_float(const FloatGemvArgs* args, cudaStream_t stream) {
+  const FloatGemvArgs& a = *args;
+  if (a.R < 1 || a.R > 16 || a.n_seg < 1 || a.n_seg > 4 || a.K <= 0 || a.K % 8 != 0 || a.ldw % 8 != 0 || a.ldw < a.K)
+    return -HE_ERR_BAD_ARG;
+  if (a.x_stride % 8 != 0 || (a.norm_w != nullptr && (a.x_dtype != 0 || a.norm_n <= 0))) return -HE_ERR_BAD_ARG;
+  const bool pair = a.seg[0].epi >= 3;
+  int items = 0;
+  for (int i = 0; i < a.n_seg; ++i) {
+    if ((a.seg[i].epi >= 3) != pair || a.seg[i].epi < 0 || a.seg[i].epi > 5 || a.seg[i].n_rows <= 0 ||
+        (pair && a.seg[i].w2 == nullptr))
+      return -HE_ERR_BAD_ARG;
+    items += (a.seg[i].n_rows + 15) / 16;
+  }
+  return pair ? launch_rows<2>(a, items, stream) : launch_rows<1>(a, items, stream);
+}
+HE_API int he_gemv_float_args_size() { return (int)sizeof(FloatGemvArgs); }
+
+static int check_moe(const FloatMoeArgs& a) {
+  if (a.k <= 0 || a.k > 32 || a.E < a.k || a.F <= 0 || a.F % 8 != 0 || (a.w1s != nullptr && (a.Fs <= 0 || a.Fs % 8 != 0)))
+    return -HE_ERR_BAD_ARG;
+  return 0;
+}
+
+HE_API int he_moe_gateup_float(const FloatMoeArgs* args, cudaStream_t stream) {
+  const FloatMoeArgs& a = *args;
+  if (a.T <= 0) return 0;
+  if (check_moe(a) != 0 || a.K % 8 != 0 || a.ldx % 8 != 0 || a.act < 3 || a.act > 5) return -HE_ERR_BAD_ARG;
+  const int F = a.w1s != nullptr && a.Fs > a.F ? a.Fs : a.F;
+  const dim3 grid((F + 15) / 16, a.T * a.k + (a.w1s != nullptr ? a.T : 0));
+  return (int)launch_pdl(moe_gateup_float_kernel, grid, dim3(NW * 32), 0, stream, a);
+}
+
+HE_API int he_moe_down_float(const FloatMoeArgs* args, cudaStream_t stream) {
+  const FloatMoeArgs& a = *args;
+  if (a.T <= 0) return 0;
+  if (check_moe(a) != 0 || a.N <= 0) return -HE_ERR_BAD_ARG;
+  return (int)launch_pdl(moe_down_float_kernel, dim3((a.N + 15) / 16, a.T), dim3(NW * 32), 0, stream, a);
+}
+HE_API int he_moe_float_args_size() { return (int)sizeof(FloatMoeArgs); }

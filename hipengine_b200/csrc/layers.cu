@@ -15,7 +15,7 @@ namespace {
 template <typename OutT>
 __global__ void __launch_bounds__(256) rmsnorm_rows_kernel(const float* __restrict__ x, const float* __restrict__ w,
                                                            OutT* __restrict__ out, int H, float eps,
-                                                           long long x_stride, long long out_stride) {
+                                                           long long x_stride, long long out_stride, int n_mean) {
   pdl_wait();      // launched with programmatic stream serialization: order after all earlier kernels
   pdl_launch();
   __shared__ float red[33];
@@ -26,7 +26,7 @@ __global__ void __launch_bounds__(256) rmsnorm_rows_kernel(const float* __restri
     ss += v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w;
   }
   ss = block_sum(ss, red);
-  const float inv = rsqrtf(ss / (float)H + eps);
+  const float inv = rsqrtf(ss / (float)n_mean + eps);    // zero-padded rows: n_mean < H real columns
   OutT* orow = out + (size_t)blockIdx.x * out_stride;
   for (int i = threadIdx.x * 4; i < H; i += blockDim.x * 4) {
     const float4 v = *reinterpret_cast<const float4*>(xr + i);
@@ -45,9 +45,15 @@ __global__ void __launch_bounds__(256) rmsnorm_rows_kernel(const float* __restri
   }
 }
 
+// act codes: 0 silu(g) * u, 1 gelu_tanh(g) * u, 2 clamped GLU with `limit`
+__device__ __forceinline__ float act_pair(float g, float u, int act, float limit) {
+  if (act == 2) return clamped_glu_f(g, u, limit);
+  return (act == 0 ? silu_f(g) : gelu_tanh_f(g)) * u;
+}
+
 // ---------------------------------------------------------------- act(gate) * up over packed [T][2F] bf16 -> [T][F] bf16
 __global__ void act_mul_kernel(const __nv_bfloat16* __restrict__ gu, __nv_bfloat16* __restrict__ out, long long T,
-                               int F, int act) {
+                               int F, int act, float limit) {
   pdl_wait();      // launched with programmatic stream serialization: order after all earlier kernels
   pdl_launch();
   const long long i = ((long long)blockIdx.x * blockDim.x + threadIdx.x) * 8;
@@ -62,16 +68,15 @@ __global__ void act_mul_kernel(const __nv_bfloat16* __restrict__ gu, __nv_bfloat
 #pragma unroll
   for (int k = 0; k < 4; ++k) {
     const float2 g = __bfloat1622float2(g2[k]), u = __bfloat1622float2(u2[k]);
-    const float a0 = act == 0 ? silu_f(g.x) : gelu_tanh_f(g.x);
-    const float a1 = act == 0 ? silu_f(g.y) : gelu_tanh_f(g.y);
-    o[k] = __floats2bfloat162_rn(a0 * u.x, a1 * u.y);
+    o[k] = __floats2bfloat162_rn(act_pair(g.x, u.x, act, limit), act_pair(g.y, u.y, act, limit));
   }
   *reinterpret_cast<uint4*>(out + i) = *reinterpret_cast<const uint4*>(o);
 }
 
-// same with the packed gate | up rows in fp32 (split-K accumulators of small batches)
-__global__ void act_mul_f32_kernel(const float* __restrict__ gu, __nv_bfloat16* __restrict__ out, long long T, int F,
-                                   int act) {
+// same with the packed gate | up rows in fp32 (split-K accumulators of small batches); bf16 or fp32 result
+template <typename OutT>
+__global__ void act_mul_f32_kernel(const float* __restrict__ gu, OutT* __restrict__ out, long long T, int F, int act,
+                                   float limit) {
   pdl_wait();      // launched with programmatic stream serialization: order after all earlier kernels
   pdl_launch();
   const long long i = ((long long)blockIdx.x * blockDim.x + threadIdx.x) * 4;
@@ -81,14 +86,15 @@ __global__ void act_mul_f32_kernel(const float* __restrict__ gu, __nv_bfloat16* 
   const float4 g = *reinterpret_cast<const float4*>(gu + (size_t)t * 2 * F + f);
   const float4 u = *reinterpret_cast<const float4*>(gu + (size_t)t * 2 * F + F + f);
   const float gx[4] = {g.x, g.y, g.z, g.w}, ux[4] = {u.x, u.y, u.z, u.w};
-  __align__(8) __nv_bfloat162 o[2];
+  float y[4];
 #pragma unroll
-  for (int k = 0; k < 2; ++k) {
-    const float a0 = act == 0 ? silu_f(gx[2 * k]) : gelu_tanh_f(gx[2 * k]);
-    const float a1 = act == 0 ? silu_f(gx[2 * k + 1]) : gelu_tanh_f(gx[2 * k + 1]);
-    o[k] = __floats2bfloat162_rn(a0 * ux[2 * k], a1 * ux[2 * k + 1]);
+  for (int k = 0; k < 4; ++k) y[k] = act_pair(gx[k], ux[k], act, limit);
+  if constexpr (sizeof(OutT) == 2) {
+    __align__(8) __nv_bfloat162 o[2] = {__floats2bfloat162_rn(y[0], y[1]), __floats2bfloat162_rn(y[2], y[3])};
+    *reinterpret_cast<uint2*>(out + i) = *reinterpret_cast<const uint2*>(o);
+  } else {
+    *reinterpret_cast<float4*>(out + i) = make_float4(y[0], y[1], y[2], y[3]);
   }
-  *reinterpret_cast<uint2*>(out + i) = *reinterpret_cast<const uint2*>(o);
 }
 
 // ---------------------------------------------------------------- residual add: h (fp32) += y (bf16)
@@ -129,6 +135,8 @@ struct QkvArgs {
   float eps;
   float q_scale;           // multiplied into Q after norm/rope (1 = none)
   int rope_denom;          // frequency spacing: inv_freq_i = theta^(-2i / rope_denom); 0 -> rope_dim
+  int d_in, dv_in;         // head widths of the projections (0 -> D): narrower heads are zero-padded to D
+  int out_f32;             // 1: q_out and kv_cache hold fp32 (the float32 compute dtype)
 };
 
 __device__ __forceinline__ float load_in(const void* p, int dtype, size_t i) {
@@ -147,17 +155,20 @@ __global__ void qkv_post_kernel(const QkvArgs a) {
   if (hh < a.H) { kind = 0; h = hh; }
   else if (hh < a.H + a.Hkv) { kind = 1; h = hh - a.H; }
   else { kind = 2; h = hh - a.H - a.Hkv; }
-  float x;
-  if (kind == 0) x = load_in(a.q, a.in_dtype, (size_t)t * a.q_stride + (size_t)h * D * (a.gated ? 2 : 1) + d);
-  else if (kind == 1) x = load_in(a.k, a.in_dtype, (size_t)t * a.k_stride + (size_t)h * D + d);
-  else x = load_in(a.v, a.in_dtype, (size_t)t * a.v_stride + (size_t)h * D + d);
+  const int din = kind == 2 ? (a.dv_in > 0 ? a.dv_in : D) : (a.d_in > 0 ? a.d_in : D);
+  float x = 0.f;
+  if (d < din) {
+    if (kind == 0) x = load_in(a.q, a.in_dtype, (size_t)t * a.q_stride + (size_t)h * din * (a.gated ? 2 : 1) + d);
+    else if (kind == 1) x = load_in(a.k, a.in_dtype, (size_t)t * a.k_stride + (size_t)h * din + d);
+    else x = load_in(a.v, a.in_dtype, (size_t)t * a.v_stride + (size_t)h * din + d);
+  }
 
   const float* nw = kind == 0 ? a.q_norm : (kind == 1 ? a.k_norm : nullptr);
   const bool do_norm = (kind < 2 && nw != nullptr) || (kind == 2 && a.v_norm);
   if (do_norm) {
     const float ss = block_sum(x * x, red);
-    x = x * rsqrtf(ss / (float)D + a.eps);
-    if (nw != nullptr) x *= nw[d];
+    x = x * rsqrtf(ss / (float)din + a.eps);
+    if (nw != nullptr && d < din) x *= nw[d];
   }
   const int p = a.pos[t];
   if (kind < 2 && a.rope_dim > 0) {
@@ -174,7 +185,9 @@ __global__ void qkv_post_kernel(const QkvArgs a) {
     }
   }
   if (kind == 0) {
-    a.q_out[((size_t)t * a.H + h) * D + d] = f32_to_bf16(x * a.q_scale);
+    const size_t qo = ((size_t)t * a.H + h) * D + d;
+    if (a.out_f32) reinterpret_cast<float*>(a.q_out)[qo] = x * a.q_scale;
+    else a.q_out[qo] = f32_to_bf16(x * a.q_scale);
     if (a.gated && a.gate_out != nullptr) {
       const float g = load_in(a.q, a.in_dtype, (size_t)t * a.q_stride + (size_t)h * D * 2 + D + d);
       a.gate_out[((size_t)t * a.H + h) * D + d] = f32_to_bf16(g);
@@ -184,7 +197,8 @@ __global__ void qkv_post_kernel(const QkvArgs a) {
     if (!HE_INDEX_OK(p / a.page, a.max_pages, HE_SITE_KV_WRITE_PAGE)) return;
     const int page_id = a.block_table[(size_t)s * a.max_pages + p / a.page];
     const size_t off = ((((size_t)page_id * 2 + (kind - 1)) * a.Hkv + h) * a.page + (p % a.page)) * D + d;
-    a.kv_cache[off] = f32_to_bf16(x);
+    if (a.out_f32) reinterpret_cast<float*>(a.kv_cache)[off] = x;
+    else a.kv_cache[off] = f32_to_bf16(x);
   }
 }
 
@@ -311,34 +325,39 @@ __global__ void advance_positions_kernel(int* pos, int* ctx_len, const int* acti
 }  // namespace
 
 HE_API int he_rmsnorm_rows(const void* x, const void* w, void* out, int out_bf16, int T, int H, float eps,
-                           long long x_stride, long long out_stride, cudaStream_t stream) {
+                           long long x_stride, long long out_stride, int n_mean, cudaStream_t stream) {
   if (T <= 0) return 0;
-  if (H % 4 != 0) return -HE_ERR_BAD_ARG;
+  if (H % 4 != 0 || n_mean <= 0 || n_mean > H) return -HE_ERR_BAD_ARG;
   if (out_bf16)
     (void)launch_pdl(rmsnorm_rows_kernel<__nv_bfloat16>, dim3(T), dim3(256), 0, stream, (const float*)x, (const float*)w, (__nv_bfloat16*)out, H,
-                                                              eps, x_stride, out_stride);
+                                                              eps, x_stride, out_stride, n_mean);
   else
     (void)launch_pdl(rmsnorm_rows_kernel<float>, dim3(T), dim3(256), 0, stream, (const float*)x, (const float*)w, (float*)out, H, eps, x_stride,
-                                                      out_stride);
+                                                      out_stride, n_mean);
   HE_LAUNCH_CHECK();
   return 0;
 }
 
-HE_API int he_act_mul(const void* gu, void* out, long long T, int F, int act, cudaStream_t stream) {
+HE_API int he_act_mul(const void* gu, void* out, long long T, int F, int act, float limit, cudaStream_t stream) {
   if (T <= 0) return 0;
   if (F % 8 != 0) return -HE_ERR_BAD_ARG;
   const long long n = T * F / 8;
   (void)launch_pdl(act_mul_kernel, dim3((unsigned)((n + 255) / 256)), dim3(256), 0, stream, (const __nv_bfloat16*)gu, (__nv_bfloat16*)out, T, F,
-                                                                   act);
+                                                                   act, limit);
   HE_LAUNCH_CHECK();
   return 0;
 }
 
-HE_API int he_act_mul_f32(const void* gu, void* out, long long T, int F, int act, cudaStream_t stream) {
+HE_API int he_act_mul_f32(const void* gu, void* out, int out_bf16, long long T, int F, int act, float limit,
+                          cudaStream_t stream) {
   if (T <= 0) return 0;
   if (F % 4 != 0) return -HE_ERR_BAD_ARG;
   const long long n = T * F / 4;
-  (void)launch_pdl(act_mul_f32_kernel, dim3((unsigned)((n + 255) / 256)), dim3(256), 0, stream, (const float*)gu, (__nv_bfloat16*)out, T, F, act);
+  const dim3 grid((unsigned)((n + 255) / 256));
+  if (out_bf16)
+    (void)launch_pdl(act_mul_f32_kernel<__nv_bfloat16>, grid, dim3(256), 0, stream, (const float*)gu, (__nv_bfloat16*)out, T, F, act, limit);
+  else
+    (void)launch_pdl(act_mul_f32_kernel<float>, grid, dim3(256), 0, stream, (const float*)gu, (float*)out, T, F, act, limit);
   HE_LAUNCH_CHECK();
   return 0;
 }
@@ -426,6 +445,32 @@ __global__ void __launch_bounds__(256) ffn_combine_kernel(float* __restrict__ h,
     h[(size_t)t * ldh + i] = (h[(size_t)t * ldh + i] + buf[i] * ic * w3[i]) * s;
 }
 
+// ---------------------------------------------------------------- looped layers: input of a pass
+// h[t] += x0[t] (the embedding output; null on the first pass) + step (one vector for all rows).  H % 4 == 0.
+__global__ void __launch_bounds__(256) resid_inject_kernel(float* __restrict__ h, const float* __restrict__ x0,
+                                                           const float* __restrict__ step, long long T, int H) {
+  pdl_wait();
+  pdl_launch();
+  const long long i = ((long long)blockIdx.x * blockDim.x + threadIdx.x) * 4;
+  if (i >= T * H) return;
+  float4 v = *reinterpret_cast<const float4*>(h + i);
+  if (x0 != nullptr) {
+    const float4 e = *reinterpret_cast<const float4*>(x0 + i);
+    v.x += e.x; v.y += e.y; v.z += e.z; v.w += e.w;
+  }
+  const float4 s = *reinterpret_cast<const float4*>(step + i % H);
+  v.x += s.x; v.y += s.y; v.z += s.z; v.w += s.w;
+  *reinterpret_cast<float4*>(h + i) = v;
+}
+
+HE_API int he_resid_inject(void* h, const void* x0, const void* step, long long T, int H, cudaStream_t stream) {
+  if (T <= 0) return 0;
+  if (H % 4 != 0 || step == nullptr) return -HE_ERR_BAD_ARG;
+  const long long n = T * H / 4;
+  return (int)launch_pdl(resid_inject_kernel, dim3((unsigned)((n + 255) / 256)), dim3(256), 0, stream, (float*)h,
+                         (const float*)x0, (const float*)step, T, H);
+}
+
 HE_API int he_norm_add(void* h, long long ldh, const void* y, int y_dtype, long long ldy, const void* w, int T, int H,
                        float eps, cudaStream_t stream) {
   if (T <= 0) return 0;
@@ -449,7 +494,8 @@ HE_API int he_ffn_combine(void* h, long long ldh, const void* d, int d_dtype, lo
 HE_API int he_qkv_post(const QkvArgs* args, int T, cudaStream_t stream) {
   const QkvArgs& a = *args;
   if (T <= 0) return 0;
-  if (a.D % 32 != 0 || a.D > 512) return -HE_ERR_BAD_ARG;
+  if (a.D % 32 != 0 || a.D > 512 || a.d_in > a.D || a.dv_in > a.D) return -HE_ERR_BAD_ARG;
+  if ((a.d_in > 0 && a.d_in < a.D) && (a.gated || a.rope_dim > 0)) return -HE_ERR_BAD_ARG;
   dim3 grid(T, a.H + 2 * a.Hkv);
   cudaError_t le = launch_pdl(qkv_post_kernel, grid, dim3(a.D), a.D * sizeof(float), stream, a);
   if (le != cudaSuccess) return (int)le;
@@ -489,9 +535,10 @@ HE_API int he_advance_positions(void* pos, void* ctx_len, const void* active, in
 namespace {
 constexpr int SG_TM = 64, SG_TN = 64, SG_TK = 16;
 __global__ void __launch_bounds__(256) small_gemm_f32_kernel(const void* __restrict__ x, int x_dtype,
-                                                             long long x_stride, const float* __restrict__ w,
+                                                             long long x_stride, const void* __restrict__ w,
+                                                             int w_dtype, long long w_stride,
                                                              float* __restrict__ out, long long out_stride, int T,
-                                                             int N, int K) {
+                                                             int N, int K, int accumulate) {
   __shared__ float xs[SG_TK][SG_TM + 1];
   __shared__ float ws[SG_TK][SG_TN + 1];
   const int t0 = blockIdx.y * SG_TM, n0 = blockIdx.x * SG_TN;
@@ -506,7 +553,7 @@ __global__ void __launch_bounds__(256) small_gemm_f32_kernel(const void* __restr
     for (int i = threadIdx.x; i < SG_TN * SG_TK; i += 256) {
       const int r = i / SG_TK, kk = i % SG_TK;
       const int n = n0 + r, k = k0 + kk;
-      ws[kk][r] = (n < N && k < K) ? w[(size_t)n * K + k] : 0.f;
+      ws[kk][r] = (n < N && k < K) ? load_in(w, w_dtype, (size_t)n * w_stride + k) : 0.f;
     }
     __syncthreads();
 #pragma unroll
@@ -526,17 +573,21 @@ __global__ void __launch_bounds__(256) small_gemm_f32_kernel(const void* __restr
 #pragma unroll
     for (int j = 0; j < 4; ++j) {
       const int t = t0 + ty * 4 + i, n = n0 + tx * 4 + j;
-      if (t < T && n < N) out[(size_t)t * out_stride + n] = acc[i][j];
+      if (t < T && n < N) {
+        float* o = out + (size_t)t * out_stride + n;
+        *o = accumulate ? *o + acc[i][j] : acc[i][j];
+      }
     }
 }
 }  // namespace
 
-HE_API int he_small_gemm_f32(const void* x, int x_dtype, long long x_stride, const void* w, void* out,
-                             long long out_stride, int T, int N, int K, cudaStream_t stream) {
+HE_API int he_small_gemm_f32(const void* x, int x_dtype, long long x_stride, const void* w, int w_dtype,
+                             long long w_stride, void* out, long long out_stride, int T, int N, int K, int accumulate,
+                             cudaStream_t stream) {
   if (T <= 0 || N <= 0) return 0;
   dim3 grid((N + SG_TN - 1) / SG_TN, (T + SG_TM - 1) / SG_TM);
-  small_gemm_f32_kernel<<<grid, 256, 0, stream>>>(x, x_dtype, x_stride, (const float*)w, (float*)out, out_stride, T, N,
-                                                  K);
+  small_gemm_f32_kernel<<<grid, 256, 0, stream>>>(x, x_dtype, x_stride, w, w_dtype, w_stride, (float*)out, out_stride, T,
+                                                  N, K, accumulate);
   HE_LAUNCH_CHECK();
   return 0;
 }

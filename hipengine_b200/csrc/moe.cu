@@ -85,6 +85,83 @@ __global__ void moe_route_kernel(const float* __restrict__ logits, long long ld,
   }
 }
 
+// Group-limited sigmoid router, one warp per token: s = sigmoid(logits); the E experts form `groups` equal groups of
+// neighbours, a group's rank is the sum of its two largest scores, the best `keep` groups stay open; the k largest
+// scores of the open groups are chosen (lower id first on equal scores), weights s / (sum + 1e-20) * scale.
+__global__ void moe_route_grouped_kernel(const float* __restrict__ logits, long long ld, int T, int E, int k, int groups,
+                                         int keep, float scale, int* __restrict__ ids, float* __restrict__ wts) {
+  extern __shared__ float route_sm[];
+  pdl_wait();
+  pdl_launch();
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int t = blockIdx.x * (blockDim.x >> 5) + warp;
+  if (t >= T) return;
+  float* s = route_sm + (size_t)warp * (E + groups);     // scores, then group ranks
+  float* gs = s + E;
+  const int size = E / groups;
+  for (int e = lane; e < E; e += 32) s[e] = 1.f / (1.f + expf(-logits[(size_t)t * ld + e]));
+  __syncwarp();
+  for (int g = lane; g < groups; g += 32) {
+    float a = -INFINITY, b = -INFINITY;                  // two largest
+    for (int i = 0; i < size; ++i) {
+      const float v = s[g * size + i];
+      if (v > a) { b = a; a = v; }
+      else if (v > b) b = v;
+    }
+    gs[g] = size > 1 ? a + b : a;
+  }
+  __syncwarp();
+  // one argmax over values[0..n) per call; the winner is taken out by the caller
+  auto pick = [&](const float* values, int n) {
+    float bv = -INFINITY;
+    int bi = 0x7fffffff;
+    for (int i = lane; i < n; i += 32)
+      if (values[i] > bv) { bv = values[i]; bi = i; }
+#pragma unroll
+    for (int off = 16; off > 0; off >>= 1) {
+      const float ov = __shfl_xor_sync(0xffffffffu, bv, off);
+      const int oi = __shfl_xor_sync(0xffffffffu, bi, off);
+      if (ov > bv || (ov == bv && oi < bi)) { bv = ov; bi = oi; }
+    }
+    return bi < n ? bi : 0;
+  };
+  const float OPEN = INFINITY;                           // mark of a kept group (ranks are at most 2)
+  if (keep < groups) {
+    for (int j = 0; j < keep; ++j) {
+      float bv = -INFINITY;
+      int bi = 0x7fffffff;
+      for (int g = lane; g < groups; g += 32)
+        if (gs[g] != OPEN && gs[g] > bv) { bv = gs[g]; bi = g; }
+#pragma unroll
+      for (int off = 16; off > 0; off >>= 1) {
+        const float ov = __shfl_xor_sync(0xffffffffu, bv, off);
+        const int oi = __shfl_xor_sync(0xffffffffu, bi, off);
+        if (ov > bv || (ov == bv && oi < bi)) { bv = ov; bi = oi; }
+      }
+      if (lane == 0 && bi < groups) gs[bi] = OPEN;
+      __syncwarp();
+    }
+    for (int e = lane; e < E; e += 32)
+      if (gs[e / size] != OPEN) s[e] = -1.f;             // closed: below every score
+    __syncwarp();
+  }
+  float sum = 0.f, my_w = 0.f;
+  int my_id = 0;
+  for (int j = 0; j < k; ++j) {
+    const int bi = pick(s, E);
+    const float v = s[bi];
+    __syncwarp();
+    if (lane == 0) s[bi] = -2.f;
+    __syncwarp();
+    if (lane == j) { my_w = v; my_id = bi; }
+    sum += v;
+  }
+  if (lane < k) {
+    ids[(size_t)t * k + lane] = my_id;
+    wts[(size_t)t * k + lane] = my_w / (sum + 1e-20f) * scale;
+  }
+}
+
 // ------------------------------------------------------------------------------------------ grouping
 // Single CTA: histogram of expert ids over the P = T*k pairs, prefix over experts with every expert's rows
 // padded to a multiple of 128, scatter.  pos[pair] = row in the sorted matrix, tile_group[tile] = expert of
@@ -405,6 +482,19 @@ HE_API int he_moe_route(const float* logits, long long ld, int T, int E, int k, 
   else (void)launch_pdl(moe_route_kernel<16>, dim3(grid), dim3(wpb * 32), 0, stream, logits, ld, T, E, k, mode, expert_scale, ids, wts);
   HE_LAUNCH_CHECK();
   return 0;
+}
+
+HE_API int he_moe_route_grouped(const float* logits, long long ld, int T, int E, int k, int groups, int keep, float scale,
+                                int* ids, float* wts, cudaStream_t stream) {
+  if (T <= 0) return 0;
+  if (groups <= 0 || E <= 0 || E % groups != 0 || keep < 1 || keep > groups || k < 1 || k > 32 ||
+      k > keep * (E / groups))
+    return -HE_ERR_BAD_ARG;
+  const int wpb = 4;
+  const size_t smem = (size_t)wpb * (E + groups) * sizeof(float);
+  if (smem > 48 * 1024) return -HE_ERR_BAD_ARG;
+  return (int)launch_pdl(moe_route_grouped_kernel, dim3((T + wpb - 1) / wpb), dim3(wpb * 32), smem, stream, logits, ld, T,
+                         E, k, groups, keep, scale, ids, wts);
 }
 
 // Upper bound of sorted rows for P pairs over E experts (every expert padded to 128 rows).

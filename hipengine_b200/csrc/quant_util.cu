@@ -146,7 +146,49 @@ __global__ void embed_kernel(const uint8_t* __restrict__ w, int qtype, long long
     out[(size_t)t * K + e] = dequant_elem(w, qtype, id, K, e) * scale;
 }
 
+// Embedding row + sinusoidal position vector, written twice: the residual and the copy that looped layers add again.
+// freq[i] = 10000^(-2i/width) in double: the angle p * freq is reduced to one turn in double before the fp32 sin / cos,
+// so late positions keep full fp32 accuracy.  Columns [K, ld) of a zero-padded row become zero.
+__global__ void embed_sinusoid_kernel(const uint8_t* __restrict__ w, int qtype, long long vocab, int K, int ld,
+                                      const int64_t* __restrict__ ids, const int* __restrict__ pos,
+                                      const double* __restrict__ freq, float* __restrict__ out,
+                                      float* __restrict__ copy, int n_tok) {
+  pdl_wait();
+  pdl_launch();
+  const int t = blockIdx.x;
+  if (t >= n_tok) return;
+  long long id = ids[t];
+  if (!HE_INDEX_OK(id, vocab, HE_SITE_EMBED_TOKEN) || id < 0 || id >= vocab) id = 0;
+  const double p = (double)pos[t];
+  const double two_pi = 6.283185307179586476925286766559;
+  for (int i = threadIdx.x; 2 * i < ld; i += blockDim.x) {
+    float v[2] = {0.f, 0.f};
+    if (2 * i < K) {
+      const double ang = p * freq[i];
+      float sn, cs;
+      sincosf((float)(ang - two_pi * rint(ang / two_pi)), &sn, &cs);
+      v[0] = dequant_elem(w, qtype, id, K, 2 * i) + sn;
+      if (2 * i + 1 < K) v[1] = dequant_elem(w, qtype, id, K, 2 * i + 1) + cs;
+    }
+#pragma unroll
+    for (int e = 0; e < 2; ++e)
+      if (2 * i + e < ld) {
+        out[(size_t)t * ld + 2 * i + e] = v[e];
+        if (copy != nullptr) copy[(size_t)t * ld + 2 * i + e] = v[e];
+      }
+  }
+}
+
 }  // namespace
+
+// out[t][:] = table[ids[t]] + sinusoidal position vector of pos[t]  (fp32 rows of `ld` columns)
+HE_API int he_embed_sinusoid(const void* w, int qtype, long long vocab, int K, int ld, const void* ids, const void* pos,
+                             const void* freq, void* out, void* copy, int n_tok, cudaStream_t stream) {
+  if (n_tok <= 0) return 0;
+  if (ld < K || freq == nullptr) return -HE_ERR_BAD_ARG;
+  return (int)launch_pdl(embed_sinusoid_kernel, dim3(n_tok), dim3(256), 0, stream, (const uint8_t*)w, qtype, vocab, K, ld,
+                         (const int64_t*)ids, (const int*)pos, (const double*)freq, (float*)out, (float*)copy, n_tok);
+}
 
 // Dequantize rows [row0, row0+rows) of a device-layout weight into bf16 [rows][K] (exact value, RNE to bf16).
 HE_API int he_dequant_bf16(const void* w, void* out, int qtype, long long row0, long long rows, long long n_total,

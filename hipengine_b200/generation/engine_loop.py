@@ -1,7 +1,8 @@
 """The resident engine loop: one tick = lifetime probes -> admission -> (prefill | decode) -> commit.
 
 Mirrors ``ResidentEngineLoop`` (``hipengine/generation/engine_loop.py:2318-4041``): policies ``protect_decode``
-(default), ``protect_ttft``, ``fair`` and ``token_budget`` (``:68``); chunked prefill; failure containment
+(default), ``protect_ttft``, ``fair`` and ``token_budget`` (``:68``), plus ``mixed`` (prompt chunks and decode rows in
+one forward pass); chunked prefill; failure containment
 (``contain_execution_failure`` ``:2869-2987``: a runner may fail only the affected rows, anything else is
 fatal); cooperative cancellation and deadlines probed before admission and after every step (``:2629-2708``).
 The loop is single-threaded and owns the runner; ``EngineService`` drives it from its driver thread.
@@ -16,7 +17,7 @@ from .runner import BaseRunner, ExecutionFailure
 from .scheduler import DECODE, FINISHED, PREFILL, GenerationAdmissionRejected, RequestState, Scheduler
 from .types import FinishDetails, GenerationRequest, TokenLogprob
 
-POLICIES = ("protect_decode", "protect_ttft", "fair", "token_budget")
+POLICIES = ("protect_decode", "protect_ttft", "fair", "token_budget", "mixed")
 
 
 class EngineLoop:
@@ -70,7 +71,9 @@ class EngineLoop:
         has_prefill = bool(self.sched.prefill_rows())
         has_decode = bool(self.sched.decode_rows())
         done = 0
-        if sc.policy == "token_budget":
+        if sc.policy == "mixed" and has_prefill and has_decode and not self._speculating():
+            done += self._run_mixed(sc.max_prefill_chunk_tokens)
+        elif sc.policy == "token_budget":
             if has_decode:
                 done += self._run_decode()
             if has_prefill:
@@ -127,6 +130,30 @@ class EngineLoop:
         except ExecutionFailure as f:
             self._contain(f)
             return 0
+        return self._commit_prefill(work, firsts, t0)
+
+    def _run_mixed(self, budget: int) -> int:
+        """Prompt chunks and every decode row as one packed forward pass: decoding never waits for a prompt, and the
+        prompt's projections carry the decode rows along."""
+        sc = self.config.scheduler
+        rows = self.sched.next_decode_work(sc.round_decode_row_budget)
+        work = self.sched.next_prefill_work(sc.max_prefill_chunk_tokens, budget)
+        t0 = time.perf_counter()
+        try:
+            res, firsts = self.runner.mixed(work, rows)
+        except ExecutionFailure as f:
+            self._contain(f)
+            return 0
+        self.sched.counters["decode_steps"] += 1
+        for rs, (tok, lp) in zip(rows, res):
+            if rs.status != FINISHED:
+                self._commit_token(rs, tok, lp)
+        return len(rows) + self._commit_prefill(work, firsts, t0)
+
+    def _speculating(self) -> bool:
+        return self.config.speculative.mode not in ("off", "", None) and self.runner.supports_mtp
+
+    def _commit_prefill(self, work, firsts, t0: float) -> int:
         n = 0
         for rs, cnt in work:
             if rs.status == FINISHED:

@@ -477,6 +477,13 @@ class EngineService:
 def build_engine(weights, backend: str, config: EngineConfig, tokenizer=None) -> EngineService:
     """weights + backend -> runner -> loop -> service."""
     eos = getattr(tokenizer, "eos_token_id", None)
+    from ..models.registry import plugin_for
+    plugin = plugin_for(weights.config.arch)
+    if backend != "cpu_reference" and config.compute_dtype not in plugin.compute_dtypes:
+        raise ValueError(f"{plugin.name}: compute dtype {config.compute_dtype!r} is not built "
+                         f"(supported: {plugin.compute_dtypes})")
+    if max(config.parallel.tp, config.parallel.ep) > 1 and not plugin.tensor_parallel and backend != "cpu_reference":
+        raise ValueError(f"{plugin.name}: tensor / expert parallel execution is not built")
     if backend == "cpu_reference":
         from .runner import CpuReferenceRunner
         runner = CpuReferenceRunner(weights, config, eos)

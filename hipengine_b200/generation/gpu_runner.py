@@ -40,7 +40,8 @@ class GpuRunner(BaseRunner):
         self.n_snap = config.kv.max_snapshots if (self.use_prefix and self.cfg.is_hybrid) else 0
         pages_per_slot = (self.max_context + self.page - 1) // self.page
         from ..config import resolve_pool_pages
-        n_pages = resolve_pool_pages(config.kv, self.cfg.kv_bytes_per_token(), self.max_slots, pages_per_slot)
+        self.kv_bytes_per_token = self.cfg.kv_bytes_per_token(4 if config.compute_dtype == "float32" else 2)
+        n_pages = resolve_pool_pages(config.kv, self.kv_bytes_per_token, self.max_slots, pages_per_slot)
         if executor is not None:
             self.ex = executor
             self.max_slots = min(self.max_slots, executor.max_slots)
@@ -51,11 +52,12 @@ class GpuRunner(BaseRunner):
             # constructing thread and the engine's driver thread on every rank but the first
             dev = torch.device("cuda", torch.cuda.current_device())
             from ..models import make_executor
-            self.ex = make_executor(weights, device=dev, max_slots=self.max_slots + self.n_snap,
+            self.ex = make_executor(weights, dtype=config.compute_dtype, device=dev, max_slots=self.max_slots + self.n_snap,
                                     max_context=self.max_context, n_pages=n_pages)
         self.device = self.ex.device
         self.pool = PagePool(n_pages, self.page)
-        self.radix = RadixCache(self.page, PrefixCompatibilityKey(self.cfg.arch, kv_storage=config.kv.storage,
+        kv_storage = "f32" if config.compute_dtype == "float32" else config.kv.storage
+        self.radix = RadixCache(self.page, PrefixCompatibilityKey(self.cfg.arch, kv_storage=kv_storage,
                                                                   page_tokens=self.page,
                                                                   rope=f"{self.cfg.rope_theta}:{self.cfg.rope_dim}"))
         self.radix.on_retain = self.pool.retain_cache
@@ -294,6 +296,46 @@ class GpuRunner(BaseRunner):
         if len(lease.pages) > before:
             self._write_block_table(rs.slot, lease, before)
 
+    # ------------------------------------------------------------------ one packed batch
+    def forward_segments(self, segs: Sequence[Tuple[int, int, Sequence[int]]]):
+        """Run (slot, first position, token ids) segments -- prompt portions and single decoded tokens alike -- as one
+        packed batch.  Returns (batch, residual rows); the pages must be in place (``_ensure_pages``)."""
+        batch = make_batch(segs, self.device)
+        self.stats["h2d_bytes"] += 8 * batch.T + 16 * batch.T
+        return batch, self.ex.forward(batch)
+
+    @torch.no_grad()
+    def mixed(self, work: List[Tuple[RequestState, int]], rows: List[RequestState]):
+        """Decode rows and prompt chunks in ONE forward pass.  Returns (results of the decode rows, first tokens of the
+        prompts that end in this step by request id)."""
+        if self.mtp is not None or self.n_snap or not work or not rows:
+            return super().mixed(work, rows)      # draft state / snapshot boundaries: the phases stay separate
+        with self.census.region("mixed"):
+            segs = []
+            for rs in rows:
+                self._ensure_pages(rs, rs.position)
+                segs.append((rs.slot, rs.position - 1, [rs.last_token]))
+                rs.telemetry.h2d_bytes += 24
+            want, idx, row = list(rows), list(range(len(rows))), len(rows)
+            for rs, n in work:
+                a, b = rs.prefilled, rs.prefilled + n
+                self._ensure_pages(rs, b)
+                segs.append((rs.slot, a, rs.req.prompt_token_ids[a:b]))
+                rs.telemetry.h2d_bytes += 24 * n
+                row += n
+                if b >= rs.prompt_len:
+                    want.append(rs)
+                    idx.append(row - 1)
+            try:
+                _, h = self.forward_segments(segs)
+                logits = self.ex.logits(h.index_select(0, torch.tensor(idx, device=self.device)))
+                res = self._sample_rows(want, logits)
+            except torch.cuda.OutOfMemoryError as exc:
+                raise ExecutionFailure([rs.rid for rs in rows] + [rs.rid for rs, _ in work], "mixed",
+                                       f"out of memory: {exc}", "partial") from exc
+            self.resident_key = ()
+            return res[:len(rows)], {rs.rid: t for rs, t in zip(want[len(rows):], res[len(rows):])}
+
     # ------------------------------------------------------------------ prefill
     def prefill(self, work: List[Tuple[RequestState, int]]) -> Dict[int, Tuple[int, Optional[TokenLogprob]]]:
         with self.census.region("prefill"):
@@ -327,9 +369,7 @@ class GpuRunner(BaseRunner):
                         segs.append((rs.slot, a, toks))
                         owners.append((rs, a, b))
                         rs.telemetry.h2d_bytes += 24 * (b - a)      # ids (int64) + slot / pos / segment (int32)
-                batch = make_batch(segs, self.device)
-                self.stats["h2d_bytes"] += 8 * batch.T + 16 * batch.T
-                h = self.ex.forward(batch)
+                batch, h = self.forward_segments(segs)
                 if self.mtp is not None:
                     self.mtp.after_prefill(batch, h)
                 row = 0
@@ -565,7 +605,7 @@ class GpuRunner(BaseRunner):
                 "resources": self.ledger.snapshot(),
                 "speculative": self.mtp.capability().as_dict() if self.mtp is not None else None,
                 "prefix_cache": self.radix.snapshot_stats(), "state_bytes": self.ex.state_bytes(),
-                "kv_bytes_per_token": self.cfg.kv_bytes_per_token(),
+                "kv_bytes_per_token": self.kv_bytes_per_token,
                 "recurrent_state_bytes_per_request": self.cfg.recurrent_state_bytes(),
                 # resident weight bytes: the quantised device layouts (there is no widened copy of any of them)
                 "weight_bytes": sum(w.data.numel() * w.data.element_size() for w in

@@ -93,6 +93,12 @@ class BaseRunner:
         return tok, lp
 
     # -- protocol defaults ---------------------------------------------------------------------------
+    def mixed(self, work, rows):
+        """One scheduling step that holds both prompt chunks and decode rows; runners that can pack them into a single
+        forward pass override this.  Returns (decode results, {request id: first token})."""
+        res = self.decode(rows) if rows else []
+        return res, (self.prefill(work) if work else {})
+
     def capacity(self) -> Dict[str, Any]:
         return {"max_slots": self.max_slots, "max_context": self.max_context}
 

@@ -105,11 +105,20 @@ class SamplingParams:
 PromptLike = Union[str, Sequence[int]]
 
 
+def _compute_dtype(name: str) -> str:
+    full = {"bf16": "bfloat16", "fp32": "float32", "f32": "float32"}.get(str(name), str(name))
+    if full not in ("bfloat16", "float32"):
+        raise ValueError(f"unknown compute dtype {name!r} (bfloat16 | float32)")
+    return full
+
+
 class LLM:
     """Load a model and generate.
 
-    ``model`` may be a GGUF path / directory, a ``ModelWeights`` object, or the name of a built-in
-    random-init geometry (``"tiny-hybrid"``, ``"qwen35-27b"``, ...; see ``models.config.NAMED_CONFIGS``).
+    ``model`` may be a GGUF path / directory, a checkpoint folder (config.json + model.safetensors), a
+    ``ModelWeights`` object, or the name of a built-in random-init geometry (``"tiny-hybrid"``, ``"qwen35-27b"``, ...;
+    see ``models.config.NAMED_CONFIGS``).  ``dtype``: compute precision, ``bfloat16`` or ``float32`` (families that
+    declare it).
     """
 
     def __init__(self, model: Any, *, backend: str = "auto", quant: Optional[str] = None,
@@ -122,7 +131,8 @@ class LLM:
                  kv_storage: str = "bf16", tensor_parallel: int = 1, expert_parallel: int = 1,
                  engine_command_timeout_seconds: float = 300.0, seed: int = 0, tokenizer: Any = None,
                  engine_config: Optional[EngineConfig] = None, device: Optional[str] = None,
-                 weights_recipe: str = "q4_k_m", expected_quant: Optional[str] = None):
+                 weights_recipe: str = "q4_k_m", expected_quant: Optional[str] = None,
+                 dtype: Optional[str] = None):
         self.model = model
         self._expected_quant = expected_quant
         self.backend = self._resolve_backend(backend, device)
@@ -139,6 +149,7 @@ class LLM:
         self.config = replace(
             base,
             max_sequence_length=int(max_sequence_length or base.max_sequence_length),
+            compute_dtype=_compute_dtype(dtype or base.compute_dtype),
             profile=self.profile,
             scheduler=replace(base.scheduler, max_active_requests=int(max_active_requests)),
             kv=replace(base.kv, storage=kv_storage, prefix_cache=prefix_cache,
@@ -209,8 +220,11 @@ class LLM:
         if isinstance(m, ModelWeights):
             self._weights = m
         elif isinstance(m, (str, Path)) and Path(str(m)).exists():
-            from .loading.model_loader import load_gguf_model
-            self._weights = load_gguf_model(m, device=dev, pin=(dev == "cuda"))
+            from .loading.model_loader import load_model
+            from .loading.safetensors_dir import is_checkpoint_dir
+            # a checkpoint folder is repacked (stacked, padded) by its executor: only the packed copy goes to the device
+            packed = is_checkpoint_dir(m)
+            self._weights = load_model(m, device="cpu" if packed else dev, pin=(dev == "cuda" and not packed))
         elif isinstance(m, str):
             from .loading.synth import build_random_model
             from .models.config import NAMED_CONFIGS

@@ -39,6 +39,9 @@ def role_of(name: str) -> str:
     parts = name.split(".")
     if parts[0] == "blk" and len(parts) > 2:
         parts = parts[2:]
+    elif parts[0][:1] == "l" and parts[0][1:].isdigit() and len(parts) > 1:
+        # folder checkpoints number layers l<i> and experts e<j>
+        parts = ["e" if p[:1] == "e" and p[1:].isdigit() else p for p in parts[1:]]
     if parts and parts[-1] in ("weight", "bias"):
         suffix = "" if parts[-1] == "weight" else ".bias"
         parts = parts[:-1]
@@ -88,6 +91,9 @@ class PlanContract:
 
 
 def _required_tensors(cfg) -> List[str]:
+    if cfg.arch == "sisisun":
+        from .sisisun import tensor_shapes
+        return list(tensor_shapes(cfg))
     need = ["token_embd.weight", "output_norm.weight"]
     for i in range(cfg.n_layers):
         need.append(f"blk.{i}.attn_norm.weight")
@@ -145,8 +151,9 @@ def memory_preflight(weights, engine_config, free_bytes: Optional[int], contract
     pages_per_slot = -(-max_ctx // kvc.page_tokens)
     n_slots = sched.max_active_requests
     from ..config import resolve_pool_pages
-    n_pages = resolve_pool_pages(kvc, cfg.kv_bytes_per_token(), n_slots, pages_per_slot)
-    kv_bytes = n_pages * kvc.page_tokens * cfg.kv_bytes_per_token()
+    kv_elem = 4 if engine_config.compute_dtype == "float32" else 2
+    n_pages = resolve_pool_pages(kvc, cfg.kv_bytes_per_token(kv_elem), n_slots, pages_per_slot)
+    kv_bytes = n_pages * kvc.page_tokens * cfg.kv_bytes_per_token(kv_elem)
     n_snap = kvc.max_snapshots if (kvc.prefix_cache != "off" and cfg.is_hybrid) else 0
     state_bytes = (n_slots + n_snap) * cfg.recurrent_state_bytes()
     # scratch of one 4096-row prefill chunk: a dozen [rows, widest projection] bf16/fp32 buffers + logits rows

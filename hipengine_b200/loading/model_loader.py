@@ -84,6 +84,11 @@ def describe_model_source(model) -> Dict[str, object]:
         return out
 
     name = str(model)
+    from .safetensors_dir import describe_checkpoint_dir, is_checkpoint_dir
+    if is_checkpoint_dir(name):
+        d = describe_checkpoint_dir(name)
+        cfg = d.pop("config", None)
+        return {**d, **(geometry(cfg) if cfg is not None else {})}
     files = discover_gguf_files(name)
     if files:
         try:
@@ -99,11 +104,20 @@ def describe_model_source(model) -> Dict[str, object]:
                 "bytes_by_block_type": dict(sorted(hist.items(), key=lambda kv: -kv[1])),
                 "name": info.get("general.name"), **geometry(cfg)}
     if Path(name).exists():
-        return {"source": "path", "path": name, "error": "no *.gguf file there"}
+        return {"source": "path", "path": name,
+                "error": "no *.gguf file there (and no config.json with model.safetensors)"}
     if name in NAMED_CONFIGS:
         return {"source": "built-in geometry (random weights)", "name": name, **geometry(NAMED_CONFIGS[name])}
     return {"source": "unknown", "error": f"{name!r} is neither a local GGUF path nor a built-in geometry "
                                           f"({sorted(NAMED_CONFIGS)})"}
+
+
+def load_model(path, device="cpu", pin: bool = False, validate: bool = True) -> ModelWeights:
+    """Weights of a local artifact: a checkpoint folder (config.json + model.safetensors) or a GGUF file / folder."""
+    from .safetensors_dir import is_checkpoint_dir, load_checkpoint_dir
+    if is_checkpoint_dir(path):
+        return load_checkpoint_dir(path, device=device, pin=pin, validate=validate)
+    return load_gguf_model(path, device=device, pin=pin, validate=validate)
 
 
 def load_gguf_model(path, device="cpu", pin: bool = False, validate: bool = True) -> ModelWeights:

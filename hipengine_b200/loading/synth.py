@@ -89,6 +89,9 @@ def build_random_model(cfg: ModelConfig, seed: int = 0, device="cpu", recipe: st
     if cfg.arch == "gemma4":
         from .gemma4 import build_random_gemma4
         return build_random_gemma4(cfg, seed=seed, device=device, recipe=recipe, std=std)
+    if cfg.arch == "sisisun":
+        from .sisisun import build_random_sisisun
+        return build_random_sisisun(cfg, seed=seed, device=device, std=std)
     b = _Builder(cfg, seed, device, recipe, std)
     base, hi = b.base_type(), b.hi_type()
     H = cfg.hidden

@@ -10,7 +10,65 @@ geometries mirror the identities the reference pins in
 from __future__ import annotations
 
 from dataclasses import dataclass, replace
-from typing import Dict, Optional, Tuple
+from typing import Dict, Optional, Tuple, Union
+
+# head widths the attention kernels are built for; narrower heads are zero-padded to the next one at load
+HEAD_WIDTHS = (64, 128, 256, 512)
+
+
+def padded_head_width(d: int) -> int:
+    for w in HEAD_WIDTHS:
+        if d <= w:
+            return w
+    raise ValueError(f"head width {d} is above the widest supported one ({HEAD_WIDTHS[-1]})")
+
+
+@dataclass(frozen=True)
+class AttentionSpec:
+    """Softmax attention of one layer, for designs whose layers are listed one by one."""
+    heads: int
+    kv_heads: int
+    dim: int                             # query / key width per head
+    vdim: int                            # value width per head
+    scale: float
+    softcap: float = 0.0                 # > 0: score <- softcap * tanh(score / softcap)
+
+    @property
+    def width(self) -> int:
+        """Width a head takes in the KV pages (both planes)."""
+        return padded_head_width(max(self.dim, self.vdim))
+
+
+@dataclass(frozen=True)
+class DenseMlpSpec:
+    ff: int
+    act: str = "silu"                    # "silu" | "gelu_tanh" | "clamped_glu"
+    limit: float = 0.0                   # clamped_glu: bound of the gate (above) and of the up branch (both sides)
+
+
+@dataclass(frozen=True)
+class MoeMlpSpec:
+    experts: int
+    top: int
+    ff: int
+    groups: int = 1                      # groups of neighbouring experts ...
+    groups_kept: int = 1                 # ... of which only the best ones may be chosen from
+    scale: float = 1.0                   # factor on the normalised routing weights
+    shared_ff: int = 0                   # > 0: shared expert, scaled per token by sigmoid(w_sg . h)
+
+
+@dataclass(frozen=True)
+class LayerSpec:
+    mixer: AttentionSpec
+    mlp: Optional[Union[DenseMlpSpec, MoeMlpSpec]] = None
+
+
+@dataclass(frozen=True)
+class LoopSpec:
+    """Layers [start, stop) run ``times`` times in a row with the same weights, every pass with its own cache."""
+    start: int
+    stop: int
+    times: int
 
 
 @dataclass(frozen=True)
@@ -57,6 +115,10 @@ class ModelConfig:
 
     swa_rope_theta: float = 10000.0      # Gemma: sliding layers rotate the whole head with this base
     global_rope_fraction: float = 0.25   # Gemma: global layers rotate this fraction of the head ("proportional")
+
+    # designs whose layers are listed one by one (``layer_specs``), some of them run repeatedly (``loop``)
+    layer_specs: Tuple[LayerSpec, ...] = ()
+    loop: Optional[LoopSpec] = None
 
     # ---- derived
     def is_global_layer(self, i: int) -> bool:
@@ -119,7 +181,21 @@ class ModelConfig:
     def scale(self) -> float:
         return self.attn_scale if self.attn_scale is not None else self.head_dim ** -0.5
 
+    def layer_runs(self) -> Tuple[Tuple[int, int], ...]:
+        """(layer, pass) in the order of execution; pass is -1 for a layer outside the loop.  A layer run, not a layer,
+        owns a KV plane."""
+        lp = self.loop
+        if lp is None:
+            return tuple((i, -1) for i in range(self.n_layers))
+        runs = [(i, -1) for i in range(lp.start)]
+        for t in range(lp.times):
+            runs += [(i, t) for i in range(lp.start, lp.stop)]
+        return tuple(runs + [(i, -1) for i in range(lp.stop, self.n_layers)])
+
     def kv_bytes_per_token(self, elem_bytes: int = 2) -> int:
+        if self.layer_specs:
+            return sum(2 * self.layer_specs[i].mixer.kv_heads * self.layer_specs[i].mixer.width * elem_bytes
+                       for i, _ in self.layer_runs())
         return self.n_full_layers * 2 * self.n_kv_heads * self.head_dim * elem_bytes
 
     def recurrent_state_bytes(self) -> int:
@@ -128,7 +204,13 @@ class ModelConfig:
         return gdn + conv
 
     def with_layers(self, n_layers: int) -> "ModelConfig":
-        return replace(self, n_layers=n_layers)
+        if not self.layer_specs:
+            return replace(self, n_layers=n_layers)
+        lp = self.loop
+        if lp is not None:
+            stop = min(lp.stop, n_layers)
+            lp = LoopSpec(lp.start, stop, lp.times) if lp.start < stop else None
+        return replace(self, n_layers=n_layers, layer_specs=self.layer_specs[:n_layers], loop=lp)
 
 
 # Tiny dense decoder of the CPU reference backend benchmark (4 layers, hidden 256, Q4_K weights).
@@ -194,6 +276,56 @@ TINY_GEMMA4 = ModelConfig(arch="gemma4", n_layers=6, hidden=256, vocab=2048, n_h
                           n_experts=8, n_experts_used=2, expert_ffn=128, final_softcap=30.0,
                           embed_scale=16.0, act="gelu_tanh", tie_embeddings=True, max_context=2048)
 
+
+def sisisun_config(hidden: int, vocab: int, layers: Tuple[LayerSpec, ...], loop: Optional[LoopSpec] = None,
+                   rms_eps: float = 1e-6, max_context: int = 262144) -> ModelConfig:
+    """``ModelConfig`` of a Sisisun model: listed layers without rotation, sinusoidal position vector at the embedding,
+    norm weights stored around zero, optional looped range.  The per-model fields of the other families are filled in
+    from the layers for reports."""
+    a = layers[0].mixer
+    moe = [l.mlp for l in layers if isinstance(l.mlp, MoeMlpSpec)]
+    dense = [l.mlp for l in layers if isinstance(l.mlp, DenseMlpSpec)]
+    for i, l in enumerate(layers):
+        if l.mixer.heads % l.mixer.kv_heads:
+            raise ValueError(f"layer {i}: {l.mixer.heads} query heads over {l.mixer.kv_heads} key/value heads")
+        if isinstance(l.mlp, MoeMlpSpec):
+            m = l.mlp
+            if m.experts % m.groups or not 1 <= m.groups_kept <= m.groups:
+                raise ValueError(f"layer {i}: {m.experts} experts in {m.groups} groups, {m.groups_kept} kept")
+            if not 1 <= m.top <= m.groups_kept * (m.experts // m.groups):
+                raise ValueError(f"layer {i}: top {m.top} of {m.groups_kept} groups of {m.experts // m.groups}")
+    if loop is not None and not (0 <= loop.start < loop.stop <= len(layers) and loop.times >= 1):
+        raise ValueError(f"loop {loop} over {len(layers)} layers")
+    return ModelConfig(
+        arch="sisisun", n_layers=len(layers), hidden=hidden, vocab=vocab, n_heads=a.heads, n_kv_heads=a.kv_heads,
+        head_dim=a.dim, ffn=max([d.ff for d in dense], default=0), rms_eps=rms_eps, rope_dim=0, qk_norm=True,
+        attn_scale=a.scale, n_experts=max([m.experts for m in moe], default=0),
+        n_experts_used=max([m.top for m in moe], default=0), expert_ffn=max([m.ff for m in moe], default=0),
+        shared_ffn=max([m.shared_ff for m in moe], default=0), layer_specs=tuple(layers), loop=loop,
+        max_context=max_context)
+
+
+# Small Sisisun geometry of the tests and the command line: unequal head widths, one layer without a feed-forward, a
+# loop that neither starts nor stops with the stack.
+_SISISUN_A = AttentionSpec(heads=4, kv_heads=2, dim=48, vdim=64, scale=0.15, softcap=20.0)
+TINY_SISISUN = sisisun_config(
+    192, 1024, (LayerSpec(_SISISUN_A, DenseMlpSpec(256, "clamped_glu", 1.5)),
+                LayerSpec(_SISISUN_A, MoeMlpSpec(12, 3, 72, groups=3, groups_kept=2, scale=1.7, shared_ff=40)),
+                LayerSpec(_SISISUN_A, None),
+                LayerSpec(_SISISUN_A, DenseMlpSpec(160, "clamped_glu", 1.5))),
+    loop=LoopSpec(1, 3, 2), max_context=8192)
+
+# Geometries at the layer sizes of deployed models, for throughput: an 8B-class dense stack and a 30B-A3B-class
+# mixture, both with a looped range.
+_SISISUN_8B_A = AttentionSpec(heads=32, kv_heads=8, dim=128, vdim=128, scale=128 ** -0.5, softcap=50.0)
+_SISISUN_30B_A = AttentionSpec(heads=32, kv_heads=4, dim=128, vdim=128, scale=128 ** -0.5, softcap=50.0)
+SISISUN_8B = sisisun_config(4096, 128256, tuple(LayerSpec(_SISISUN_8B_A, DenseMlpSpec(14336, "clamped_glu", 7.0))
+                                                for _ in range(32)), loop=LoopSpec(8, 16, 2))
+SISISUN_30B_MOE = sisisun_config(2048, 151936, tuple(
+    LayerSpec(_SISISUN_30B_A, MoeMlpSpec(128, 8, 768, groups=8, groups_kept=4, scale=2.5, shared_ff=768))
+    for _ in range(48)), loop=LoopSpec(12, 24, 2))
+
+
 @dataclass(frozen=True)
 class AssistantConfig:
     """Gemma 4 assistant (MTP) head: a separate four-block draft model with no K/V projections of its own.  Every
@@ -258,4 +390,7 @@ NAMED_CONFIGS: Dict[str, ModelConfig] = {
     "tiny-hybrid-mtp": replace(TINY_HYBRID, nextn_layers=1),
     "qwen35-35b-a3b": QWEN35_35B_A3B,
     "gemma4-26b-a4b": GEMMA4_26B_A4B,
+    "tiny-sisisun": TINY_SISISUN,
+    "sisisun-8b": SISISUN_8B,
+    "sisisun-30b-moe": SISISUN_30B_MOE,
 }

@@ -74,11 +74,12 @@ class DecodeGraphRunner:
         ex = self.ex
         b = self.batch(rows, max_ctx)
         h = ex.forward(b, defer_resid=True)
+        hid = self.hidden[:rows] if ex.keeps_hidden else None
         if greedy:
-            ex.head_greedy(h, self.next_ids[:rows], logits_out=self.logits[:rows], hidden_out=self.hidden[:rows])
+            ex.head_greedy(h, self.next_ids[:rows], logits_out=self.logits[:rows], hidden_out=hid)
             self.publish(rows)
         else:
-            ex.logits(h, out=self.logits[:rows], hidden_out=self.hidden[:rows])
+            ex.logits(h, out=self.logits[:rows], hidden_out=hid)
 
     def publish(self, rows: int) -> None:
         """next_ids -> tokens, advance positions (device side)."""

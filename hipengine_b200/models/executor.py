@@ -136,6 +136,8 @@ class _Scratch:
 
 
 class HybridExecutor:
+    keeps_hidden = True           # decode steps also store the post-norm hidden rows
+
     def __init__(self, weights: ModelWeights, device="cuda", max_slots: int = 4, max_context: int = 4608,
                  n_pages: Optional[int] = None, gemm_impl: Optional[str] = None):
         self.cfg = cfg = weights.config
@@ -236,6 +238,10 @@ class HybridExecutor:
                                                  dtype=torch.float32, device=dev)
                 self.gdn_state[i] = torch.zeros(self.max_slots, cfg.ssm_v_heads, cfg.ssm_state, cfg.ssm_state,
                                                 dtype=torch.float32, device=dev)
+        self._alloc_tables()
+
+    def _alloc_tables(self) -> None:
+        dev = self.device
         # default identity paging: slot s owns pages [1 + s*mp, 1 + (s+1)*mp); page 0 is a scratch sink
         mp = self.max_pages_per_slot
         bt = torch.arange(self.max_slots * mp, dtype=torch.int32).reshape(self.max_slots, mp) + 1

@@ -76,13 +76,7 @@ class Gemma4Executor(HybridExecutor):
         for i in range(cfg.n_layers):
             self.kv[i] = torch.zeros(self.n_pages, 2, cfg.layer_kv_heads(i), PAGE, cfg.layer_head_dim(i),
                                      dtype=torch.bfloat16, device=dev)
-        mp = self.max_pages_per_slot
-        bt = torch.arange(self.max_slots * mp, dtype=torch.int32).reshape(self.max_slots, mp) + 1
-        if self.n_pages < self.max_slots * mp + 1:
-            bt = bt.clamp(max=self.n_pages - 1)
-        self.block_table = bt.to(dev)
-        self.am_v = torch.empty(GEMV_MAX_ROWS * 64 * 64, dtype=torch.float32, device=dev)
-        self.am_i = torch.empty(GEMV_MAX_ROWS * 64 * 64, dtype=torch.int32, device=dev)
+        self._alloc_tables()
 
     def _rope(self, i: int):
         cfg = self.cfg

@@ -10,7 +10,7 @@ from __future__ import annotations
 from dataclasses import dataclass
 from typing import Any, Dict, List, Optional, Tuple
 
-from .config import ModelConfig
+from .config import ModelConfig, MoeMlpSpec
 
 
 @dataclass(frozen=True)
@@ -26,6 +26,8 @@ class ModelPlugin:
     kv_storage: Tuple[str, ...] = ("bf16",)
     tensor_parallel: bool = True
     expert_parallel: bool = False
+    compute_dtypes: Tuple[str, ...] = ("bfloat16",)
+    native_sources: Tuple[str, ...] = ()        # csrc files a build for this family alone needs (empty: all of them)
     notes: str = ""
 
     def layer_sequence(self, cfg: ModelConfig) -> List[str]:
@@ -46,11 +48,17 @@ class ModelPlugin:
                              "widened_block_types": list(self.widened_block_types), "chat_template": self.chat_template,
                              "speculative_providers": list(self.speculative_providers),
                              "kv_storage": list(self.kv_storage), "tensor_parallel": self.tensor_parallel,
-                             "expert_parallel": self.expert_parallel, "notes": self.notes}
+                             "expert_parallel": self.expert_parallel, "compute_dtypes": list(self.compute_dtypes),
+                             "notes": self.notes}
         if cfg is not None:
             seq = self.layer_sequence(cfg)
             d["layers"] = {k: seq.count(k) for k in sorted(set(seq))}
             d["ffn"] = "moe" if cfg.is_moe else "dense"
+            if cfg.layer_specs:
+                kinds = ["none" if l.mlp is None else "moe" if isinstance(l.mlp, MoeMlpSpec) else "dense"
+                         for l in cfg.layer_specs]
+                d["ffn"] = {k: kinds.count(k) for k in sorted(set(kinds))}
+                d["layer_runs"] = len(cfg.layer_runs())
             providers = list(self.speculative_providers)
             if "mtp" in providers and cfg.arch != "gemma4" and cfg.nextn_layers == 0:
                 providers.remove("mtp")                         # this checkpoint carries no NextN block
@@ -73,6 +81,14 @@ PLUGINS: Tuple[ModelPlugin, ...] = (
                 tensor_parallel=False,
                 notes="5 sliding-window layers : 1 global layer, dense GeGLU branch beside top-k experts; the MTP "
                       "drafter is the separate gemma4-assistant artifact"),
+    ModelPlugin("sisisun", ("sisisun",), "hipengine_b200.models.sisisun.SisisunExecutor", default_quant="bf16",
+                native_block_types=("BF16",), widened_block_types=(), kv_storage=("bf16", "f32"),
+                tensor_parallel=False, compute_dtypes=("bfloat16", "float32"),
+                native_sources=("attn_decode.cu", "attn_prefill.cu", "exact_f32.cu", "gemm_sm100.cu", "gemv_float.cu",
+                                "layers.cu", "moe.cu", "quant_util.cu", "runtime.cpp", "sampling.cu"),
+                notes="layers listed one by one: attention without rotation, soft-capped scores, dense (clamped GLU) or "
+                      "group-limited sigmoid-routed experts; a range of layers may run several times; checkpoints are "
+                      "folders with config.json and model.safetensors"),
 )
 
 

@@ -1,0 +1,348 @@
+"""Sisisun executor: listed attention layers without rotation, dense / expert feed-forwards, looped layer ranges.
+
+Reuses the hybrid executor's scratch, paged KV pool, projection dispatch, decode-graph and prefill-graph plumbing and
+replaces the weight packing and the layer walk:
+  * weights stay bfloat16.  q | k | v and gate | up are stacked at load, experts are stacked per layer, norm weights are
+    stored as 1 + w, widths that are not a multiple of eight and head widths the attention kernels do not have are
+    zero-padded (zeros change no result; the norms average over the real width);
+  * the KV planes belong to layer RUNS: every pass of a looped range attends only to what the same pass wrote;
+  * up to 16 rows (decode steps, short portions) run on the streaming bf16 GEMV with the norm and the activation fused
+    into it, more rows on the tcgen05 GEMM (split over K up to 128 rows); experts go through the selected-expert kernels
+    or the grouped GEMM by the same rule;
+  * ``dtype="float32"`` runs the same walk on fp32 CUDA-core kernels with fp32 activations and fp32 KV pages.
+In both modes residual, norms, scores, softmax, router and positions are fp32.  Oracle: ``ref/sisisun.py``.
+"""
+from __future__ import annotations
+
+from dataclasses import dataclass
+from typing import Callable, List, Optional, Tuple
+
+import torch
+
+from ..loading.weights import ModelWeights
+from ..ops import kernels as K
+from ..ops.kernels import DeviceWeight
+from ..quant.ggml import GGMLType
+from .config import AttentionSpec, DenseMlpSpec, MoeMlpSpec
+from .executor import PAGE, BatchDesc, HybridExecutor
+
+# segments of up to this many rows attend through the split-K decode kernel, longer ones through the flash kernel
+DECODE_SEG_ROWS = 8
+EXACT, FEW, MANY = "exact", "few", "many"       # kernel routes of a forward
+
+
+def _up8(n: int) -> int:
+    return -(-n // 8) * 8
+
+
+def _pad(t: torch.Tensor, rows: int, cols: int) -> torch.Tensor:
+    if t.shape == (rows, cols):
+        return t
+    out = torch.zeros(rows, cols, dtype=t.dtype, device=t.device)
+    out[:t.shape[0], :t.shape[1]] = t
+    return out
+
+
+@dataclass
+class _Layer:
+    norm1: torch.Tensor                          # fp32 [Hp], 1 + w
+    norm2: Optional[torch.Tensor]
+    qkv: DeviceWeight                            # [q | k | v rows, Hp]
+    q_norm: torch.Tensor                         # fp32 [dim]
+    k_norm: torch.Tensor
+    o: DeviceWeight                              # [Hp, heads * D]
+    gate_up: Optional[DeviceWeight] = None       # dense: [gate | up rows, Hp]
+    down: Optional[DeviceWeight] = None          # dense: [Hp, F]
+    router: Optional[DeviceWeight] = None        # [experts (+ shared gate), Hp], rows padded to eight
+    e_gate_up: Optional[DeviceWeight] = None     # [experts * (gate | up), Hp]
+    e_down: Optional[DeviceWeight] = None        # [experts * Hp, F]
+    s_gate_up: Optional[DeviceWeight] = None
+    s_down: Optional[DeviceWeight] = None
+
+
+class SisisunExecutor(HybridExecutor):
+    keeps_hidden = False
+
+    def __init__(self, weights: ModelWeights, dtype: str = "bfloat16", **kw):
+        if dtype not in ("bfloat16", "float32"):
+            raise ValueError(f"compute dtype {dtype!r} (bfloat16 | float32)")
+        self.exact = dtype == "float32"
+        self.act_dtype = torch.float32 if self.exact else torch.bfloat16
+        self.on_layer_run: Optional[Callable[[int, torch.Tensor], None]] = None    # (run, residual rows) observer
+        super().__init__(weights, **kw)
+
+    # ------------------------------------------------------------------ weights
+    def _load(self, weights: ModelWeights) -> None:
+        cfg, dev = self.cfg, self.device
+        self.hp = hp = _up8(cfg.hidden)
+
+        def mat(name: str) -> torch.Tensor:
+            t = weights[name]
+            if t.ggml_type == GGMLType.BF16:
+                return t.raw.to(dev).reshape(-1).view(torch.bfloat16).reshape(t.shape)
+            return t.dequant(dev).to(torch.bfloat16)
+
+        def put(name: str, t: torch.Tensor) -> DeviceWeight:
+            w = self.dw[name] = DeviceWeight(int(GGMLType.BF16), t.shape[0], t.shape[1], t.contiguous())
+            return w
+
+        def norm(name: str) -> torch.Tensor:
+            v = torch.zeros(hp, dtype=torch.float32, device=dev)
+            v[:cfg.hidden] = 1.0 + mat(name).float()
+            self.f32[name] = v
+            return v
+
+        def gate_up(p: str, ff: int) -> torch.Tensor:
+            fp = _up8(ff)
+            return torch.cat([_pad(mat(p + "gate"), fp, hp), _pad(mat(p + "up"), fp, hp)], 0)
+
+        def glu(name: str, p: str, ff: int) -> Tuple[DeviceWeight, DeviceWeight]:
+            return put(name + "gate_up", gate_up(p, ff)), put(name + "down", _pad(mat(p + "down"), hp, _up8(ff)))
+
+        self.layers: List[_Layer] = []
+        for i, spec in enumerate(cfg.layer_specs):
+            a, m, p = spec.mixer, spec.mlp, f"l{i}."
+            qkv = torch.cat([mat(p + "mix.q"), mat(p + "mix.k"), mat(p + "mix.v")], 0)
+            o = torch.zeros(hp, a.heads, a.width, dtype=torch.bfloat16, device=dev)
+            o[:cfg.hidden, :, :a.vdim] = mat(p + "mix.o").reshape(cfg.hidden, a.heads, a.vdim)
+            for s in ("q.norm", "k.norm"):
+                self.f32[p + "mix." + s] = mat(p + "mix." + s).float().contiguous()
+            L = _Layer(norm(p + "norm1"), norm(p + "norm2") if m is not None else None,
+                       put(p + "qkv", _pad(qkv, _up8(qkv.shape[0]), hp)), self.f32[p + "mix.q.norm"],
+                       self.f32[p + "mix.k.norm"], put(p + "o", o.reshape(hp, -1)))
+            if isinstance(m, DenseMlpSpec):
+                L.gate_up, L.down = glu(p, p + "mlp.", m.ff)
+            elif isinstance(m, MoeMlpSpec):
+                fp = _up8(m.ff)
+                gu = torch.empty(m.experts * 2 * fp, hp, dtype=torch.bfloat16, device=dev)
+                dn = torch.empty(m.experts * hp, fp, dtype=torch.bfloat16, device=dev)
+                for e in range(m.experts):
+                    gu[e * 2 * fp:(e + 1) * 2 * fp] = gate_up(p + f"mlp.e{e}.", m.ff)
+                    dn[e * hp:(e + 1) * hp] = _pad(mat(p + f"mlp.e{e}.down"), hp, fp)
+                L.e_gate_up, L.e_down = put(p + "experts.gate_up", gu), put(p + "experts.down", dn)
+                rows = [mat(p + "mlp.router")]
+                if m.shared_ff:
+                    L.s_gate_up, L.s_down = glu(p + "shared.", p + "mlp.shared.", m.shared_ff)
+                    rows.append(mat(p + "mlp.shared.sg"))
+                r = torch.cat(rows, 0)
+                L.router = put(p + "router", _pad(r, _up8(r.shape[0]), hp))
+            self.layers.append(L)
+        self.embed_w = put("token_embd.weight", mat("embed"))
+        self.head_w = put("output.weight", _pad(mat("head"), cfg.vocab, hp))
+        norm("final.norm")
+        self.runs = cfg.layer_runs()
+        self.loop_step: Optional[torch.Tensor] = None
+        if cfg.loop is not None:
+            self.loop_step = _pad(mat("loop.step").float(), cfg.loop.times, hp).contiguous()
+        i = torch.arange((cfg.hidden + 1) // 2, dtype=torch.float64)
+        self.pos_freq = torch.pow(torch.tensor(10000.0, dtype=torch.float64), -2.0 * i / cfg.hidden).to(dev)
+
+    # ------------------------------------------------------------------ state: one KV plane per layer run
+    def _alloc_state(self) -> None:
+        dev = self.device
+        self.conv_state, self.gdn_state = {}, {}
+        self.kv = {}
+        for run, (i, _) in enumerate(self.runs):
+            a = self.cfg.layer_specs[i].mixer
+            self.kv[run] = torch.zeros(self.n_pages, 2, a.kv_heads, PAGE, a.width, dtype=self.act_dtype, device=dev)
+        self._alloc_tables()
+
+    # ------------------------------------------------------------------ dispatch
+    def _resid_buffer(self, T: int) -> torch.Tensor:
+        return self.scratch.get("h", (T, self.hp), torch.float32)
+
+    def _norm_rows(self, h: torch.Tensor, w: torch.Tensor) -> torch.Tensor:
+        xn = self.scratch.get("xn", (h.shape[0], self.hp), self.act_dtype)
+        return K.rmsnorm_rows(h, w, xn, self.cfg.rms_eps, n_mean=self.cfg.hidden)
+
+    def _route(self, T: int) -> str:
+        return EXACT if self.exact else FEW if T <= K.FLOAT_GEMV_MAX_ROWS else MANY
+
+    def _in_proj(self, h: torch.Tensor, norm_w: torch.Tensor, w: DeviceWeight, name: str, route: str,
+                 xn: Optional[torch.Tensor] = None) -> torch.Tensor:
+        """norm(h) @ W^T (fp32, or bf16 rows for large batches); ``xn``: the normalised rows when they exist already."""
+        T, cfg = h.shape[0], self.cfg
+        if route == FEW:
+            out = self.scratch.get(name + "_f32", (T, w.n_rows), torch.float32)
+            K.gemv_float(h, [(w.data, None, out, K.EPI_F32)], norm_w=norm_w, eps=cfg.rms_eps, norm_n=cfg.hidden)
+            return out
+        if xn is None:
+            with self._stage("norm"):
+                xn = self._norm_rows(h, norm_w)
+        if route == EXACT:
+            return K.small_gemm_f32(xn, w.data, self.scratch.get(name + "_f32", (T, w.n_rows), torch.float32))
+        return self._proj(xn, w, name, name)
+
+    def _add_proj(self, x: torch.Tensor, w: DeviceWeight, h: torch.Tensor, route: str) -> None:
+        """h += x @ W^T."""
+        if route == EXACT:
+            K.small_gemm_f32(x, w.data, h, add=True)
+        elif route == FEW:
+            K.gemv_float(x, [(w.data, None, h, K.EPI_ADD_F32)])
+        else:
+            self._out_big(x, w, h, "o")
+
+    # ------------------------------------------------------------------ layers
+    def _attention(self, run: int, i: int, h: torch.Tensor, b: BatchDesc, route: str) -> None:
+        cfg, sc, L = self.cfg, self.scratch, self.layers[i]
+        a, T = cfg.layer_specs[i].mixer, b.T
+        with self._stage("attn_qkv_gemm"):
+            qkv = self._in_proj(h, L.norm1, L.qkv, "qkv", route)
+        nq, nk = a.heads * a.dim, a.kv_heads * a.dim
+        q_out = sc.get("q_out", (T, a.heads, a.width), self.act_dtype)
+        K.qkv_post(qkv[:, :nq], qkv[:, nq:nq + nk], qkv[:, nq + nk:], L.q_norm, L.k_norm, q_out, None, self.kv[run],
+                   self.block_table, b.slot, b.pos, a.heads, a.kv_heads, a.width, PAGE, False, 0, 1.0, cfg.rms_eps,
+                   d_in=a.dim, dv_in=a.vdim)
+        out = sc.get("attn_out", (T, a.heads * a.width), self.act_dtype)
+        with self._stage("attn_core"):
+            self._attend_run(run, a, q_out, b, out)
+        with self._stage("out_gemm"):
+            self._add_proj(out, L.o, h, route)
+
+    def _attend_run(self, run: int, a: AttentionSpec, q: torch.Tensor, b: BatchDesc, out: torch.Tensor) -> None:
+        D, kv = a.width, self.kv[run]
+        if self.exact:
+            K.attn_exact(q, kv, self.block_table, b.slot, b.ctx_len, out, a.heads, a.kv_heads, D, PAGE, a.scale,
+                         a.softcap)
+            return
+        from ..ops import attention as A
+
+        def decode(r0: int, r1: int, ctx: int) -> None:
+            split_len, max_splits = K.attn_decode_split(ctx, r1 - r0, a.kv_heads)
+            part = self.scratch.get("attn_part", (K.attn_decode_scratch_floats(r1 - r0, a.heads, max_splits, D),),
+                                    torch.float32)
+            K.attn_decode(q[r0:r1], None, kv, self.block_table, b.slot[r0:r1], b.ctx_len[r0:r1], part, out[r0:r1],
+                          a.heads, a.kv_heads, D, PAGE, split_len, max_splits, a.scale, softcap=a.softcap)
+
+        if b.segs_host is None:
+            decode(0, b.T, b.max_ctx)
+            return
+        # neighbouring segments of the same kind share a launch: prompt portions the flash kernel, single tokens and
+        # short portions the split-K kernel
+        flash = A.flash_prefill_available(D)
+        s, r0 = 0, 0
+        while s < len(b.segs_host):
+            long = flash and b.segs_host[s][2] > DECODE_SEG_ROWS
+            e, r1, ctx = s, r0, 1
+            while e < len(b.segs_host) and (flash and b.segs_host[e][2] > DECODE_SEG_ROWS) == long:
+                _, p0, n = b.segs_host[e]
+                ctx, r1, e = max(ctx, p0 + n), r1 + n, e + 1
+            if long:
+                A.flash_prefill_segs(q, None, kv, self.block_table, b.seg_start[s:], b.seg_slot[s:], b.pos,
+                                     [n for _, _, n in b.segs_host[s:e]], out, a.heads, a.kv_heads, D, PAGE, a.scale,
+                                     softcap=a.softcap)
+            else:
+                for c0 in range(r0, r1, 512):       # bounds the split-K scratch of long segments of very wide heads
+                    decode(c0, min(r1, c0 + 512), ctx)
+            s, r0 = e, r1
+
+    def _dense(self, L: _Layer, m: DenseMlpSpec, h: torch.Tensor, route: str) -> None:
+        T, F = h.shape[0], L.down.n_cols
+        act = self.scratch.get("ffn_act", (T, F), self.act_dtype)
+        if route == FEW:
+            gu = L.gate_up.data
+            K.gemv_float(h, [(gu[:F], gu[F:], act, K.EPI_OF_ACT[m.act])], norm_w=L.norm2, eps=self.cfg.rms_eps,
+                         norm_n=self.cfg.hidden, limit=m.limit)
+        else:
+            with self._stage("ffn_gateup_gemm"):
+                gu = self._in_proj(h, L.norm2, L.gate_up, "ffn_gu", route)
+            with self._stage("act_mul"):
+                K.act_mul(gu, act, m.act, m.limit)
+        with self._stage("ffn_down_gemm"):
+            self._add_proj(act, L.down, h, route)
+
+    def _experts(self, L: _Layer, m: MoeMlpSpec, h: torch.Tensor, route: str) -> None:
+        from ..ops import gemm as GM
+        sc, cfg, T, E, k = self.scratch, self.cfg, h.shape[0], m.experts, m.top
+        F = L.e_down.n_cols
+        xn = None
+        if route != FEW:
+            with self._stage("norm"):
+                xn = self._norm_rows(h, L.norm2)
+        if route == MANY:
+            logits = GM.gemm_bf16(xn, L.router.data, sc.get("moe_logits_f32", (T, L.router.n_rows), torch.float32))
+        else:
+            logits = self._in_proj(h, L.norm2, L.router, "moe_logits", route, xn=xn)
+        ids = sc.get("moe_ids", (T, k), torch.int32)
+        wts = sc.get("moe_wts", (T, k), torch.float32)
+        K.moe_route_grouped(logits, k, ids, wts, E, m.groups, m.groups_kept, m.scale)
+        sg = logits[:, E:E + 1] if m.shared_ff else None
+        s_gu = L.s_gate_up.data if m.shared_ff else None
+        s_dn = L.s_down.data if m.shared_ff else None
+        if route != MANY:
+            rows = sc.get("moe_act", (T * k, F), self.act_dtype)
+            rows_s = sc.get("moe_act_sh", (T, L.s_down.n_cols), self.act_dtype) if m.shared_ff else None
+            if route == EXACT:
+                K.moe_exact(xn, ids, wts, L.e_gate_up.data, L.e_down.data, E, rows, h, sg, s_gu, s_dn, rows_s)
+                return
+            K.moe_gateup_float(h, L.norm2, cfg.rms_eps, cfg.hidden, ids, wts, L.e_gate_up.data, E, rows, sg, s_gu, rows_s)
+            K.moe_down_float(rows, ids, L.e_down.data, E, h, rows_s, s_dn)
+            return
+        P = T * k
+        bound = K.moe_sorted_rows_bound(P, E)
+        pos = sc.get("moe_pos", (P,), torch.int32)
+        tiles = sc.get("moe_tiles", (bound // 128,), torch.int32)
+        K.moe_group(ids, E, pos, tiles, sc.get("moe_meta", (4,), torch.int32))
+        xs = sc.get("moe_xs", (bound, self.hp), torch.bfloat16)
+        K.moe_gather(xn, pos, k, xs)
+        gu = sc.get("moe_gu", (bound, 2 * F), torch.bfloat16)
+        GM.gemm_bf16_grouped(xs, L.e_gate_up.data, gu, E, tiles)
+        act = sc.get("moe_act_g", (bound, F), torch.bfloat16)
+        K.act_mul(gu, act, "silu")
+        ys = sc.get("moe_ys", (bound, self.hp), torch.bfloat16)
+        GM.gemm_bf16_grouped(act, L.e_down.data, ys, E, tiles)
+        ysh = None
+        if m.shared_ff:
+            gus = self._proj(xn, L.s_gate_up, "moe_gus", "g")
+            acts = sc.get("moe_acts", (T, L.s_down.n_cols), torch.bfloat16)
+            K.act_mul(gus, acts, "silu")
+            ysh = self._gemm(acts, L.s_down, sc.get("y_bf", (T, self.hp), torch.bfloat16), tag="d")
+        K.moe_combine(h, ys, pos, wts, k, ysh, sg)
+
+    # ------------------------------------------------------------------ whole model
+    def forward(self, b: BatchDesc, journal: Optional[dict] = None, h_out: Optional[torch.Tensor] = None,
+                defer_resid: bool = False) -> torch.Tensor:
+        cfg, T = self.cfg, b.T
+        route = self._route(T)
+        direct = h_out is not None and h_out.shape[1] == self.hp and h_out.is_contiguous()
+        h = h_out if direct else self._resid_buffer(T)
+        lp = cfg.loop
+        x0 = self.scratch.get("embed_out", (T, self.hp), torch.float32) if lp is not None and lp.times > 1 else None
+        K.embed_sinusoid(self.embed_w, b.tokens, b.pos, self.pos_freq, h, x0)
+        for run, (i, t) in enumerate(self.runs):
+            if t >= 0 and i == lp.start:
+                K.resid_inject(h, x0 if t > 0 else None, self.loop_step[t])
+            self._attention(run, i, h, b, route)
+            m = cfg.layer_specs[i].mlp
+            if isinstance(m, DenseMlpSpec):
+                self._dense(self.layers[i], m, h, route)
+            elif isinstance(m, MoeMlpSpec):
+                self._experts(self.layers[i], m, h, route)
+            if self.on_layer_run is not None:
+                self.on_layer_run(run, h[:, :cfg.hidden])
+        if h_out is not None and not direct:
+            h_out.copy_(h[:, :cfg.hidden])
+            return h_out
+        return h
+
+    def logits(self, h_rows: torch.Tensor, out: Optional[torch.Tensor] = None,
+               hidden_out: Optional[torch.Tensor] = None) -> torch.Tensor:
+        cfg, R = self.cfg, h_rows.shape[0]
+        if h_rows.shape[1] != self.hp:
+            h_rows = _pad(h_rows, R, self.hp)
+        norm_w = self.f32["final.norm"]
+        if out is None:
+            out = self.scratch.get("logits", (R, cfg.vocab), torch.float32)
+        if hidden_out is not None:
+            hid = self.scratch.get("hidden_rows", (R, self.hp), torch.float32)
+            hidden_out.copy_(K.rmsnorm_rows(h_rows, norm_w, hid, cfg.rms_eps, n_mean=cfg.hidden)[:, :cfg.hidden])
+        if self._route(R) == FEW:
+            K.gemv_float(h_rows, [(self.head_w.data, None, out, K.EPI_F32)], norm_w=norm_w, eps=cfg.rms_eps,
+                         norm_n=cfg.hidden)
+            return out
+        xn = self.scratch.get("xn_head", (R, self.hp), self.act_dtype)
+        K.rmsnorm_rows(h_rows, norm_w, xn, cfg.rms_eps, n_mean=cfg.hidden)
+        if self.exact:
+            return K.small_gemm_f32(xn, self.head_w.data, out)
+        from ..ops import gemm as GM
+        return GM.gemm_bf16(xn, self.head_w.data, out)

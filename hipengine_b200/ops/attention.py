@@ -15,6 +15,23 @@ def flash_prefill_available(head_dim: int) -> bool:
         return False
 
 
+FLASH_TILE_ROWS = 64
+
+
+def flash_prefill_segs(q, gate, kv_cache, block_table, seg_start, seg_slot, pos, seg_rows, out, H, Hkv, D, page, scale,
+                       window: int = 0, softcap: float = 0.0) -> None:
+    """``flash_prefill`` for several segments in one launch: ``seg_start`` (device, n + 1 absolute row offsets),
+    ``seg_slot`` (device), ``pos`` (device, per row) and ``seg_rows`` (host row counts, sizes the grid)."""
+    tiles = sum(-(-n // FLASH_TILE_ROWS) for n in seg_rows)
+    N.check(N.lib().he_flash_prefill_segs(
+        C.c_void_p(q.data_ptr()), C.c_void_p(None if gate is None else gate.data_ptr()),
+        C.c_void_p(kv_cache.data_ptr()), C.c_void_p(block_table.data_ptr()), C.c_int(block_table.shape[1]),
+        C.c_void_p(seg_start.data_ptr()), C.c_void_p(seg_slot.data_ptr()), C.c_void_p(pos.data_ptr()),
+        C.c_int(len(seg_rows)), C.c_int(tiles), C.c_void_p(out.data_ptr()), C.c_int(H), C.c_int(Hkv), C.c_int(D),
+        C.c_int(page), C.c_float(scale), C.c_int(window), C.c_float(softcap),
+        C.c_void_p(torch.cuda.current_stream().cuda_stream)), "he_flash_prefill_segs")
+
+
 def flash_prefill(q, gate, kv_cache, block_table, slot: int, pos0: int, out, H, Hkv, D, page, scale,
                   window: int = 0) -> None:
     """Causal paged GQA attention over one segment's rows (append-then-attend) with the sigmoid gate fused.

@@ -50,7 +50,7 @@ class _QkvArgs(C.Structure):
                 ("slot", c_vp), ("pos", c_vp), ("max_pages", C.c_int),
                 ("H", C.c_int), ("Hkv", C.c_int), ("D", C.c_int), ("page", C.c_int), ("gated", C.c_int),
                 ("rope_dim", C.c_int), ("theta", C.c_float), ("eps", C.c_float), ("q_scale", C.c_float),
-                ("rope_denom", C.c_int)]
+                ("rope_denom", C.c_int), ("d_in", C.c_int), ("dv_in", C.c_int), ("out_f32", C.c_int)]
 
 
 class _ConvArgs(C.Structure):
@@ -77,7 +77,7 @@ class _AttnDecArgs(C.Structure):
                 ("ctx_len", c_vp), ("partial", c_vp), ("out", c_vp),
                 ("R", C.c_int), ("H", C.c_int), ("Hkv", C.c_int), ("D", C.c_int), ("page", C.c_int),
                 ("max_pages", C.c_int), ("split_len", C.c_int), ("max_splits", C.c_int), ("window", C.c_int),
-                ("scale", C.c_float), ("status", c_vp)]
+                ("scale", C.c_float), ("status", c_vp), ("softcap", C.c_float)]
 
 
 class _GdnDecodeArgs(C.Structure):
@@ -102,6 +102,36 @@ class _MoeSelArgs(C.Structure):
                 ("expert_lo", C.c_int), ("expert_n", C.c_int)]
 
 
+class _FloatGemvSeg(C.Structure):
+    _fields_ = [("w", c_vp), ("w2", c_vp), ("out", c_vp), ("out_stride", c_ll), ("n_rows", C.c_int), ("epi", C.c_int)]
+
+
+class _FloatGemvArgs(C.Structure):
+    _fields_ = [("seg", _FloatGemvSeg * 4), ("n_seg", C.c_int), ("K", C.c_int), ("ldw", c_ll), ("R", C.c_int),
+                ("x_dtype", C.c_int), ("x", c_vp), ("x_stride", c_ll), ("norm_w", c_vp), ("eps", C.c_float),
+                ("norm_n", C.c_int), ("limit", C.c_float)]
+
+
+class _FloatMoeArgs(C.Structure):
+    _fields_ = [("x", c_vp), ("ldx", c_ll), ("norm_w", c_vp), ("eps", C.c_float), ("norm_n", C.c_int), ("ids", c_vp),
+                ("wts", c_vp), ("sg", c_vp), ("ld_sg", c_ll), ("w1", c_vp), ("w1s", c_vp), ("E", C.c_int),
+                ("T", C.c_int), ("k", C.c_int), ("K", C.c_int), ("F", C.c_int), ("Fs", C.c_int), ("N", C.c_int),
+                ("act", C.c_int), ("limit", C.c_float), ("rows", c_vp), ("rows_s", c_vp), ("h", c_vp), ("ldh", c_ll)]
+
+
+class _ExactAttnArgs(C.Structure):
+    _fields_ = [("q", c_vp), ("kv_cache", c_vp), ("block_table", c_vp), ("slot", c_vp), ("ctx_len", c_vp),
+                ("out", c_vp), ("R", C.c_int), ("H", C.c_int), ("Hkv", C.c_int), ("D", C.c_int), ("page", C.c_int),
+                ("max_pages", C.c_int), ("scale", C.c_float), ("softcap", C.c_float)]
+
+
+class _ExactMoeArgs(C.Structure):
+    _fields_ = [("x", c_vp), ("ldx", c_ll), ("ids", c_vp), ("wts", c_vp), ("sg", c_vp), ("ld_sg", c_ll),
+                ("w1", c_vp), ("w1s", c_vp), ("E", C.c_int), ("T", C.c_int), ("k", C.c_int), ("K", C.c_int),
+                ("F", C.c_int), ("Fs", C.c_int), ("N", C.c_int), ("rows", c_vp), ("rows_s", c_vp), ("h", c_vp),
+                ("ldh", c_ll)]
+
+
 _CHECKED = False
 
 
@@ -111,12 +141,16 @@ def _check_abi() -> None:
     if _CHECKED:
         return
     L = N.lib()
-    pairs = [("he_gemv_args_size", _GemvArgs), ("he_qkv_args_size", _QkvArgs), ("he_conv_args_size", _ConvArgs),
+    pairs = [("he_gemv_float_args_size", _FloatGemvArgs), ("he_moe_float_args_size", _FloatMoeArgs),
+             ("he_exact_attn_args_size", _ExactAttnArgs), ("he_exact_moe_args_size", _ExactMoeArgs),
+             ("he_gemv_args_size", _GemvArgs), ("he_qkv_args_size", _QkvArgs), ("he_conv_args_size", _ConvArgs),
              ("he_gdn_prep_args_size", _GdnPrepArgs), ("he_gdn_scan_args_size", _GdnScanArgs),
              ("he_attn_dec_args_size", _AttnDecArgs), ("he_moe_sel_args_size", _MoeSelArgs),
              ("he_gdn_decode_args_size", _GdnDecodeArgs), ("he_gdn_chunk_args_size", _GdnChunkArgs),
              ("he_gemv_comm_size", GemvComm)]
     for fn, st in pairs:
+        if not hasattr(L, fn):           # a library built from a subset of the sources
+            continue
         got = getattr(L, fn)()
         if got != C.sizeof(st):
             raise RuntimeError(f"ABI mismatch for {st.__name__}: C={got} Python={C.sizeof(st)}")
@@ -339,24 +373,32 @@ def embed(w: DeviceWeight, ids: torch.Tensor, out: torch.Tensor, scale: float = 
 
 # ----------------------------------------------------------------------------- row-wise layers
 
-def rmsnorm_rows(x: torch.Tensor, w: Optional[torch.Tensor], out: torch.Tensor, eps: float = 1e-6) -> torch.Tensor:
+def rmsnorm_rows(x: torch.Tensor, w: Optional[torch.Tensor], out: torch.Tensor, eps: float = 1e-6,
+                 n_mean: int = 0) -> torch.Tensor:
+    """``n_mean``: columns the mean square is taken over when the rows are zero-padded (0: all of them)."""
     T, H = x.shape
     assert x.dtype == torch.float32
     N.check(N.lib().he_rmsnorm_rows(c_vp(x.data_ptr()), c_vp(_p(w)), c_vp(out.data_ptr()),
                                     C.c_int(1 if out.dtype == torch.bfloat16 else 0), C.c_int(T), C.c_int(H),
-                                    C.c_float(eps), c_ll(x.stride(0)), c_ll(out.stride(0)), _stream()),
-            "he_rmsnorm_rows")
+                                    C.c_float(eps), c_ll(x.stride(0)), c_ll(out.stride(0)), C.c_int(n_mean or H),
+                                    _stream()), "he_rmsnorm_rows")
     return out
 
 
-def act_mul(gu: torch.Tensor, out: torch.Tensor, act: str = "silu") -> torch.Tensor:
+ACT_CODES = {"silu": 0, "gelu_tanh": 1, "clamped_glu": 2}
+
+
+def act_mul(gu: torch.Tensor, out: torch.Tensor, act: str = "silu", limit: float = 0.0) -> torch.Tensor:
+    """Packed rows [gate | up] -> act(gate) * up; ``clamped_glu`` bounds both branches by ``limit``."""
     T, F2 = gu.shape
+    code = C.c_int(ACT_CODES[act])
     if gu.dtype == torch.float32:
-        N.check(N.lib().he_act_mul_f32(c_vp(gu.data_ptr()), c_vp(out.data_ptr()), c_ll(T), C.c_int(F2 // 2),
-                                       C.c_int(0 if act == "silu" else 1), _stream()), "he_act_mul")
+        N.check(N.lib().he_act_mul_f32(c_vp(gu.data_ptr()), c_vp(out.data_ptr()),
+                                       C.c_int(1 if out.dtype == torch.bfloat16 else 0), c_ll(T), C.c_int(F2 // 2), code,
+                                       C.c_float(limit), _stream()), "he_act_mul")
         return out
-    N.check(N.lib().he_act_mul(c_vp(gu.data_ptr()), c_vp(out.data_ptr()), c_ll(T), C.c_int(F2 // 2),
-                               C.c_int(0 if act == "silu" else 1), _stream()), "he_act_mul")
+    N.check(N.lib().he_act_mul(c_vp(gu.data_ptr()), c_vp(out.data_ptr()), c_ll(T), C.c_int(F2 // 2), code,
+                               C.c_float(limit), _stream()), "he_act_mul")
     return out
 
 
@@ -370,8 +412,12 @@ def qkv_post(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, q_norm, k_norm, 
              gate_out: Optional[torch.Tensor], kv_cache: torch.Tensor, block_table: torch.Tensor,
              slot: torch.Tensor, pos: torch.Tensor, H: int, Hkv: int, D: int, page: int, gated: bool,
              rope_dim: int, theta: float, eps: float, q_scale: float = 1.0, v_norm: bool = False,
-             rope_denom: int = 0) -> None:
+             rope_denom: int = 0, d_in: int = 0, dv_in: int = 0) -> None:
+    """``d_in`` / ``dv_in``: head widths of the projected q, k / v rows when they are narrower than the cache's ``D``
+    (the rest is written as zeros; the norms average over the real width).  fp32 ``q_out`` and ``kv_cache`` are written
+    without rounding."""
     _check_abi()
+    assert q_out.dtype == kv_cache.dtype
     T = q.shape[0]
     a = _QkvArgs()
     a.q, a.k, a.v = q.data_ptr(), k.data_ptr(), v.data_ptr()
@@ -385,6 +431,7 @@ def qkv_post(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, q_norm, k_norm, 
     a.H, a.Hkv, a.D, a.page, a.gated = H, Hkv, D, page, int(gated)
     a.rope_dim, a.theta, a.eps, a.q_scale = rope_dim, theta, eps, q_scale
     a.rope_denom = rope_denom
+    a.d_in, a.dv_in, a.out_f32 = d_in, dv_in, int(q_out.dtype == torch.float32)
     N.check(N.lib().he_qkv_post(C.byref(a), C.c_int(T), _stream()), "he_qkv_post")
 
 
@@ -490,7 +537,8 @@ def attn_decode_scratch_floats(R: int, H: int, max_splits: int, D: int) -> int:
 
 def attn_decode(q: torch.Tensor, gate: Optional[torch.Tensor], kv_cache: torch.Tensor, block_table: torch.Tensor,
                 slot: torch.Tensor, ctx_len: torch.Tensor, partial: torch.Tensor, out: torch.Tensor, H: int, Hkv: int,
-                D: int, page: int, split_len: int, max_splits: int, scale: float, window: int = 0) -> None:
+                D: int, page: int, split_len: int, max_splits: int, scale: float, window: int = 0,
+                softcap: float = 0.0) -> None:
     _check_abi()
     a = _AttnDecArgs()
     a.q, a.gate, a.kv_cache = q.data_ptr(), _p(gate), kv_cache.data_ptr()
@@ -500,6 +548,7 @@ def attn_decode(q: torch.Tensor, gate: Optional[torch.Tensor], kv_cache: torch.T
     a.max_pages = block_table.shape[1]
     a.split_len, a.max_splits, a.window, a.scale = split_len, max_splits, window, scale
     a.status = status_tensor(q.device).data_ptr()
+    a.softcap = softcap
     assert partial.numel() >= attn_decode_scratch_floats(a.R, H, max_splits, D)
     N.check(N.lib().he_attn_decode(C.byref(a), _stream()), "he_attn_decode")
 
@@ -540,6 +589,16 @@ def moe_route(logits: torch.Tensor, k: int, ids: torch.Tensor, wts: torch.Tensor
     N.check(N.lib().he_moe_route(c_vp(logits.data_ptr()), c_ll(logits.stride(0)), C.c_int(T), C.c_int(E), C.c_int(k),
                                  C.c_int(mode), c_vp(_p(expert_scale)), c_vp(ids.data_ptr()), c_vp(wts.data_ptr()),
                                  _stream()), "he_moe_route")
+
+
+def moe_route_grouped(logits: torch.Tensor, k: int, ids: torch.Tensor, wts: torch.Tensor, n_experts: int, groups: int,
+                      keep: int, scale: float) -> None:
+    """Sigmoid router limited to the best ``keep`` of ``groups`` groups of neighbouring experts; weights are the chosen
+    scores over their sum, times ``scale``."""
+    N.check(N.lib().he_moe_route_grouped(c_vp(logits.data_ptr()), c_ll(logits.stride(0)), C.c_int(logits.shape[0]),
+                                         C.c_int(n_experts), C.c_int(k), C.c_int(groups), C.c_int(keep),
+                                         C.c_float(scale), c_vp(ids.data_ptr()), c_vp(wts.data_ptr()), _stream()),
+            "he_moe_route_grouped")
 
 
 def moe_sorted_rows_bound(P: int, E: int) -> int:
@@ -614,6 +673,121 @@ def moe_down_sel(act_rows: torch.Tensor, ids: torch.Tensor, wts: torch.Tensor, w
     ``expert_range`` = (lo, hi) restricts the sum to the local experts of an expert-parallel rank."""
     _moe_sel("he_moe_down_sel", act_rows, None, 0.0, ids, wts, w_down, None, n_out, h, "silu",
              expert_range=expert_range)
+
+
+# ----------------------------------------------------------------------------- bfloat16 weights, few rows
+
+FLOAT_GEMV_MAX_ROWS = 16
+EPI_CLAMPED_GLU = 5
+EPI_OF_ACT = {"silu": EPI_SILU_MUL, "gelu_tanh": EPI_GELU_MUL, "clamped_glu": EPI_CLAMPED_GLU}
+
+
+def gemv_float(x: torch.Tensor, segs: Sequence[Tuple[torch.Tensor, Optional[torch.Tensor], torch.Tensor, int]],
+               norm_w: Optional[torch.Tensor] = None, eps: float = 1e-6, norm_n: int = 0, limit: float = 0.0) -> None:
+    """1..16 rows times bf16 weights: ``segs`` are (w [N, K], w2 or None, out, epilogue).  fp32 rows may have the RMS
+    norm fused (mean over ``norm_n`` columns)."""
+    _check_abi()
+    _check_device(x)
+    R, Kc = x.shape
+    a = _FloatGemvArgs()
+    a.n_seg, a.K, a.R = len(segs), segs[0][0].shape[1], R
+    a.ldw = segs[0][0].stride(0)
+    assert Kc == a.K, (Kc, a.K)
+    for i, (w, w2, out, epi) in enumerate(segs):
+        sg = a.seg[i]
+        assert w.dtype == torch.bfloat16 and w.stride(0) == a.ldw and w.shape[1] == a.K
+        assert out.dtype == (torch.float32 if epi in (EPI_F32, EPI_ADD_F32) else torch.bfloat16)
+        sg.w, sg.w2, sg.out = w.data_ptr(), _p(w2), out.data_ptr()
+        sg.out_stride, sg.n_rows, sg.epi = out.stride(0), w.shape[0], epi
+    a.x_dtype, a.x, a.x_stride = _dt(x), x.data_ptr(), x.stride(0)
+    a.norm_w, a.eps, a.norm_n, a.limit = _p(norm_w), eps, norm_n or Kc, limit
+    N.check(N.lib().he_gemv_float(C.byref(a), _stream()), "he_gemv_float")
+
+
+def moe_gateup_float(h: torch.Tensor, norm_w: torch.Tensor, eps: float, norm_n: int, ids: torch.Tensor,
+                     wts: torch.Tensor, w_gu: torch.Tensor, n_experts: int, rows: torch.Tensor,
+                     sg: Optional[torch.Tensor] = None, w_gu_shared: Optional[torch.Tensor] = None,
+                     rows_shared: Optional[torch.Tensor] = None, act: str = "silu", limit: float = 0.0) -> None:
+    """Selected experts, few tokens: ``rows`` [T*k, F] = weight * act(Wg xn) * (Wu xn) in bf16, and ``rows_shared``
+    [T, Fs] the same for the shared expert with weight sigmoid(sg).  ``w_gu`` stacks [gate | up] rows per expert."""
+    _check_abi()
+    a = _FloatMoeArgs()
+    a.x, a.ldx, a.norm_w, a.eps, a.norm_n = h.data_ptr(), h.stride(0), norm_w.data_ptr(), eps, norm_n
+    a.ids, a.wts, a.sg, a.ld_sg = ids.data_ptr(), wts.data_ptr(), _p(sg), sg.stride(0) if sg is not None else 0
+    a.w1, a.w1s = w_gu.data_ptr(), _p(w_gu_shared)
+    a.E, a.T, a.k, a.K = n_experts, ids.shape[0], ids.shape[1], w_gu.shape[1]
+    a.F, a.Fs = rows.shape[1], rows_shared.shape[1] if rows_shared is not None else 0
+    a.act, a.limit, a.rows, a.rows_s = EPI_OF_ACT[act], limit, rows.data_ptr(), _p(rows_shared)
+    assert w_gu.is_contiguous() and rows.is_contiguous() and w_gu.shape[0] == 2 * n_experts * a.F
+    N.check(N.lib().he_moe_gateup_float(C.byref(a), _stream()), "he_moe_gateup_float")
+
+
+def moe_down_float(rows: torch.Tensor, ids: torch.Tensor, w_down: torch.Tensor, n_experts: int, h: torch.Tensor,
+                   rows_shared: Optional[torch.Tensor] = None, w_down_shared: Optional[torch.Tensor] = None) -> None:
+    """h[t] += sum_j Wd[ids[t, j]] rows[t*k + j] (+ Wd_shared rows_shared[t]); the weights are already in the rows."""
+    _check_abi()
+    a = _FloatMoeArgs()
+    a.ids, a.w1, a.w1s = ids.data_ptr(), w_down.data_ptr(), _p(w_down_shared)
+    a.E, a.T, a.k, a.N = n_experts, ids.shape[0], ids.shape[1], w_down.shape[0] // n_experts
+    a.F, a.Fs = rows.shape[1], rows_shared.shape[1] if rows_shared is not None else 0
+    a.rows, a.rows_s, a.h, a.ldh = rows.data_ptr(), _p(rows_shared), h.data_ptr(), h.stride(0)
+    assert w_down.is_contiguous() and w_down.shape[1] == a.F
+    N.check(N.lib().he_moe_down_float(C.byref(a), _stream()), "he_moe_down_float")
+
+
+# ----------------------------------------------------------------------------- float32 compute dtype
+
+def attn_exact(q: torch.Tensor, kv_cache: torch.Tensor, block_table: torch.Tensor, slot: torch.Tensor,
+               ctx_len: torch.Tensor, out: torch.Tensor, H: int, Hkv: int, D: int, page: int, scale: float,
+               softcap: float = 0.0) -> None:
+    """Causal attention of any rows over fp32 pages, fp32 throughout."""
+    _check_abi()
+    assert q.dtype == kv_cache.dtype == out.dtype == torch.float32
+    a = _ExactAttnArgs()
+    a.q, a.kv_cache, a.block_table = q.data_ptr(), kv_cache.data_ptr(), block_table.data_ptr()
+    a.slot, a.ctx_len, a.out = slot.data_ptr(), ctx_len.data_ptr(), out.data_ptr()
+    a.R, a.H, a.Hkv, a.D, a.page, a.max_pages = q.shape[0], H, Hkv, D, page, block_table.shape[1]
+    a.scale, a.softcap = scale, softcap
+    N.check(N.lib().he_attn_exact(C.byref(a), _stream()), "he_attn_exact")
+
+
+def moe_exact(xn: torch.Tensor, ids: torch.Tensor, wts: torch.Tensor, w_gu: torch.Tensor, w_down: torch.Tensor,
+              n_experts: int, rows: torch.Tensor, h: torch.Tensor, sg: Optional[torch.Tensor] = None,
+              w_gu_shared: Optional[torch.Tensor] = None, w_down_shared: Optional[torch.Tensor] = None,
+              rows_shared: Optional[torch.Tensor] = None) -> None:
+    """Selected SiLU experts (and the shared one) of normalised fp32 rows, added to ``h``; fp32 throughout."""
+    _check_abi()
+    a = _ExactMoeArgs()
+    a.x, a.ldx, a.ids, a.wts = xn.data_ptr(), xn.stride(0), ids.data_ptr(), wts.data_ptr()
+    a.sg, a.ld_sg = _p(sg), sg.stride(0) if sg is not None else 0
+    a.w1, a.w1s = w_gu.data_ptr(), _p(w_gu_shared)
+    a.E, a.T, a.k, a.K, a.N = n_experts, ids.shape[0], ids.shape[1], w_gu.shape[1], w_down.shape[0] // n_experts
+    a.F, a.Fs = rows.shape[1], rows_shared.shape[1] if rows_shared is not None else 0
+    a.rows, a.rows_s, a.h, a.ldh = rows.data_ptr(), _p(rows_shared), h.data_ptr(), h.stride(0)
+    N.check(N.lib().he_moe_gateup_exact(C.byref(a), _stream()), "he_moe_gateup_exact")
+    a.w1, a.w1s = w_down.data_ptr(), _p(w_down_shared)
+    N.check(N.lib().he_moe_down_exact(C.byref(a), _stream()), "he_moe_down_exact")
+
+
+# ----------------------------------------------------------------------------- looped layers, position vectors
+
+def embed_sinusoid(w: "DeviceWeight", ids: torch.Tensor, pos: torch.Tensor, freq: torch.Tensor, out: torch.Tensor,
+                   copy: Optional[torch.Tensor] = None) -> None:
+    """out[t] = table[ids[t]] + sinusoidal position vector of pos[t] (fp32, zero-padded to the row width); ``copy``
+    receives the same rows.  ``freq`` float64 [width / 2]."""
+    _check_device(out)
+    assert ids.dtype == torch.int64 and out.dtype == torch.float32 and out.is_contiguous() and freq.dtype == torch.float64
+    N.check(N.lib().he_embed_sinusoid(c_vp(w.ptr), C.c_int(w.qtype), c_ll(w.n_rows), C.c_int(w.n_cols),
+                                      C.c_int(out.shape[1]), c_vp(ids.data_ptr()), c_vp(pos.data_ptr()),
+                                      c_vp(freq.data_ptr()), c_vp(out.data_ptr()), c_vp(_p(copy)),
+                                      C.c_int(ids.numel()), _stream()), "he_embed_sinusoid")
+
+
+def resid_inject(h: torch.Tensor, x0: Optional[torch.Tensor], step: torch.Tensor) -> None:
+    """h += x0 (when given) + step, before a pass of a looped range."""
+    assert h.dtype == torch.float32 and h.is_contiguous() and step.dtype == torch.float32
+    N.check(N.lib().he_resid_inject(c_vp(h.data_ptr()), c_vp(_p(x0)), c_vp(step.data_ptr()), c_ll(h.shape[0]),
+                                    C.c_int(h.shape[1]), _stream()), "he_resid_inject")
 
 
 # ----------------------------------------------------------------------------- speculative decoding
@@ -714,12 +888,14 @@ def softcap_(x: torch.Tensor, cap: float) -> None:
     N.check(N.lib().he_softcap(c_vp(x.data_ptr()), c_ll(x.numel()), C.c_float(cap), _stream()), "he_softcap")
 
 
-def small_gemm_f32(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor) -> torch.Tensor:
-    """out[T, N] (fp32) = x[T, K] @ w[N, K]^T with fp32 weights (router / ssm_alpha / ssm_beta at prefill)."""
+def small_gemm_f32(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, add: bool = False) -> torch.Tensor:
+    """out[T, N] (fp32) = (or +=) x[T, K] @ w[N, K]^T in fp32 arithmetic; w fp32 (router / ssm_alpha / ssm_beta at
+    prefill) or bf16 (the float32 compute dtype)."""
     T, K = x.shape
     Nn = w.shape[0]
-    assert w.dtype == torch.float32 and out.dtype == torch.float32
+    assert out.dtype == torch.float32 and w.shape[1] == K
     N.check(N.lib().he_small_gemm_f32(c_vp(x.data_ptr()), C.c_int(_dt(x)), c_ll(x.stride(0)), c_vp(w.data_ptr()),
-                                      c_vp(out.data_ptr()), c_ll(out.stride(0)), C.c_int(T), C.c_int(Nn), C.c_int(K),
-                                      _stream()), "he_small_gemm_f32")
+                                      C.c_int(_dt(w)), c_ll(w.stride(0)), c_vp(out.data_ptr()), c_ll(out.stride(0)),
+                                      C.c_int(T), C.c_int(Nn), C.c_int(K), C.c_int(int(add)), _stream()),
+            "he_small_gemm_f32")
     return out

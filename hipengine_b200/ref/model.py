@@ -52,6 +52,10 @@ class RefModel:
             self._gemma = Gemma4Ref(self)
         else:
             self._gemma = None
+        self._listed = None
+        if self.cfg.arch == "sisisun":
+            from .sisisun import SisisunRef
+            self._listed = SisisunRef(weights.metadata["config"], self.w)
 
     # -- helpers
     def W(self, i: int, slot: str) -> torch.Tensor:
@@ -60,8 +64,8 @@ class RefModel:
     def lin(self, x: torch.Tensor, w: torch.Tensor) -> torch.Tensor:
         return x.to(self.dtype) @ w.t()
 
-    def new_state(self) -> RefState:
-        return RefState()
+    def new_state(self):
+        return self._listed.new_state() if self._listed is not None else RefState()
 
     # -- layers
     def full_attention(self, i: int, x: torch.Tensor, st: RefState, pos: torch.Tensor,
@@ -151,6 +155,8 @@ class RefModel:
         """Run ``tokens`` (1-D ids) after the ``st.pos`` tokens already consumed.  Returns post-norm hidden [T, H]."""
         if self._gemma is not None:
             return self._gemma.forward_hidden(tokens, st)
+        if self._listed is not None:
+            return self._listed.forward_hidden(tokens, st)
         cfg = self.cfg
         T = tokens.shape[0]
         pos = torch.arange(st.pos, st.pos + T, device=self.device)
@@ -167,7 +173,9 @@ class RefModel:
         return R.rmsnorm(h, self.w["output_norm.weight"], cfg.rms_eps)
 
     def logits_from_hidden(self, hidden: torch.Tensor) -> torch.Tensor:
-        head = self.w.get("output.weight", self.w["token_embd.weight"])
+        if self._listed is not None:
+            return self._listed.logits(hidden)
+        head = self.w.get("output.weight", self.w.get("token_embd.weight"))
         lg = hidden.to(self.dtype) @ head.t()
         if self.cfg.final_softcap > 0:
             lg = self.cfg.final_softcap * torch.tanh(lg / self.cfg.final_softcap)

@@ -14,7 +14,10 @@ from typing import List, Optional
 
 def build_parser() -> argparse.ArgumentParser:
     ap = argparse.ArgumentParser(prog="hipengine-b200 serve", description="OpenAI-compatible server on sm_100a")
-    ap.add_argument("--model", required=True, help="GGUF file / directory, or a built-in random-init geometry name")
+    ap.add_argument("--model", required=True, help="GGUF file / directory, a folder with config.json and "
+                                                     "model.safetensors, or a built-in random-init geometry name")
+    ap.add_argument("--dtype", default="bfloat16", choices=["bfloat16", "float32"],
+                    help="compute precision (float32: families that declare it)")
     ap.add_argument("--backend", default="auto", choices=["auto", "cuda_sm100a", "cpu_reference"])
     ap.add_argument("--execution-profile", default="production", choices=["strict", "production", "batch_invariant", "fast"])
     ap.add_argument("--served-model-name", default=None)
@@ -55,7 +58,7 @@ def build_parser() -> argparse.ArgumentParser:
     ap.add_argument("--prefix-snapshot-interval", type=int, default=2048)
     ap.add_argument("--prefix-max-snapshots", type=int, default=16)
     ap.add_argument("--prefill-decode-policy", default="protect_decode",
-                    choices=["protect_decode", "protect_ttft", "fair", "token_budget"])
+                    choices=["protect_decode", "protect_ttft", "fair", "token_budget", "mixed"])
     ap.add_argument("--max-prefill-chunk-tokens", type=int, default=4096)
     ap.add_argument("--round-prefill-token-budget", type=int, default=4096)
     ap.add_argument("--round-decode-row-budget", type=int, default=64)
@@ -84,6 +87,7 @@ def configs_from_args(a):
     from .api import ServerConfig
     eng = EngineConfig(
         max_sequence_length=a.max_context_tokens, use_cuda_graphs=not a.no_cuda_graphs,
+        compute_dtype=a.dtype,
         scheduler=SchedulerConfig(policy=a.prefill_decode_policy, max_prefill_chunk_tokens=a.max_prefill_chunk_tokens,
                                   round_prefill_token_budget=a.round_prefill_token_budget,
                                   round_decode_row_budget=a.round_decode_row_budget,
