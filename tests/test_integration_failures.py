@@ -165,7 +165,7 @@ def test_stream_many_interleaves_requests_and_delivers_every_token_once():
         eng.close()
 
 
-@pytest.mark.parametrize("policy", ["protect_decode", "protect_ttft", "fair", "token_budget"])
+@pytest.mark.parametrize("policy", ["protect_decode", "protect_ttft", "fair", "token_budget", "mixed"])
 @pytest.mark.parametrize("prefix,spec_depth", [("radix", 0), ("off", 0), ("radix", 3)])
 def test_churn_of_submits_cancels_and_contained_failures_leaves_the_books_balanced(policy, prefix, spec_depth):
     """Sixty requests with shared prefixes arrive at random, a third are cancelled at random moments (pending, in
