@@ -21,13 +21,15 @@ from ..quant.ggml import GGMLType
 from .gguf import GGUFModelInfo, GGUFReader, discover_gguf_files, scan_gguf
 from .weights import ModelWeights, QTensor, expected_tensor_names
 
-SUPPORTED_ARCHS = ("qwen35", "qwen35moe", "qwen3", "qwen3moe", "llama", "gemma4")
+GGUF_ARCHS = ("qwen35", "qwen35moe", "qwen3", "qwen3moe", "llama", "gemma4")
+FOLDER_ARCHS = ("sisisun",)                  # checkpoint folders (``safetensors_dir.py``)
+SUPPORTED_ARCHS = GGUF_ARCHS + FOLDER_ARCHS
 
 
 def config_from_gguf(info: GGUFModelInfo) -> ModelConfig:
     a = info.architecture
-    if a not in SUPPORTED_ARCHS:
-        raise ValueError(f"unsupported GGUF architecture {a!r}; supported: {SUPPORTED_ARCHS}")
+    if a not in GGUF_ARCHS:
+        raise ValueError(f"unsupported GGUF architecture {a!r}; supported: {GGUF_ARCHS}")
     g = lambda k, d=None: info.metadata.get(f"{a}.{k}", d)
     hidden = int(g("embedding_length"))
     n_heads = int(g("attention.head_count"))
