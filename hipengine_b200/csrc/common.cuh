@@ -134,6 +134,10 @@ __device__ __forceinline__ float gelu_tanh_f(float x) {
   const float k = 0.7978845608028654f;
   return 0.5f * x * (1.f + tanhf(k * (x + 0.044715f * x * x * x)));
 }
+__device__ __forceinline__ float relu2_f(float x) {
+  x = fmaxf(x, 0.f);
+  return x * x;
+}
 // min(g, limit) * sigmoid(1.702 min(g, limit)) * (clamp(u, -limit, limit) + 1)
 __device__ __forceinline__ float clamped_glu_f(float g, float u, float limit) {
   g = fminf(g, limit);

@@ -43,9 +43,9 @@ constexpr int NTHREADS_FUSED_Q = NTHREADS_FUSED + 32 * (1 + N_UNPACK_WARPS);
 struct GemmArgs {
   void* C;
   long long ldc;        // elements
-  const float* resid;   // unused (reserved)
+  const float* col_scale;   // epi 2: factor per output column, or null
   int M, N, K;
-  int epi;              // 0: bf16 store, 1: fp32 store, 2: fp32 += (C is fp32, in place)
+  int epi;              // 0: bf16 store, 1: fp32 store, 2: fp32 += (C is fp32, in place), 6: bf16 store of relu(v)^2
   int* status;
   // grouped mode (MoE experts): M-tile tm multiplies rows [tm*BM, +BM) of A with the weight block
   // B[tile_group[tm] * N .. +N); a negative group marks an unused tile.  Null for a plain GEMM.
@@ -642,7 +642,15 @@ __device__ __forceinline__ void gemm_body(const CUtensorMap& tmA, const CUtensor
         } else
         if (row < g.M && col0 < g.N) {
           const int ncols = min(32, g.N - col0);
-          if (g.epi == 0) {
+          if (g.epi == 6) {
+#pragma unroll
+            for (int e = 0; e < 32; ++e) r[e] = __float_as_uint(he::relu2_f(__uint_as_float(r[e])));
+          } else if (g.epi == 2 && g.col_scale != nullptr) {
+#pragma unroll
+            for (int e = 0; e < 32; ++e)
+              if (e < ncols) r[e] = __float_as_uint(__uint_as_float(r[e]) * __ldg(g.col_scale + col0 + e));
+          }
+          if (g.epi == 0 || g.epi == 6) {
             __nv_bfloat16* dst = reinterpret_cast<__nv_bfloat16*>(g.C) + (size_t)row * g.ldc + col0;
             if (ncols == 32 && ((reinterpret_cast<uintptr_t>(dst) & 15) == 0)) {
 #pragma unroll
@@ -868,19 +876,19 @@ constexpr size_t SMEM_Q = STAGES_Q * STAGE_BYTES + QSTAGES * Q_STAGE_BYTES + siz
 }  // namespace
 
 // C[M][N] = A[M][K] (bf16, row stride lda) * B[N][K]^T (bf16, row stride ldb).
-// epi: 0 bf16 store, 1 fp32 store, 2 fp32 accumulate into C.  `status` (device int, may be null) receives a
-// non-zero code if a bounded wait inside the kernel gave up.
+// epi: 0 bf16 store, 1 fp32 store, 2 fp32 accumulate into C (times col_scale[n] when given), 6 bf16 store of relu(v)^2.
+// `status` (device int, may be null) receives a non-zero code if a bounded wait inside the kernel gave up.
 HE_API int he_gemm_bf16(const void* A, long long lda, const void* B, long long ldb, void* C, long long ldc, int M,
-                        int N, int K, int epi, void* status, int num_sms, cudaStream_t stream) {
+                        int N, int K, int epi, const void* col_scale, void* status, int num_sms, cudaStream_t stream) {
   if (M <= 0 || N <= 0 || K <= 0) return 0;
-  if (K % 8 != 0) return -HE_ERR_BAD_ARG;
+  if (K % 8 != 0 || !(epi == 0 || epi == 1 || epi == 2 || epi == 6)) return -HE_ERR_BAD_ARG;
   CUtensorMap tmA, tmB;
   int rc = make_map(&tmA, A, M, K, lda, BM);
   if (rc != 0) return rc;
   rc = make_map(&tmB, B, N, K, ldb, BN);
   if (rc != 0) return rc;
   GemmArgs g = {};
-  g.C = C; g.ldc = ldc; g.resid = nullptr; g.M = M; g.N = N; g.K = K; g.epi = epi; g.status = (int*)status;
+  g.C = C; g.ldc = ldc; g.col_scale = (const float*)col_scale; g.M = M; g.N = N; g.K = K; g.epi = epi; g.status = (int*)status;
   g.tile_group = nullptr;
   g.k_splits = 1;
   g.split_stride = 0;
@@ -924,7 +932,7 @@ HE_API int he_gemm_bf16_allreduce(const void* A, long long lda, const void* B, l
   rc = make_map(&tmB, B, N, K, ldb, BN);
   if (rc != 0) return rc;
   GemmArgs g = {};
-  g.C = nullptr; g.ldc = 0; g.resid = nullptr; g.M = M; g.N = N; g.K = K; g.epi = 5; g.status = (int*)status;
+  g.C = nullptr; g.ldc = 0; g.col_scale = nullptr; g.M = M; g.N = N; g.K = K; g.epi = 5; g.status = (int*)status;
   g.tile_group = nullptr;
   g.k_splits = 1;
   g.split_stride = 0;
@@ -955,7 +963,7 @@ HE_API int he_gemm_bf16_grouped(const void* A, long long lda, const void* B, lon
   rc = make_map(&tmB, B, (long long)n_groups * N, K, ldb, BN);
   if (rc != 0) return rc;
   GemmArgs g = {};
-  g.C = C; g.ldc = ldc; g.resid = nullptr; g.M = M; g.N = N; g.K = K; g.epi = epi; g.status = (int*)status;
+  g.C = C; g.ldc = ldc; g.col_scale = nullptr; g.M = M; g.N = N; g.K = K; g.epi = epi; g.status = (int*)status;
   g.tile_group = tile_group;
   g.k_splits = 1;
   g.split_stride = 0;
@@ -976,9 +984,11 @@ HE_API int he_gemm_bf16_grouped(const void* A, long long lda, const void* B, lon
 // the weight instead of one CTA per 256 output columns.  C must already hold the value to add to (e.g. the
 // residual stream).  k_splits <= 0 picks a split that gives about one tile per SM.
 namespace {
-// out[m][n] (+)= sum over splits, in split order (deterministic).  mode 0: fp32 store, 1: fp32 add in place.
+// out[m][n] (+)= sum over splits, in split order (deterministic).  mode 0: fp32 store, 1: fp32 add in place (of the sum
+// times col_scale[n] when given), 2: bf16 store of relu(sum)^2.
 __global__ void splitk_reduce_kernel(const float* __restrict__ part, long long split_stride, int k_splits,
-                                     float* __restrict__ out, long long ldo, int M, int N, int mode) {
+                                     void* __restrict__ out_v, long long ldo, int M, int N, int mode,
+                                     const float* __restrict__ col_scale) {
   const long long i = ((long long)blockIdx.x * blockDim.x + threadIdx.x) * 4;
   if (i >= (long long)M * N) return;
   const int m = (int)(i / N), n = (int)(i % N);
@@ -987,8 +997,19 @@ __global__ void splitk_reduce_kernel(const float* __restrict__ part, long long s
     const float4 v = *reinterpret_cast<const float4*>(part + (size_t)k * split_stride + (size_t)m * N + n);
     s.x += v.x; s.y += v.y; s.z += v.z; s.w += v.w;
   }
-  float4* o = reinterpret_cast<float4*>(out + (size_t)m * ldo + n);
+  if (mode == 2) {
+    __align__(8) __nv_bfloat162 b[2] = {__floats2bfloat162_rn(he::relu2_f(s.x), he::relu2_f(s.y)),
+                                        __floats2bfloat162_rn(he::relu2_f(s.z), he::relu2_f(s.w))};
+    *reinterpret_cast<uint2*>(reinterpret_cast<__nv_bfloat16*>(out_v) + (size_t)m * ldo + n) =
+        *reinterpret_cast<const uint2*>(b);
+    return;
+  }
+  float4* o = reinterpret_cast<float4*>(reinterpret_cast<float*>(out_v) + (size_t)m * ldo + n);
   if (mode == 1) {
+    if (col_scale != nullptr) {
+      const float4 c = *reinterpret_cast<const float4*>(col_scale + n);
+      s.x *= c.x; s.y *= c.y; s.z *= c.z; s.w *= c.w;
+    }
     const float4 h = *o;
     s.x += h.x; s.y += h.y; s.z += h.z; s.w += h.w;
   }
@@ -998,7 +1019,8 @@ __global__ void splitk_reduce_kernel(const float* __restrict__ part, long long s
 
 // Deterministic split-K: partial tiles go to `partials` ([k_splits][M][N] fp32, caller scratch of at least
 // he_gemm_splitk_scratch_floats(M, N, K) floats), then one pass sums them in split order into `out`
-// (mode 0: store, 1: add in place -- the residual add).  Same use as he_gemm_bf16_splitk, bit-reproducible.
+// (mode 0: store, 1: add in place -- the residual add, with an optional factor per column --, 2: bf16 squared ReLU).  Same
+// use as he_gemm_bf16_splitk, bit-reproducible.
 HE_API long long he_gemm_splitk_plan(int M, int N, int K, int num_sms) {
   const int tiles = ((M + BM - 1) / BM) * ((N + BN - 1) / BN);
   const int k_blocks = (K + BK - 1) / BK;
@@ -1010,10 +1032,10 @@ HE_API long long he_gemm_splitk_plan(int M, int N, int K, int num_sms) {
 }
 
 HE_API int he_gemm_bf16_splitk_det(const void* A, long long lda, const void* B, long long ldb, void* partials,
-                                   void* out, long long ldo, int M, int N, int K, int mode, void* status,
-                                   int num_sms, cudaStream_t stream) {
+                                   void* out, long long ldo, int M, int N, int K, int mode, const void* col_scale,
+                                   void* status, int num_sms, cudaStream_t stream) {
   if (M <= 0 || N <= 0 || K <= 0) return 0;
-  if (K % 8 != 0 || N % 4 != 0) return -HE_ERR_BAD_ARG;
+  if (K % 8 != 0 || N % 4 != 0 || mode < 0 || mode > 2) return -HE_ERR_BAD_ARG;
   CUtensorMap tmA, tmB;
   int rc = make_map(&tmA, A, M, K, lda, BM);
   if (rc != 0) return rc;
@@ -1021,7 +1043,7 @@ HE_API int he_gemm_bf16_splitk_det(const void* A, long long lda, const void* B, 
   if (rc != 0) return rc;
   const int k_splits = (int)he_gemm_splitk_plan(M, N, K, num_sms);
   GemmArgs g = {};
-  g.C = partials; g.ldc = N; g.resid = nullptr; g.M = M; g.N = N; g.K = K; g.epi = 4; g.status = (int*)status;
+  g.C = partials; g.ldc = N; g.col_scale = nullptr; g.M = M; g.N = N; g.K = K; g.epi = 4; g.status = (int*)status;
   g.tile_group = nullptr;
   g.k_splits = k_splits;
   g.split_stride = (long long)M * N;
@@ -1034,7 +1056,8 @@ HE_API int he_gemm_bf16_splitk_det(const void* A, long long lda, const void* B, 
   HE_LAUNCH_CHECK();
   const long long n4 = ((long long)M * N + 3) / 4;
   splitk_reduce_kernel<<<(unsigned)((n4 + 255) / 256), 256, 0, stream>>>((const float*)partials, g.split_stride,
-                                                                        k_splits, (float*)out, ldo, M, N, mode);
+                                                                        k_splits, out, ldo, M, N, mode,
+                                                                        (const float*)col_scale);
   HE_LAUNCH_CHECK();
   return 0;
 }
@@ -1056,7 +1079,7 @@ HE_API int he_gemm_bf16_splitk(const void* A, long long lda, const void* B, long
   const int kb_per = (k_blocks + k_splits - 1) / k_splits;
   k_splits = (k_blocks + kb_per - 1) / kb_per;            // no empty split
   GemmArgs g = {};
-  g.C = C; g.ldc = ldc; g.resid = nullptr; g.M = M; g.N = N; g.K = K; g.epi = 3; g.status = (int*)status;
+  g.C = C; g.ldc = ldc; g.col_scale = nullptr; g.M = M; g.N = N; g.K = K; g.epi = 3; g.status = (int*)status;
   g.tile_group = nullptr;
   g.k_splits = k_splits;
   g.split_stride = 0;
@@ -1093,7 +1116,7 @@ HE_API int he_gemm_q_allreduce(const void* A, long long lda, const void* B, int 
   rc = make_qmaps(&q, B, qtype, b_rows, K);
   if (rc != 0) return rc;
   GemmArgs g = {};
-  g.C = nullptr; g.ldc = 0; g.resid = nullptr; g.M = M; g.N = N; g.K = K; g.epi = 5; g.status = (int*)status;
+  g.C = nullptr; g.ldc = 0; g.col_scale = nullptr; g.M = M; g.N = N; g.K = K; g.epi = 5; g.status = (int*)status;
   g.tile_group = nullptr;
   g.k_splits = 1;
   g.split_stride = 0;

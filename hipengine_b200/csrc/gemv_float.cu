@@ -8,7 +8,10 @@
 // requested before the kernel waits for its predecessor.
 //   norm      : RMS norm needs no separate pass: sum over k of w[k] (x[k] g[k]) is scaled by 1/rms(x) at the end, and
 //               every warp accumulates the squares of the columns it reads anyway (fp32)
-//   epilogue  : fp32 / bf16 store, fp32 residual add, or act(gate) * up (SiLU, tanh-GELU, clamped GLU)
+//   epilogue  : fp32 / bf16 store, fp32 residual add, squared ReLU, or act(gate) * up (SiLU, tanh-GELU, clamped GLU)
+//   batches   : grid.y repeats the product with other weights and rows (one small matrix per attention head)
+//   sums      : the two output projections of a layer whose sublayers run side by side are one launch: each has its own
+//               rows and columns, both accumulators get their per-column factors and meet in the residual add
 // The expert forms add an indirection: grid.y is a (token, expert) pair or a token, the weight base comes from the
 // routed expert id, and the down projection walks the concatenated columns of all selected experts (and the shared
 // one), which adds the k expert outputs in a fixed order inside the accumulator.
@@ -20,9 +23,10 @@ struct FloatGemvSeg {
   const __nv_bfloat16* w;
   const __nv_bfloat16* w2;   // gate/up pair: the up rows
   void* out;
+  const void* x;             // activation rows of this segment (same type and stride as FloatGemvArgs::x); null: those
   long long out_stride;
   int n_rows;
-  int epi;                   // 0 f32, 1 bf16, 2 f32 +=, 3 silu(g)*u, 4 gelu_tanh(g)*u, 5 clamped GLU (all bf16)
+  int epi;                   // 0 f32, 1 bf16, 2 f32 +=, 3 silu(g)*u, 4 gelu_tanh(g)*u, 5 clamped GLU, 6 relu(v)^2 (3..6 bf16)
 };
 
 struct FloatGemvArgs {
@@ -38,6 +42,19 @@ struct FloatGemvArgs {
   float eps;
   int norm_n;                // columns the mean square is taken over (zero-padded rows are wider)
   float limit;               // epi 5
+  int n_batch;               // grid.y; every pointer advances by its stride (elements) per batch
+  long long w_bs, x_bs, out_bs;
+};
+
+struct FloatSumArgs {        // out[r][n] += sum over i of scale_i[n] * (x_i[r] . w_i[n]),  bf16 rows and weights
+  const __nv_bfloat16* w[2];
+  const __nv_bfloat16* x[2];
+  const float* scale[2];     // null: 1
+  long long ldw[2], x_stride[2];
+  int K[2];                  // multiples of 8; K[1] = 0: one product
+  float* out;
+  long long out_stride;
+  int n_rows, R;
 };
 
 struct FloatMoeArgs {
@@ -208,16 +225,21 @@ __global__ void __launch_bounds__(NW * 32, 2) gemv_float_kernel(const __grid_con
   }
   const FloatGemvSeg& sg = a.seg[si];
   const int row0 = item * 16;
+  const size_t bt = blockIdx.y;
+  const size_t x_off = bt * a.x_bs, o_off = bt * a.out_bs;
+  const void* xs = sg.x != nullptr ? sg.x : a.x;
+  xs = XF32 ? (const void*)(reinterpret_cast<const float*>(xs) + x_off)
+            : (const void*)(reinterpret_cast<const __nv_bfloat16*>(xs) + x_off);
   const __nv_bfloat16* wrow[MT][2];
 #pragma unroll
   for (int hf = 0; hf < 2; ++hf) {
-    const size_t off = (size_t)min(row0 + g + 8 * hf, sg.n_rows - 1) * a.ldw + 8 * c;
+    const size_t off = bt * a.w_bs + (size_t)min(row0 + g + 8 * hf, sg.n_rows - 1) * a.ldw + 8 * c;
     wrow[0][hf] = sg.w + off;
     if constexpr (MT == 2) wrow[1][hf] = sg.w2 + off;
   }
   float acc[MT][NT][4] = {};
   float ss[NT] = {};
-  product<MT, NT, XF32, true>(wrow, a.K, a.x, a.x_stride, a.R, a.norm_w, acc, ss);
+  product<MT, NT, XF32, true>(wrow, a.K, xs, a.x_stride, a.R, a.norm_w, acc, ss);
   store_partials<MT, NT>(sm, acc, ss);
   __syncthreads();
   for (int o = threadIdx.x; o < 16 * NT * 8; o += NW * 32) {
@@ -225,17 +247,57 @@ __global__ void __launch_bounds__(NW * 32, 2) gemv_float_kernel(const __grid_con
     if (col >= a.R || n >= sg.n_rows) continue;
     const float inv = a.norm_w != nullptr ? inv_rms_of<MT, NT>(sm, col, a.norm_n, a.eps) : 1.f;
     const float v = sum_partials<MT, NT>(sm, row, col) * inv;
-    const size_t off = (size_t)col * sg.out_stride + n;
+    const size_t off = o_off + (size_t)col * sg.out_stride + n;
     if constexpr (MT == 2) {
       const float u = sum_partials<MT, NT>(sm, 16 + row, col) * inv;
       reinterpret_cast<__nv_bfloat16*>(sg.out)[off] = f32_to_bf16(glu_f(v, u, sg.epi, a.limit));
     } else if (sg.epi == 0) {
       reinterpret_cast<float*>(sg.out)[off] = v;
-    } else if (sg.epi == 1) {
-      reinterpret_cast<__nv_bfloat16*>(sg.out)[off] = f32_to_bf16(v);
+    } else if (sg.epi == 1 || sg.epi == 6) {
+      reinterpret_cast<__nv_bfloat16*>(sg.out)[off] = f32_to_bf16(sg.epi == 6 ? relu2_f(v) : v);
     } else {
       reinterpret_cast<float*>(sg.out)[off] += v;
     }
+  }
+}
+
+// grid: items of 16 output columns
+template <int NT>
+__global__ void __launch_bounds__(NW * 32, 2) gemv_sum_kernel(const __grid_constant__ FloatSumArgs a) {
+  __shared__ Tile<1, NT> sm;
+  pdl_launch();
+  const int lane = threadIdx.x & 31, g = lane >> 2, c = lane & 3;
+  const int row0 = blockIdx.x * 16;
+  const int ra = min(row0 + g, a.n_rows - 1), rb = min(row0 + g + 8, a.n_rows - 1);
+  const __nv_bfloat16* wrow[1][2] = {{a.w[0] + (size_t)ra * a.ldw[0] + 8 * c, a.w[0] + (size_t)rb * a.ldw[0] + 8 * c}};
+  float acc[1][NT][4] = {};
+  float ss[NT] = {};
+  product<1, NT, false, true>(wrow, a.K[0], a.x[0], a.x_stride[0], a.R, nullptr, acc, ss);
+  if (a.scale[0] != nullptr) {
+    const float sa = a.scale[0][ra], sb = a.scale[0][rb];
+#pragma unroll
+    for (int n = 0; n < NT; ++n) {
+      acc[0][n][0] *= sa; acc[0][n][1] *= sa;
+      acc[0][n][2] *= sb; acc[0][n][3] *= sb;
+    }
+  }
+  if (a.K[1] > 0) {
+    wrow[0][0] = a.w[1] + (size_t)ra * a.ldw[1] + 8 * c;
+    wrow[0][1] = a.w[1] + (size_t)rb * a.ldw[1] + 8 * c;
+    float acc2[1][NT][4] = {};
+    product<1, NT, false, false>(wrow, a.K[1], a.x[1], a.x_stride[1], a.R, nullptr, acc2, ss);
+    const float sa = a.scale[1] != nullptr ? a.scale[1][ra] : 1.f, sb = a.scale[1] != nullptr ? a.scale[1][rb] : 1.f;
+#pragma unroll
+    for (int n = 0; n < NT; ++n) {
+      acc[0][n][0] += sa * acc2[0][n][0]; acc[0][n][1] += sa * acc2[0][n][1];
+      acc[0][n][2] += sb * acc2[0][n][2]; acc[0][n][3] += sb * acc2[0][n][3];
+    }
+  }
+  store_partials<1, NT>(sm, acc, ss);
+  __syncthreads();
+  for (int o = threadIdx.x; o < 16 * NT * 8; o += NW * 32) {
+    const int row = o & 15, col = o >> 4, n = row0 + row;
+    if (col < a.R && n < a.n_rows) a.out[(size_t)col * a.out_stride + n] += sum_partials<1, NT>(sm, row, col);
   }
 }
 
@@ -335,7 +397,7 @@ __global__ void __launch_bounds__(NW * 32, 2) moe_down_float_kernel(const __grid
 template <int MT>
 int launch_rows(const FloatGemvArgs& a, int items, cudaStream_t stream) {
   cudaError_t e;
-  const dim3 grid(items), block(NW * 32);
+  const dim3 grid(items, a.n_batch > 1 ? a.n_batch : 1), block(NW * 32);
   if (a.x_dtype == 0) {
     e = a.R <= 8 ? launch_pdl(gemv_float_kernel<MT, 1, true>, grid, block, 0, stream, a)
                  : launch_pdl(gemv_float_kernel<MT, 2, true>, grid, block, 0, stream, a);
@@ -349,16 +411,18 @@ int launch_rows(const FloatGemvArgs& a, int items, cudaStream_t stream) {
 }  // namespace
 
 // Rows of x (fp32 with an optional fused RMS norm, or bf16) times up to four bf16 weight segments of the same width.
-// All segments of a launch are plain (epi 0..2) or all are gate/up pairs (epi 3..5).
+// All segments of a launch are plain (epi 0..2, 6) or all are gate/up pairs (epi 3..5).
 HE_API int he_gemv_float(const FloatGemvArgs* args, cudaStream_t stream) {
   const FloatGemvArgs& a = *args;
   if (a.R < 1 || a.R > 16 || a.n_seg < 1 || a.n_seg > 4 || a.K <= 0 || a.K % 8 != 0 || a.ldw % 8 != 0 || a.ldw < a.K)
     return -HE_ERR_BAD_ARG;
   if (a.x_stride % 8 != 0 || (a.norm_w != nullptr && (a.x_dtype != 0 || a.norm_n <= 0))) return -HE_ERR_BAD_ARG;
-  const bool pair = a.seg[0].epi >= 3;
+  const auto is_pair = [](int epi) { return epi >= 3 && epi <= 5; };
+  const bool pair = is_pair(a.seg[0].epi);
+  if (a.n_batch > 65535 || a.w_bs % 8 != 0 || a.x_bs % 8 != 0) return -HE_ERR_BAD_ARG;
   int items = 0;
   for (int i = 0; i < a.n_seg; ++i) {
-    if ((a.seg[i].epi >= 3) != pair || a.seg[i].epi < 0 || a.seg[i].epi > 5 || a.seg[i].n_rows <= 0 ||
+    if (is_pair(a.seg[i].epi) != pair || a.seg[i].epi < 0 || a.seg[i].epi > 6 || a.seg[i].n_rows <= 0 ||
         (pair && a.seg[i].w2 == nullptr))
       return -HE_ERR_BAD_ARG;
     items += (a.seg[i].n_rows + 15) / 16;
@@ -366,6 +430,17 @@ HE_API int he_gemv_float(const FloatGemvArgs* args, cudaStream_t stream) {
   return pair ? launch_rows<2>(a, items, stream) : launch_rows<1>(a, items, stream);
 }
 HE_API int he_gemv_float_args_size() { return (int)sizeof(FloatGemvArgs); }
+
+HE_API int he_gemv_sum(const FloatSumArgs* args, cudaStream_t stream) {
+  const FloatSumArgs& a = *args;
+  if (a.R < 1 || a.R > 16 || a.n_rows <= 0 || a.K[0] <= 0 || a.K[1] < 0) return -HE_ERR_BAD_ARG;
+  for (int i = 0; i < (a.K[1] > 0 ? 2 : 1); ++i)
+    if (a.K[i] % 8 != 0 || a.ldw[i] % 8 != 0 || a.ldw[i] < a.K[i] || a.x_stride[i] % 8 != 0) return -HE_ERR_BAD_ARG;
+  const dim3 grid((a.n_rows + 15) / 16), block(NW * 32);
+  return (int)(a.R <= 8 ? launch_pdl(gemv_sum_kernel<1>, grid, block, 0, stream, a)
+                        : launch_pdl(gemv_sum_kernel<2>, grid, block, 0, stream, a));
+}
+HE_API int he_gemv_sum_args_size() { return (int)sizeof(FloatSumArgs); }
 
 static int check_moe(const FloatMoeArgs& a) {
   if (a.k <= 0 || a.k > 32 || a.E < a.k || a.F <= 0 || a.F % 8 != 0 || (a.w1s != nullptr && (a.Fs <= 0 || a.Fs % 8 != 0)))

@@ -45,6 +45,80 @@ __global__ void __launch_bounds__(256) rmsnorm_rows_kernel(const float* __restri
   }
 }
 
+// ---------------------------------------------------------------- RMSNorm rows + token shift
+// h[t] = norm(x[t]) and hs[t] = h[t] + shift * (h[t-1] - h[t]) for packed segments; the row before a segment's first one is
+// the slot's state (zeros for a new request).  The CTA of that first row also replaces the state with the segment's last
+// normalised row (recomputed here), so the only reader and the only writer of a state row are the same threads.  With a
+// journal (verify chains) the state stays and every row's h is recorded instead.
+struct NormShiftArgs {
+  const float* x;            // [T][ldx] residual rows
+  long long ldx;
+  const float* w;            // [H] norm gains (zero in padded columns)
+  const float* shift;        // [H]
+  float* state;              // [n_slots][H]
+  float* journal;            // [T][H] or null
+  const int* seg_start;      // [n_seg + 1]
+  const int* seg_slot;       // [n_seg]
+  const int* tok_seg;        // [T]
+  void* h;                   // [T][H] bf16 or fp32
+  void* hs;
+  int T, H, n_mean, out_bf16, n_slots;
+  float eps;
+};
+
+template <typename OutT>
+__device__ __forceinline__ void store4(OutT* p, float4 v) {
+  if constexpr (sizeof(OutT) == 2) {
+    __align__(8) __nv_bfloat162 b[2] = {__floats2bfloat162_rn(v.x, v.y), __floats2bfloat162_rn(v.z, v.w)};
+    *reinterpret_cast<uint2*>(p) = *reinterpret_cast<const uint2*>(b);
+  } else {
+    *reinterpret_cast<float4*>(p) = v;
+  }
+}
+__device__ __forceinline__ float sq4(float4 v) { return v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w; }
+__device__ __forceinline__ float4 mul4(float4 v, float4 g, float s) {
+  return make_float4(v.x * s * g.x, v.y * s * g.y, v.z * s * g.z, v.w * s * g.w);
+}
+
+template <typename OutT>
+__global__ void __launch_bounds__(256) norm_shift_kernel(const NormShiftArgs a) {
+  pdl_wait();
+  pdl_launch();
+  __shared__ float red[33];
+  const int t = blockIdx.x, seg = a.tok_seg[t], first = a.seg_start[seg], last = a.seg_start[seg + 1] - 1;
+  const int slot = a.seg_slot[seg];
+  if (!HE_INDEX_OK(slot, a.n_slots, HE_SITE_STATE_SLOT)) return;
+  const bool head = t == first, upd = head && a.journal == nullptr;
+  const float* xt = a.x + (size_t)t * a.ldx;
+  const float* xp = head ? xt : xt - a.ldx;
+  const float* xl = a.x + (size_t)last * a.ldx;
+  float st = 0.f, sp = 0.f, sl = 0.f;
+  for (int i = threadIdx.x * 4; i < a.H; i += 1024) {
+    st += sq4(*reinterpret_cast<const float4*>(xt + i));
+    if (!head) sp += sq4(*reinterpret_cast<const float4*>(xp + i));
+    if (upd && last != t) sl += sq4(*reinterpret_cast<const float4*>(xl + i));
+  }
+  const float n = (float)a.n_mean;
+  const float it = rsqrtf(block_sum(st, red) / n + a.eps);
+  float ip = 0.f, il = it;                   // conditions are uniform over the CTA
+  if (!head) ip = rsqrtf(block_sum(sp, red) / n + a.eps);
+  if (upd && last != t) il = rsqrtf(block_sum(sl, red) / n + a.eps);
+  float* state = a.state + (size_t)slot * a.H;
+  OutT* ho = reinterpret_cast<OutT*>(a.h) + (size_t)t * a.H;
+  OutT* so = reinterpret_cast<OutT*>(a.hs) + (size_t)t * a.H;
+  for (int i = threadIdx.x * 4; i < a.H; i += 1024) {
+    const float4 g = *reinterpret_cast<const float4*>(a.w + i), s = *reinterpret_cast<const float4*>(a.shift + i);
+    const float4 h = mul4(*reinterpret_cast<const float4*>(xt + i), g, it);
+    const float4 p = head ? *reinterpret_cast<const float4*>(state + i)
+                          : mul4(*reinterpret_cast<const float4*>(xp + i), g, ip);
+    store4(ho + i, h);
+    store4(so + i, make_float4(h.x + (p.x - h.x) * s.x, h.y + (p.y - h.y) * s.y, h.z + (p.z - h.z) * s.z,
+                               h.w + (p.w - h.w) * s.w));
+    if (upd) *reinterpret_cast<float4*>(state + i) = mul4(*reinterpret_cast<const float4*>(xl + i), g, il);
+    if (a.journal != nullptr) *reinterpret_cast<float4*>(a.journal + (size_t)t * a.H + i) = h;
+  }
+}
+
 // act codes: 0 silu(g) * u, 1 gelu_tanh(g) * u, 2 clamped GLU with `limit`
 __device__ __forceinline__ float act_pair(float g, float u, int act, float limit) {
   if (act == 2) return clamped_glu_f(g, u, limit);
@@ -338,6 +412,15 @@ HE_API int he_rmsnorm_rows(const void* x, const void* w, void* out, int out_bf16
   return 0;
 }
 
+HE_API int he_norm_shift(const NormShiftArgs* args, cudaStream_t stream) {
+  const NormShiftArgs& a = *args;
+  if (a.T <= 0) return 0;
+  if (a.H % 4 != 0 || a.ldx % 4 != 0 || a.n_mean <= 0 || a.n_mean > a.H) return -HE_ERR_BAD_ARG;
+  return (int)(a.out_bf16 ? launch_pdl(norm_shift_kernel<__nv_bfloat16>, dim3(a.T), dim3(256), 0, stream, a)
+                          : launch_pdl(norm_shift_kernel<float>, dim3(a.T), dim3(256), 0, stream, a));
+}
+HE_API int he_norm_shift_args_size() { return (int)sizeof(NormShiftArgs); }
+
 HE_API int he_act_mul(const void* gu, void* out, long long T, int F, int act, float limit, cudaStream_t stream) {
   if (T <= 0) return 0;
   if (F % 8 != 0) return -HE_ERR_BAD_ARG;
@@ -531,29 +614,35 @@ HE_API int he_advance_positions(void* pos, void* ctx_len, const void* active, in
 }
 
 // ---------------------------------------------------------------- skinny fp32 GEMM: out[T][N] = x[T][K] * W[N][K]^T
-// For the few projections whose weights stay F32 in GGUF files (router, ssm_alpha/beta) at prefill row counts.
+// For the few projections whose weights stay F32 in GGUF files (router, ssm_alpha/beta) at prefill row counts, and every
+// projection of the float32 compute dtype.  grid.z repeats the product at the batch strides (one matrix per head).
+// mode 0: store, 1: add (times col_scale[n] when given), 2: store relu(v)^2.
 namespace {
 constexpr int SG_TM = 64, SG_TN = 64, SG_TK = 16;
 __global__ void __launch_bounds__(256) small_gemm_f32_kernel(const void* __restrict__ x, int x_dtype,
                                                              long long x_stride, const void* __restrict__ w,
                                                              int w_dtype, long long w_stride,
                                                              float* __restrict__ out, long long out_stride, int T,
-                                                             int N, int K, int accumulate) {
+                                                             int N, int K, int mode,
+                                                             const float* __restrict__ col_scale, long long x_bs,
+                                                             long long w_bs, long long out_bs) {
   __shared__ float xs[SG_TK][SG_TM + 1];
   __shared__ float ws[SG_TK][SG_TN + 1];
   const int t0 = blockIdx.y * SG_TM, n0 = blockIdx.x * SG_TN;
+  const size_t x0 = (size_t)blockIdx.z * x_bs, w0 = (size_t)blockIdx.z * w_bs;
+  out += (size_t)blockIdx.z * out_bs;
   const int tx = threadIdx.x % 16, ty = threadIdx.x / 16;  // 16 x 16 threads, 4x4 outputs each
   float acc[4][4] = {};
   for (int k0 = 0; k0 < K; k0 += SG_TK) {
     for (int i = threadIdx.x; i < SG_TM * SG_TK; i += 256) {
       const int r = i / SG_TK, kk = i % SG_TK;
       const int t = t0 + r, k = k0 + kk;
-      xs[kk][r] = (t < T && k < K) ? load_in(x, x_dtype, (size_t)t * x_stride + k) : 0.f;
+      xs[kk][r] = (t < T && k < K) ? load_in(x, x_dtype, x0 + (size_t)t * x_stride + k) : 0.f;
     }
     for (int i = threadIdx.x; i < SG_TN * SG_TK; i += 256) {
       const int r = i / SG_TK, kk = i % SG_TK;
       const int n = n0 + r, k = k0 + kk;
-      ws[kk][r] = (n < N && k < K) ? load_in(w, w_dtype, (size_t)n * w_stride + k) : 0.f;
+      ws[kk][r] = (n < N && k < K) ? load_in(w, w_dtype, w0 + (size_t)n * w_stride + k) : 0.f;
     }
     __syncthreads();
 #pragma unroll
@@ -575,19 +664,22 @@ __global__ void __launch_bounds__(256) small_gemm_f32_kernel(const void* __restr
       const int t = t0 + ty * 4 + i, n = n0 + tx * 4 + j;
       if (t < T && n < N) {
         float* o = out + (size_t)t * out_stride + n;
-        *o = accumulate ? *o + acc[i][j] : acc[i][j];
+        const float v = acc[i][j];
+        *o = mode == 1 ? *o + (col_scale != nullptr ? v * col_scale[n] : v) : mode == 2 ? relu2_f(v) : v;
       }
     }
 }
 }  // namespace
 
 HE_API int he_small_gemm_f32(const void* x, int x_dtype, long long x_stride, const void* w, int w_dtype,
-                             long long w_stride, void* out, long long out_stride, int T, int N, int K, int accumulate,
+                             long long w_stride, void* out, long long out_stride, int T, int N, int K, int mode,
+                             const void* col_scale, int n_batch, long long x_bs, long long w_bs, long long out_bs,
                              cudaStream_t stream) {
   if (T <= 0 || N <= 0) return 0;
-  dim3 grid((N + SG_TN - 1) / SG_TN, (T + SG_TM - 1) / SG_TM);
+  if (mode < 0 || mode > 2 || n_batch < 1 || n_batch > 65535) return -HE_ERR_BAD_ARG;
+  dim3 grid((N + SG_TN - 1) / SG_TN, (T + SG_TM - 1) / SG_TM, n_batch);
   small_gemm_f32_kernel<<<grid, 256, 0, stream>>>(x, x_dtype, x_stride, w, w_dtype, w_stride, (float*)out, out_stride, T,
-                                                  N, K, accumulate);
+                                                  N, K, mode, (const float*)col_scale, x_bs, w_bs, out_bs);
   HE_LAUNCH_CHECK();
   return 0;
 }

@@ -135,15 +135,15 @@ __global__ void dequant_bf16_kernel(const uint8_t* __restrict__ w, __nv_bfloat16
 }
 
 __global__ void embed_kernel(const uint8_t* __restrict__ w, int qtype, long long vocab, int K,
-                             const int64_t* __restrict__ ids, float* __restrict__ out, float scale, int n_tok) {
+                             const int64_t* __restrict__ ids, float* __restrict__ out, float scale, int n_tok, int ld) {
   pdl_wait();      // launched with programmatic stream serialization: order after all earlier kernels
   pdl_launch();
   const int t = blockIdx.x;
   if (t >= n_tok) return;
   long long id = ids[t];
   if (!HE_INDEX_OK(id, vocab, HE_SITE_EMBED_TOKEN) || id < 0 || id >= vocab) id = 0;
-  for (int e = threadIdx.x; e < K; e += blockDim.x)
-    out[(size_t)t * K + e] = dequant_elem(w, qtype, id, K, e) * scale;
+  for (int e = threadIdx.x; e < ld; e += blockDim.x)
+    out[(size_t)t * ld + e] = e < K ? dequant_elem(w, qtype, id, K, e) * scale : 0.f;
 }
 
 // Embedding row + sinusoidal position vector, written twice: the residual and the copy that looped layers add again.
@@ -202,12 +202,13 @@ HE_API int he_dequant_bf16(const void* w, void* out, int qtype, long long row0, 
   return 0;
 }
 
-// out[t][:] = dequant(table[ids[t]]) * scale   (fp32 residual stream rows)
+// out[t][:] = dequant(table[ids[t]]) * scale   (fp32 residual stream rows of `ld` >= K columns, zeros past K)
 HE_API int he_embed(const void* w, int qtype, long long vocab, int K, const void* ids, void* out, float scale,
-                    int n_tok, cudaStream_t stream) {
+                    int n_tok, int ld, cudaStream_t stream) {
   if (n_tok <= 0) return 0;
+  if (ld < K) return -HE_ERR_BAD_ARG;
   (void)launch_pdl(embed_kernel, dim3(n_tok), dim3(256), 0, stream, (const uint8_t*)w, qtype, vocab, K, (const int64_t*)ids, (float*)out, scale,
-                                          n_tok);
+                                          n_tok, ld);
   HE_LAUNCH_CHECK();
   return 0;
 }

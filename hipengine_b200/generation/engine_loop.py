@@ -71,7 +71,8 @@ class EngineLoop:
         has_prefill = bool(self.sched.prefill_rows())
         has_decode = bool(self.sched.decode_rows())
         done = 0
-        if sc.policy == "mixed" and has_prefill and has_decode and not self._speculating():
+        if (sc.policy == "mixed" and has_prefill and has_decode and not self._speculating()
+                and self.runner.packs_mixed()):
             done += self._run_mixed(sc.max_prefill_chunk_tokens)
         elif sc.policy == "token_budget":
             if has_decode:
@@ -89,7 +90,7 @@ class EngineLoop:
                 done += self._run_prefill(sc.max_prefill_chunk_tokens * sc.fair_prefill_burst_chunks, round_robin=True)
             elif has_decode:
                 done += self._run_decode()
-        else:  # protect_decode: resident rows never wait behind more than one prefill chunk
+        else:  # protect_decode (and mixed where it cannot pack): resident rows wait behind one prefill chunk at most
             if has_decode:
                 done += self._run_decode()
             if has_prefill:

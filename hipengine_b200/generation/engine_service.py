@@ -500,7 +500,7 @@ def build_engine(weights, backend: str, config: EngineConfig, tokenizer=None) ->
             raise RuntimeError(f"tensor/expert parallel size {want} needs a {want}-process job "
                                f"(python -m torch.distributed.run --nproc-per-node {want} ...); this job has "
                                f"{ctx.world} process(es)")
-        n_snap = config.kv.max_snapshots if (config.kv.prefix_cache != "off" and weights.config.is_hybrid) else 0
+        n_snap = config.kv.max_snapshots if (config.kv.prefix_cache != "off" and weights.config.has_recurrent_state) else 0
         max_ctx = min(config.max_sequence_length, weights.config.max_context)
         pages_per_slot = (max_ctx + config.kv.page_tokens - 1) // config.kv.page_tokens
         n_slots = config.scheduler.max_active_requests

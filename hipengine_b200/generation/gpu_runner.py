@@ -37,7 +37,7 @@ class GpuRunner(BaseRunner):
         self.page = config.kv.page_tokens
         assert self.page == PAGE, "the attention kernels are built for 16-token pages"
         self.use_prefix = config.kv.prefix_cache != "off"
-        self.n_snap = config.kv.max_snapshots if (self.use_prefix and self.cfg.is_hybrid) else 0
+        self.n_snap = config.kv.max_snapshots if (self.use_prefix and self.cfg.has_recurrent_state) else 0
         pages_per_slot = (self.max_context + self.page - 1) // self.page
         from ..config import resolve_pool_pages
         self.kv_bytes_per_token = self.cfg.kv_bytes_per_token(4 if config.compute_dtype == "float32" else 2)
@@ -168,7 +168,7 @@ class GpuRunner(BaseRunner):
         gets a snapshot slot (its block may be cold too, or still cached with its snapshot slot recycled).
         Returns the number of tokens by which the usable prefix grew."""
         from ..kvcache.tiering import prefix_key, restore_is_worthwhile
-        page, hybrid = self.page, self.cfg.is_hybrid
+        page, hybrid = self.page, self.cfg.has_recurrent_state
         limit = (len(prompt) - 1) // page
         present = self.radix.match(prompt, require_snapshot=False)      # blocks whose pages are still in the pool
         b0 = present.tokens // page
@@ -254,10 +254,10 @@ class GpuRunner(BaseRunner):
         except ResourceUnavailable:
             return False
         prompt = rs.req.prompt_token_ids
-        match = self.radix.match(prompt, require_snapshot=self.cfg.is_hybrid) if self.use_prefix else None
+        match = self.radix.match(prompt, require_snapshot=self.cfg.has_recurrent_state) if self.use_prefix else None
         if self.cold is not None and len(self.cold) and match is not None:
             if self._restore_from_cold(prompt, match.tokens):
-                match = self.radix.match(prompt, require_snapshot=self.cfg.is_hybrid)
+                match = self.radix.match(prompt, require_snapshot=self.cfg.has_recurrent_state)
         shared = match.pages if match and match.tokens else []
         try:
             lease = self.pool.admit(rs.rid, total, shared_prefix=shared, now_tokens=rs.prompt_len)
@@ -274,7 +274,7 @@ class GpuRunner(BaseRunner):
         if self.mtp is not None:
             self.mtp.reset_slot(slot)
         if shared:
-            if self.cfg.is_hybrid and match.snapshot is not None:
+            if self.cfg.has_recurrent_state and match.snapshot is not None:
                 self._copy_state(match.snapshot, slot)
             rs.prefilled = rs.cached_tokens = match.tokens
             self.stats["prefix_hits"] += 1
@@ -304,37 +304,79 @@ class GpuRunner(BaseRunner):
         self.stats["h2d_bytes"] += 8 * batch.T + 16 * batch.T
         return batch, self.ex.forward(batch)
 
+    def packs_mixed(self) -> bool:
+        return self.ex.packs_mixed and self.mtp is None
+
     @torch.no_grad()
     def mixed(self, work: List[Tuple[RequestState, int]], rows: List[RequestState]):
-        """Decode rows and prompt chunks in ONE forward pass.  Returns (results of the decode rows, first tokens of the
-        prompts that end in this step by request id)."""
-        if self.mtp is not None or self.n_snap or not work or not rows:
-            return super().mixed(work, rows)      # draft state / snapshot boundaries: the phases stay separate
+        """Decode rows and prompt chunks in ONE forward pass (chunks that cross a snapshot boundary go on after it in
+        passes of their own).  Returns (results of the decode rows, first tokens of the prompts that end in this step by
+        request id)."""
         with self.census.region("mixed"):
-            segs = []
-            for rs in rows:
-                self._ensure_pages(rs, rs.position)
-                segs.append((rs.slot, rs.position - 1, [rs.last_token]))
-                rs.telemetry.h2d_bytes += 24
-            want, idx, row = list(rows), list(range(len(rows))), len(rows)
-            for rs, n in work:
-                a, b = rs.prefilled, rs.prefilled + n
-                self._ensure_pages(rs, b)
-                segs.append((rs.slot, a, rs.req.prompt_token_ids[a:b]))
-                rs.telemetry.h2d_bytes += 24 * n
-                row += n
-                if b >= rs.prompt_len:
-                    want.append(rs)
-                    idx.append(row - 1)
             try:
-                _, h = self.forward_segments(segs)
-                logits = self.ex.logits(h.index_select(0, torch.tensor(idx, device=self.device)))
-                res = self._sample_rows(want, logits)
+                return self._mixed_impl(work, rows)
             except torch.cuda.OutOfMemoryError as exc:
                 raise ExecutionFailure([rs.rid for rs in rows] + [rs.rid for rs, _ in work], "mixed",
                                        f"out of memory: {exc}", "partial") from exc
-            self.resident_key = ()
-            return res[:len(rows)], {rs.rid: t for rs, t in zip(want[len(rows):], res[len(rows):])}
+            finally:
+                self.resident_key = ()
+
+    def _mixed_impl(self, work: List[Tuple[RequestState, int]], rows: List[RequestState]):
+        segs = []
+        for rs in rows:
+            self._ensure_pages(rs, rs.position)
+            segs.append((rs.slot, rs.position - 1, [rs.last_token]))
+            rs.telemetry.h2d_bytes += 24
+        plans = self._chunk_plans(work)
+        res: List[Tuple[int, Optional[TokenLogprob]]] = []
+        firsts: Dict[int, Tuple[int, Optional[TokenLogprob]]] = {}
+        for k in range(max(len(p) for p in plans)):
+            part, owners = self._chunk_round(work, plans, k)
+            carried = rows if k == 0 else []
+            _, h = self.forward_segments((segs if k == 0 else []) + part)
+            want, idx, row = list(carried), list(range(len(carried))), len(carried)
+            for rs, a, b in owners:
+                row += b - a
+                if b >= rs.prompt_len:
+                    want.append(rs)
+                    idx.append(row - 1)
+                self._snapshot_at(rs, b)
+            if want:
+                got = self._sample_rows(want, self.ex.logits(h.index_select(0, torch.tensor(idx, device=self.device))))
+                res += got[:len(carried)]
+                firsts.update({rs.rid: t for rs, t in zip(want[len(carried):], got[len(carried):])})
+        return res, firsts
+
+    # ------------------------------------------------------------------ prompt chunks
+    def _chunk_plans(self, work: List[Tuple[RequestState, int]]) -> List[List[Tuple[int, int]]]:
+        """Every chunk as (start, end) parts that end at the snapshot boundaries inside it."""
+        interval = self.config.kv.snapshot_interval_tokens if self.n_snap else 0
+        plans: List[List[Tuple[int, int]]] = []
+        for rs, n in work:
+            cur, end, parts = rs.prefilled, rs.prefilled + n, []
+            while cur < end:
+                nxt = min(end, (cur // interval + 1) * interval) if interval else end
+                parts.append((cur, nxt))
+                cur = nxt
+            plans.append(parts)
+        return plans
+
+    def _chunk_round(self, work, plans, k: int):
+        """Part ``k`` of every chunk that has one: (segments, (request, start, end) owners); their pages are in place."""
+        segs, owners = [], []
+        for (rs, _), parts in zip(work, plans):
+            if k < len(parts):
+                a, b = parts[k]
+                self._ensure_pages(rs, b)
+                segs.append((rs.slot, a, rs.req.prompt_token_ids[a:b]))
+                owners.append((rs, a, b))
+                rs.telemetry.h2d_bytes += 24 * (b - a)      # ids (int64) + slot / pos / segment (int32)
+        return segs, owners
+
+    def _snapshot_at(self, rs: RequestState, n_tokens: int) -> None:
+        interval = self.config.kv.snapshot_interval_tokens if self.n_snap else 0
+        if interval and n_tokens % interval == 0 and n_tokens < rs.prompt_len:
+            self._snapshot(rs, n_tokens)
 
     # ------------------------------------------------------------------ prefill
     def prefill(self, work: List[Tuple[RequestState, int]]) -> Dict[int, Tuple[int, Optional[TokenLogprob]]]:
@@ -344,31 +386,12 @@ class GpuRunner(BaseRunner):
     @torch.no_grad()
     def _prefill_impl(self, work: List[Tuple[RequestState, int]]) -> Dict[int, Tuple[int, Optional[TokenLogprob]]]:
         out: Dict[int, Tuple[int, Optional[TokenLogprob]]] = {}
-        interval = self.config.kv.snapshot_interval_tokens if self.n_snap else 0
         # split every chunk at snapshot boundaries, then run the sub-chunks round by round as packed batches
-        plans: List[List[Tuple[int, int]]] = []
-        for rs, n in work:
-            cur, end, parts = rs.prefilled, rs.prefilled + n, []
-            while cur < end:
-                nxt = end
-                if interval:
-                    b = (cur // interval + 1) * interval
-                    nxt = min(end, b)
-                parts.append((cur, nxt))
-                cur = nxt
-            plans.append(parts)
+        plans = self._chunk_plans(work)
         rounds = max(len(p) for p in plans)
         try:
             for r in range(rounds):
-                segs, owners = [], []
-                for (rs, n), parts in zip(work, plans):
-                    if r < len(parts):
-                        a, b = parts[r]
-                        self._ensure_pages(rs, b)
-                        toks = rs.req.prompt_token_ids[a:b]
-                        segs.append((rs.slot, a, toks))
-                        owners.append((rs, a, b))
-                        rs.telemetry.h2d_bytes += 24 * (b - a)      # ids (int64) + slot / pos / segment (int32)
+                segs, owners = self._chunk_round(work, plans, r)
                 batch, h = self.forward_segments(segs)
                 if self.mtp is not None:
                     self.mtp.after_prefill(batch, h)
@@ -378,8 +401,7 @@ class GpuRunner(BaseRunner):
                     row += b - a
                     if b >= rs.prompt_len:
                         last_rows.append((rs, row - 1))
-                    if interval and b % interval == 0 and b < rs.prompt_len:
-                        self._snapshot(rs, b)
+                    self._snapshot_at(rs, b)
                 if last_rows:
                     idx = torch.tensor([i for _, i in last_rows], device=self.device)
                     logits = self.ex.logits(h.index_select(0, idx))
@@ -388,7 +410,8 @@ class GpuRunner(BaseRunner):
                         out[rs.rid] = t
         except torch.cuda.OutOfMemoryError as exc:
             raise ExecutionFailure([rs.rid for rs, _ in work], "prefill", f"out of memory: {exc}", "partial") from exc
-        self.resident_key = ()
+        finally:
+            self.resident_key = ()
         return out
 
     def _snapshot(self, rs: RequestState, n_tokens: int) -> None:
@@ -562,7 +585,7 @@ class GpuRunner(BaseRunner):
     def release(self, rs: RequestState) -> None:
         lease: Optional[KVLease] = rs.runner_data
         if lease is not None:
-            if self.use_prefix and not self.cfg.is_hybrid and rs.prefilled >= self.page:
+            if self.use_prefix and not self.cfg.has_recurrent_state and rs.prefilled >= self.page:
                 n = (min(rs.prefilled, rs.prompt_len) // self.page) * self.page
                 self.radix.insert(rs.req.prompt_token_ids[:n], lease.pages[:n // self.page])
             self.pool.release(rs.rid)

@@ -93,11 +93,11 @@ class BaseRunner:
         return tok, lp
 
     # -- protocol defaults ---------------------------------------------------------------------------
-    def mixed(self, work, rows):
-        """One scheduling step that holds both prompt chunks and decode rows; runners that can pack them into a single
-        forward pass override this.  Returns (decode results, {request id: first token})."""
-        res = self.decode(rows) if rows else []
-        return res, (self.prefill(work) if work else {})
+    def packs_mixed(self) -> bool:
+        """Can ``mixed(work, rows)`` run prompt chunks and decode rows as one forward pass, returning (decode results,
+        {request id: first token})?  Otherwise the loop runs the two phases one after the other, each committed before
+        the next may fail."""
+        return False
 
     def capacity(self) -> Dict[str, Any]:
         return {"max_slots": self.max_slots, "max_context": self.max_context}

@@ -91,9 +91,9 @@ class PlanContract:
 
 
 def _required_tensors(cfg) -> List[str]:
-    if cfg.arch == "sisisun":
-        from .sisisun import tensor_shapes
-        return list(tensor_shapes(cfg))
+    if cfg.layer_specs:
+        from .folder_family import family_module
+        return list(family_module(cfg).tensor_shapes(cfg))
     need = ["token_embd.weight", "output_norm.weight"]
     for i in range(cfg.n_layers):
         need.append(f"blk.{i}.attn_norm.weight")
@@ -118,7 +118,7 @@ def plan_contract(weights) -> PlanContract:
         rows = 1
         for d in t.shape[:-1]:
             rows *= int(d)
-        cols = int(t.shape[-1])
+        cols = int(t.shape[-1]) if t.shape else 1
         if qt in IN_PLACE:
             mode = "in_place"
             nbytes = int(t.raw.numel())
@@ -154,7 +154,7 @@ def memory_preflight(weights, engine_config, free_bytes: Optional[int], contract
     kv_elem = 4 if engine_config.compute_dtype == "float32" else 2
     n_pages = resolve_pool_pages(kvc, cfg.kv_bytes_per_token(kv_elem), n_slots, pages_per_slot)
     kv_bytes = n_pages * kvc.page_tokens * cfg.kv_bytes_per_token(kv_elem)
-    n_snap = kvc.max_snapshots if (kvc.prefix_cache != "off" and cfg.is_hybrid) else 0
+    n_snap = kvc.max_snapshots if (kvc.prefix_cache != "off" and cfg.has_recurrent_state) else 0
     state_bytes = (n_slots + n_snap) * cfg.recurrent_state_bytes()
     # scratch of one 4096-row prefill chunk: a dozen [rows, widest projection] bf16/fp32 buffers + logits rows
     widest = max(cfg.hidden, 2 * getattr(cfg, "ffn", cfg.hidden), getattr(cfg, "linear_qkv_width", 0) or 0)

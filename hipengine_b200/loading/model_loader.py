@@ -17,12 +17,13 @@ import numpy as np
 import torch
 
 from ..models.config import ModelConfig
+from ..models.registry import PLUGINS
 from ..quant.ggml import GGMLType
 from .gguf import GGUFModelInfo, GGUFReader, discover_gguf_files, scan_gguf
 from .weights import ModelWeights, QTensor, expected_tensor_names
 
 GGUF_ARCHS = ("qwen35", "qwen35moe", "qwen3", "qwen3moe", "llama", "gemma4")
-FOLDER_ARCHS = ("sisisun",)                  # checkpoint folders (``safetensors_dir.py``)
+FOLDER_ARCHS = tuple(a for p in PLUGINS if p.folder_reader for a in p.architectures)     # ``safetensors_dir.py``
 SUPPORTED_ARCHS = GGUF_ARCHS + FOLDER_ARCHS
 
 

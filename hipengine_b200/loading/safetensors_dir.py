@@ -1,13 +1,14 @@
 """Checkpoint folders: ``config.json`` beside ``model.safetensors``.
 
 A safetensors file is an 8-byte little-endian header length, that many bytes of JSON (name -> dtype, shape,
-data_offsets into the rest) and the tensor bytes.  The model family is chosen by ``architecture`` in config.json; each
-family contributes a reader of its configuration and the list of tensors it needs.
+data_offsets into the rest) and the tensor bytes.  The registry finds the model family by ``architecture`` in config.json
+and names the module with its configuration reader and tensor list (``folder_family.py``).
 """
 from __future__ import annotations
 
 import json
 import struct
+from importlib import import_module
 from pathlib import Path
 from typing import Any, Dict, Optional, Tuple
 
@@ -93,18 +94,19 @@ def config_of(path):
     """(``ModelConfig``, decoded config.json) of a checkpoint folder."""
     with open(Path(path) / CONFIG_FILE) as f:
         raw = json.load(f)
-    arch = str(raw.get("architecture", ""))
-    if arch == "Sisisun":
-        from .sisisun import config_from_json
-        return config_from_json(raw), raw
-    raise ValueError(f"unsupported architecture {arch!r} in {path}/{CONFIG_FILE}; supported: ('Sisisun',)")
+    from ..models.registry import folder_plugin
+    try:
+        plugin = folder_plugin(str(raw.get("architecture", "")))
+    except KeyError as e:
+        raise ValueError(f"{path}/{CONFIG_FILE}: {e.args[0]}") from None
+    return import_module(plugin.folder_reader).config_from_json(raw), raw
 
 
 def load_checkpoint_dir(path, device="cpu", pin: bool = False, validate: bool = True) -> ModelWeights:
     cfg, raw = config_of(path)
     tensors = read_tensors(Path(path) / TENSOR_FILE, device, pin)
     if validate:
-        from .sisisun import check_tensors
+        from .folder_family import check_tensors
         check_tensors(cfg, {n: t.shape for n, t in tensors.items()})
     return ModelWeights(cfg, tensors, {"general.architecture": cfg.arch, "general.name": str(path), "config": raw})
 

@@ -6,13 +6,11 @@ with ``.mix.q.norm`` / ``.mix.k.norm``, ``.norm2`` and either ``.mlp.gate/up/dow
 """
 from __future__ import annotations
 
-from typing import Any, Dict, List, Mapping, Optional, Sequence, Tuple
+from typing import Any, Dict, List, Mapping, Optional, Tuple
 
-import torch
-
-from ..models.config import (AttentionSpec, DenseMlpSpec, LayerSpec, LoopSpec, ModelConfig, MoeMlpSpec, sisisun_config)
-from ..quant.ggml import GGMLType
-from .weights import ModelWeights, QTensor
+from ..models.config import AttentionSpec, DenseMlpSpec, LayerSpec, ModelConfig, MoeMlpSpec, sisisun_config
+from .folder_family import build_random_folder, loop_from_json, loop_to_json
+from .weights import ModelWeights
 
 
 # ----------------------------------------------------------------------------- configuration
@@ -41,9 +39,7 @@ def config_from_json(c: Mapping[str, Any]) -> ModelConfig:
             AttentionSpec(int(m["heads"]), int(m["kv_heads"]), int(m["dim"]), int(m["vdim"]), float(m["scale"]),
                           float(m.get("softcap") or 0.0)),
             _mlp_from_json(i, l.get("mlp"))))
-    lp = c.get("loop")
-    loop = LoopSpec(int(lp["start"]), int(lp["stop"]), int(lp["times"])) if lp else None
-    return sisisun_config(int(c["width"]), int(c["vocab"]), tuple(layers), loop, rms_eps=float(c["norm"]["eps"]))
+    return sisisun_config(int(c["width"]), int(c["vocab"]), tuple(layers), loop_from_json(c), rms_eps=float(c["norm"]["eps"]))
 
 
 def config_to_json(cfg: ModelConfig) -> Dict[str, Any]:
@@ -60,9 +56,8 @@ def config_to_json(cfg: ModelConfig) -> Dict[str, Any]:
         layers.append({"type": "attention", "mlp": mlp,
                        "mixer": {"heads": a.heads, "kv_heads": a.kv_heads, "dim": a.dim, "vdim": a.vdim,
                                  "scale": a.scale, "softcap": a.softcap}})
-    lp = cfg.loop
     return {"architecture": "Sisisun", "vocab": cfg.vocab, "width": cfg.hidden, "norm": {"eps": cfg.rms_eps},
-            "layers": layers, "loop": {"start": lp.start, "stop": lp.stop, "times": lp.times} if lp else None}
+            "layers": layers, "loop": loop_to_json(cfg.loop)}
 
 
 # ----------------------------------------------------------------------------- tensors
@@ -100,34 +95,5 @@ def tensor_shapes(cfg: ModelConfig) -> Dict[str, Tuple[int, ...]]:
     return out
 
 
-def check_tensors(cfg: ModelConfig, have: Mapping[str, Sequence[int]]) -> None:
-    bad = [f"{n}: expected {list(s)}, found {list(have[n]) if n in have else 'nothing'}"
-           for n, s in tensor_shapes(cfg).items() if n not in have or tuple(have[n]) != tuple(s)]
-    if bad:
-        raise KeyError(f"checkpoint does not match its configuration: {'; '.join(bad[:6])}"
-                       + (f" and {len(bad) - 6} more" if len(bad) > 6 else ""))
-
-
-def weights_from_tensors(cfg: ModelConfig, tensors: Mapping[str, torch.Tensor]) -> ModelWeights:
-    """``ModelWeights`` over in-memory bfloat16 tensors under their checkpoint names."""
-    check_tensors(cfg, {n: t.shape for n, t in tensors.items()})
-    out = {}
-    for n, t in tensors.items():
-        b = t.to(torch.bfloat16).contiguous()
-        out[n] = QTensor(n, GGMLType.BF16, tuple(b.shape), b.reshape(-1, b.shape[-1]).view(torch.uint8))
-    return ModelWeights(cfg, out, {"general.architecture": cfg.arch, "general.name": "sisisun",
-                                   "config": config_to_json(cfg)})
-
-
 def build_random_sisisun(cfg: ModelConfig, seed: int = 0, device="cpu", std: float = 0.02) -> ModelWeights:
-    gen = torch.Generator(device=torch.device(device))
-    gen.manual_seed(seed)
-    tensors: Dict[str, torch.Tensor] = {}
-    for n, shape in tensor_shapes(cfg).items():
-        t = torch.randn(*shape, generator=gen, device=device, dtype=torch.float32) * std
-        if n.endswith(("q.norm", "k.norm")):
-            t = 1.0 + t
-        tensors[n] = t.to(torch.bfloat16)
-    w = weights_from_tensors(cfg, tensors)
-    w.metadata["general.name"] = f"random-init sisisun seed={seed}"
-    return w
+    return build_random_folder(cfg, seed, device, std, lambda n, t: 1.0 + t if n.endswith(("q.norm", "k.norm")) else t)

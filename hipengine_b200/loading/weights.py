@@ -37,7 +37,7 @@ class QTensor:
 
     @property
     def n_cols(self) -> int:
-        return self.shape[-1]
+        return self.shape[-1] if self.shape else 1       # a single number has an empty shape
 
     @property
     def n_rows(self) -> int:

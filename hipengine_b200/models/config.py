@@ -9,6 +9,7 @@ geometries mirror the identities the reference pins in
 """
 from __future__ import annotations
 
+import math
 from dataclasses import dataclass, replace
 from typing import Dict, Optional, Tuple, Union
 
@@ -39,10 +40,95 @@ class AttentionSpec:
         return padded_head_width(max(self.dim, self.vdim))
 
 
+    @property
+    def cache_elems(self) -> int:
+        """Elements a token takes in the layer's cache plane."""
+        return 2 * self.kv_heads * self.width
+
+
+@dataclass(frozen=True)
+class YarnSpec:
+    """Context extension of a rotary table: slow pairs are slowed down by ``factor``, fast ones are kept."""
+    factor: float
+    original: float                      # context the unscaled table was made for
+    fast: float                          # turns over that context from which a pair counts as fast ...
+    slow: float                          # ... and below which as slow
+
+
+@dataclass(frozen=True)
+class RotarySpec:
+    """Rotation of neighbouring pairs (2i, 2i + 1) by position * base^(-2i / dims)."""
+    dims: int
+    base: float
+    yarn: Optional[YarnSpec] = None
+
+    def table(self) -> Tuple[Tuple[float, ...], float]:
+        """(angular frequency per pair, amplitude of sine and cosine)."""
+        freq = [self.base ** (-2.0 * i / self.dims) for i in range(self.dims // 2)]
+        y = self.yarn
+        if y is None:
+            return tuple(freq), 1.0
+        at = lambda turns: self.dims * math.log(y.original / (2 * math.pi * turns)) / (2 * math.log(self.base))
+        lo, hi = max(math.floor(at(y.fast)), 0), min(math.ceil(at(y.slow)), self.dims - 1)
+        for i, f in enumerate(freq):
+            slow = min(max((i - lo) / max(hi - lo, 0.001), 0.0), 1.0)
+            freq[i] = f * (slow / y.factor + 1.0 - slow)
+        return tuple(freq), 0.1 * math.log(y.factor) + 1.0
+
+
+# bounds of the latent attention kernels: padded latent columns, and those plus the padded rotated part
+LATENT_MAX_RANK = 1024
+LATENT_MAX_ROW = 1280
+
+
+def round_up(n: int, m: int) -> int:
+    return -(-n // m) * m
+
+
+@dataclass(frozen=True)
+class LatentAttentionSpec:
+    """Attention whose keys and values are linear maps of one latent row per token (plus a rotated key part shared by
+    all heads); only the latent and the rotated part are cached."""
+    heads: int
+    dim: int                             # unrotated query / key width per head
+    rot_dim: int                         # rotated query / key width per head
+    vdim: int
+    kv_rank: int                         # latent width
+    scale: float
+    rot: RotarySpec
+    q_rank: int = 0                      # > 0: queries go through a normalised latent of this width
+    window: int = 0                      # > 0: only the last ``window`` positions are visible
+    sink: bool = False                   # a learned term per head in the softmax denominator
+
+    @property
+    def rank_cols(self) -> int:
+        """Columns of the latent in a cache row (zero-padded)."""
+        return round_up(self.kv_rank, 16)
+
+    @property
+    def row_cols(self) -> int:
+        """Columns of a cache row: latent, then the rotated part, zero-padded."""
+        return round_up(self.rank_cols + self.rot_dim, 32)
+
+    @property
+    def cache_elems(self) -> int:
+        return self.row_cols
+
+    def check(self) -> None:
+        if min(self.heads, self.dim, self.vdim, self.kv_rank) < 1 or self.rot_dim < 2 or self.rot_dim % 2:
+            raise ValueError(f"latent attention of {self.heads} heads, {self.dim} + {self.rot_dim} / {self.vdim} wide, "
+                             f"latent {self.kv_rank}")
+        if self.rot.dims != self.rot_dim:
+            raise ValueError(f"rotary table over {self.rot.dims} dimensions for a rotated part of {self.rot_dim}")
+        if self.rank_cols > LATENT_MAX_RANK or self.row_cols > LATENT_MAX_ROW:
+            raise ValueError(f"latent of {self.kv_rank} + {self.rot_dim} columns is above the widest supported one "
+                             f"({LATENT_MAX_RANK}, {LATENT_MAX_ROW} with the rotated part)")
+
+
 @dataclass(frozen=True)
 class DenseMlpSpec:
     ff: int
-    act: str = "silu"                    # "silu" | "gelu_tanh" | "clamped_glu"
+    act: str = "silu"                    # gated: "silu" | "gelu_tanh" | "clamped_glu"; ungated: "relu2"
     limit: float = 0.0                   # clamped_glu: bound of the gate (above) and of the up branch (both sides)
 
 
@@ -59,8 +145,10 @@ class MoeMlpSpec:
 
 @dataclass(frozen=True)
 class LayerSpec:
-    mixer: AttentionSpec
+    mixer: Union[AttentionSpec, LatentAttentionSpec]
     mlp: Optional[Union[DenseMlpSpec, MoeMlpSpec]] = None
+    parallel: bool = False               # both sublayers read one norm and are added together
+    token_shift: bool = False            # the mixer reads a mix of this token's and the previous token's normalised row
 
 
 @dataclass(frozen=True)
@@ -119,6 +207,7 @@ class ModelConfig:
     # designs whose layers are listed one by one (``layer_specs``), some of them run repeatedly (``loop``)
     layer_specs: Tuple[LayerSpec, ...] = ()
     loop: Optional[LoopSpec] = None
+    residual_mult: float = 1.0           # factor on what a layer adds to the residual
 
     # ---- derived
     def is_global_layer(self, i: int) -> bool:
@@ -137,6 +226,11 @@ class ModelConfig:
     @property
     def is_hybrid(self) -> bool:
         return self.full_attention_interval > 0
+
+    @property
+    def has_recurrent_state(self) -> bool:
+        """Does a request carry state besides its cache pages (prefix reuse then needs snapshots of it)?"""
+        return self.is_hybrid or any(l.token_shift for l in self.layer_specs)
 
     @property
     def is_moe(self) -> bool:
@@ -194,11 +288,12 @@ class ModelConfig:
 
     def kv_bytes_per_token(self, elem_bytes: int = 2) -> int:
         if self.layer_specs:
-            return sum(2 * self.layer_specs[i].mixer.kv_heads * self.layer_specs[i].mixer.width * elem_bytes
-                       for i, _ in self.layer_runs())
+            return sum(self.layer_specs[i].mixer.cache_elems * elem_bytes for i, _ in self.layer_runs())
         return self.n_full_layers * 2 * self.n_kv_heads * self.head_dim * elem_bytes
 
     def recurrent_state_bytes(self) -> int:
+        if self.layer_specs:
+            return sum(4 * round_up(self.hidden, 8) for i, _ in self.layer_runs() if self.layer_specs[i].token_shift)
         gdn = self.n_linear_layers * self.ssm_v_heads * self.ssm_state * self.ssm_state * 4
         conv = self.n_linear_layers * self.linear_qkv_width * self.conv_kernel * 4
         return gdn + conv
@@ -326,6 +421,50 @@ SISISUN_30B_MOE = sisisun_config(2048, 151936, tuple(
     for _ in range(48)), loop=LoopSpec(12, 24, 2))
 
 
+def milutar_config(hidden: int, vocab: int, layers: Tuple[LayerSpec, ...], loop: Optional[LoopSpec] = None,
+                   rms_eps: float = 1e-6, residual_mult: float = 1.0, max_context: int = 262144) -> ModelConfig:
+    """``ModelConfig`` of a Milutar model: parallel layers with token shift and layer scale over latent attention, norms
+    with a single gain, optional looped range."""
+    if not layers:
+        raise ValueError("a model needs layers")
+    for i, l in enumerate(layers):
+        try:
+            l.mixer.check()
+        except ValueError as e:
+            raise ValueError(f"layer {i}: {e}") from None
+    if loop is not None and not (0 <= loop.start < loop.stop <= len(layers) and loop.times >= 1):
+        raise ValueError(f"loop {loop} over {len(layers)} layers")
+    a = layers[0].mixer
+    return ModelConfig(
+        arch="milutar", n_layers=len(layers), hidden=hidden, vocab=vocab, n_heads=a.heads, n_kv_heads=1,
+        head_dim=a.dim + a.rot_dim, ffn=max([l.mlp.ff for l in layers if l.mlp is not None], default=0), rms_eps=rms_eps,
+        rope_theta=a.rot.base, rope_dim=a.rot_dim, attn_scale=a.scale, layer_specs=tuple(layers), loop=loop,
+        residual_mult=residual_mult, max_context=max_context)
+
+
+def _milutar_layer(mixer: LatentAttentionSpec, ff: int) -> LayerSpec:
+    return LayerSpec(mixer, DenseMlpSpec(ff, "relu2") if ff else None, parallel=True, token_shift=True)
+
+
+# Small Milutar geometry of the tests and the command line: both kinds of attention, unequal widths, a layer without a
+# feed-forward, a loop inside the stack.
+_MILUTAR_W = LatentAttentionSpec(heads=3, dim=40, rot_dim=24, vdim=48, kv_rank=72, scale=0.125, window=50,
+                                 rot=RotarySpec(24, 5000.0, YarnSpec(4.0, 512.0, 20.0, 1.5)))
+_MILUTAR_F = LatentAttentionSpec(heads=5, dim=24, rot_dim=8, vdim=32, kv_rank=48, scale=0.18, q_rank=56, sink=True,
+                                 rot=RotarySpec(8, 100000.0))
+TINY_MILUTAR = milutar_config(
+    200, 1024, (_milutar_layer(_MILUTAR_W, 232), _milutar_layer(_MILUTAR_F, 184), _milutar_layer(_MILUTAR_W, 0),
+                _milutar_layer(_MILUTAR_F, 184)), loop=LoopSpec(1, 3, 2), residual_mult=0.6, max_context=8192)
+
+# Geometry at the layer sizes of a deployed model, for throughput: an 8B-class width with 512-wide latents.
+_MILUTAR_8B_W = LatentAttentionSpec(heads=32, dim=128, rot_dim=64, vdim=128, kv_rank=512, scale=192 ** -0.5, window=4096,
+                                    rot=RotarySpec(64, 50000.0, YarnSpec(16.0, 8192.0, 24.0, 2.0)))
+_MILUTAR_8B_F = LatentAttentionSpec(heads=32, dim=128, rot_dim=64, vdim=128, kv_rank=512, scale=192 ** -0.5, q_rank=1536,
+                                    sink=True, rot=RotarySpec(64, 2e6))
+MILUTAR_8B = milutar_config(4096, 128256, tuple(_milutar_layer(_MILUTAR_8B_F if i % 4 == 3 else _MILUTAR_8B_W, 20480)
+                                                for i in range(28)), loop=LoopSpec(8, 16, 2), residual_mult=0.5)
+
+
 @dataclass(frozen=True)
 class AssistantConfig:
     """Gemma 4 assistant (MTP) head: a separate four-block draft model with no K/V projections of its own.  Every
@@ -393,4 +532,6 @@ NAMED_CONFIGS: Dict[str, ModelConfig] = {
     "tiny-sisisun": TINY_SISISUN,
     "sisisun-8b": SISISUN_8B,
     "sisisun-30b-moe": SISISUN_30B_MOE,
+    "tiny-milutar": TINY_MILUTAR,
+    "milutar-8b": MILUTAR_8B,
 }

@@ -137,6 +137,7 @@ class _Scratch:
 
 class HybridExecutor:
     keeps_hidden = True           # decode steps also store the post-norm hidden rows
+    packs_mixed = False           # can decode rows ride in a prompt's forward without costing more than a step of their own
 
     def __init__(self, weights: ModelWeights, device="cuda", max_slots: int = 4, max_context: int = 4608,
                  n_pages: Optional[int] = None, gemm_impl: Optional[str] = None):
@@ -628,23 +629,16 @@ class HybridExecutor:
         return out
 
     def alloc_journal(self, rows: int) -> dict:
-        """Per-verify-row recurrent state journals for every linear-attention layer."""
-        cfg = self.cfg
-        j = {"conv": {}, "gdn": {}}
-        for i in self.conv_state:
-            j["conv"][i] = torch.empty(rows, cfg.linear_qkv_width, cfg.conv_kernel - 1, dtype=torch.float32,
-                                       device=self.device)
-            j["gdn"][i] = torch.empty(rows, cfg.ssm_v_heads, cfg.ssm_state, cfg.ssm_state, dtype=torch.float32,
-                                      device=self.device)
-        return j
+        """Per-verify-row recurrent state journals for every layer that has such state."""
+        like = lambda d: {i: torch.empty(rows, *t.shape[1:], dtype=torch.float32, device=self.device)
+                          for i, t in d.items()}
+        return {"conv": like(self.conv_state), "gdn": like(self.gdn_state)}
 
     def commit_journal(self, journal: dict, seg_slot: torch.Tensor, commit_row: torch.Tensor) -> None:
-        """state[seg_slot[s]] = journal[commit_row[s]] for every linear layer (speculative commit)."""
-        cfg = self.cfg
-        for i, st in self.conv_state.items():
-            K.state_commit(st, journal["conv"][i], seg_slot, commit_row, cfg.linear_qkv_width * (cfg.conv_kernel - 1))
-            K.state_commit(self.gdn_state[i], journal["gdn"][i], seg_slot, commit_row,
-                           cfg.ssm_v_heads * cfg.ssm_state * cfg.ssm_state)
+        """state[seg_slot[s]] = journal[commit_row[s]] for every layer with recurrent state (speculative commit)."""
+        for kind, states in (("conv", self.conv_state), ("gdn", self.gdn_state)):
+            for i, st in states.items():
+                K.state_commit(st, journal[kind][i], seg_slot, commit_row, st[0].numel())
 
     def greedy(self, logits: torch.Tensor, out_ids: torch.Tensor) -> torch.Tensor:
         return K.argmax_rows(logits, self.am_v, self.am_i, out_ids)

@@ -1,0 +1,167 @@
+"""Common base of the designs whose layers are listed one by one (``ModelConfig.layer_specs``), some of them run repeatedly.
+
+On top of the hybrid executor (scratch, paged pool, block tables, decode and prefill graphs, journals) it holds what these
+families share:
+  * bfloat16 weights; widths that are no multiple of eight are zero-padded at load (norms average over the real width);
+  * one cache plane per layer RUN: every pass of a looped range attends only to what the same pass wrote;
+  * per-slot recurrent rows (token shift) per layer run, kept where the hybrid executor keeps its convolution windows, so
+    admission, snapshots, the cold tier, graph warm-up and speculative commits treat them alike;
+  * three kernel routes by row count: fp32, up to 16 rows (streaming GEMV), more (tcgen05 GEMM, split over K up to 128 rows).
+"""
+from __future__ import annotations
+
+from typing import Callable, Optional
+
+import torch
+
+from ..loading.weights import ModelWeights
+from ..ops import kernels as K
+from ..ops.kernels import DeviceWeight
+from ..quant.ggml import GGMLType
+from .executor import PAGE, BatchDesc, HybridExecutor
+
+# segments of up to this many rows attend through the split-K decode kernel, longer ones through the flash kernel
+DECODE_SEG_ROWS = 8
+EXACT, FEW, MANY = "exact", "few", "many"       # kernel routes of a forward
+
+
+def up8(n: int) -> int:
+    return -(-n // 8) * 8
+
+
+def pad2(t: torch.Tensor, rows: int, cols: int) -> torch.Tensor:
+    """``t`` in the upper left corner of a zero [rows, cols] matrix."""
+    if t.shape == (rows, cols):
+        return t
+    out = torch.zeros(rows, cols, dtype=t.dtype, device=t.device)
+    out[:t.shape[0], :t.shape[1]] = t
+    return out
+
+
+class ListedExecutor(HybridExecutor):
+    keeps_hidden = False
+    packs_mixed = True             # prompt portions and decode rows of one step run as one forward
+
+    def __init__(self, weights: ModelWeights, dtype: str = "bfloat16", **kw):
+        if dtype not in ("bfloat16", "float32"):
+            raise ValueError(f"compute dtype {dtype!r} (bfloat16 | float32)")
+        self.exact = dtype == "float32"
+        self.act_dtype = torch.float32 if self.exact else torch.bfloat16
+        self.on_layer_run: Optional[Callable[[int, torch.Tensor], None]] = None    # (run, residual rows) observer
+        super().__init__(weights, **kw)
+
+    # ------------------------------------------------------------------ weights
+    def _load(self, weights: ModelWeights) -> None:
+        self.weights_in = weights
+        self.hp = up8(self.cfg.hidden)
+        self.runs = self.cfg.layer_runs()
+        self._load_layers()
+        self.embed_w = self._put("token_embd.weight", self._mat("embed"))
+        self.head_w = self._put("output.weight", pad2(self._mat("head"), self.cfg.vocab, self.hp))
+        self.f32["final.norm"] = self._norm_weight("final.norm")
+        self.loop_step: Optional[torch.Tensor] = None
+        if self.cfg.loop is not None:
+            self.loop_step = pad2(self._mat("loop.step").float(), self.cfg.loop.times, self.hp).contiguous()
+        del self.weights_in
+
+    def _load_layers(self) -> None:
+        raise NotImplementedError
+
+    def _norm_weight(self, name: str) -> torch.Tensor:
+        """fp32 gains [hp] of a norm over the residual width (zero in padded columns)."""
+        raise NotImplementedError
+
+    def _mat(self, name: str) -> torch.Tensor:
+        t = self.weights_in[name]
+        if t.ggml_type == GGMLType.BF16:
+            return t.raw.to(self.device).reshape(-1).view(torch.bfloat16).reshape(t.shape)
+        return t.dequant(self.device).to(torch.bfloat16)
+
+    def _put(self, name: str, t: torch.Tensor) -> DeviceWeight:
+        w = self.dw[name] = DeviceWeight(int(GGMLType.BF16), t.shape[0], t.shape[1], t.contiguous())
+        return w
+
+    def _vec(self, name: str, width: int, factor: float = 1.0) -> torch.Tensor:
+        """A vector as fp32, times ``factor``, zero-padded to ``width``."""
+        t = self._mat(name).float().reshape(-1)
+        v = torch.zeros(width, dtype=torch.float32, device=self.device)
+        v[:t.numel()] = t * factor
+        self.f32[name] = v
+        return v
+
+    # ------------------------------------------------------------------ state: one cache plane per layer run
+    def _alloc_state(self) -> None:
+        dev = self.device
+        self.conv_state, self.gdn_state, self.kv = {}, {}, {}
+        for run, (i, _) in enumerate(self.runs):
+            spec = self.cfg.layer_specs[i]
+            self.kv[run] = torch.zeros(*self._plane_shape(spec.mixer), dtype=self.act_dtype, device=dev)
+            if spec.token_shift:
+                self.conv_state[run] = torch.zeros(self.max_slots, self.hp, 1, dtype=torch.float32, device=dev)
+        self._alloc_tables()
+
+    def _plane_shape(self, mixer):
+        return self.n_pages, 2, mixer.kv_heads, PAGE, mixer.width
+
+    # ------------------------------------------------------------------ dispatch
+    def _resid_buffer(self, T: int) -> torch.Tensor:
+        return self.scratch.get("h", (T, self.hp), torch.float32)
+
+    def _norm_rows(self, h: torch.Tensor, w: torch.Tensor) -> torch.Tensor:
+        xn = self.scratch.get("xn", (h.shape[0], self.hp), self.act_dtype)
+        return K.rmsnorm_rows(h, w, xn, self.cfg.rms_eps, n_mean=self.cfg.hidden)
+
+    def _route(self, T: int) -> str:
+        return EXACT if self.exact else FEW if T <= K.FLOAT_GEMV_MAX_ROWS else MANY
+
+    # ------------------------------------------------------------------ whole model
+    def _embed(self, b: BatchDesc, h: torch.Tensor, copy: Optional[torch.Tensor]) -> None:
+        raise NotImplementedError
+
+    def _layer_run(self, run: int, i: int, h: torch.Tensor, b: BatchDesc, route: str, journal: Optional[dict]) -> None:
+        raise NotImplementedError
+
+    readds_embedding = False       # later passes of a loop start from x + the embedding output
+
+    def forward(self, b: BatchDesc, journal: Optional[dict] = None, h_out: Optional[torch.Tensor] = None,
+                defer_resid: bool = False) -> torch.Tensor:
+        cfg, T = self.cfg, b.T
+        route = self._route(T)
+        direct = h_out is not None and h_out.shape[1] == self.hp and h_out.is_contiguous()
+        h = h_out if direct else self._resid_buffer(T)
+        lp = cfg.loop
+        again = self.readds_embedding and lp is not None and lp.times > 1
+        x0 = self.scratch.get("embed_out", (T, self.hp), torch.float32) if again else None
+        self._embed(b, h, x0)
+        for run, (i, t) in enumerate(self.runs):
+            if t >= 0 and i == lp.start:
+                K.resid_inject(h, x0 if t > 0 else None, self.loop_step[t])
+            self._layer_run(run, i, h, b, route, journal)
+            if self.on_layer_run is not None:
+                self.on_layer_run(run, h[:, :cfg.hidden])
+        if h_out is not None and not direct:
+            h_out.copy_(h[:, :cfg.hidden])
+            return h_out
+        return h
+
+    def logits(self, h_rows: torch.Tensor, out: Optional[torch.Tensor] = None,
+               hidden_out: Optional[torch.Tensor] = None) -> torch.Tensor:
+        cfg, R = self.cfg, h_rows.shape[0]
+        if h_rows.shape[1] != self.hp:
+            h_rows = pad2(h_rows, R, self.hp)
+        norm_w = self.f32["final.norm"]
+        if out is None:
+            out = self.scratch.get("logits", (R, cfg.vocab), torch.float32)
+        if hidden_out is not None:
+            hid = self.scratch.get("hidden_rows", (R, self.hp), torch.float32)
+            hidden_out.copy_(K.rmsnorm_rows(h_rows, norm_w, hid, cfg.rms_eps, n_mean=cfg.hidden)[:, :cfg.hidden])
+        if self._route(R) == FEW:
+            K.gemv_float(h_rows, [(self.head_w.data, None, out, K.EPI_F32)], norm_w=norm_w, eps=cfg.rms_eps,
+                         norm_n=cfg.hidden)
+            return out
+        xn = self.scratch.get("xn_head", (R, self.hp), self.act_dtype)
+        K.rmsnorm_rows(h_rows, norm_w, xn, cfg.rms_eps, n_mean=cfg.hidden)
+        if self.exact:
+            return K.small_gemm_f32(xn, self.head_w.data, out)
+        from ..ops import gemm as GM
+        return GM.gemm_bf16(xn, self.head_w.data, out)

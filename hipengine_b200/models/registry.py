@@ -28,13 +28,18 @@ class ModelPlugin:
     expert_parallel: bool = False
     compute_dtypes: Tuple[str, ...] = ("bfloat16",)
     native_sources: Tuple[str, ...] = ()        # csrc files a build for this family alone needs (empty: all of them)
+    folder_architecture: str = ""               # ``architecture`` of its checkpoint folders (config.json), if it has any
+    folder_reader: str = ""                     # module with their configuration reader and tensor list
+    reference: str = ""                         # plain reference of a folder family: class over (config.json, tensors)
     notes: str = ""
 
     def layer_sequence(self, cfg: ModelConfig) -> List[str]:
         """One word per layer of ``cfg``: ``linear`` (Gated-DeltaNet), ``full``, ``sliding`` or ``global``."""
         out = []
         for i in range(cfg.n_layers):
-            if cfg.arch == "gemma4":
+            if cfg.layer_specs:
+                out.append("sliding" if getattr(cfg.layer_specs[i].mixer, "window", 0) else "full")
+            elif cfg.arch == "gemma4":
                 out.append("global" if cfg.is_global_layer(i) else "sliding")
             elif cfg.is_hybrid:
                 out.append("full" if cfg.is_full_attention_layer(i) else "linear")
@@ -86,9 +91,21 @@ PLUGINS: Tuple[ModelPlugin, ...] = (
                 tensor_parallel=False, compute_dtypes=("bfloat16", "float32"),
                 native_sources=("attn_decode.cu", "attn_prefill.cu", "exact_f32.cu", "gemm_sm100.cu", "gemv_float.cu",
                                 "layers.cu", "moe.cu", "quant_util.cu", "runtime.cpp", "sampling.cu"),
+                folder_architecture="Sisisun", folder_reader="hipengine_b200.loading.sisisun",
+                reference="hipengine_b200.ref.sisisun.SisisunRef",
                 notes="layers listed one by one: attention without rotation, soft-capped scores, dense (clamped GLU) or "
                       "group-limited sigmoid-routed experts; a range of layers may run several times; checkpoints are "
                       "folders with config.json and model.safetensors"),
+    ModelPlugin("milutar", ("milutar",), "hipengine_b200.models.milutar.MilutarExecutor", default_quant="bf16",
+                native_block_types=("BF16",), widened_block_types=(), kv_storage=("bf16", "f32"),
+                tensor_parallel=False, compute_dtypes=("bfloat16", "float32"),
+                native_sources=("gemm_sm100.cu", "gemv_float.cu", "latent_attn.cu", "latent_prefill.cu", "layers.cu",
+                                "quant_util.cu", "runtime.cpp", "sampling.cu"),
+                folder_architecture="Milutar", folder_reader="hipengine_b200.loading.milutar",
+                reference="hipengine_b200.ref.milutar.MilutarRef",
+                notes="layers listed one by one: latent attention (windowed, or causal with a softmax sink and a query "
+                      "latent) beside a squared-ReLU feed-forward on one norm, token shift, layer scale; a range of layers "
+                      "may run several times; checkpoints are folders with config.json and model.safetensors"),
 )
 
 
@@ -98,6 +115,22 @@ def plugin_for(arch: str) -> ModelPlugin:
             return p
     known = sorted(a for p in PLUGINS for a in p.architectures)
     raise KeyError(f"no model plugin for architecture {arch!r}; supported: {known}")
+
+
+def folder_plugin(architecture: str) -> ModelPlugin:
+    """Family of a checkpoint folder by its ``architecture``."""
+    for p in PLUGINS:
+        if p.folder_architecture and p.folder_architecture == architecture:
+            return p
+    known = [p.folder_architecture for p in PLUGINS if p.folder_architecture]
+    raise KeyError(f"unsupported architecture {architecture!r}; supported: {known}")
+
+
+def load_object(path: str):
+    """The class a plugin names by its import path."""
+    from importlib import import_module
+    mod, name = path.rsplit(".", 1)
+    return getattr(import_module(mod), name)
 
 
 def supported_architectures() -> List[str]:

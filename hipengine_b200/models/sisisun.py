@@ -1,11 +1,9 @@
 """Sisisun executor: listed attention layers without rotation, dense / expert feed-forwards, looped layer ranges.
 
-Reuses the hybrid executor's scratch, paged KV pool, projection dispatch, decode-graph and prefill-graph plumbing and
-replaces the weight packing and the layer walk:
-  * weights stay bfloat16.  q | k | v and gate | up are stacked at load, experts are stacked per layer, norm weights are
-    stored as 1 + w, widths that are not a multiple of eight and head widths the attention kernels do not have are
-    zero-padded (zeros change no result; the norms average over the real width);
-  * the KV planes belong to layer RUNS: every pass of a looped range attends only to what the same pass wrote;
+The base (``listed.py``) holds the planes per layer run, the routes and the walk over runs; here are the weight packing and
+the sublayers:
+  * q | k | v and gate | up are stacked at load, experts are stacked per layer, norm weights are stored as 1 + w, head widths
+    the attention kernels do not have are zero-padded;
   * up to 16 rows (decode steps, short portions) run on the streaming bf16 GEMV with the norm and the activation fused
     into it, more rows on the tcgen05 GEMM (split over K up to 128 rows); experts go through the selected-expert kernels
     or the grouped GEMM by the same rule;
@@ -15,33 +13,15 @@ In both modes residual, norms, scores, softmax, router and positions are fp32.  
 from __future__ import annotations
 
 from dataclasses import dataclass
-from typing import Callable, List, Optional, Tuple
+from typing import List, Optional, Tuple
 
 import torch
 
-from ..loading.weights import ModelWeights
 from ..ops import kernels as K
 from ..ops.kernels import DeviceWeight
-from ..quant.ggml import GGMLType
 from .config import AttentionSpec, DenseMlpSpec, MoeMlpSpec
-from .executor import PAGE, BatchDesc, HybridExecutor
-
-# segments of up to this many rows attend through the split-K decode kernel, longer ones through the flash kernel
-DECODE_SEG_ROWS = 8
-EXACT, FEW, MANY = "exact", "few", "many"       # kernel routes of a forward
-
-
-def _up8(n: int) -> int:
-    return -(-n // 8) * 8
-
-
-def _pad(t: torch.Tensor, rows: int, cols: int) -> torch.Tensor:
-    if t.shape == (rows, cols):
-        return t
-    out = torch.zeros(rows, cols, dtype=t.dtype, device=t.device)
-    out[:t.shape[0], :t.shape[1]] = t
-    return out
-
+from .executor import PAGE, BatchDesc
+from .listed import DECODE_SEG_ROWS, EXACT, FEW, MANY, ListedExecutor, pad2, up8
 
 @dataclass
 class _Layer:
@@ -60,44 +40,25 @@ class _Layer:
     s_down: Optional[DeviceWeight] = None
 
 
-class SisisunExecutor(HybridExecutor):
-    keeps_hidden = False
-
-    def __init__(self, weights: ModelWeights, dtype: str = "bfloat16", **kw):
-        if dtype not in ("bfloat16", "float32"):
-            raise ValueError(f"compute dtype {dtype!r} (bfloat16 | float32)")
-        self.exact = dtype == "float32"
-        self.act_dtype = torch.float32 if self.exact else torch.bfloat16
-        self.on_layer_run: Optional[Callable[[int, torch.Tensor], None]] = None    # (run, residual rows) observer
-        super().__init__(weights, **kw)
+class SisisunExecutor(ListedExecutor):
+    readds_embedding = True
 
     # ------------------------------------------------------------------ weights
-    def _load(self, weights: ModelWeights) -> None:
-        cfg, dev = self.cfg, self.device
-        self.hp = hp = _up8(cfg.hidden)
+    def _norm_weight(self, name: str) -> torch.Tensor:
+        v = torch.zeros(self.hp, dtype=torch.float32, device=self.device)
+        v[:self.cfg.hidden] = 1.0 + self._mat(name).float()
+        self.f32[name] = v
+        return v
 
-        def mat(name: str) -> torch.Tensor:
-            t = weights[name]
-            if t.ggml_type == GGMLType.BF16:
-                return t.raw.to(dev).reshape(-1).view(torch.bfloat16).reshape(t.shape)
-            return t.dequant(dev).to(torch.bfloat16)
-
-        def put(name: str, t: torch.Tensor) -> DeviceWeight:
-            w = self.dw[name] = DeviceWeight(int(GGMLType.BF16), t.shape[0], t.shape[1], t.contiguous())
-            return w
-
-        def norm(name: str) -> torch.Tensor:
-            v = torch.zeros(hp, dtype=torch.float32, device=dev)
-            v[:cfg.hidden] = 1.0 + mat(name).float()
-            self.f32[name] = v
-            return v
+    def _load_layers(self) -> None:
+        cfg, dev, hp, mat, put, norm = self.cfg, self.device, self.hp, self._mat, self._put, self._norm_weight
 
         def gate_up(p: str, ff: int) -> torch.Tensor:
-            fp = _up8(ff)
-            return torch.cat([_pad(mat(p + "gate"), fp, hp), _pad(mat(p + "up"), fp, hp)], 0)
+            fp = up8(ff)
+            return torch.cat([pad2(mat(p + "gate"), fp, hp), pad2(mat(p + "up"), fp, hp)], 0)
 
         def glu(name: str, p: str, ff: int) -> Tuple[DeviceWeight, DeviceWeight]:
-            return put(name + "gate_up", gate_up(p, ff)), put(name + "down", _pad(mat(p + "down"), hp, _up8(ff)))
+            return put(name + "gate_up", gate_up(p, ff)), put(name + "down", pad2(mat(p + "down"), hp, up8(ff)))
 
         self.layers: List[_Layer] = []
         for i, spec in enumerate(cfg.layer_specs):
@@ -108,56 +69,29 @@ class SisisunExecutor(HybridExecutor):
             for s in ("q.norm", "k.norm"):
                 self.f32[p + "mix." + s] = mat(p + "mix." + s).float().contiguous()
             L = _Layer(norm(p + "norm1"), norm(p + "norm2") if m is not None else None,
-                       put(p + "qkv", _pad(qkv, _up8(qkv.shape[0]), hp)), self.f32[p + "mix.q.norm"],
+                       put(p + "qkv", pad2(qkv, up8(qkv.shape[0]), hp)), self.f32[p + "mix.q.norm"],
                        self.f32[p + "mix.k.norm"], put(p + "o", o.reshape(hp, -1)))
             if isinstance(m, DenseMlpSpec):
                 L.gate_up, L.down = glu(p, p + "mlp.", m.ff)
             elif isinstance(m, MoeMlpSpec):
-                fp = _up8(m.ff)
+                fp = up8(m.ff)
                 gu = torch.empty(m.experts * 2 * fp, hp, dtype=torch.bfloat16, device=dev)
                 dn = torch.empty(m.experts * hp, fp, dtype=torch.bfloat16, device=dev)
                 for e in range(m.experts):
                     gu[e * 2 * fp:(e + 1) * 2 * fp] = gate_up(p + f"mlp.e{e}.", m.ff)
-                    dn[e * hp:(e + 1) * hp] = _pad(mat(p + f"mlp.e{e}.down"), hp, fp)
+                    dn[e * hp:(e + 1) * hp] = pad2(mat(p + f"mlp.e{e}.down"), hp, fp)
                 L.e_gate_up, L.e_down = put(p + "experts.gate_up", gu), put(p + "experts.down", dn)
                 rows = [mat(p + "mlp.router")]
                 if m.shared_ff:
                     L.s_gate_up, L.s_down = glu(p + "shared.", p + "mlp.shared.", m.shared_ff)
                     rows.append(mat(p + "mlp.shared.sg"))
                 r = torch.cat(rows, 0)
-                L.router = put(p + "router", _pad(r, _up8(r.shape[0]), hp))
+                L.router = put(p + "router", pad2(r, up8(r.shape[0]), hp))
             self.layers.append(L)
-        self.embed_w = put("token_embd.weight", mat("embed"))
-        self.head_w = put("output.weight", _pad(mat("head"), cfg.vocab, hp))
-        norm("final.norm")
-        self.runs = cfg.layer_runs()
-        self.loop_step: Optional[torch.Tensor] = None
-        if cfg.loop is not None:
-            self.loop_step = _pad(mat("loop.step").float(), cfg.loop.times, hp).contiguous()
         i = torch.arange((cfg.hidden + 1) // 2, dtype=torch.float64)
         self.pos_freq = torch.pow(torch.tensor(10000.0, dtype=torch.float64), -2.0 * i / cfg.hidden).to(dev)
 
-    # ------------------------------------------------------------------ state: one KV plane per layer run
-    def _alloc_state(self) -> None:
-        dev = self.device
-        self.conv_state, self.gdn_state = {}, {}
-        self.kv = {}
-        for run, (i, _) in enumerate(self.runs):
-            a = self.cfg.layer_specs[i].mixer
-            self.kv[run] = torch.zeros(self.n_pages, 2, a.kv_heads, PAGE, a.width, dtype=self.act_dtype, device=dev)
-        self._alloc_tables()
-
     # ------------------------------------------------------------------ dispatch
-    def _resid_buffer(self, T: int) -> torch.Tensor:
-        return self.scratch.get("h", (T, self.hp), torch.float32)
-
-    def _norm_rows(self, h: torch.Tensor, w: torch.Tensor) -> torch.Tensor:
-        xn = self.scratch.get("xn", (h.shape[0], self.hp), self.act_dtype)
-        return K.rmsnorm_rows(h, w, xn, self.cfg.rms_eps, n_mean=self.cfg.hidden)
-
-    def _route(self, T: int) -> str:
-        return EXACT if self.exact else FEW if T <= K.FLOAT_GEMV_MAX_ROWS else MANY
-
     def _in_proj(self, h: torch.Tensor, norm_w: torch.Tensor, w: DeviceWeight, name: str, route: str,
                  xn: Optional[torch.Tensor] = None) -> torch.Tensor:
         """norm(h) @ W^T (fp32, or bf16 rows for large batches); ``xn``: the normalised rows when they exist already."""
@@ -300,49 +234,13 @@ class SisisunExecutor(HybridExecutor):
         K.moe_combine(h, ys, pos, wts, k, ysh, sg)
 
     # ------------------------------------------------------------------ whole model
-    def forward(self, b: BatchDesc, journal: Optional[dict] = None, h_out: Optional[torch.Tensor] = None,
-                defer_resid: bool = False) -> torch.Tensor:
-        cfg, T = self.cfg, b.T
-        route = self._route(T)
-        direct = h_out is not None and h_out.shape[1] == self.hp and h_out.is_contiguous()
-        h = h_out if direct else self._resid_buffer(T)
-        lp = cfg.loop
-        x0 = self.scratch.get("embed_out", (T, self.hp), torch.float32) if lp is not None and lp.times > 1 else None
-        K.embed_sinusoid(self.embed_w, b.tokens, b.pos, self.pos_freq, h, x0)
-        for run, (i, t) in enumerate(self.runs):
-            if t >= 0 and i == lp.start:
-                K.resid_inject(h, x0 if t > 0 else None, self.loop_step[t])
-            self._attention(run, i, h, b, route)
-            m = cfg.layer_specs[i].mlp
-            if isinstance(m, DenseMlpSpec):
-                self._dense(self.layers[i], m, h, route)
-            elif isinstance(m, MoeMlpSpec):
-                self._experts(self.layers[i], m, h, route)
-            if self.on_layer_run is not None:
-                self.on_layer_run(run, h[:, :cfg.hidden])
-        if h_out is not None and not direct:
-            h_out.copy_(h[:, :cfg.hidden])
-            return h_out
-        return h
+    def _embed(self, b: BatchDesc, h: torch.Tensor, copy: Optional[torch.Tensor]) -> None:
+        K.embed_sinusoid(self.embed_w, b.tokens, b.pos, self.pos_freq, h, copy)
 
-    def logits(self, h_rows: torch.Tensor, out: Optional[torch.Tensor] = None,
-               hidden_out: Optional[torch.Tensor] = None) -> torch.Tensor:
-        cfg, R = self.cfg, h_rows.shape[0]
-        if h_rows.shape[1] != self.hp:
-            h_rows = _pad(h_rows, R, self.hp)
-        norm_w = self.f32["final.norm"]
-        if out is None:
-            out = self.scratch.get("logits", (R, cfg.vocab), torch.float32)
-        if hidden_out is not None:
-            hid = self.scratch.get("hidden_rows", (R, self.hp), torch.float32)
-            hidden_out.copy_(K.rmsnorm_rows(h_rows, norm_w, hid, cfg.rms_eps, n_mean=cfg.hidden)[:, :cfg.hidden])
-        if self._route(R) == FEW:
-            K.gemv_float(h_rows, [(self.head_w.data, None, out, K.EPI_F32)], norm_w=norm_w, eps=cfg.rms_eps,
-                         norm_n=cfg.hidden)
-            return out
-        xn = self.scratch.get("xn_head", (R, self.hp), self.act_dtype)
-        K.rmsnorm_rows(h_rows, norm_w, xn, cfg.rms_eps, n_mean=cfg.hidden)
-        if self.exact:
-            return K.small_gemm_f32(xn, self.head_w.data, out)
-        from ..ops import gemm as GM
-        return GM.gemm_bf16(xn, self.head_w.data, out)
+    def _layer_run(self, run: int, i: int, h: torch.Tensor, b: BatchDesc, route: str, journal: Optional[dict]) -> None:
+        self._attention(run, i, h, b, route)
+        m = self.cfg.layer_specs[i].mlp
+        if isinstance(m, DenseMlpSpec):
+            self._dense(self.layers[i], m, h, route)
+        elif isinstance(m, MoeMlpSpec):
+            self._experts(self.layers[i], m, h, route)

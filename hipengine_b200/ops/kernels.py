@@ -103,13 +103,26 @@ class _MoeSelArgs(C.Structure):
 
 
 class _FloatGemvSeg(C.Structure):
-    _fields_ = [("w", c_vp), ("w2", c_vp), ("out", c_vp), ("out_stride", c_ll), ("n_rows", C.c_int), ("epi", C.c_int)]
+    _fields_ = [("w", c_vp), ("w2", c_vp), ("out", c_vp), ("x", c_vp), ("out_stride", c_ll), ("n_rows", C.c_int),
+                ("epi", C.c_int)]
 
 
 class _FloatGemvArgs(C.Structure):
     _fields_ = [("seg", _FloatGemvSeg * 4), ("n_seg", C.c_int), ("K", C.c_int), ("ldw", c_ll), ("R", C.c_int),
                 ("x_dtype", C.c_int), ("x", c_vp), ("x_stride", c_ll), ("norm_w", c_vp), ("eps", C.c_float),
-                ("norm_n", C.c_int), ("limit", C.c_float)]
+                ("norm_n", C.c_int), ("limit", C.c_float), ("n_batch", C.c_int), ("w_bs", c_ll), ("x_bs", c_ll),
+                ("out_bs", c_ll)]
+
+
+class _FloatSumArgs(C.Structure):
+    _fields_ = [("w", c_vp * 2), ("x", c_vp * 2), ("scale", c_vp * 2), ("ldw", c_ll * 2), ("x_stride", c_ll * 2),
+                ("K", C.c_int * 2), ("out", c_vp), ("out_stride", c_ll), ("n_rows", C.c_int), ("R", C.c_int)]
+
+
+class _NormShiftArgs(C.Structure):
+    _fields_ = [("x", c_vp), ("ldx", c_ll), ("w", c_vp), ("shift", c_vp), ("state", c_vp), ("journal", c_vp),
+                ("seg_start", c_vp), ("seg_slot", c_vp), ("tok_seg", c_vp), ("h", c_vp), ("hs", c_vp), ("T", C.c_int),
+                ("H", C.c_int), ("n_mean", C.c_int), ("out_bf16", C.c_int), ("n_slots", C.c_int), ("eps", C.c_float)]
 
 
 class _FloatMoeArgs(C.Structure):
@@ -142,6 +155,7 @@ def _check_abi() -> None:
         return
     L = N.lib()
     pairs = [("he_gemv_float_args_size", _FloatGemvArgs), ("he_moe_float_args_size", _FloatMoeArgs),
+             ("he_gemv_sum_args_size", _FloatSumArgs), ("he_norm_shift_args_size", _NormShiftArgs),
              ("he_exact_attn_args_size", _ExactAttnArgs), ("he_exact_moe_args_size", _ExactMoeArgs),
              ("he_gemv_args_size", _GemvArgs), ("he_qkv_args_size", _QkvArgs), ("he_conv_args_size", _ConvArgs),
              ("he_gdn_prep_args_size", _GdnPrepArgs), ("he_gdn_scan_args_size", _GdnScanArgs),
@@ -365,9 +379,11 @@ def _check_device(t: torch.Tensor) -> None:
 
 def embed(w: DeviceWeight, ids: torch.Tensor, out: torch.Tensor, scale: float = 1.0) -> torch.Tensor:
     _check_device(out)
-    assert ids.dtype == torch.int64 and out.dtype == torch.float32
+    """Embedding rows as fp32; rows of ``out`` wider than the table are zero-padded."""
+    assert ids.dtype == torch.int64 and out.dtype == torch.float32 and out.is_contiguous()
     N.check(N.lib().he_embed(c_vp(w.ptr), C.c_int(w.qtype), c_ll(w.n_rows), C.c_int(w.n_cols), c_vp(ids.data_ptr()),
-                             c_vp(out.data_ptr()), C.c_float(scale), C.c_int(ids.numel()), _stream()), "he_embed")
+                             c_vp(out.data_ptr()), C.c_float(scale), C.c_int(ids.numel()), C.c_int(out.shape[-1]),
+                             _stream()), "he_embed")
     return out
 
 
@@ -678,14 +694,14 @@ def moe_down_sel(act_rows: torch.Tensor, ids: torch.Tensor, wts: torch.Tensor, w
 # ----------------------------------------------------------------------------- bfloat16 weights, few rows
 
 FLOAT_GEMV_MAX_ROWS = 16
-EPI_CLAMPED_GLU = 5
+EPI_CLAMPED_GLU, EPI_RELU2 = 5, 6
 EPI_OF_ACT = {"silu": EPI_SILU_MUL, "gelu_tanh": EPI_GELU_MUL, "clamped_glu": EPI_CLAMPED_GLU}
 
 
-def gemv_float(x: torch.Tensor, segs: Sequence[Tuple[torch.Tensor, Optional[torch.Tensor], torch.Tensor, int]],
+def gemv_float(x: torch.Tensor, segs: Sequence[Tuple],
                norm_w: Optional[torch.Tensor] = None, eps: float = 1e-6, norm_n: int = 0, limit: float = 0.0) -> None:
-    """1..16 rows times bf16 weights: ``segs`` are (w [N, K], w2 or None, out, epilogue).  fp32 rows may have the RMS
-    norm fused (mean over ``norm_n`` columns)."""
+    """1..16 rows times bf16 weights: ``segs`` are (w [N, K], w2 or None, out, epilogue[, rows of its own instead of
+    ``x``]).  fp32 rows may have the RMS norm fused (mean over ``norm_n`` columns)."""
     _check_abi()
     _check_device(x)
     R, Kc = x.shape
@@ -693,8 +709,11 @@ def gemv_float(x: torch.Tensor, segs: Sequence[Tuple[torch.Tensor, Optional[torc
     a.n_seg, a.K, a.R = len(segs), segs[0][0].shape[1], R
     a.ldw = segs[0][0].stride(0)
     assert Kc == a.K, (Kc, a.K)
-    for i, (w, w2, out, epi) in enumerate(segs):
+    for i, (w, w2, out, epi, *own) in enumerate(segs):
         sg = a.seg[i]
+        if own:
+            assert own[0].dtype == x.dtype and own[0].shape == x.shape and own[0].stride(0) == x.stride(0)
+            sg.x = own[0].data_ptr()
         assert w.dtype == torch.bfloat16 and w.stride(0) == a.ldw and w.shape[1] == a.K
         assert out.dtype == (torch.float32 if epi in (EPI_F32, EPI_ADD_F32) else torch.bfloat16)
         sg.w, sg.w2, sg.out = w.data_ptr(), _p(w2), out.data_ptr()
@@ -702,6 +721,58 @@ def gemv_float(x: torch.Tensor, segs: Sequence[Tuple[torch.Tensor, Optional[torc
     a.x_dtype, a.x, a.x_stride = _dt(x), x.data_ptr(), x.stride(0)
     a.norm_w, a.eps, a.norm_n, a.limit = _p(norm_w), eps, norm_n or Kc, limit
     N.check(N.lib().he_gemv_float(C.byref(a), _stream()), "he_gemv_float")
+
+
+def gemv_float_batched(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor) -> None:
+    """out[r, b, :N] = x[r, b] @ w[b]^T for every b: ``x`` [R, B, K] (fp32 or bf16, R of any size), ``w`` [B, N, K] bf16,
+    ``out`` [R, B, >= N] fp32 or bf16.  Views with strides are fine; columns of ``out`` past N are not touched."""
+    _check_abi()
+    _check_device(x)
+    R, B, Kc = x.shape
+    assert w.dtype == torch.bfloat16 and w.shape[0] == B and w.shape[2] == Kc and w.stride(2) == x.stride(2) == 1
+    for r0 in range(0, R, FLOAT_GEMV_MAX_ROWS):
+        xr, o = x[r0:r0 + FLOAT_GEMV_MAX_ROWS], out[r0:r0 + FLOAT_GEMV_MAX_ROWS]
+        a = _FloatGemvArgs()
+        a.n_seg, a.K, a.R, a.ldw, a.n_batch = 1, Kc, xr.shape[0], w.stride(1), B
+        a.w_bs, a.x_bs, a.out_bs = w.stride(0), x.stride(1), out.stride(1)
+        sg = a.seg[0]
+        sg.w, sg.out, sg.out_stride, sg.n_rows = w.data_ptr(), o.data_ptr(), out.stride(0), w.shape[1]
+        sg.epi = EPI_F32 if out.dtype == torch.float32 else EPI_BF16
+        a.x_dtype, a.x, a.x_stride, a.norm_n = _dt(x), xr.data_ptr(), x.stride(0), Kc
+        N.check(N.lib().he_gemv_float(C.byref(a), _stream()), "he_gemv_float")
+
+
+def gemv_sum(h: torch.Tensor, parts: Sequence[Tuple[torch.Tensor, torch.Tensor, Optional[torch.Tensor]]]) -> None:
+    """h[r, n] += sum over one or two (x, w, scale) of scale[n] * (x[r] . w[n]); bf16 rows and weights, 1..16 rows."""
+    _check_abi()
+    _check_device(h)
+    assert 1 <= len(parts) <= 2 and h.dtype == torch.float32
+    a = _FloatSumArgs()
+    for i, (x, w, scale) in enumerate(parts):
+        assert x.dtype == w.dtype == torch.bfloat16 and x.shape == (h.shape[0], w.shape[1]) and w.shape[0] == parts[0][1].shape[0]
+        a.w[i], a.x[i], a.scale[i] = w.data_ptr(), x.data_ptr(), _p(scale)
+        a.ldw[i], a.x_stride[i], a.K[i] = w.stride(0), x.stride(0), w.shape[1]
+    a.out, a.out_stride, a.n_rows, a.R = h.data_ptr(), h.stride(0), parts[0][1].shape[0], h.shape[0]
+    N.check(N.lib().he_gemv_sum(C.byref(a), _stream()), "he_gemv_sum")
+
+
+def norm_shift(x: torch.Tensor, w: torch.Tensor, shift: torch.Tensor, state: torch.Tensor, seg_start: torch.Tensor,
+               seg_slot: torch.Tensor, tok_seg: torch.Tensor, h: torch.Tensor, hs: torch.Tensor, eps: float, n_mean: int,
+               journal: Optional[torch.Tensor] = None) -> None:
+    """h = RMSNorm(x) * w, hs[t] = h[t] + shift * (h[t-1] - h[t]) inside every segment; the row before a segment is
+    ``state[slot]``, which then takes the segment's last row (with ``journal`` every row goes there and the state stays)."""
+    _check_abi()
+    T, H = x.shape
+    assert x.dtype == w.dtype == shift.dtype == state.dtype == torch.float32 and h.dtype == hs.dtype
+    assert h.is_contiguous() and hs.is_contiguous() and h.shape == hs.shape == x.shape
+    assert state.is_contiguous() and state.numel() == state.shape[0] * H and w.numel() == shift.numel() == H
+    a = _NormShiftArgs()
+    a.x, a.ldx, a.w, a.shift = x.data_ptr(), x.stride(0), w.data_ptr(), shift.data_ptr()
+    a.state, a.journal, a.n_slots = state.data_ptr(), _p(journal), state.shape[0]
+    a.seg_start, a.seg_slot, a.tok_seg = seg_start.data_ptr(), seg_slot.data_ptr(), tok_seg.data_ptr()
+    a.h, a.hs, a.T, a.H, a.n_mean, a.eps = h.data_ptr(), hs.data_ptr(), T, H, n_mean, eps
+    a.out_bf16 = int(h.dtype == torch.bfloat16)
+    N.check(N.lib().he_norm_shift(C.byref(a), _stream()), "he_norm_shift")
 
 
 def moe_gateup_float(h: torch.Tensor, norm_w: torch.Tensor, eps: float, norm_n: int, ids: torch.Tensor,
@@ -888,14 +959,21 @@ def softcap_(x: torch.Tensor, cap: float) -> None:
     N.check(N.lib().he_softcap(c_vp(x.data_ptr()), c_ll(x.numel()), C.c_float(cap), _stream()), "he_softcap")
 
 
-def small_gemm_f32(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, add: bool = False) -> torch.Tensor:
-    """out[T, N] (fp32) = (or +=) x[T, K] @ w[N, K]^T in fp32 arithmetic; w fp32 (router / ssm_alpha / ssm_beta at
-    prefill) or bf16 (the float32 compute dtype)."""
-    T, K = x.shape
-    Nn = w.shape[0]
-    assert out.dtype == torch.float32 and w.shape[1] == K
+GEMM_STORE, GEMM_ADD, GEMM_RELU2 = 0, 1, 2
+
+
+def small_gemm_f32(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, add: bool = False, mode: int = GEMM_STORE,
+                   col_scale: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """out[T, N] (fp32) = (or +=, or relu(.)^2 of) x[T, K] @ w[N, K]^T in fp32 arithmetic; w fp32 (router / ssm_alpha /
+    ssm_beta at prefill) or bf16 (the float32 compute dtype).  ``col_scale`` [N] multiplies what is added.  Three-dimensional
+    operands x [T, B, K], w [B, N, K], out [T, B, N] are B products."""
+    mode = GEMM_ADD if add else mode
+    assert out.dtype == torch.float32 and w.shape[-1] == x.shape[-1] and (col_scale is None or mode == GEMM_ADD)
+    B = x.shape[1] if x.dim() == 3 else 1
+    bs = (x.stride(1), w.stride(0), out.stride(1)) if x.dim() == 3 else (0, 0, 0)
     N.check(N.lib().he_small_gemm_f32(c_vp(x.data_ptr()), C.c_int(_dt(x)), c_ll(x.stride(0)), c_vp(w.data_ptr()),
-                                      C.c_int(_dt(w)), c_ll(w.stride(0)), c_vp(out.data_ptr()), c_ll(out.stride(0)),
-                                      C.c_int(T), C.c_int(Nn), C.c_int(K), C.c_int(int(add)), _stream()),
+                                      C.c_int(_dt(w)), c_ll(w.stride(-2)), c_vp(out.data_ptr()), c_ll(out.stride(0)),
+                                      C.c_int(x.shape[0]), C.c_int(w.shape[-2]), C.c_int(x.shape[-1]), C.c_int(mode),
+                                      c_vp(_p(col_scale)), C.c_int(B), c_ll(bs[0]), c_ll(bs[1]), c_ll(bs[2]), _stream()),
             "he_small_gemm_f32")
     return out

@@ -53,9 +53,9 @@ class RefModel:
         else:
             self._gemma = None
         self._listed = None
-        if self.cfg.arch == "sisisun":
-            from .sisisun import SisisunRef
-            self._listed = SisisunRef(weights.metadata["config"], self.w)
+        if self.cfg.layer_specs:
+            from ..models.registry import load_object, plugin_for
+            self._listed = load_object(plugin_for(self.cfg.arch).reference)(weights.metadata["config"], self.w)
 
     # -- helpers
     def W(self, i: int, slot: str) -> torch.Tensor:

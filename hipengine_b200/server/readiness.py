@@ -32,7 +32,7 @@ def kv_capability(cfg, kv_cfg) -> Dict[str, Any]:
                          else "CUDA-core split-K",
         "prefill_kernel": "flash (mma.sync)" if hd in (64, 128, 256) else "row-wise decode kernel",
         "prefix_cache": getattr(kv_cfg, "prefix_cache", "off"),
-        "recurrent_state_snapshots": bool(getattr(cfg, "is_hybrid", False)),
+        "recurrent_state_snapshots": bool(getattr(cfg, "has_recurrent_state", False)),
         "sliding_window": bool(getattr(cfg, "sliding_window", 0)),
         "cold_tier": True,
     }

@@ -3,7 +3,8 @@ import json
 
 import torch
 
-from hipengine_b200.loading.sisisun import config_from_json, tensor_shapes, weights_from_tensors
+from hipengine_b200.loading.folder_family import weights_from_tensors
+from hipengine_b200.loading.sisisun import config_from_json, tensor_shapes
 from hipengine_b200.ref.sisisun import SisisunRef, route
 
 
