@@ -122,13 +122,13 @@ def main() -> int:
                          "packed step per token (continuous-batching steady state)")
     ap.add_argument("--no-mtp", action="store_true", help="N = 1: skip the speculative (NextN depth 3) cycle figures")
     ap.add_argument("--mtp-depth", type=int, default=3)
-    ap.add_argument("--beside", default=None, choices=["sisisun"],
+    ap.add_argument("--beside", default=None, choices=["sisisun", "milutar"],
                     help="instead of the workload above: kernels and models of this family beside the closest other "
                          "family at equal size (one JSON line per row)")
     args = ap.parse_args()
     if args.beside:
         from hipengine_b200.benchmark.families import main as families_main
-        return families_main([])
+        return families_main([args.beside])
     if args.impl == "reference":
         return reference_arm(args)
     if args.warmup < 3 and not args.layers:

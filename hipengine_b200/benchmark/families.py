@@ -1,10 +1,10 @@
 """A family beside its closest existing one at equal size: kernel by kernel against the roofline, then whole models.
 
-    python bench.py --beside sisisun            # what this module prints, as one JSON line per row
-    python -m hipengine_b200.benchmark.families [--kernels-only | --models-only]
+    python bench.py --beside sisisun|milutar    # what this module prints, as one JSON line per row
+    python -m hipengine_b200.benchmark.families [family] [--kernels-only | --models-only]
 
-Each kernel row gives the new design's kernel and the like kernel of the closest model (the Qwen3-shaped dense / MoE
-decoder on the hybrid executor), their device times and the fraction of the measured peak that bounds them: HBM for the
+Each kernel row gives the new design's kernel and the like kernel of the closest model (Sisisun beside the Qwen3-shaped
+dense / MoE decoder on the hybrid executor, Milutar beside Sisisun, ``latent_rows.py``), their device times and the fraction of the measured peak that bounds them: HBM for the
 weight or KV streams (every format counts its own bytes), the bf16 tensor peak for the large products.  Operands are
 rotated through more than the L2 holds.  Weights are random.
 """
@@ -17,6 +17,7 @@ from typing import Callable, Dict, List, Optional
 
 import torch
 
+from ..utils.nvml_sampler import NvmlSampler, decode_reasons
 from .micro import peaks, time_launches
 
 L2_POOL = 300e6
@@ -286,16 +287,28 @@ def model_rows(emit: Callable[[Dict], None]) -> None:
 
 def main(argv: Optional[List[str]] = None) -> int:
     ap = argparse.ArgumentParser(prog="families")
+    ap.add_argument("family", nargs="?", default="sisisun", choices=["sisisun", "milutar"])
     ap.add_argument("--kernels-only", action="store_true")
     ap.add_argument("--models-only", action="store_true")
     a = ap.parse_args(argv)
 
     def emit(r: Dict) -> None:
         print(json.dumps(r), flush=True)
-    if not a.models_only:
-        kernel_rows(emit)
-    if not a.kernels_only:
-        model_rows(emit)
+    if a.family == "milutar":
+        from . import latent_rows as rows
+    else:
+        rows = sys.modules[__name__]
+    with NvmlSampler(device_index=torch.cuda.current_device(), interval_s=0.02) as clocks:
+        def emit_clocked(r: Dict) -> None:
+            """The row with the clocks and throttle reasons sampled since the last one."""
+            seen, clocks.samples = clocks.samples, []
+            mhz = sorted(s.sm_mhz for s in seen if s.sm_mhz is not None)
+            reasons = sorted({n for s in seen for n in decode_reasons(s.reasons)})
+            emit({**r, "sm_mhz": mhz[len(mhz) // 2] if mhz else None, "clock_reasons": reasons})
+        if not a.models_only:
+            rows.kernel_rows(emit_clocked)
+        if not a.kernels_only:
+            rows.model_rows(emit_clocked)
     return 0
 
 

@@ -60,7 +60,7 @@ def build_random_folder(cfg: ModelConfig, seed: int = 0, device="cpu", std: floa
     gen.manual_seed(seed)
     tensors: Dict[str, torch.Tensor] = {}
     for n, shape in family_module(cfg).tensor_shapes(cfg).items():
-        t = torch.randn(*shape, generator=gen, device=device, dtype=torch.float32) * std
+        t = torch.randn(tuple(shape), generator=gen, device=device, dtype=torch.float32) * std
         tensors[n] = (adjust(n, t) if adjust is not None else t).to(torch.bfloat16)
     w = weights_from_tensors(cfg, tensors)
     w.metadata["general.name"] = f"random-init {cfg.arch} seed={seed}"
