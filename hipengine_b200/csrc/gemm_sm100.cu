@@ -24,6 +24,7 @@ constexpr int STAGE_BYTES = A_BYTES + B_BYTES;
 constexpr int ACC_COLS = BN;           // fp32 columns per accumulator
 constexpr int TMEM_COLS = 512;
 constexpr int NTHREADS = 192;
+constexpr int EPI_STAGE_BYTES = 4 * 32 * 128;   // per epilogue warp: 32 rows x 128 bytes of output on their way to full lines
 constexpr int NTHREADS_FUSED = 320;    // + 4 collective warps (fused GEMM -> all-reduce kernel)
 
 // Quantised-B mode (QM): the weight stays in its GGUF-derived device layout (Q4_K 144-byte blocks, Q6_K 224-byte
@@ -399,6 +400,120 @@ __device__ __forceinline__ void unpack_q80(const uint8_t* qst, uint8_t* bstage, 
 
 __device__ __forceinline__ int q_kb_per_stage(int qtype) { return qtype == HE_Q4_K ? 4 : 2; }
 
+// Epilogue of one warp: rows [row0, row0 + 32) x columns [col_lo, col_lo + BN) of the accumulator at TMEM address `t_row`.
+// A lane holds a row, so stores straight from the registers would touch 32 lines at a time: 128 bytes per row go through
+// shared memory (16-byte chunks permuted by row: no bank conflicts) and leave as full lines, four rows per instruction.
+__device__ __forceinline__ void store_tile(const GemmArgs& g, uint8_t* stage, uint32_t t_row, int row0, int col_lo, int ks,
+                                           bool empty_split) {
+  const int lane = threadIdx.x & 31;
+  const bool bf = g.epi == 0 || g.epi == 6;
+  const int step = bf ? 64 : 32, ch = lane & 7, rq = lane >> 3;
+#pragma unroll 1
+  for (int c0 = 0; c0 < BN; c0 += step) {
+    const int col0 = col_lo + c0;
+    if (col0 >= g.N) break;
+    uint32_t r[32];
+    tmem_ld_32x32(t_row + c0, r);
+    tmem_ld_wait();
+    if (bf) {
+#pragma unroll
+      for (int half = 0; half < 2; ++half) {
+        if (half == 1) {
+          tmem_ld_32x32(t_row + c0 + 32, r);
+          tmem_ld_wait();
+        }
+        if (g.epi == 6) {
+#pragma unroll
+          for (int e = 0; e < 32; ++e) r[e] = __float_as_uint(he::relu2_f(__uint_as_float(r[e])));
+        }
+#pragma unroll
+        for (int v = 0; v < 4; ++v) {
+          uint4 pk;
+          uint32_t* pw = reinterpret_cast<uint32_t*>(&pk);
+#pragma unroll
+          for (int e = 0; e < 4; ++e) {
+            __nv_bfloat162 h = __floats2bfloat162_rn(__uint_as_float(r[v * 8 + 2 * e]), __uint_as_float(r[v * 8 + 2 * e + 1]));
+            pw[e] = *reinterpret_cast<uint32_t*>(&h);
+          }
+          *reinterpret_cast<uint4*>(stage + lane * 128 + (((half * 4 + v) ^ (lane & 7)) << 4)) = pk;
+        }
+      }
+    } else {
+#pragma unroll
+      for (int v = 0; v < 8; ++v)
+        *reinterpret_cast<uint4*>(stage + lane * 128 + ((v ^ (lane & 7)) << 4)) =
+            make_uint4(r[4 * v], r[4 * v + 1], r[4 * v + 2], r[4 * v + 3]);
+    }
+    __syncwarp();
+    const int per = bf ? 8 : 4, col = col0 + ch * per, left = g.N - col;     // this lane's columns, in four-row steps
+    if (left > 0) {
+      if (bf) {
+        __nv_bfloat16* base = reinterpret_cast<__nv_bfloat16*>(g.C) + col;
+#pragma unroll
+        for (int it = 0; it < 8; ++it) {
+          const int rl = it * 4 + rq, row = row0 + rl;
+          if (row >= g.M) break;
+          const uint4 v = *reinterpret_cast<const uint4*>(stage + rl * 128 + ((ch ^ (rl & 7)) << 4));
+          __nv_bfloat16* dst = base + (size_t)row * g.ldc;
+          if (left >= 8 && (reinterpret_cast<uintptr_t>(dst) & 15) == 0) {
+            *reinterpret_cast<uint4*>(dst) = v;
+          } else {
+            const __nv_bfloat16* x = reinterpret_cast<const __nv_bfloat16*>(&v);
+#pragma unroll
+            for (int e = 0; e < 8; ++e)
+              if (e < left) dst[e] = x[e];
+          }
+        }
+      } else {
+        float* base = reinterpret_cast<float*>(g.C) + col + (g.epi == 4 ? (size_t)ks * (size_t)g.split_stride : (size_t)0);
+        const bool vec = left >= 4 && ((reinterpret_cast<uintptr_t>(base) | (uintptr_t)(g.ldc * 4)) & 15) == 0;
+        float4 sc = make_float4(1.f, 1.f, 1.f, 1.f);
+        if (g.epi == 2 && g.col_scale != nullptr) {
+          sc.x = __ldg(g.col_scale + col);
+          if (left > 1) sc.y = __ldg(g.col_scale + col + 1);
+          if (left > 2) sc.z = __ldg(g.col_scale + col + 2);
+          if (left > 3) sc.w = __ldg(g.col_scale + col + 3);
+        }
+        float4 old[8];
+        if (g.epi == 2 && vec) {
+#pragma unroll
+          for (int it = 0; it < 8; ++it) {
+            const int row = row0 + it * 4 + rq;
+            if (row < g.M) old[it] = *reinterpret_cast<const float4*>(base + (size_t)row * g.ldc);
+          }
+        }
+#pragma unroll
+        for (int it = 0; it < 8; ++it) {
+          const int rl = it * 4 + rq, row = row0 + rl;
+          if (row >= g.M) break;
+          float4 v = *reinterpret_cast<const float4*>(stage + rl * 128 + ((ch ^ (rl & 7)) << 4));
+          v.x *= sc.x; v.y *= sc.y; v.z *= sc.z; v.w *= sc.w;
+          float* dst = base + (size_t)row * g.ldc;
+          if (g.epi == 3) {
+            if (!empty_split) {
+              const float x[4] = {v.x, v.y, v.z, v.w};
+#pragma unroll
+              for (int e = 0; e < 4; ++e)
+                if (e < left) atomicAdd(dst + e, x[e]);
+            }
+          } else if (vec) {
+            if (g.epi == 2) {
+              v.x += old[it].x; v.y += old[it].y; v.z += old[it].z; v.w += old[it].w;
+            }
+            *reinterpret_cast<float4*>(dst) = v;
+          } else {
+            const float x[4] = {v.x, v.y, v.z, v.w};
+#pragma unroll
+            for (int e = 0; e < 4; ++e)
+              if (e < left) dst[e] = g.epi == 2 ? dst[e] + x[e] : x[e];
+          }
+        }
+      }
+    }
+    __syncwarp();
+  }
+}
+
 template <bool FUSE, bool QM>
 __device__ __forceinline__ void gemm_body(const CUtensorMap& tmA, const CUtensorMap& tmB, const CUtensorMap& tmQ1,
                                           const CUtensorMap& tmQ2, const GemmArgs& g, const FuseArgs* f) {
@@ -407,7 +522,9 @@ __device__ __forceinline__ void gemm_body(const CUtensorMap& tmA, const CUtensor
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~(uintptr_t)1023);
   constexpr int NST = QM ? STAGES_Q : STAGES;
   uint8_t* qring = smem + NST * STAGE_BYTES;                     // QM only: QSTAGES x Q_STAGE_BYTES
-  Barriers* bar = reinterpret_cast<Barriers*>(smem + NST * STAGE_BYTES + (QM ? QSTAGES * Q_STAGE_BYTES : 0));
+  uint8_t* epi_stage = smem + NST * STAGE_BYTES;                 // plain kernel only
+  Barriers* bar = reinterpret_cast<Barriers*>(smem + NST * STAGE_BYTES + (QM ? QSTAGES * Q_STAGE_BYTES : 0) +
+                                              (!FUSE && !QM ? EPI_STAGE_BYTES : 0));
   volatile int* abort_flag = &bar->abort_flag;
   constexpr int WARP_Q = FUSE ? 10 : 6;                          // QM: raw-block producer warp, then the unpack warps
 
@@ -599,15 +716,13 @@ __device__ __forceinline__ void gemm_body(const CUtensorMap& tmA, const CUtensor
       const uint32_t acc_ph = (tcount >> 1) & 1;
       if (!mbar_wait(&bar->acc_full[acc], acc_ph, abort_flag, g.status, 104)) break;
       tc_fence_after();
-      const int row = tm * BM + q * 32 + lane;
       const uint32_t t_row = tmem_base + acc * ACC_COLS + ((uint32_t)(q * 32) << 16);
+      if constexpr (FUSE) {
 #pragma unroll 1
-      for (int c = 0; c < BN / 32; ++c) {
-        uint32_t r[32];
-        tmem_ld_32x32(t_row + c * 32, r);
-        tmem_ld_wait();
-        const int col0 = tn * BN + c * 32;
-        if constexpr (FUSE) {
+        for (int c = 0; c < BN / 32; ++c) {
+          uint32_t r[32];
+          tmem_ld_32x32(t_row + c * 32, r);
+          tmem_ld_wait();
           // partial quarter -> the owner's stage slot; rows and columns past M / N are zeros (zero-filled operand
           // tiles), so the whole tile is stored and no bound is needed
           uint4 pk[4];
@@ -639,62 +754,9 @@ __device__ __forceinline__ void gemm_body(const CUtensorMap& tmA, const CUtensor
 #pragma unroll
             for (int v = 0; v < 4; ++v) *reinterpret_cast<uint4*>(dst + v * 256) = pk[v];
           }
-        } else
-        if (row < g.M && col0 < g.N) {
-          const int ncols = min(32, g.N - col0);
-          if (g.epi == 6) {
-#pragma unroll
-            for (int e = 0; e < 32; ++e) r[e] = __float_as_uint(he::relu2_f(__uint_as_float(r[e])));
-          } else if (g.epi == 2 && g.col_scale != nullptr) {
-#pragma unroll
-            for (int e = 0; e < 32; ++e)
-              if (e < ncols) r[e] = __float_as_uint(__uint_as_float(r[e]) * __ldg(g.col_scale + col0 + e));
-          }
-          if (g.epi == 0 || g.epi == 6) {
-            __nv_bfloat16* dst = reinterpret_cast<__nv_bfloat16*>(g.C) + (size_t)row * g.ldc + col0;
-            if (ncols == 32 && ((reinterpret_cast<uintptr_t>(dst) & 15) == 0)) {
-#pragma unroll
-              for (int v = 0; v < 4; ++v) {
-                uint4 pk;
-                uint32_t* pw = reinterpret_cast<uint32_t*>(&pk);
-#pragma unroll
-                for (int e = 0; e < 4; ++e) {
-                  __nv_bfloat162 h = __floats2bfloat162_rn(__uint_as_float(r[v * 8 + 2 * e]),
-                                                           __uint_as_float(r[v * 8 + 2 * e + 1]));
-                  pw[e] = *reinterpret_cast<uint32_t*>(&h);
-                }
-                *reinterpret_cast<uint4*>(dst + v * 8) = pk;
-              }
-            } else {
-              for (int e = 0; e < ncols; ++e) dst[e] = __float2bfloat16_rn(__uint_as_float(r[e]));
-            }
-          } else {
-            float* dst = reinterpret_cast<float*>(g.C) + (size_t)row * g.ldc + col0 +
-                         (g.epi == 4 ? (size_t)ks_e * (size_t)g.split_stride : (size_t)0);
-            const bool vec = ncols == 32 && (reinterpret_cast<uintptr_t>(dst) & 15) == 0;
-            if ((g.epi == 1 || g.epi == 4) && vec) {
-#pragma unroll
-              for (int v = 0; v < 8; ++v)
-                reinterpret_cast<float4*>(dst)[v] =
-                    make_float4(__uint_as_float(r[4 * v]), __uint_as_float(r[4 * v + 1]), __uint_as_float(r[4 * v + 2]),
-                                __uint_as_float(r[4 * v + 3]));
-            } else if (g.epi == 2 && vec) {
-#pragma unroll
-              for (int v = 0; v < 8; ++v) {
-                float4 o = reinterpret_cast<float4*>(dst)[v];
-                o.x += __uint_as_float(r[4 * v]); o.y += __uint_as_float(r[4 * v + 1]);
-                o.z += __uint_as_float(r[4 * v + 2]); o.w += __uint_as_float(r[4 * v + 3]);
-                reinterpret_cast<float4*>(dst)[v] = o;
-              }
-            } else if (g.epi == 1 || g.epi == 4) {
-              for (int e = 0; e < ncols; ++e) dst[e] = __uint_as_float(r[e]);
-            } else if (g.epi == 2) {
-              for (int e = 0; e < ncols; ++e) dst[e] += __uint_as_float(r[e]);
-            } else if (!empty_split) {
-              for (int e = 0; e < ncols; ++e) atomicAdd(dst + e, __uint_as_float(r[e]));
-            }
-          }
         }
+      } else {
+        store_tile(g, epi_stage + q * 32 * 128, t_row, tm * BM + q * 32, tn * BN, ks_e, empty_split);
       }
       tc_fence_before();
       __syncwarp();
@@ -871,6 +933,7 @@ int make_qmaps(QMaps* q, const void* B, int qtype, long long rows, int K) {
   return -HE_ERR_BAD_ARG;
 }
 
+constexpr size_t SMEM_PLAIN = STAGES * STAGE_BYTES + EPI_STAGE_BYTES + sizeof(Barriers) + 1024;
 constexpr size_t SMEM_Q = STAGES_Q * STAGE_BYTES + QSTAGES * Q_STAGE_BYTES + sizeof(Barriers) + 1024;
 
 }  // namespace
@@ -894,7 +957,7 @@ HE_API int he_gemm_bf16(const void* A, long long lda, const void* B, long long l
   g.split_stride = 0;
   g.qtype = 0;
   g.kb_per = 0;
-  const size_t smem = STAGES * STAGE_BYTES + sizeof(Barriers) + 1024;
+  const size_t smem = SMEM_PLAIN;
   // the attribute is per device: set it on every call (cheap) rather than once per process
   cudaError_t e = cudaFuncSetAttribute(gemm_bf16_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
   if (e != cudaSuccess) return (int)e;
@@ -969,7 +1032,7 @@ HE_API int he_gemm_bf16_grouped(const void* A, long long lda, const void* B, lon
   g.split_stride = 0;
   g.qtype = 0;
   g.kb_per = 0;
-  const size_t smem = STAGES * STAGE_BYTES + sizeof(Barriers) + 1024;
+  const size_t smem = SMEM_PLAIN;
   cudaError_t e = cudaFuncSetAttribute(gemm_bf16_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
   if (e != cudaSuccess) return (int)e;
   const int tiles = ((M + BM - 1) / BM) * ((N + BN - 1) / BN);
@@ -1047,7 +1110,7 @@ HE_API int he_gemm_bf16_splitk_det(const void* A, long long lda, const void* B, 
   g.tile_group = nullptr;
   g.k_splits = k_splits;
   g.split_stride = (long long)M * N;
-  const size_t smem = STAGES * STAGE_BYTES + sizeof(Barriers) + 1024;
+  const size_t smem = SMEM_PLAIN;
   cudaError_t e = cudaFuncSetAttribute(gemm_bf16_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
   if (e != cudaSuccess) return (int)e;
   const int tiles = ((M + BM - 1) / BM) * ((N + BN - 1) / BN);
@@ -1083,7 +1146,7 @@ HE_API int he_gemm_bf16_splitk(const void* A, long long lda, const void* B, long
   g.tile_group = nullptr;
   g.k_splits = k_splits;
   g.split_stride = 0;
-  const size_t smem = STAGES * STAGE_BYTES + sizeof(Barriers) + 1024;
+  const size_t smem = SMEM_PLAIN;
   cudaError_t e = cudaFuncSetAttribute(gemm_bf16_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
   if (e != cudaSuccess) return (int)e;
   const int total = tiles * k_splits;

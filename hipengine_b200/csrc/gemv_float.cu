@@ -163,22 +163,22 @@ __device__ __forceinline__ float inv_rms_of(const Tile<MT, NT>& sm, int col, int
   return rsqrtf(s / (float)n + eps);
 }
 
-// acc += W[16 MT rows][K] x[K][8 NT]: this warp's units.  wrow[m][half] points at column 8c of row (g + 8 half) of tile m.
+// acc += W[16 MT rows][K] x[K][8 NT]: this warp's units (every STEP-th one).  wrow[m][half] points at column 8c of row (g + 8 half) of tile m.
 // EARLY: the weights do not depend on earlier kernels, so the first batch is requested before griddepcontrol.wait.
-template <int MT, int NT, bool XF32, bool EARLY>
+template <int MT, int NT, bool XF32, bool EARLY, int STEP = NW>
 __device__ __forceinline__ void product(const __nv_bfloat16* const (&wrow)[MT][2], int K, const void* x,
                                         long long x_stride, int R, const float* norm_w, float (&acc)[MT][NT][4],
                                         float (&ss)[NT]) {
   constexpr int UN = MT == 1 ? 4 : 2;                    // units in flight per warp: 16 x 16 bytes per lane
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, g = lane >> 2, c = lane & 3;
-  const int units = (K + UK - 1) / UK;
+  const int units = (K + UK - 1) / UK, first = STEP == NW ? warp : 0;
   uint4 A[UN][2][MT][2];
   auto load_a = [&](int u0) {
 #pragma unroll
     for (int i = 0; i < UN; ++i)
 #pragma unroll
       for (int s = 0; s < 2; ++s) {
-        const int k = (u0 + i * NW) * UK + s * 32;
+        const int k = (u0 + i * STEP) * UK + s * 32;
         const bool live = k + 8 * c < K;
 #pragma unroll
         for (int m = 0; m < MT; ++m)
@@ -188,16 +188,16 @@ __device__ __forceinline__ void product(const __nv_bfloat16* const (&wrow)[MT][2
       }
   };
   if (EARLY) {
-    load_a(warp);
+    load_a(first);
     pdl_wait();
   }
-  for (int u0 = warp; u0 < units; u0 += UN * NW) {
-    if (!EARLY || u0 != warp) load_a(u0);
+  for (int u0 = first; u0 < units; u0 += UN * STEP) {
+    if (!EARLY || u0 != first) load_a(u0);
 #pragma unroll
     for (int i = 0; i < UN; ++i)
 #pragma unroll
       for (int s = 0; s < 2; ++s) {
-        const int k = (u0 + i * NW) * UK + s * 32 + 8 * c;
+        const int k = (u0 + i * STEP) * UK + s * 32 + 8 * c;
 #pragma unroll
         for (int n = 0; n < NT; ++n) {
           const int r = n * 8 + g;
@@ -259,6 +259,36 @@ __global__ void __launch_bounds__(NW * 32, 2) gemv_float_kernel(const __grid_con
       reinterpret_cast<float*>(sg.out)[off] += v;
     }
   }
+}
+
+// Short rows (K too small to share between the warps of a CTA): every warp owns 16 output columns and all of K.
+// grid (ceil(n_rows / 128), batches), one segment, plain store
+template <int NT, bool XF32>
+__global__ void __launch_bounds__(NW * 32, 2) gemv_short_kernel(const __grid_constant__ FloatGemvArgs a) {
+  pdl_launch();
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, g = lane >> 2, c = lane & 3;
+  const FloatGemvSeg& sg = a.seg[0];
+  const size_t bt = blockIdx.y;
+  const int row0 = (blockIdx.x * NW + warp) * 16;
+  if (row0 >= sg.n_rows) return;
+  const void* xs = XF32 ? (const void*)(reinterpret_cast<const float*>(a.x) + bt * a.x_bs)
+                        : (const void*)(reinterpret_cast<const __nv_bfloat16*>(a.x) + bt * a.x_bs);
+  const __nv_bfloat16* w0 = sg.w + bt * a.w_bs + 8 * c;
+  const __nv_bfloat16* wrow[1][2] = {{w0 + (size_t)min(row0 + g, sg.n_rows - 1) * a.ldw,
+                                      w0 + (size_t)min(row0 + g + 8, sg.n_rows - 1) * a.ldw}};
+  float acc[1][NT][4] = {};
+  float ss[NT] = {};
+  product<1, NT, XF32, true, 1>(wrow, a.K, xs, a.x_stride, a.R, nullptr, acc, ss);
+#pragma unroll
+  for (int n = 0; n < NT; ++n)
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      const int row = row0 + g + (e >> 1) * 8, col = n * 8 + 2 * c + (e & 1);
+      if (row >= sg.n_rows || col >= a.R) continue;
+      const size_t off = bt * a.out_bs + (size_t)col * sg.out_stride + row;
+      if (sg.epi == 0) reinterpret_cast<float*>(sg.out)[off] = acc[0][n][e];
+      else reinterpret_cast<__nv_bfloat16*>(sg.out)[off] = f32_to_bf16(acc[0][n][e]);
+    }
 }
 
 // grid: items of 16 output columns
@@ -426,6 +456,14 @@ HE_API int he_gemv_float(const FloatGemvArgs* args, cudaStream_t stream) {
         (pair && a.seg[i].w2 == nullptr))
       return -HE_ERR_BAD_ARG;
     items += (a.seg[i].n_rows + 15) / 16;
+  }
+  if (a.n_seg == 1 && a.norm_w == nullptr && a.seg[0].epi <= 1 && a.seg[0].x == nullptr && a.K <= 4 * UK && a.n_batch > 1) {
+    const dim3 grid((a.seg[0].n_rows + NW * 16 - 1) / (NW * 16), a.n_batch), block(NW * 32);
+    if (a.x_dtype == 0)
+      return (int)(a.R <= 8 ? launch_pdl(gemv_short_kernel<1, true>, grid, block, 0, stream, a)
+                            : launch_pdl(gemv_short_kernel<2, true>, grid, block, 0, stream, a));
+    return (int)(a.R <= 8 ? launch_pdl(gemv_short_kernel<1, false>, grid, block, 0, stream, a)
+                          : launch_pdl(gemv_short_kernel<2, false>, grid, block, 0, stream, a));
   }
   return pair ? launch_rows<2>(a, items, stream) : launch_rows<1>(a, items, stream);
 }

@@ -34,7 +34,7 @@ struct LatentDecArgs {
   const int* block_table;
   const int* slot;           // [R]
   const int* ctx_len;        // [R] keys up to and including the row's own
-  float* partial;            // [R][H][max_splits][rank_cols + 2]
+  float* partial;            // [R][H][max_splits][rank_cols], then (maximum, sum) [R][H][max_splits][2]
   void* out;                 // [R][H][rank_cols]
   const float* sink;         // [H] or null: one more term in the softmax denominator
   int R, H, W, rank_cols, page, max_pages, split_len, max_splits, window;
@@ -161,26 +161,29 @@ __device__ __forceinline__ void mma_bf16(float (&c)[4], const uint32_t (&a)[4], 
 }
 __device__ __forceinline__ uint32_t smem_addr(const void* p) { return (uint32_t)__cvta_generic_to_shared(p); }
 
-constexpr int DEC_WARPS = 8;
+constexpr int DEC_WARPS = 16;
 
 template <int MT, int TK>
 __host__ __device__ inline size_t dec_smem(int W) {
-  return (size_t)(MT * 16 + 2 * TK) * (W * 2 + 16) + (size_t)MT * 16 * ((TK + 4) * 4 + (TK * 2 + 16)) + MT * 16 * 3 * 4;
+  return (size_t)(MT * 16 + 2 * TK) * (W * 2 + 16) +
+         (size_t)MT * 16 * ((256 / TK) * (TK + 4) * 4 + (TK * 2 + 16)) + MT * 16 * 3 * 4;
 }
 
 // One CTA per (key span, chunk of up to 16 MT heads, row).  Tiles of TK latent rows are double-buffered with cp.async (rows
-// padded by 16 bytes: conflict-free ldmatrix); per tile: scores (a warp takes eight keys), running maximum and sum per head,
-// then the weighted sum (a warp owns every eighth block of 16 latent columns, up to NB blocks).
+// padded by 16 bytes: conflict-free ldmatrix).  Per tile: partial scores (the warps split 16-key groups and the columns, so
+// the queries are read from shared memory TK / 16 times and not once per warp), running maximum and sum per head, then the
+// weighted sum (a warp owns every sixteenth block of 16 latent columns, up to NB blocks).
 template <int MT, int NB, int TK>
 __global__ void __launch_bounds__(DEC_WARPS * 32) latent_decode_kernel(const LatentDecArgs a) {
   extern __shared__ __align__(16) uint8_t smem[];
   constexpr int MR = MT * 16, SP = TK + 4, PP = TK * 2 + 16;
+  constexpr int KG = TK / 16, KS = DEC_WARPS / KG;        // key groups, column shares
   const int pitch = a.W * 2 + 16, chunks16 = a.W / 8;
   uint8_t* q_s = smem;                                    // [MR][pitch]
   uint8_t* kv_s = q_s + (size_t)MR * pitch;               // [2][TK][pitch]
   uint8_t* p_s = kv_s + (size_t)2 * TK * pitch;           // [MR][PP] bf16 weights
-  float* sc = reinterpret_cast<float*>(p_s + MR * PP);    // [MR][SP]
-  float* m_s = sc + MR * SP;
+  float* sc = reinterpret_cast<float*>(p_s + MR * PP);    // [KS][MR][SP] partial scores
+  float* m_s = sc + KS * MR * SP;
   float* l_s = m_s + MR;
   float* corr_s = l_s + MR;
   const int sp = blockIdx.x, r = blockIdx.z, per = (a.H + gridDim.y - 1) / gridDim.y, h0 = blockIdx.y * per;
@@ -221,7 +224,7 @@ __global__ void __launch_bounds__(DEC_WARPS * 32) latent_decode_kernel(const Lat
     corr_s[tid] = 0.f;
   }
 
-  const int n_blk = a.rank_cols / 16;
+  const int n_blk = a.rank_cols / 16, kg = warp % KG, kq = warp / KG;
   float o[MT][NB][2][4];
 #pragma unroll
   for (int m = 0; m < MT; ++m)
@@ -237,45 +240,56 @@ __global__ void __launch_bounds__(DEC_WARPS * 32) latent_decode_kernel(const Lat
     cp_async_wait<1>();
     __syncthreads();
     const uint8_t* kt = kv_s + (size_t)buf * TK * pitch;
-    // ---- scores of eight keys per warp
-    for (int nb = warp; nb < TK / 8; nb += DEC_WARPS) {
+    // ---- partial scores of 16 keys over this warp's columns (every KS-th group of 32)
+    {
       float s[MT][2][4];
 #pragma unroll
       for (int m = 0; m < MT; ++m)
 #pragma unroll
         for (int e = 0; e < 4; ++e) s[m][0][e] = s[m][1][e] = 0.f;
-      const uint32_t k_addr = smem_addr(kt + (size_t)(nb * 8 + (lane & 7)) * pitch + (lane >> 3) * 16);
+      const uint32_t k_addr = smem_addr(kt + (size_t)(kg * 16 + (lane & 7)) * pitch + (lane >> 3) * 16);
       const uint32_t q_addr = smem_addr(q_s + (size_t)(lane & 15) * pitch + (lane >> 4) * 16);
-#pragma unroll 4
-      for (int ks = 0; ks < a.W / 32; ++ks) {
-        uint32_t kf[4];
-        ldsm_x4(k_addr + ks * 64, kf);
+      if (kg * 16 < live) {
+#pragma unroll 2
+        for (int ks = kq; ks < a.W / 32; ks += KS) {
+          uint32_t ka[4], kb[4];
+          ldsm_x4(k_addr + ks * 64, ka);
+          ldsm_x4(k_addr + 8 * pitch + ks * 64, kb);
 #pragma unroll
-        for (int m = 0; m < MT; ++m) {
-          uint32_t qa[4], qb[4];
-          ldsm_x4(q_addr + m * 16 * pitch + ks * 64, qa);
-          ldsm_x4(q_addr + m * 16 * pitch + ks * 64 + 32, qb);
-          mma_bf16(s[m][0], qa, kf[0], kf[1]);
-          mma_bf16(s[m][1], qb, kf[2], kf[3]);
+          for (int m = 0; m < MT; ++m) {
+            uint32_t qa[4], qb[4];
+            ldsm_x4(q_addr + m * 16 * pitch + ks * 64, qa);
+            ldsm_x4(q_addr + m * 16 * pitch + ks * 64 + 32, qb);
+            mma_bf16(s[m][0], qa, ka[0], ka[1]);
+            mma_bf16(s[m][1], qa, kb[0], kb[1]);
+            mma_bf16(s[m][0], qb, ka[2], ka[3]);
+            mma_bf16(s[m][1], qb, kb[2], kb[3]);
+          }
         }
       }
-      const int col = nb * 8 + 2 * c;
+      float* dst = sc + (size_t)kq * MR * SP + kg * 16 + 2 * c;
 #pragma unroll
       for (int m = 0; m < MT; ++m)
 #pragma unroll
-        for (int e = 0; e < 4; ++e) {
-          const int k = col + (e & 1);
-          sc[(m * 16 + g + (e >> 1) * 8) * SP + k] = k < live ? (s[m][0][e] + s[m][1][e]) * a.scale : -INFINITY;
+        for (int b = 0; b < 2; ++b) {
+          *reinterpret_cast<float2*>(dst + (m * 16 + g) * SP + b * 8) = make_float2(s[m][b][0], s[m][b][1]);
+          *reinterpret_cast<float2*>(dst + (m * 16 + g + 8) * SP + b * 8) = make_float2(s[m][b][2], s[m][b][3]);
         }
     }
     __syncthreads();
     // ---- running maximum and sum per head
-    for (int h = warp; h < gc; h += DEC_WARPS) {
+#pragma unroll
+    for (int hh = 0; hh < MT; ++hh) {
+      const int h = warp + hh * DEC_WARPS;
+      if (h >= gc) break;
       float v[TK / 32], mx = m_s[h];
       const float m_old = mx;
 #pragma unroll
       for (int i = 0; i < TK / 32; ++i) {
-        v[i] = sc[h * SP + i * 32 + lane];
+        float x = 0.f;
+#pragma unroll
+        for (int k = 0; k < KS; ++k) x += sc[(k * MR + h) * SP + i * 32 + lane];
+        v[i] = i * 32 + lane < live ? x * a.scale : -INFINITY;
         mx = fmaxf(mx, v[i]);
       }
       mx = warp_max(mx);
@@ -332,12 +346,11 @@ __global__ void __launch_bounds__(DEC_WARPS * 32) latent_decode_kernel(const Lat
     }
     __syncthreads();
   }
-  const int stride = a.rank_cols + 2;
-  float* part = a.partial + (((size_t)r * a.H + h0) * a.max_splits + sp) * stride;
-  const size_t head_stride = (size_t)a.max_splits * stride;
+  float* part = a.partial + (((size_t)r * a.H + h0) * a.max_splits + sp) * a.rank_cols;
+  const size_t head_stride = (size_t)a.max_splits * a.rank_cols;
   if (tid < gc) {
-    part[tid * head_stride + a.rank_cols] = m_s[tid];
-    part[tid * head_stride + a.rank_cols + 1] = l_s[tid];
+    float2* ml = reinterpret_cast<float2*>(a.partial + (size_t)a.R * a.H * head_stride);
+    ml[((size_t)r * a.H + h0 + tid) * a.max_splits + sp] = make_float2(m_s[tid], l_s[tid]);
   }
 #pragma unroll
   for (int m = 0; m < MT; ++m)
@@ -356,53 +369,73 @@ __global__ void __launch_bounds__(DEC_WARPS * 32) latent_decode_kernel(const Lat
     }
 }
 
-// grid (H, R): merge the spans, add the sink to the denominator, round to bf16
-__global__ void __launch_bounds__(128) latent_reduce_kernel(const LatentDecArgs a) {
+// grid (H, R, ceil(rank_cols / 128)): merge the spans (the eight warps take them in turn, a lane owns four columns), add the
+// sink to the denominator, round to bf16
+constexpr int RED_WARPS = 8;
+__global__ void __launch_bounds__(RED_WARPS * 32) latent_reduce_kernel(const LatentDecArgs a) {
   extern __shared__ float wsm[];     // [max_splits]
   __shared__ float red[33];
+  __shared__ float4 acc_s[RED_WARPS][32];
   pdl_wait();
   pdl_launch();
-  const int h = blockIdx.x, r = blockIdx.y, stride = a.rank_cols + 2;
+  const int h = blockIdx.x, r = blockIdx.y, lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
   const int ctx = a.ctx_len[r];
   const int start = (a.window > 0 && ctx > a.window) ? ctx - a.window : 0;
   const int ns = min((ctx - start + a.split_len - 1) / a.split_len, a.max_splits);
-  const float* pb = a.partial + ((size_t)r * a.H + h) * a.max_splits * stride;
+  const size_t row = ((size_t)r * a.H + h) * a.max_splits;
+  const float2* ml = reinterpret_cast<const float2*>(a.partial + (size_t)a.R * a.H * a.max_splits * a.rank_cols) + row;
+  const int d = blockIdx.z * 128 + lane * 4;
+  const float* pb = a.partial + row * a.rank_cols + d;
+  const bool mine = d < a.rank_cols;
+  // the first spans' columns are requested before their weights are known
+  constexpr int AHEAD = 4;
+  float4 x[AHEAD];
+#pragma unroll
+  for (int u = 0; u < AHEAD; ++u) {
+    const int s = warp + u * RED_WARPS;
+    x[u] = mine && s < ns ? *reinterpret_cast<const float4*>(pb + (size_t)s * a.rank_cols) : make_float4(0.f, 0.f, 0.f, 0.f);
+  }
   float m = a.sink != nullptr ? a.sink[h] : -INFINITY;
   const float sk = m;
-  for (int s = threadIdx.x; s < ns; s += 128) {
-    const float ms = pb[(size_t)s * stride + a.rank_cols];
-    wsm[s] = ms;
-    m = fmaxf(m, ms);
-  }
+  for (int s = threadIdx.x; s < ns; s += RED_WARPS * 32) m = fmaxf(m, ml[s].x);
   m = block_max(m, red);
   float den = 0.f;
-  for (int s = threadIdx.x; s < ns; s += 128) {
-    const float w = __expf(wsm[s] - m);
+  for (int s = threadIdx.x; s < ns; s += RED_WARPS * 32) {
+    const float2 v = ml[s];
+    const float w = __expf(v.x - m);
     wsm[s] = w;
-    den += w * pb[(size_t)s * stride + a.rank_cols + 1];
+    den += w * v.y;
   }
   den = block_sum(den, red);         // its barriers also publish wsm
   if (a.sink != nullptr) den += __expf(sk - m);
-  const float inv = den > 0.f ? 1.f / den : 0.f;
-  __nv_bfloat16* out = reinterpret_cast<__nv_bfloat16*>(a.out) + ((size_t)r * a.H + h) * a.rank_cols;
-  for (int d = threadIdx.x * 2; d < a.rank_cols; d += 256) {
-    float2 v[4] = {};
-    int s = 0;
-    for (; s + 4 <= ns; s += 4)
+  float4 acc = make_float4(0.f, 0.f, 0.f, 0.f);
+  for (int s0 = warp; s0 < ns; s0 += AHEAD * RED_WARPS) {
+    if (s0 != warp) {
 #pragma unroll
-      for (int u = 0; u < 4; ++u) {
-        const float2 x = *reinterpret_cast<const float2*>(pb + (size_t)(s + u) * stride + d);
-        v[u].x += wsm[s + u] * x.x;
-        v[u].y += wsm[s + u] * x.y;
+      for (int u = 0; u < AHEAD; ++u) {
+        const int s = s0 + u * RED_WARPS;
+        x[u] = mine && s < ns ? *reinterpret_cast<const float4*>(pb + (size_t)s * a.rank_cols) : make_float4(0.f, 0.f, 0.f, 0.f);
       }
-    for (; s < ns; ++s) {
-      const float2 x = *reinterpret_cast<const float2*>(pb + (size_t)s * stride + d);
-      v[0].x += wsm[s] * x.x;
-      v[0].y += wsm[s] * x.y;
     }
-    *reinterpret_cast<__nv_bfloat162*>(out + d) =
-        __floats2bfloat162_rn(((v[0].x + v[1].x) + (v[2].x + v[3].x)) * inv, ((v[0].y + v[1].y) + (v[2].y + v[3].y)) * inv);
+#pragma unroll
+    for (int u = 0; u < AHEAD; ++u) {
+      const int s = s0 + u * RED_WARPS;
+      const float w = s < ns ? wsm[s] : 0.f;
+      acc.x += w * x[u].x; acc.y += w * x[u].y; acc.z += w * x[u].z; acc.w += w * x[u].w;
+    }
   }
+  acc_s[warp][lane] = acc;
+  __syncthreads();
+  if (warp != 0 || !mine) return;
+#pragma unroll
+  for (int w = 1; w < RED_WARPS; ++w) {
+    const float4 v = acc_s[w][lane];
+    acc.x += v.x; acc.y += v.y; acc.z += v.z; acc.w += v.w;
+  }
+  const float inv = den > 0.f ? 1.f / den : 0.f;
+  __align__(8) __nv_bfloat162 b[2] = {__floats2bfloat162_rn(acc.x * inv, acc.y * inv), __floats2bfloat162_rn(acc.z * inv, acc.w * inv)};
+  *reinterpret_cast<uint2*>(reinterpret_cast<__nv_bfloat16*>(a.out) + ((size_t)r * a.H + h) * a.rank_cols + d) =
+      *reinterpret_cast<const uint2*>(b);
 }
 
 // ---------------------------------------------------------------- fp32: one CTA per (row, head)
@@ -497,6 +530,16 @@ int launch_decode(const LatentDecArgs& a, cudaStream_t stream) {
   return (int)launch_pdl(latent_decode_kernel<MT, NB, TK>, grid, dim3(DEC_WARPS * 32), smem, stream, a);
 }
 
+// Tiles of 64 keys and 32 heads where they fit and the spans are whole tiles, else smaller ones.
+template <int NB>
+int pick_decode(const LatentDecArgs& a, cudaStream_t stream) {
+  const bool big = a.split_len % 64 == 0;
+  if (a.H > 16 && big && dec_smem<2, 64>(a.W) <= 227 * 1024) return launch_decode<2, NB, 64>(a, stream);
+  if (a.H > 16 && dec_smem<2, 32>(a.W) <= 227 * 1024) return launch_decode<2, NB, 32>(a, stream);
+  if (big && dec_smem<1, 64>(a.W) <= 227 * 1024) return launch_decode<1, NB, 64>(a, stream);
+  return launch_decode<1, NB, 32>(a, stream);
+}
+
 }  // namespace
 
 HE_API int he_latent_post(const LatentPostArgs* args, cudaStream_t stream) {
@@ -525,14 +568,13 @@ HE_API int he_latent_decode(const LatentDecArgs* args, cudaStream_t stream) {
   if (a.R <= 0) return 0;
   if (check_decode(a) != 0 || a.split_len <= 0 || a.max_splits <= 0 || a.R > 65535) return -HE_ERR_BAD_ARG;
   const int nb = (a.rank_cols / 16 + DEC_WARPS - 1) / DEC_WARPS;
-  const bool wide = a.H > 16 && dec_smem<2, 64>(a.W) <= 227 * 1024, narrow = dec_smem<1, 64>(a.W) <= 227 * 1024;
   int rc;
-  if (nb <= 1) rc = wide ? launch_decode<2, 1, 64>(a, stream) : narrow ? launch_decode<1, 1, 64>(a, stream) : launch_decode<1, 1, 32>(a, stream);
-  else if (nb <= 2) rc = wide ? launch_decode<2, 2, 64>(a, stream) : narrow ? launch_decode<1, 2, 64>(a, stream) : launch_decode<1, 2, 32>(a, stream);
-  else if (nb <= 4) rc = wide ? launch_decode<2, 4, 64>(a, stream) : narrow ? launch_decode<1, 4, 64>(a, stream) : launch_decode<1, 4, 32>(a, stream);
-  else rc = launch_decode<1, 8, 32>(a, stream);
+  if (nb <= 1) rc = pick_decode<1>(a, stream);
+  else if (nb <= 2) rc = pick_decode<2>(a, stream);
+  else rc = launch_decode<1, 4, 32>(a, stream);
   if (rc != 0) return rc;
-  return (int)launch_pdl(latent_reduce_kernel, dim3(a.H, a.R), dim3(128), (size_t)a.max_splits * sizeof(float), stream, a);
+  return (int)launch_pdl(latent_reduce_kernel, dim3(a.H, a.R, (a.rank_cols + 127) / 128), dim3(RED_WARPS * 32),
+                         (size_t)a.max_splits * sizeof(float), stream, a);
 }
 HE_API int he_latent_dec_args_size() { return (int)sizeof(LatentDecArgs); }
 

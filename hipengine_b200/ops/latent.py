@@ -83,16 +83,21 @@ def latent_post(down: torch.Tensor, q: torch.Tensor, norm_w: torch.Tensor, freq:
 
 
 def decode_split(span: int, rows: int, heads: int, W: int) -> Tuple[int, int]:
-    """(split_len, max_splits): spans of whole 64-key tiles so that rows x head chunks x spans fill the SMs about once (wide
-    rows, one CTA per SM) or several times (narrow rows)."""
-    chunks = -(-heads // 32) if heads > 16 else 1
-    per_sm = max(1, min(4, int(220e3 // ((160 if heads > 16 else 144) * (2 * W + 16)))))
-    split = -(-(span * max(rows, 1) * chunks) // (148 * per_sm))
-    split = max(64, -(-split // 64) * 64)
+    """(split_len, max_splits): the spans of all rows and head chunks fill the SMs about once (wide rows: one CTA per SM) or
+    a few times (narrow rows), without a last round of a few stragglers.  Spans are whole tiles of 64 keys, or single tiles
+    of 32 where even those leave SMs idle."""
+    chunks, tile_rows = (-(-heads // 32), 32) if heads > 16 else (1, 16)
+    per_sm = max(1, min(4, int(227e3 // ((tile_rows + 128) * (2 * W + 16) + tile_rows * 1300))))
+    slots, jobs = 148 * per_sm, max(rows, 1) * chunks
+    if span * jobs <= 32 * slots:
+        return 32, max(1, -(-span // 32))
+    spans = max(1, slots // jobs)                    # whole rounds: every job gets the same number of spans
+    split = max(64, -(-(-(-span // spans)) // 64) * 64)
     return split, max(1, -(-span // split))
 
 
 def decode_scratch_floats(rows: int, heads: int, max_splits: int, rank_cols: int) -> int:
+    """Span sums, then their (maximum, sum) pairs."""
     return rows * heads * max_splits * (rank_cols + 2)
 
 

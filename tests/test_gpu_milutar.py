@@ -239,7 +239,7 @@ def test_latent_space_attention(heads, rank, rd, window, sink, exact):
         assert not out[:, :, rank:].any()
         return
     span = min(300, window) if window else 300
-    for split in (64, 128, 192, 1024):
+    for split in (32, 64, 96, 128, 192, 1024):
         ns = -(-span // split)
         part = torch.full((LA.decode_scratch_floats(n, heads, ns, rc),), float("nan"), device="cuda")
         LA.latent_decode(ql, cache, bt, slot, ctx, part, out, rc, scale, split, ns, window, skc)
