@@ -130,20 +130,26 @@ def attention_prefill(T: int, window: int = 0) -> List[Dict]:
     q, out = _bf(T, H, DIM + RD) * 20, torch.empty(T, H * VDIM, device="cuda", dtype=torch.bfloat16)
     start, slot = torch.tensor([0, T], dtype=torch.int32, device="cuda"), torch.zeros(1, dtype=torch.int32, device="cuda")
     pos, lat = torch.arange(T, dtype=torch.int32, device="cuda"), torch.empty(T, W, device="cuda", dtype=torch.bfloat16)
-    ukv, kv = _bf(H * (DIM + VDIM), RANK), [_bf(T, H * (DIM + VDIM)) for _ in range(n)]
+    ukv, kx, v = _bf(H * (DIM + VDIM), RANK), [_bf(T, H * DIM) for _ in range(n)], [_bf(H * VDIM, T) for _ in range(n)]
     sink = torch.zeros(H, device="cuda")
-    ms = time_launches(lambda i: LA.latent_prefill(q, kv[i], lat, start, pos, [T], out, H, 0, H, DIM, VDIM, RANK,
-                                                   (DIM + RD) ** -0.5, window, sink), n)
+    lat.zero_()
+    ms, reg = (time_launches(lambda i: LA.latent_prefill(q, kx[i], v[i] if tc else v[i].view(T, -1), lat, start, pos, [T], out, H, 0,
+                                                         H, DIM, VDIM, RANK, (DIM + RD) ** -0.5, window, sink, transposed=tc), n)
+               for tc in (True, False))
     G, D = 8, 128
     pages = -(-T // 16)
     kvl, q2 = [_bf(pages + 1, 2, G, 16, D) * 20 for _ in range(n)], _bf(T, H, D) * 20
     lms = time_launches(lambda i: A.flash_prefill(q2, None, kvl[i], bt, 0, 0, out, H, G, D, 16, D ** -0.5, window), n)
     seen = float(T) * T / 2 if not window else float(window) * (T - window / 2)
-    rows = [_row(f"expanded attention T {T} heads {H} x {DIM + RD}/{VDIM}" + (f" window {window}" if window else ""), "bf16", ms,
-                 2.0 * seen * H * (DIM + RD + VDIM), "flash prefill", lms, 2.0 * seen * H * 2 * D)]
+    rows = [_row(f"expanded attention{form}, T {T} heads {H} x {DIM + RD}/{VDIM}" + (f" window {window}" if window else ""),
+                 "bf16", t, 2.0 * seen * H * (DIM + RD + VDIM), "flash prefill", lms, 2.0 * seen * H * 2 * D)
+            for form, t in (("", ms), (" (register form)", reg))]
     if not window:
         fl = 2.0 * T * H * (DIM + VDIM) * RANK
-        gm = time_launches(lambda i: GM.gemm_bf16(lat, ukv, kv[i]) if False else GM.gemm_bf16(lat[:, :RANK], ukv, kv[i]), n)
+        def expand(i):
+            GM.gemm_bf16(lat[:, :RANK], ukv[:H * DIM], kx[i])
+            GM.gemm_bf16(ukv[H * DIM:], lat[:, :RANK], v[i])
+        gm = time_launches(expand, n)
         x, w2 = _bf(T, 4096), _bf(4096, 4096)
         y = torch.empty(T, 4096, device="cuda", dtype=torch.bfloat16)
         lm = time_launches(lambda i: GM.gemm_bf16(x, w2, y), n)

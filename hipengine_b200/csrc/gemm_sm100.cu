@@ -11,8 +11,12 @@
 // reference, which use 16x16x16 WMMA with one wave per block).
 #include "common.cuh"
 #include "sm100.cuh"
+#include "tmap.cuh"
 
 using namespace sm100;
+using he::EncodeTiledFn;
+using he::get_encode;
+using he::make_map;
 
 namespace {
 
@@ -855,37 +859,6 @@ gemm_q_allreduce_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_co
 }
 
 // ---------------------------------------------------------------- host side: tensor maps
-typedef CUresult (*EncodeTiledFn)(CUtensorMap*, CUtensorMapDataType, cuuint32_t, void*, const cuuint64_t*,
-                                  const cuuint64_t*, const cuuint32_t*, const cuuint32_t*, CUtensorMapInterleave,
-                                  CUtensorMapSwizzle, CUtensorMapL2promotion, CUtensorMapFloatOOBfill);
-
-EncodeTiledFn get_encode() {
-  static EncodeTiledFn fn = nullptr;
-  if (fn == nullptr) {
-    void* p = nullptr;
-    cudaDriverEntryPointQueryResult qres;
-    if (cudaGetDriverEntryPoint("cuTensorMapEncodeTiled", &p, cudaEnableDefault, &qres) == cudaSuccess &&
-        qres == cudaDriverEntryPointSuccess)
-      fn = reinterpret_cast<EncodeTiledFn>(p);
-  }
-  return fn;
-}
-
-// 2-D bf16 row-major [rows][cols] with row stride `ld` elements; box = {BK cols, box_rows rows}; 128B swizzle.
-int make_map(CUtensorMap* m, const void* ptr, long long rows, long long cols, long long ld, int box_rows) {
-  EncodeTiledFn enc = get_encode();
-  if (enc == nullptr) return -HE_ERR_BAD_ARG;
-  if ((reinterpret_cast<uintptr_t>(ptr) & 15) != 0 || (ld * 2) % 16 != 0) return -HE_ERR_BAD_ARG;
-  cuuint64_t dims[2] = {(cuuint64_t)cols, (cuuint64_t)rows};
-  cuuint64_t strides[1] = {(cuuint64_t)ld * 2};
-  cuuint32_t box[2] = {(cuuint32_t)BK, (cuuint32_t)box_rows};
-  cuuint32_t estr[2] = {1, 1};
-  CUresult r = enc(m, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, const_cast<void*>(ptr), dims, strides, box, estr,
-                   CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B,
-                   CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
-  return r == CUDA_SUCCESS ? 0 : 1000 + (int)r;
-}
-
 // Byte-typed 2-D map over quantised weight rows: [rows][row_bytes] uint8, box = {box_bytes, BN rows}, no swizzle.
 int make_byte_map(CUtensorMap* m, const void* ptr, long long rows, long long row_bytes, int box_bytes) {
   EncodeTiledFn enc = get_encode();

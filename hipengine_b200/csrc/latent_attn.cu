@@ -6,7 +6,7 @@
 // rotated part, its value another linear map of the latent.  Decode never builds them: the key map is moved onto the query
 // (q_lat = [W_k^T q | rotated q], W columns) and the value map behind the weighted sum, so all heads of a request attend to
 // one W-wide row per token, which is read once and serves as key and value.
-#include "common.cuh"
+#include "latent_segs.cuh"
 
 using namespace he;
 
@@ -497,27 +497,28 @@ __global__ void __launch_bounds__(EX_THREADS) latent_exact_kernel(const LatentDe
 }
 
 // ---------------------------------------------------------------- cache rows of long portions, side by side
-// Segment s contributes the keys its rows can see: positions [max(0, first - window + 1), last], in segment order.
+// Segment s contributes the keys its rows can see, in segment order, padded with zero rows (latent_segs.cuh).
 __global__ void __launch_bounds__(256) latent_gather_kernel(const LatentGatherArgs a) {
   pdl_wait();
   pdl_launch();
   const int lane = threadIdx.x & 31, row = blockIdx.x * 8 + (threadIdx.x >> 5);
   if (row >= a.keys) return;
+  uint4* dst = reinterpret_cast<uint4*>(a.out + (size_t)row * a.W);
   int k = row;
   for (int s = 0; s < a.n_seg; ++s) {
-    const int r0 = a.seg_start[s], p0 = a.pos[r0];
-    const int lo = a.window > 0 ? max(0, p0 - a.window + 1) : 0, n = p0 + (a.seg_start[s + 1] - r0) - lo;
-    if (k < n) {
-      const int p = lo + k, pi = p / a.page;
+    const LatentSeg g = latent_seg(a.seg_start, a.pos, s, a.window, 0);
+    if (k < g.keys) {
+      const int p = g.lo + k, pi = p / a.page;
       const int* bt = a.block_table + (size_t)a.seg_slot[s] * a.max_pages;
       const int pg = bt[HE_INDEX_OK(pi, a.max_pages, HE_SITE_ATTN_DECODE_PAGE) ? pi : 0];
       const uint4* src = reinterpret_cast<const uint4*>(a.cache + ((size_t)pg * a.page + p % a.page) * a.W);
-      uint4* dst = reinterpret_cast<uint4*>(a.out + (size_t)row * a.W);
       for (int i = lane; i < a.W / 8; i += 32) dst[i] = src[i];
       return;
     }
-    k -= n;
+    k -= latent_seg_rows(g);
+    if (k < 0) break;                                    // padding of this segment
   }
+  for (int i = lane; i < a.W / 8; i += 32) dst[i] = make_uint4(0u, 0u, 0u, 0u);
 }
 
 template <int MT, int NB, int TK>

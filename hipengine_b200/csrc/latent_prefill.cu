@@ -1,26 +1,14 @@
 // Prefill form of latent attention: long prompt portions attend with full keys and values.
 //
-// The latents of every visible key lie side by side (latent_gather_kernel), one tensor-core GEMM has expanded them to
-// [key][head][dn key columns | dv value columns], and the rotated key part is read from the gathered latent row itself, so it
-// exists once and not per head.  Flash-style single pass: a CTA owns 64 MT query rows of one head (4 warps x MT x 16 rows),
+// The latents of every visible key lie side by side (latent_gather_kernel), tensor-core GEMMs have expanded them to keys
+// [key][head][dn] and values [key][head][dv], and the rotated key part is read from the gathered latent row itself, so it
+// exists once and not per head.  This form takes any head shape up to 256 columns; latent_prefill_tc.cu has the common ones.  Flash-style single pass: a CTA owns 64 MT query rows of one head (4 warps x MT x 16 rows),
 // streams 32-key tiles with cp.async (double buffered), keeps running maximum / sum per row and the output in registers;
 // mma.sync m16n8k16 with fp32 accumulation.  Causal, optionally only the last `window` keys, optionally with a learned term
 // per head in the softmax denominator.  Segments of several requests share a launch.
-#include "common.cuh"
+#include "latent_segs.cuh"
 
 using namespace he;
-
-struct LatentPrefillArgs {
-  const __nv_bfloat16* q;      // [T][H][qd], rotated: [dn | rotated, zero-padded]
-  const __nv_bfloat16* kv;     // [keys][n_heads][dn + dv]
-  const __nv_bfloat16* lat;    // [keys][W], rotated key part from column rank_cols
-  const float* sink;           // [H] or null
-  const int* seg_start;        // [n_seg + 1] absolute rows of q / out
-  const int* pos;              // [rows]
-  __nv_bfloat16* out;          // [T][H * dv]
-  int n_seg, tiles, H, head0, n_heads, dn, dv, qd, W, rank_cols, window;
-  float scale;
-};
 
 namespace {
 
@@ -64,28 +52,18 @@ __global__ void __launch_bounds__(NTHR) latent_prefill_kernel(const __grid_const
   __nv_bfloat16* sQ = sm;                    // [BM][LK]
   __nv_bfloat16* sK = sQ + BM * LK;          // [2][BN][LK]
   __nv_bfloat16* sV = sK + 2 * BN * LK;      // [2][BN][LV]
-  int qt = gridDim.x - 1 - blockIdx.x;       // heavy (late) tiles first
-  int s = 0, key_row0 = 0;                   // first gathered row of the segment
-  int row0 = 0, T = 0, pos0 = 0, lo = 0;
-  for (; s < a.n_seg; ++s) {
-    row0 = a.seg_start[s];
-    T = a.seg_start[s + 1] - row0;
-    pos0 = a.pos[row0];
-    lo = a.window > 0 ? max(0, pos0 - a.window + 1) : 0;
-    const int tiles = (T + BM - 1) / BM;
-    if (qt < tiles) break;
-    qt -= tiles;
-    key_row0 += pos0 + T - lo;
-  }
-  if (s == a.n_seg) return;
+  LatentSeg seg;
+  int qt;
+  if (!latent_find_tile<BM>(a.seg_start, a.pos, a.n_seg, a.window, (int)gridDim.x - 1 - (int)blockIdx.x, seg, qt)) return;
+  const int row0 = seg.row0, T = seg.T, pos0 = seg.pos0, lo = seg.lo, key_row0 = seg.key0;
   const int hl = blockIdx.y, h = a.head0 + hl;
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, c = lane & 3;
   const int t0 = qt * BM, rows = min(BM, T - t0);
   const int kv_end = pos0 + t0 + rows;                                              // keys [kv_begin, kv_end)
   const int kv_begin = a.window > 0 ? max(lo, pos0 + t0 - a.window + 1) : 0;
   const int n_tiles = (kv_end - kv_begin + BN - 1) / BN;
-  const int hw = a.dn + a.dv, dn8 = a.dn / 8, qd8 = a.qd / 8, dv8 = a.dv / 8;
-  const size_t kv_ld = (size_t)a.n_heads * hw;
+  const int dn8 = a.dn / 8, qd8 = a.qd / 8, dv8 = a.dv / 8;
+  const size_t k_ld = (size_t)a.n_heads * a.dn, v_ld = (size_t)a.n_heads * a.dv;
 
   auto load_kv = [&](int tile, int buf) {
     const int k0 = kv_begin + tile * BN;
@@ -94,7 +72,7 @@ __global__ void __launch_bounds__(NTHR) latent_prefill_kernel(const __grid_const
     for (int i = tid; i < BN * CK; i += NTHR) {
       const int r = i / CK, ch = i % CK, p = k0 + r;
       const size_t kr = key_row0 + min(p, kv_end - 1) - lo;
-      const __nv_bfloat16* src = ch < dn8 ? a.kv + kr * kv_ld + (size_t)hl * hw + ch * 8
+      const __nv_bfloat16* src = ch < dn8 ? a.kx + kr * k_ld + (size_t)hl * a.dn + ch * 8
                                           : a.lat + kr * a.W + a.rank_cols + (ch < qd8 ? (ch - dn8) * 8 : 0);
       cp_async16(sK + ((size_t)buf * BN + r) * LK + ch * 8, src, p < kv_end && ch < qd8);
     }
@@ -102,7 +80,7 @@ __global__ void __launch_bounds__(NTHR) latent_prefill_kernel(const __grid_const
     for (int i = tid; i < BN * CV; i += NTHR) {
       const int r = i / CV, ch = i % CV, p = k0 + r;
       const size_t kr = key_row0 + min(p, kv_end - 1) - lo;
-      const __nv_bfloat16* src = a.kv + kr * kv_ld + (size_t)hl * hw + a.dn + (ch < dv8 ? ch * 8 : 0);
+      const __nv_bfloat16* src = a.v + kr * v_ld + (size_t)hl * a.dv + (ch < dv8 ? ch * 8 : 0);
       cp_async16(sV + ((size_t)buf * BN + r) * LV + ch * 8, src, p < kv_end && ch < dv8);
     }
   };

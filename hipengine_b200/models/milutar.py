@@ -6,7 +6,8 @@ The base (``listed.py``) holds the planes per layer run, the recurrent rows, the
                  segment reads its own input); more rows: tcgen05 GEMMs with the activation in the epilogue;
   cache          latent norm, rotation and page write in one kernel; a page row is [latent | rotated key part];
   attention      single rows and short portions in latent space (the key map moved onto the query, the value map behind the
-                 sum), long portions with keys and values expanded once per launch by a GEMM;
+                 sum), long portions with keys and values expanded once per launch by GEMMs: the common head shapes on
+                 tcgen05 with accumulators in tensor memory, the others on a register kernel;
   output         both output projections with their per-channel factors: one launch for few rows, two accumulating GEMMs
                  otherwise.
 ``dtype="float32"`` runs the same walk, in latent space throughout, on fp32 CUDA-core kernels and fp32 pages.  In both modes
@@ -27,6 +28,7 @@ from .executor import PAGE, BatchDesc
 from .listed import DECODE_SEG_ROWS, EXACT, FEW, MANY, ListedExecutor, pad2, up8
 
 EXPANDED_KV_BYTES = 1 << 30       # expanded keys and values of a launch: above this the heads are taken in groups
+TC_MIN_ROWS = 65                  # longest portion from which the tensor-memory form (256-row tiles) is taken
 LATENT_ROWS = 512                 # rows per latent-space launch (bounds its split-K scratch)
 
 
@@ -40,7 +42,8 @@ class _Layer:
     in_w: DeviceWeight                     # [query (or query latent) rows | latent and rotated key rows, hp]
     n_q: int                               # rows of its first part
     kv_norm: torch.Tensor                  # fp32 [rank_cols]
-    ukv: DeviceWeight                      # [heads * (dn key rows | dv value rows), rank_cols]
+    uk: DeviceWeight                       # [heads * dn, rank_cols]
+    uv: DeviceWeight                       # [heads * dv, rank_cols]
     uk_t: torch.Tensor                     # [heads, rank_cols, dn]: the key map from the query's side
     freq: torch.Tensor                     # float64 [rot_dim / 2]
     amp: float
@@ -52,9 +55,6 @@ class _Layer:
     up: Optional[DeviceWeight] = None      # [ff padded, hp]
     down: Optional[DeviceWeight] = None    # [hp, ff padded]
     s2: Optional[torch.Tensor] = None
-
-    def uv(self, heads: int) -> torch.Tensor:
-        return self.ukv.data.view(heads, self.dn + self.dv, -1)[:, self.dn:]
 
 
 class MilutarExecutor(ListedExecutor):
@@ -98,7 +98,7 @@ class MilutarExecutor(ListedExecutor):
             L = _Layer(self._norm_weight(p + "norm1"), self._vec(p + "shift", hp), dn, dv, dn + rr,
                        put(p + "in", torch.cat([first, down], 0)), first.shape[0],
                        self._vec(p + "mix.dkv.norm", a.rank_cols),
-                       put(p + "ukv", torch.cat([uk, uv], 1).reshape(a.heads * (dn + dv), a.rank_cols)), uk_t,
+                       put(p + "uk", uk.reshape(-1, a.rank_cols)), put(p + "uv", uv.reshape(-1, a.rank_cols)), uk_t,
                        torch.tensor(freq, dtype=torch.float64, device=self.device), amp, put(p + "o", o.reshape(hp, -1)),
                        self._vec(p + "ls1", hp, cfg.residual_mult))
             if a.q_rank:
@@ -230,23 +230,27 @@ class MilutarExecutor(ListedExecutor):
             split_len, n_splits = LA.decode_split(min(ctx, a.window) if a.window else ctx, R, H, a.row_cols)
             part = self.scratch.get("attn_part", (LA.decode_scratch_floats(R, H, n_splits, rank),), torch.float32)
             LA.latent_decode(*args, part, o_lat, rank, a.scale, split_len, n_splits, a.window, L.sink)
-        mul(o_lat, L.uv(H), out[r0:r1].view(R, H, L.dv))
+        mul(o_lat, L.uv.data.view(H, L.dv, rank), out[r0:r1].view(R, H, L.dv))
 
     def _expanded(self, a: LatentAttentionSpec, L: _Layer, kv: torch.Tensor, q: torch.Tensor, b: BatchDesc, s: int, e: int,
                   out: torch.Tensor) -> None:
         """Segments s..e with full keys and values, expanded from the cache rows they can see."""
         from ..ops import gemm as GM
-        segs, hw, H = b.segs_host[s:e], L.dn + L.dv, a.heads
-        keys = LA.visible_keys(segs, a.window)
+        segs, H = b.segs_host[s:e], a.heads
+        keys, rows = LA.gathered_rows(segs, a.window), [n for _, _, n in segs]
+        tc = LA.prefill_tc_ok(L.dn, L.qd, L.dv) and max(rows) >= TC_MIN_ROWS and a.scale > 0
         lat = self.scratch.get("lat_keys", (keys, a.row_cols), torch.bfloat16)
         LA.latent_gather(kv, self.block_table, b.seg_start[s:], b.seg_slot[s:], b.pos, e - s, a.window, lat)
-        group = max(1, min(H, EXPANDED_KV_BYTES // (keys * hw * 2)))
+        group = max(1, min(H, EXPANDED_KV_BYTES // (keys * (L.dn + L.dv) * 2)))
+        c = lat[:, :a.rank_cols]
         for h0 in range(0, H, group):
             n = min(group, H - h0)
-            full = self.scratch.get("lat_kv", (keys, n * hw), torch.bfloat16)
-            GM.gemm_bf16(lat[:, :a.rank_cols], L.ukv.data[h0 * hw:(h0 + n) * hw], full)
-            LA.latent_prefill(q, full, lat, b.seg_start[s:], b.pos, [r for _, _, r in segs], out, H, h0, n, L.dn, L.dv,
-                              a.rank_cols, a.scale, a.window, L.sink)
+            uk, uv = L.uk.data[h0 * L.dn:(h0 + n) * L.dn], L.uv.data[h0 * L.dv:(h0 + n) * L.dv]
+            kx = GM.gemm_bf16(c, uk, self.scratch.get("lat_kx", (keys, n * L.dn), torch.bfloat16))
+            v = self.scratch.get("lat_v", (n * L.dv, keys) if tc else (keys, n * L.dv), torch.bfloat16)
+            GM.gemm_bf16(*((uv, c) if tc else (c, uv)), v)
+            LA.latent_prefill(q, kx, v, lat, b.seg_start[s:], b.pos, rows, out, H, h0, n, L.dn, L.dv, a.rank_cols, a.scale,
+                              a.window, L.sink, transposed=tc)
 
     # ------------------------------------------------------------------ whole model
     def _embed(self, b: BatchDesc, h: torch.Tensor, copy: Optional[torch.Tensor]) -> None:

@@ -99,8 +99,8 @@ PLUGINS: Tuple[ModelPlugin, ...] = (
     ModelPlugin("milutar", ("milutar",), "hipengine_b200.models.milutar.MilutarExecutor", default_quant="bf16",
                 native_block_types=("BF16",), widened_block_types=(), kv_storage=("bf16", "f32"),
                 tensor_parallel=False, compute_dtypes=("bfloat16", "float32"),
-                native_sources=("gemm_sm100.cu", "gemv_float.cu", "latent_attn.cu", "latent_prefill.cu", "layers.cu",
-                                "quant_util.cu", "runtime.cpp", "sampling.cu"),
+                native_sources=("gemm_sm100.cu", "gemv_float.cu", "latent_attn.cu", "latent_prefill.cu", "latent_prefill_tc.cu",
+                                "layers.cu", "quant_util.cu", "runtime.cpp", "sampling.cu"),
                 folder_architecture="Milutar", folder_reader="hipengine_b200.loading.milutar",
                 reference="hipengine_b200.ref.milutar.MilutarRef",
                 notes="layers listed one by one: latent attention (windowed, or causal with a softmax sink and a query "

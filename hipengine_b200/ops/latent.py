@@ -1,4 +1,4 @@
-"""Launchers of the latent attention kernels (``csrc/latent_attn.cu``, ``csrc/latent_prefill.cu``).
+"""Launchers of the latent attention kernels (``csrc/latent_attn.cu``, ``latent_prefill.cu``, ``latent_prefill_tc.cu``).
 
 A cache plane is ``[n_pages, page, W]`` in bf16 (fp32 for the float32 compute dtype): latent columns, then the rotated key
 part, zero-padded.
@@ -11,7 +11,7 @@ from typing import Optional, Sequence, Tuple
 import torch
 
 from ..core import native as N
-from .kernels import _check_device, _dt, _p, _stream
+from .kernels import _check_device, _dt, _p, _stream, status_tensor
 
 c_vp, c_ll, c_int = C.c_void_p, C.c_longlong, C.c_int
 
@@ -38,12 +38,13 @@ class _GatherArgs(C.Structure):
 
 
 class _PrefillArgs(C.Structure):
-    _fields_ = [("q", c_vp), ("kv", c_vp), ("lat", c_vp), ("sink", c_vp), ("seg_start", c_vp), ("pos", c_vp),
-                ("out", c_vp), ("n_seg", c_int), ("tiles", c_int), ("H", c_int), ("head0", c_int), ("n_heads", c_int),
-                ("dn", c_int), ("dv", c_int), ("qd", c_int), ("W", c_int), ("rank_cols", c_int), ("window", c_int),
-                ("scale", C.c_float)]
+    _fields_ = [("q", c_vp), ("kx", c_vp), ("v", c_vp), ("lat", c_vp), ("sink", c_vp), ("seg_start", c_vp), ("pos", c_vp),
+                ("out", c_vp), ("status", c_vp), ("n_seg", c_int), ("tiles", c_int), ("H", c_int), ("head0", c_int),
+                ("n_heads", c_int), ("dn", c_int), ("dv", c_int), ("qd", c_int), ("W", c_int), ("rank_cols", c_int),
+                ("window", c_int), ("rows", c_int), ("keys", c_int), ("scale", C.c_float)]
 
 
+SEG_ALIGN = 8             # gathered rows of a segment are padded to a multiple of this
 _ABI_OK = False
 
 
@@ -133,14 +134,15 @@ def latent_exact(q: torch.Tensor, cache: torch.Tensor, block_table: torch.Tensor
     N.check(_lib().he_latent_exact(C.byref(a), _stream()), "he_latent_exact")
 
 
-def visible_keys(segs: Sequence[Tuple[int, int, int]], window: int) -> int:
-    """Cache rows that (slot, first position, rows) segments can see in total."""
-    return sum(p0 + n - (max(0, p0 - window + 1) if window > 0 else 0) for _, p0, n in segs)
+def gathered_rows(segs: Sequence[Tuple[int, int, int]], window: int) -> int:
+    """Rows of the gathered keys of (slot, first position, rows) segments: what each can see, padded."""
+    seen = (p0 + n - (max(0, p0 - window + 1) if window > 0 else 0) for _, p0, n in segs)
+    return sum(-(-n // SEG_ALIGN) * SEG_ALIGN for n in seen)
 
 
 def latent_gather(cache: torch.Tensor, block_table: torch.Tensor, seg_start: torch.Tensor, seg_slot: torch.Tensor,
                   pos: torch.Tensor, n_seg: int, window: int, out: torch.Tensor) -> None:
-    """The cache rows the segments can see, side by side in segment order: ``out`` [keys, W]."""
+    """The cache rows the segments can see, side by side in segment order: ``out`` [``gathered_rows``, W]."""
     a = _GatherArgs()
     a.cache, a.block_table, a.seg_start = cache.data_ptr(), block_table.data_ptr(), seg_start.data_ptr()
     a.seg_slot, a.pos, a.out, a.n_seg, a.keys = seg_slot.data_ptr(), pos.data_ptr(), out.data_ptr(), n_seg, out.shape[0]
@@ -149,25 +151,36 @@ def latent_gather(cache: torch.Tensor, block_table: torch.Tensor, seg_start: tor
     N.check(_lib().he_latent_gather(C.byref(a), _stream()), "he_latent_gather")
 
 
+TC_TILE_ROWS = 256
+
+
 def prefill_tile_rows(q_cols: int, dv: int) -> int:
-    """Query rows per tile of the prefill kernel for this head shape (0: it has none)."""
+    """Query rows per tile of the register form of prefill for this head shape (0: it has none)."""
     return int(_lib().he_latent_prefill_tile_rows(c_int(q_cols), c_int(dv)))
 
 
-def latent_prefill(q: torch.Tensor, kv: torch.Tensor, lat: torch.Tensor, seg_start: torch.Tensor, pos: torch.Tensor,
-                   seg_rows: Sequence[int], out: torch.Tensor, heads: int, head0: int, n_heads: int, dn: int, dv: int,
-                   rank_cols: int, scale: float, window: int = 0, sink: Optional[torch.Tensor] = None) -> None:
-    """Heads head0 .. head0 + n_heads of the segments' rows: ``q`` [T, heads, q_cols] rotated queries, ``kv``
-    [keys, n_heads * (dn + dv)] expanded keys and values of the rows gathered into ``lat``; ``out`` [T, heads * dv]."""
-    a = _PrefillArgs()
-    qd = q.shape[2]
-    assert q.is_contiguous() and kv.is_contiguous() and out.is_contiguous() and lat.is_contiguous()
-    assert kv.shape == (lat.shape[0], n_heads * (dn + dv)) and out.shape[1] == heads * dv and q.shape[1] == heads
-    a.q, a.kv, a.lat, a.sink = q.data_ptr(), kv.data_ptr(), lat.data_ptr(), _p(sink)
+def prefill_tc_ok(dn: int, q_cols: int, dv: int) -> bool:
+    """Does the tensor-memory form take this head shape?"""
+    return bool(_lib().he_latent_prefill_tc_ok(c_int(dn), c_int(q_cols), c_int(dv)))
+
+
+def latent_prefill(q: torch.Tensor, kx: torch.Tensor, v: torch.Tensor, lat: torch.Tensor, seg_start: torch.Tensor,
+                   pos: torch.Tensor, seg_rows: Sequence[int], out: torch.Tensor, heads: int, head0: int, n_heads: int,
+                   dn: int, dv: int, rank_cols: int, scale: float, window: int = 0, sink: Optional[torch.Tensor] = None,
+                   transposed: bool = False) -> None:
+    """Heads head0 .. head0 + n_heads of the segments' rows: ``q`` [T, heads, q_cols] rotated queries, ``kx``
+    [keys, n_heads * dn] and ``v`` [keys, n_heads * dv] expanded from the rows gathered into ``lat``; ``out``
+    [T, heads * dv].  ``transposed``: ``v`` is [n_heads * dv, keys] and the tensor-memory form runs."""
+    a, keys, qd = _PrefillArgs(), lat.shape[0], q.shape[2]
+    assert q.is_contiguous() and kx.is_contiguous() and v.is_contiguous() and out.is_contiguous() and lat.is_contiguous()
+    assert kx.shape == (keys, n_heads * dn) and out.shape == (q.shape[0], heads * dv) and q.shape[1] == heads
+    assert v.shape == ((n_heads * dv, keys) if transposed else (keys, n_heads * dv))
+    a.q, a.kx, a.v, a.lat, a.sink = q.data_ptr(), kx.data_ptr(), v.data_ptr(), lat.data_ptr(), _p(sink)
     a.seg_start, a.pos, a.out, a.n_seg = seg_start.data_ptr(), pos.data_ptr(), out.data_ptr(), len(seg_rows)
-    bm = prefill_tile_rows(qd, dv)
+    bm = TC_TILE_ROWS if transposed else prefill_tile_rows(qd, dv)
     assert bm > 0
-    a.tiles = sum(-(-n // bm) for n in seg_rows)
+    a.tiles, a.status = sum(-(-n // bm) for n in seg_rows), status_tensor(q.device).data_ptr()
     a.H, a.head0, a.n_heads, a.dn, a.dv, a.qd = heads, head0, n_heads, dn, dv, qd
-    a.W, a.rank_cols, a.window, a.scale = lat.shape[1], rank_cols, window, scale
-    N.check(_lib().he_latent_prefill(C.byref(a), _stream()), "he_latent_prefill")
+    a.W, a.rank_cols, a.window, a.scale, a.rows, a.keys = lat.shape[1], rank_cols, window, scale, q.shape[0], keys
+    fn = "he_latent_prefill_tc" if transposed else "he_latent_prefill"
+    N.check(getattr(_lib(), fn)(C.byref(a), _stream()), fn)

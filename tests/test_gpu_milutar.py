@@ -250,15 +250,16 @@ def test_latent_space_attention(heads, rank, rd, window, sink, exact):
 
 @pytest.mark.parametrize("window,sink", [(0, True), (0, False), (1, True), (33, False), (40, True), (1000, False)])
 @pytest.mark.parametrize("heads,dim,rd,dv,rank", [(3, 20, 12, 28, 44), (2, 64, 40, 64, 72), (4, 64, 64, 96, 64),
-                                                  (2, 128, 64, 128, 136), (2, 150, 50, 136, 80), (1, 8, 2, 8, 16)])
+                                                  (2, 128, 64, 128, 136), (2, 150, 50, 136, 80), (1, 8, 2, 8, 16),
+                                                  (3, 60, 18, 122, 48), (2, 128, 8, 64, 512)])
 def test_expanded_attention(heads, dim, rd, dv, rank, window, sink):
     """Portions of several requests (different slots, pages and starts) in one launch, heads in groups, against the plain
     equations; the keys just inside and just outside a window stand out."""
     from hipengine_b200.ops import gemm as G
     from hipengine_b200.ops import latent as LA
     up8 = lambda n: -(-n // 8) * 8
-    segs = [(2, 0, 150), (0, 37, 9), (1, 128, 70)]                            # slot, first position, rows
-    ctxs = [46, 198, 150]
+    segs = [(2, 0, 300), (0, 37, 9), (1, 128, 270)]                           # slot, first position, rows
+    ctxs = [46, 398, 300]
     cache, bt, lats, rots, rc, W = _latent_cache(ctxs, rank, rd, rank + dim, BF, [20, 140, 60])
     g, T = _gen(2), sum(n for _, _, n in segs)
     dn, dvp, qd = up8(dim), up8(dv), up8(dim) + up8(rd)
@@ -272,41 +273,77 @@ def test_expanded_attention(heads, dim, rd, dv, rank, window, sink):
         row += n
     qp = torch.zeros(T, heads, qd)
     qp[:, :, :dim], qp[:, :, dn:dn + rd] = q[:, :, :dim], q[:, :, dim:]
-    ukv = torch.zeros(heads, dn + dvp, rc)
-    ukv[:, :dim, :rank], ukv[:, dn:dn + dv, :rank] = wk.view(heads, dim, rank), wv.view(heads, dv, rank)
-    ukv = ukv.view(-1, rc).to(BF).cuda()
+    uk, uv = torch.zeros(heads, dn, rc), torch.zeros(heads, dvp, rc)
+    uk[:, :dim, :rank], uv[:, :dv, :rank] = wk.view(heads, dim, rank), wv.view(heads, dv, rank)
+    uk, uv = (x.view(-1, rc).to(BF).cuda() for x in (uk, uv))
     starts = [0]
     for _, _, n in segs:
         starts.append(starts[-1] + n)
     pos = _i32([p for _, p0, n in segs for p in range(p0, p0 + n)])
     start, slot = _i32(starts), _i32([s for s, _, _ in segs])
-    keys = LA.visible_keys(segs, window)
-    lat = torch.full((keys, W), float("nan"), dtype=BF, device="cuda")
-    LA.latent_gather(cache, bt, start, slot, pos, len(segs), window, lat)
-    lo = [max(0, p0 - window + 1) if window else 0 for _, p0, _ in segs]
-    _close(lat[:, :rank], torch.cat([lats[s][a:p0 + n] for (s, p0, n), a in zip(segs, lo)]), 0.0)
-    out = torch.full((T, heads * dvp), 7.0, dtype=BF, device="cuda")
-    for group in {heads, 1}:
+    qc, skc = qp.to(BF).cuda(), sk.cuda() if sink else None
+
+    def run(first, group, tc, out):
+        """Segments first.. with ``group`` heads a launch."""
+        sub = segs[first:]
+        keys = LA.gathered_rows(sub, window)
+        lat = torch.full((keys, W), float("nan"), dtype=BF, device="cuda")
+        LA.latent_gather(cache, bt, start[first:], slot[first:], pos, len(sub), window, lat)
+        at = 0
+        for s, p0, n in sub:
+            a = max(0, p0 - window + 1) if window else 0
+            _close(lat[at:at + p0 + n - a, :rank], lats[s][a:p0 + n], 0.0)
+            at += -(-(p0 + n - a) // 8) * 8
+            assert not lat[at - (-(p0 + n - a) % 8):at].any()
+        assert at == keys
         for h0 in range(0, heads, group):
             n = min(group, heads - h0)
-            kv = torch.empty(keys, n * (dn + dvp), dtype=BF, device="cuda")
-            G.gemm_bf16(lat[:, :rc], ukv[h0 * (dn + dvp):(h0 + n) * (dn + dvp)], kv)
-            LA.latent_prefill(qp.to(BF).cuda(), kv, lat, start, pos, [n for _, _, n in segs], out, heads, h0, n, dn, dvp, rc,
-                              scale, window, sk.cuda() if sink else None)
+            kx, v = torch.empty(keys, n * dn, dtype=BF, device="cuda"), torch.empty(keys * n * dvp, dtype=BF, device="cuda")
+            v = v.view(n * dvp, keys) if tc else v.view(keys, n * dvp)
+            G.gemm_bf16(lat[:, :rc], uk[h0 * dn:(h0 + n) * dn], kx)
+            G.gemm_bf16(*((uv[h0 * dvp:(h0 + n) * dvp], lat[:, :rc]) if tc else (lat[:, :rc], uv[h0 * dvp:(h0 + n) * dvp])), v)
+            LA.latent_prefill(qc, kx, v, lat, start[first:], pos, [n for _, _, n in sub], out, heads, h0, n, dn, dvp, rc, scale,
+                              window, skc, transposed=tc)
         G.check_status()
-        o = out.view(T, heads, dvp)
-        _close(o[:, :, :dv], torch.cat(want).view(T, heads, dv), 0.03)
-        assert not o[:, :, dv:].any()
-    # the later segments alone read the same rows
-    part = torch.full_like(out, 7.0)
-    keys2 = LA.visible_keys(segs[1:], window)
-    LA.latent_gather(cache, bt, start[1:], slot[1:], pos, 2, window, lat[:keys2])
-    kv = torch.empty(keys2, heads * (dn + dvp), dtype=BF, device="cuda")
-    G.gemm_bf16(lat[:keys2, :rc], ukv, kv)
-    LA.latent_prefill(qp.to(BF).cuda(), kv, lat[:keys2], start[1:], pos, [9, 70], part, heads, 0, heads, dn, dvp, rc, scale,
-                      window, sk.cuda() if sink else None)
-    assert bool((part[:150] == 7.0).all())
-    _close(part[150:].view(79, heads, dvp)[:, :, :dv], torch.cat(want[1:]).view(79, heads, dv), 0.03)
+
+    full_want = torch.cat(want).view(T, heads, dv)
+    for tc in (False, True):
+        if tc and not LA.prefill_tc_ok(dn, qd, dvp):
+            continue
+        for group in sorted({heads, 1}):
+            out = torch.full((T, heads * dvp), 7.0, dtype=BF, device="cuda")
+            run(0, group, tc, out)
+            _close(out.view(T, heads, dvp)[:, :, :dv], full_want, 0.03)
+            assert not out.view(T, heads, dvp)[:, :, dv:].any()
+        out = torch.full((T, heads * dvp), 7.0, dtype=BF, device="cuda")
+        run(1, heads, tc, out)                                                # the later segments alone
+        assert bool((out[:300] == 7.0).all())
+        _close(out[300:].view(T - 300, heads, dvp)[:, :, :dv], full_want[300:], 0.03)
+
+
+def test_growing_scores_in_the_tensor_memory_form():
+    """Scores that rise key by key by far more than the tolerated growth, then fall: the accumulators are rescaled on the way
+    and the last keys weigh nothing, in both tiles of a pair."""
+    from hipengine_b200.ops import latent as LA
+    T, H, dn, dv, rc, W = 300, 2, 64, 64, 16, 32
+    g = _gen(3)
+    k = torch.cat([torch.linspace(0, 40, 200), torch.linspace(40, -40, 100)])
+    q, kx, v = torch.zeros(T, H, 72), torch.zeros(T, H, dn), torch.randn(T, H, dv, generator=g).to(BF).float()
+    q[:, 0, 0], q[:, 1, 0], kx[:, :, 0] = 1.0, -1.0, k[:, None]
+    kx, lat = kx.to(BF).float(), torch.zeros(T, W)
+    want = torch.zeros(T, H, dv)
+    for h in range(H):
+        s = (q[:, h, :dn] @ kx[:, h].t()) * 3.0
+        want[:, h] = R.softmax_with_sink(s, R.visible_keys(torch.arange(T), T)) @ v[:, h]
+    out = torch.zeros(T, H * dv, dtype=BF, device="cuda")
+    keys = LA.gathered_rows([(0, 0, T)], 0)
+    pad = lambda x: torch.cat([x, torch.zeros(keys - T, *x.shape[1:])])
+    c = lambda x: x.to(BF).cuda()
+    LA.latent_prefill(c(q), c(pad(kx.reshape(T, -1))), c(pad(v.reshape(T, -1)).t().contiguous()), c(pad(lat)), _i32([0, T]),
+                      torch.arange(T, dtype=torch.int32, device="cuda"), [T], out, H, 0, H, dn, dv, rc, 3.0, transposed=True)
+    from hipengine_b200.ops import kernels as K
+    K.check_status()
+    _close(out.view(T, H, dv), want, 0.02)
 
 
 # ----------------------------------------------------------------------------- whole models
