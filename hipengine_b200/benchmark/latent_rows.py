@@ -172,9 +172,9 @@ def attention_decode(ctx: int, R: int, heads: int = H) -> Dict:
     cache, bt = _pages(ctx, R, n, W)
     q, out = _bf(R, heads, W) * 20, torch.empty(R, heads, RANK, device="cuda", dtype=torch.bfloat16)
     slot, cl = torch.arange(R, dtype=torch.int32, device="cuda"), torch.full((R,), ctx, dtype=torch.int32, device="cuda")
-    sl, ns = LA.decode_split(ctx, R, heads, W)
-    part = torch.empty(LA.decode_scratch_floats(R, heads, ns, RANK), device="cuda")
-    ms = time_launches(lambda i: LA.latent_decode(q, cache[i], bt, slot, cl, part, out, RANK, 0.07, sl, ns), n)
+    plan = LA.decode_plan(ctx, R, heads, W)
+    part = torch.empty(plan.scratch_floats(R, heads, RANK), device="cuda")
+    ms = time_launches(lambda i: LA.latent_decode(q, cache[i], bt, slot, cl, part, out, RANK, 0.07, plan), n)
     del cache
     G, D = max(1, heads // 4), 128
     nl = _variants(R * ctx * 2 * G * D * 2)

@@ -419,6 +419,21 @@ __device__ __forceinline__ void store_tile(const GemmArgs& g, uint8_t* stage, ui
     uint32_t r[32];
     tmem_ld_32x32(t_row + c0, r);
     tmem_ld_wait();
+    if (g.epi == 4) {
+      // split-K partials: few rows, one tile per CTA, nothing to overlap with -- the detour would only add latency
+      float* dst = reinterpret_cast<float*>(g.C) + (size_t)(row0 + lane) * g.ldc + col0 + (size_t)ks * (size_t)g.split_stride;
+      if (row0 + lane < g.M) {
+        if (g.N - col0 >= 32 && (reinterpret_cast<uintptr_t>(dst) & 15) == 0) {
+#pragma unroll
+          for (int v = 0; v < 8; ++v) *reinterpret_cast<uint4*>(dst + 4 * v) = make_uint4(r[4 * v], r[4 * v + 1], r[4 * v + 2], r[4 * v + 3]);
+        } else {
+#pragma unroll
+          for (int e = 0; e < 32; ++e)
+            if (e < g.N - col0) dst[e] = __uint_as_float(r[e]);
+        }
+      }
+      continue;
+    }
     if (bf) {
 #pragma unroll
       for (int half = 0; half < 2; ++half) {
@@ -469,7 +484,7 @@ __device__ __forceinline__ void store_tile(const GemmArgs& g, uint8_t* stage, ui
           }
         }
       } else {
-        float* base = reinterpret_cast<float*>(g.C) + col + (g.epi == 4 ? (size_t)ks * (size_t)g.split_stride : (size_t)0);
+        float* base = reinterpret_cast<float*>(g.C) + col;
         const bool vec = left >= 4 && ((reinterpret_cast<uintptr_t>(base) | (uintptr_t)(g.ldc * 4)) & 15) == 0;
         float4 sc = make_float4(1.f, 1.f, 1.f, 1.f);
         if (g.epi == 2 && g.col_scale != nullptr) {

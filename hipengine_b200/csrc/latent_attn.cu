@@ -7,6 +7,7 @@
 // (q_lat = [W_k^T q | rotated q], W columns) and the value map behind the weighted sum, so all heads of a request attend to
 // one W-wide row per token, which is read once and serves as key and value.
 #include "latent_segs.cuh"
+#include "sm100.cuh"
 
 using namespace he;
 
@@ -34,11 +35,13 @@ struct LatentDecArgs {
   const int* block_table;
   const int* slot;           // [R]
   const int* ctx_len;        // [R] keys up to and including the row's own
-  float* partial;            // [R][H][max_splits][rank_cols], then (maximum, sum) [R][H][max_splits][2]
+  float* partial;            // more than one cluster per row: [R][H][clusters][rank_cols], then (maximum, sum) pairs
   void* out;                 // [R][H][rank_cols]
   const float* sink;         // [H] or null: one more term in the softmax denominator
-  int R, H, W, rank_cols, page, max_pages, split_len, max_splits, window;
+  int R, H, W, rank_cols, page, max_pages, window;
+  int spans, cluster, tile;  // CTAs per row and head chunk, how many of them merge on chip, keys per tile (32 or 64)
   float scale;
+  int* status;               // a bounded wait that gave up records its code here (split form)
 };
 
 struct LatentGatherArgs {
@@ -72,6 +75,19 @@ __global__ void __launch_bounds__(256) latent_post_kernel(const LatentPostArgs a
   pdl_wait();
   pdl_launch();
   const int t = blockIdx.x, p = a.pos[t], half = a.rot_dim / 2;
+  // the latent row and the page are requested before anything waits for them
+  constexpr int PER = 4;                                   // latents up to 1024 wide
+  const size_t in0 = (size_t)t * a.down_stride;
+  float lat[PER] = {};
+  int pg = 0;
+  const int pi = p / a.page;
+  const bool page_ok = HE_INDEX_OK(pi, a.max_pages, HE_SITE_KV_WRITE_PAGE);
+  if (blockIdx.y == 0) {
+#pragma unroll
+    for (int k = 0; k < PER; ++k)
+      if (threadIdx.x + 256 * k < a.rank) lat[k] = load_in(a.down, a.down_dtype, in0 + threadIdx.x + 256 * k);
+    if (page_ok) pg = a.block_table[(size_t)a.slot[t] * a.max_pages + pi];
+  }
   for (int i = threadIdx.x; i < half; i += 256) {
     // the angle is reduced to one turn in double, so late positions keep full fp32 accuracy
     const double two_pi = 6.283185307179586476925286766559;
@@ -81,19 +97,17 @@ __global__ void __launch_bounds__(256) latent_post_kernel(const LatentPostArgs a
     cs[i] = make_float2(c * a.amp, sn * a.amp);
   }
   if (blockIdx.y == 0) {
-    const size_t in0 = (size_t)t * a.down_stride;
     float ss = 0.f;
-    for (int i = threadIdx.x; i < a.rank; i += 256) {
-      const float v = load_in(a.down, a.down_dtype, in0 + i);
-      ss += v * v;
-    }
+#pragma unroll
+    for (int k = 0; k < PER; ++k) ss += lat[k] * lat[k];
     const float inv = rsqrtf(block_sum(ss, red) / (float)a.rank + a.eps);     // its barriers also publish cs
-    const int pi = p / a.page;
-    if (!HE_INDEX_OK(pi, a.max_pages, HE_SITE_KV_WRITE_PAGE)) return;
-    const int pg = a.block_table[(size_t)a.slot[t] * a.max_pages + pi];
+    if (!page_ok) return;
     OutT* row = reinterpret_cast<OutT*>(a.cache) + ((size_t)pg * a.page + p % a.page) * a.W;
-    for (int i = threadIdx.x; i < a.rank_cols; i += 256)
-      row[i] = from_f32<OutT>(i < a.rank ? load_in(a.down, a.down_dtype, in0 + i) * inv * a.norm_w[i] : 0.f);
+#pragma unroll
+    for (int k = 0; k < PER; ++k) {
+      const int i = threadIdx.x + 256 * k;
+      if (i < a.rank_cols) row[i] = from_f32<OutT>(i < a.rank ? lat[k] * inv * a.norm_w[i] : 0.f);
+    }
     for (int i = threadIdx.x; 2 * i < a.W - a.rank_cols; i += 256) {
       float u = 0.f, v = 0.f;
       if (i < half) {
@@ -139,13 +153,6 @@ __global__ void __launch_bounds__(256) latent_post_kernel(const LatentPostArgs a
 }
 
 // ---------------------------------------------------------------- split-K attention of single rows
-__device__ __forceinline__ void cp_async16(void* smem, const void* gmem) {
-  const uint32_t s = (uint32_t)__cvta_generic_to_shared(smem);
-  asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(s), "l"(gmem) : "memory");
-}
-__device__ __forceinline__ void cp_async_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
-template <int N>
-__device__ __forceinline__ void cp_async_wait() { asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory"); }
 __device__ __forceinline__ void ldsm_x4(uint32_t addr, uint32_t (&r)[4]) {
   asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];"
                : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr));
@@ -169,10 +176,48 @@ __host__ __device__ inline size_t dec_smem(int W) {
          (size_t)MT * 16 * ((256 / TK) * (TK + 4) * 4 + (TK * 2 + 16)) + MT * 16 * 3 * 4;
 }
 
-// One CTA per (key span, chunk of up to 16 MT heads, row).  Tiles of TK latent rows are double-buffered with cp.async (rows
-// padded by 16 bytes: conflict-free ldmatrix).  Per tile: partial scores (the warps split 16-key groups and the columns, so
+__device__ __forceinline__ uint32_t cluster_rank() {
+  uint32_t v;
+  asm volatile("mov.u32 %0, %%cluster_ctarank;" : "=r"(v));
+  return v;
+}
+__device__ __forceinline__ void cluster_arrive() { asm volatile("barrier.cluster.arrive.release.aligned;" ::: "memory"); }
+__device__ __forceinline__ void cluster_wait() { asm volatile("barrier.cluster.wait.acquire.aligned;" ::: "memory"); }
+// shared-memory address `addr` of this CTA as seen in CTA `rank` of the cluster
+__device__ __forceinline__ uint32_t map_peer(uint32_t addr, uint32_t rank) {
+  uint32_t v;
+  asm volatile("mapa.shared::cluster.u32 %0, %1, %2;" : "=r"(v) : "r"(addr), "r"(rank));
+  return v;
+}
+__device__ __forceinline__ float ld_peer(uint32_t addr) {
+  float v;
+  asm volatile("ld.shared::cluster.f32 %0, [%1];" : "=f"(v) : "r"(addr) : "memory");
+  return v;
+}
+__device__ __forceinline__ float4 ld_peer4(uint32_t addr) {
+  float4 v;
+  asm volatile("ld.shared::cluster.v4.f32 {%0,%1,%2,%3}, [%4];" : "=f"(v.x), "=f"(v.y), "=f"(v.z), "=f"(v.w) : "r"(addr) : "memory");
+  return v;
+}
+__device__ __forceinline__ void store_bf16x4(__nv_bfloat16* dst, float4 v, float f) {
+  __align__(8) __nv_bfloat162 b[2] = {__floats2bfloat162_rn(v.x * f, v.y * f), __floats2bfloat162_rn(v.z * f, v.w * f)};
+  *reinterpret_cast<uint2*>(dst) = *reinterpret_cast<const uint2*>(b);
+}
+
+__device__ __forceinline__ void bulk_row(void* smem_dst, const void* gsrc, uint32_t bytes, uint64_t* bar) {
+  asm volatile("cp.async.bulk.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1], %2, [%3];"
+               :
+               : "r"(smem_addr(smem_dst)), "l"(gsrc), "r"(bytes), "r"(smem_addr(bar))
+               : "memory");
+}
+
+// One CTA per (key span, chunk of up to 16 MT heads, row).  A row's visible keys are cut into `spans` equal spans of whole
+// tiles, from its own context, so a launch sized for longer contexts stays balanced.  Tiles of TK latent rows are double-buffered: a lane
+// copies one whole row in bulk (rows padded by 16 bytes: conflict-free ldmatrix).  Per tile: partial scores (the warps split 16-key groups and the columns, so
 // the queries are read from shared memory TK / 16 times and not once per warp), running maximum and sum per head, then the
 // weighted sum (a warp owns every sixteenth block of 16 latent columns, up to NB blocks).
+// Merge: the CTAs of a cluster leave their sums in shared memory and each adds up one share of the columns over all of them
+// (distributed shared memory).  With one cluster per row that is the result; with several, latent_reduce_kernel merges theirs.
 template <int MT, int NB, int TK>
 __global__ void __launch_bounds__(DEC_WARPS * 32) latent_decode_kernel(const LatentDecArgs a) {
   extern __shared__ __align__(16) uint8_t smem[];
@@ -190,28 +235,36 @@ __global__ void __launch_bounds__(DEC_WARPS * 32) latent_decode_kernel(const Lat
   const int gc = min(per, a.H - h0);
   pdl_wait();
   pdl_launch();
-  if (gc <= 0) return;
+  if (gc <= 0) return;                                    // the whole cluster: it shares the head chunk
   const int ctx = a.ctx_len[r];
   const int start = (a.window > 0 && ctx > a.window) ? ctx - a.window : 0;
-  const int k0 = start + sp * a.split_len;
-  if (k0 >= ctx) return;
-  const int n = min(a.split_len, ctx - k0), n_tiles = (n + TK - 1) / TK;
+  const int tiles = (ctx - start + TK - 1) / TK, span = (tiles + a.spans - 1) / a.spans * TK;
+  const int k0 = start + sp * span;
+  const int n = max(0, min(span, ctx - k0)), n_tiles = (n + TK - 1) / TK;
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g = lane >> 2, c = lane & 3;
   const int* bt = a.block_table + (size_t)a.slot[r] * a.max_pages;
   const __nv_bfloat16* cache = reinterpret_cast<const __nv_bfloat16*>(a.cache);
 
-  auto load_tile = [&](int t, int buf) {
-    for (int i = warp; i < TK; i += DEC_WARPS) {
-      const int pos = k0 + min(t * TK + i, n - 1);        // rows past the span repeat its last key; their weight is zero
-      const int pi = pos / a.page;
-      const int pg = bt[HE_INDEX_OK(pi, a.max_pages, HE_SITE_ATTN_DECODE_PAGE) ? pi : 0];
-      const __nv_bfloat16* src = cache + ((size_t)pg * a.page + pos % a.page) * a.W;
-      uint8_t* dst = kv_s + ((size_t)buf * TK + i) * pitch;
-      for (int ch = lane; ch < chunks16; ch += 32) cp_async16(dst + ch * 16, src + ch * 8);
-    }
+  __shared__ uint64_t full_s[2];
+  __shared__ int abort_s;
+  if (tid == 0) {
+    sm100::mbar_init(&full_s[0], 1);
+    sm100::mbar_init(&full_s[1], 1);
+    abort_s = 0;
+    sm100::mbar_fence_init();
+  }
+  __syncthreads();
+  const int page_log2 = 31 - __clz(a.page);               // pages are powers of two (checked by the launcher)
+  const auto load_tile = [&](int t, int buf) {
+    if (tid >= TK) return;
+    const int pos = k0 + min(t * TK + tid, n - 1);        // rows past the span repeat its last key; their weight is zero
+    const int pi = pos >> page_log2;
+    const int pg = bt[HE_INDEX_OK(pi, a.max_pages, HE_SITE_ATTN_DECODE_PAGE) ? pi : 0];
+    if (tid == 0) sm100::mbar_expect_tx(&full_s[buf], (uint32_t)TK * a.W * 2);
+    bulk_row(kv_s + ((size_t)buf * TK + tid) * pitch, cache + (((size_t)pg << page_log2) + (pos & (a.page - 1))) * a.W, a.W * 2,
+             &full_s[buf]);
   };
-  load_tile(0, 0);
-  cp_async_commit();
+  if (n > 0) load_tile(0, 0);
   const __nv_bfloat16* q = reinterpret_cast<const __nv_bfloat16*>(a.q) + ((size_t)r * a.H + h0) * a.W;
   for (int i = warp; i < MR; i += DEC_WARPS)
     for (int ch = lane; ch < chunks16; ch += 32)
@@ -236,9 +289,14 @@ __global__ void __launch_bounds__(DEC_WARPS * 32) latent_decode_kernel(const Lat
   for (int t = 0; t < n_tiles; ++t) {
     const int buf = t & 1, live = min(TK, n - t * TK);
     if (t + 1 < n_tiles) load_tile(t + 1, buf ^ 1);
-    cp_async_commit();
-    cp_async_wait<1>();
-    __syncthreads();
+    const bool landed = sm100::mbar_wait(&full_s[buf], (t >> 1) & 1, &abort_s, a.status, 501);
+    if (__syncthreads_or(!landed)) {
+      // give up: no copy may still be in flight when the buffers are written below
+      if (t + 1 < n_tiles)
+        for (uint32_t w = 0; w < sm100::WAIT_LIMIT && !sm100::mbar_try_wait(&full_s[buf ^ 1], ((t + 1) >> 1) & 1); ++w) {}
+      __syncthreads();
+      break;
+    }
     const uint8_t* kt = kv_s + (size_t)buf * TK * pitch;
     // ---- partial scores of 16 keys over this warp's columns (every KS-th group of 32)
     {
@@ -277,31 +335,46 @@ __global__ void __launch_bounds__(DEC_WARPS * 32) latent_decode_kernel(const Lat
         }
     }
     __syncthreads();
-    // ---- running maximum and sum per head
-#pragma unroll
-    for (int hh = 0; hh < MT; ++hh) {
-      const int h = warp + hh * DEC_WARPS;
-      if (h >= gc) break;
-      float v[TK / 32], mx = m_s[h];
+    // ---- running maximum and sum per head: half a warp per head
+    for (int h = warp * 2 + (lane >> 4); h < MR; h += DEC_WARPS * 2) {
+      const int k = (lane & 15) * (TK / 16);              // this lane's neighbouring keys
+      float v[TK / 16], mx = m_s[h];
       const float m_old = mx;
 #pragma unroll
-      for (int i = 0; i < TK / 32; ++i) {
-        float x = 0.f;
+      for (int i = 0; i < TK / 16; ++i) v[i] = 0.f;
 #pragma unroll
-        for (int k = 0; k < KS; ++k) x += sc[(k * MR + h) * SP + i * 32 + lane];
-        v[i] = i * 32 + lane < live ? x * a.scale : -INFINITY;
+      for (int q = 0; q < KS; ++q) {
+        const float* src = sc + (q * MR + h) * SP + k;
+        if constexpr (TK == 64) {
+          const float4 x = *reinterpret_cast<const float4*>(src);
+          v[0] += x.x; v[1] += x.y; v[2] += x.z; v[3] += x.w;
+        } else {
+          const float2 x = *reinterpret_cast<const float2*>(src);
+          v[0] += x.x; v[1] += x.y;
+        }
+      }
+#pragma unroll
+      for (int i = 0; i < TK / 16; ++i) {
+        v[i] = k + i < live ? v[i] * a.scale : -INFINITY;
         mx = fmaxf(mx, v[i]);
       }
-      mx = warp_max(mx);
+#pragma unroll
+      for (int d = 8; d > 0; d >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, d));
       float l = 0.f;
 #pragma unroll
-      for (int i = 0; i < TK / 32; ++i) {
-        const float w = __expf(v[i] - mx);
-        l += w;
-        reinterpret_cast<__nv_bfloat16*>(p_s + h * PP)[i * 32 + lane] = f32_to_bf16(w);
+      for (int i = 0; i < TK / 16; ++i) {
+        v[i] = __expf(v[i] - mx);
+        l += v[i];
       }
-      l = warp_sum(l);
-      if (lane == 0) {
+      uint32_t* dst = reinterpret_cast<uint32_t*>(p_s + h * PP) + k / 2;
+#pragma unroll
+      for (int i = 0; i < TK / 32; ++i) {
+        __nv_bfloat162 b = __floats2bfloat162_rn(v[2 * i], v[2 * i + 1]);
+        dst[i] = *reinterpret_cast<uint32_t*>(&b);
+      }
+#pragma unroll
+      for (int d = 8; d > 0; d >>= 1) l += __shfl_xor_sync(0xffffffffu, l, d);
+      if ((lane & 15) == 0) {
         const float cr = __expf(m_old - mx);
         corr_s[h] = cr;
         l_s[h] = l_s[h] * cr + l;
@@ -346,12 +419,10 @@ __global__ void __launch_bounds__(DEC_WARPS * 32) latent_decode_kernel(const Lat
     }
     __syncthreads();
   }
-  float* part = a.partial + (((size_t)r * a.H + h0) * a.max_splits + sp) * a.rank_cols;
-  const size_t head_stride = (size_t)a.max_splits * a.rank_cols;
-  if (tid < gc) {
-    float2* ml = reinterpret_cast<float2*>(a.partial + (size_t)a.R * a.H * head_stride);
-    ml[((size_t)r * a.H + h0 + tid) * a.max_splits + sp] = make_float2(m_s[tid], l_s[tid]);
-  }
+  // ---- merge.  This CTA's sums go where its tiles were (every warp is past its last tile).
+  __syncthreads();
+  float* o_s = reinterpret_cast<float*>(kv_s);            // [MR][rank_cols]
+  float* w_s = sc;                                        // [cluster or clusters][MR] weights, then [MR] sums
 #pragma unroll
   for (int m = 0; m < MT; ++m)
 #pragma unroll
@@ -360,30 +431,89 @@ __global__ void __launch_bounds__(DEC_WARPS * 32) latent_decode_kernel(const Lat
       if (blk >= n_blk) continue;
 #pragma unroll
       for (int hf = 0; hf < 2; ++hf) {
-        const int h = m * 16 + g + hf * 8;
-        if (h >= gc) continue;
-        float* dst = part + h * head_stride + blk * 16 + 2 * c;
+        float* dst = o_s + (size_t)(m * 16 + g + hf * 8) * a.rank_cols + blk * 16 + 2 * c;
         *reinterpret_cast<float2*>(dst) = make_float2(o[m][j][0][2 * hf], o[m][j][0][2 * hf + 1]);
         *reinterpret_cast<float2*>(dst + 8) = make_float2(o[m][j][1][2 * hf], o[m][j][1][2 * hf + 1]);
       }
     }
+  const int C = a.cluster, cl = sp / C, n_cl = a.spans / C;
+  const uint32_t me = C > 1 ? cluster_rank() : 0u;
+  if (C > 1) {
+    cluster_arrive();
+    cluster_wait();
+  } else {
+    __syncthreads();
+  }
+  const int share = ((a.rank_cols + C - 1) / C + 3) / 4 * 4, d0 = (int)me * share, d1 = min(a.rank_cols, d0 + share);
+  const int quads = max(0, d1 - d0) / 4;
+  __shared__ float M_s[MR], L_s[MR];
+  float* pl_s = w_s + 128 * MR;                           // peers' sums, then nothing
+  if (tid < C * MR) {
+    const int p = tid / MR, h = tid % MR;
+    w_s[tid] = ld_peer(map_peer(smem_addr(m_s + h), p));
+    pl_s[tid] = ld_peer(map_peer(smem_addr(l_s + h), p));
+  }
+  __syncthreads();
+  if (tid < gc) {
+    float M = -INFINITY, L = 0.f;
+    for (int p = 0; p < C; ++p) M = fmaxf(M, w_s[p * MR + tid]);
+    for (int p = 0; p < C; ++p) {
+      const float mp = w_s[p * MR + tid], w = mp == -INFINITY ? 0.f : __expf(mp - M);
+      w_s[p * MR + tid] = w;
+      L += w * pl_s[p * MR + tid];
+    }
+    M_s[tid] = M;
+    L_s[tid] = L;
+  }
+  __syncthreads();
+  __nv_bfloat16* out = reinterpret_cast<__nv_bfloat16*>(a.out) + ((size_t)r * a.H + h0) * a.rank_cols + d0;
+  float* part = a.partial + (((size_t)r * a.H + h0) * n_cl + cl) * a.rank_cols + d0;
+  const size_t head_stride = (size_t)n_cl * a.rank_cols;
+  for (int e = tid; e < gc * quads; e += DEC_WARPS * 32) {
+    const int h = e / quads, d = (e % quads) * 4;
+    float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+    const uint32_t src = smem_addr(o_s + (size_t)h * a.rank_cols + d0 + d);
+    float4 x[8];
+#pragma unroll
+    for (int p = 0; p < 8; ++p) x[p] = p < C ? ld_peer4(map_peer(src, p)) : make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+    for (int p = 0; p < 8; ++p) {
+      const float w = p < C ? w_s[p * MR + h] : 0.f;      // an idle CTA's sums are zeros
+      v.x += w * x[p].x; v.y += w * x[p].y; v.z += w * x[p].z; v.w += w * x[p].w;
+    }
+    if (n_cl == 1) {
+      float f = 1.f, L = L_s[h];
+      if (a.sink != nullptr) {
+        const float sk = a.sink[h0 + h], mn = fmaxf(M_s[h], sk);
+        f = __expf(M_s[h] - mn);
+        L = L * f + __expf(sk - mn);
+      }
+      store_bf16x4(out + (size_t)h * a.rank_cols + d, v, L > 0.f ? f / L : 0.f);
+    } else {
+      *reinterpret_cast<float4*>(part + h * head_stride + d) = v;
+    }
+  }
+  __syncwarp();
+  if (C > 1) cluster_arrive();                            // done with the peers' shared memory
+  if (n_cl > 1 && me == 0 && tid < gc) {
+    float2* ml = reinterpret_cast<float2*>(a.partial + (size_t)a.R * a.H * head_stride);
+    ml[((size_t)r * a.H + h0 + tid) * n_cl + cl] = make_float2(M_s[tid], L_s[tid]);
+  }
+  if (C > 1) cluster_wait();
 }
 
-// grid (H, R, ceil(rank_cols / 128)): merge the spans (the eight warps take them in turn, a lane owns four columns), add the
+// grid (H, R, ceil(rank_cols / 128)): merge the clusters' sums (the eight warps take them in turn, a lane owns four columns), add the
 // sink to the denominator, round to bf16
-constexpr int RED_WARPS = 8;
+constexpr int RED_WARPS = 8, MAX_CLUSTERS = 128;
 __global__ void __launch_bounds__(RED_WARPS * 32) latent_reduce_kernel(const LatentDecArgs a) {
-  extern __shared__ float wsm[];     // [max_splits]
-  __shared__ float red[33];
+  __shared__ float red[33], wsm[MAX_CLUSTERS];
   __shared__ float4 acc_s[RED_WARPS][32];
   pdl_wait();
   pdl_launch();
   const int h = blockIdx.x, r = blockIdx.y, lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
-  const int ctx = a.ctx_len[r];
-  const int start = (a.window > 0 && ctx > a.window) ? ctx - a.window : 0;
-  const int ns = min((ctx - start + a.split_len - 1) / a.split_len, a.max_splits);
-  const size_t row = ((size_t)r * a.H + h) * a.max_splits;
-  const float2* ml = reinterpret_cast<const float2*>(a.partial + (size_t)a.R * a.H * a.max_splits * a.rank_cols) + row;
+  const int ns = a.spans / a.cluster;
+  const size_t row = ((size_t)r * a.H + h) * ns;
+  const float2* ml = reinterpret_cast<const float2*>(a.partial + (size_t)a.R * a.H * ns * a.rank_cols) + row;
   const int d = blockIdx.z * 128 + lane * 4;
   const float* pb = a.partial + row * a.rank_cols + d;
   const bool mine = d < a.rank_cols;
@@ -402,7 +532,7 @@ __global__ void __launch_bounds__(RED_WARPS * 32) latent_reduce_kernel(const Lat
   float den = 0.f;
   for (int s = threadIdx.x; s < ns; s += RED_WARPS * 32) {
     const float2 v = ml[s];
-    const float w = __expf(v.x - m);
+    const float w = v.x == -INFINITY ? 0.f : __expf(v.x - m);      // an idle cluster
     wsm[s] = w;
     den += w * v.y;
   }
@@ -432,10 +562,8 @@ __global__ void __launch_bounds__(RED_WARPS * 32) latent_reduce_kernel(const Lat
     const float4 v = acc_s[w][lane];
     acc.x += v.x; acc.y += v.y; acc.z += v.z; acc.w += v.w;
   }
-  const float inv = den > 0.f ? 1.f / den : 0.f;
-  __align__(8) __nv_bfloat162 b[2] = {__floats2bfloat162_rn(acc.x * inv, acc.y * inv), __floats2bfloat162_rn(acc.z * inv, acc.w * inv)};
-  *reinterpret_cast<uint2*>(reinterpret_cast<__nv_bfloat16*>(a.out) + ((size_t)r * a.H + h) * a.rank_cols + d) =
-      *reinterpret_cast<const uint2*>(b);
+  store_bf16x4(reinterpret_cast<__nv_bfloat16*>(a.out) + ((size_t)r * a.H + h) * a.rank_cols + d, acc,
+               den > 0.f ? 1.f / den : 0.f);
 }
 
 // ---------------------------------------------------------------- fp32: one CTA per (row, head)
@@ -524,20 +652,32 @@ __global__ void __launch_bounds__(256) latent_gather_kernel(const LatentGatherAr
 template <int MT, int NB, int TK>
 int launch_decode(const LatentDecArgs& a, cudaStream_t stream) {
   const size_t smem = dec_smem<MT, TK>(a.W);
-  if (smem > 227 * 1024) return -HE_ERR_BAD_ARG;
+  if (smem > 226 * 1024) return -HE_ERR_BAD_ARG;          // a few hundred bytes are static
   cudaError_t e = cudaFuncSetAttribute(latent_decode_kernel<MT, NB, TK>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
   if (e != cudaSuccess) return (int)e;
-  const dim3 grid(a.max_splits, (a.H + MT * 16 - 1) / (MT * 16), a.R);
-  return (int)launch_pdl(latent_decode_kernel<MT, NB, TK>, grid, dim3(DEC_WARPS * 32), smem, stream, a);
+  cudaLaunchConfig_t cfg = {};
+  cfg.gridDim = dim3(a.spans, (a.H + MT * 16 - 1) / (MT * 16), a.R);
+  cfg.blockDim = dim3(DEC_WARPS * 32);
+  cfg.dynamicSmemBytes = smem;
+  cfg.stream = stream;
+  cudaLaunchAttribute attr[2];
+  attr[0].id = cudaLaunchAttributeClusterDimension;
+  attr[0].val.clusterDim.x = a.cluster;
+  attr[0].val.clusterDim.y = attr[0].val.clusterDim.z = 1;
+  attr[1].id = cudaLaunchAttributeProgrammaticStreamSerialization;
+  attr[1].val.programmaticStreamSerializationAllowed = 1;
+  cfg.attrs = attr;
+  cfg.numAttrs = pdl_enabled() ? 2 : 1;
+  return (int)cudaLaunchKernelEx(&cfg, latent_decode_kernel<MT, NB, TK>, a);
 }
 
 // Tiles of 64 keys and 32 heads where they fit and the spans are whole tiles, else smaller ones.
 template <int NB>
 int pick_decode(const LatentDecArgs& a, cudaStream_t stream) {
-  const bool big = a.split_len % 64 == 0;
-  if (a.H > 16 && big && dec_smem<2, 64>(a.W) <= 227 * 1024) return launch_decode<2, NB, 64>(a, stream);
-  if (a.H > 16 && dec_smem<2, 32>(a.W) <= 227 * 1024) return launch_decode<2, NB, 32>(a, stream);
-  if (big && dec_smem<1, 64>(a.W) <= 227 * 1024) return launch_decode<1, NB, 64>(a, stream);
+  const bool big = a.tile == 64;
+  if (a.H > 16 && big && dec_smem<2, 64>(a.W) <= 226 * 1024) return launch_decode<2, NB, 64>(a, stream);
+  if (a.H > 16 && dec_smem<2, 32>(a.W) <= 226 * 1024) return launch_decode<2, NB, 32>(a, stream);
+  if (big && dec_smem<1, 64>(a.W) <= 226 * 1024) return launch_decode<1, NB, 64>(a, stream);
   return launch_decode<1, NB, 32>(a, stream);
 }
 
@@ -546,7 +686,7 @@ int pick_decode(const LatentDecArgs& a, cudaStream_t stream) {
 HE_API int he_latent_post(const LatentPostArgs* args, cudaStream_t stream) {
   const LatentPostArgs& a = *args;
   if (a.T <= 0) return 0;
-  if (a.rot_dim % 2 != 0 || a.dn % 2 != 0 || a.q_cols % 2 != 0 || a.q_cols < a.dn + a.rot_dim || a.rank > a.rank_cols ||
+  if (a.rank_cols > 1024 || a.rot_dim % 2 != 0 || a.dn % 2 != 0 || a.q_cols % 2 != 0 || a.q_cols < a.dn + a.rot_dim || a.rank > a.rank_cols ||
       a.W < a.rank_cols + a.rot_dim || (a.W - a.rank_cols) % 2 != 0)
     return -HE_ERR_BAD_ARG;
   if (a.q_out == a.q && (a.q_dtype == 0) != (a.out_f32 != 0)) return -HE_ERR_BAD_ARG;
@@ -563,19 +703,18 @@ static int check_decode(const LatentDecArgs& a) {
   return 0;
 }
 
-// Scratch: R * H * max_splits * (rank_cols + 2) floats in `partial`.
+// With more than one cluster per row (spans > cluster): `partial` holds R * H * (spans / cluster) * (rank_cols + 2) floats.
 HE_API int he_latent_decode(const LatentDecArgs* args, cudaStream_t stream) {
   const LatentDecArgs& a = *args;
   if (a.R <= 0) return 0;
-  if (check_decode(a) != 0 || a.split_len <= 0 || a.max_splits <= 0 || a.R > 65535) return -HE_ERR_BAD_ARG;
+  if (check_decode(a) != 0 || a.cluster < 1 || a.cluster > 8 || a.spans < a.cluster || a.spans % a.cluster != 0 ||
+      a.spans / a.cluster > MAX_CLUSTERS || (a.tile != 32 && a.tile != 64) || a.R > 65535)
+    return -HE_ERR_BAD_ARG;
+  if ((a.spans > a.cluster && a.partial == nullptr) || a.page <= 0 || (a.page & (a.page - 1)) != 0) return -HE_ERR_BAD_ARG;
   const int nb = (a.rank_cols / 16 + DEC_WARPS - 1) / DEC_WARPS;
-  int rc;
-  if (nb <= 1) rc = pick_decode<1>(a, stream);
-  else if (nb <= 2) rc = pick_decode<2>(a, stream);
-  else rc = launch_decode<1, 4, 32>(a, stream);
-  if (rc != 0) return rc;
-  return (int)launch_pdl(latent_reduce_kernel, dim3(a.H, a.R, (a.rank_cols + 127) / 128), dim3(RED_WARPS * 32),
-                         (size_t)a.max_splits * sizeof(float), stream, a);
+  const int rc = nb <= 1 ? pick_decode<1>(a, stream) : nb <= 2 ? pick_decode<2>(a, stream) : launch_decode<1, 4, 32>(a, stream);
+  if (rc != 0 || a.spans == a.cluster) return rc;
+  return (int)launch_pdl(latent_reduce_kernel, dim3(a.H, a.R, (a.rank_cols + 127) / 128), dim3(RED_WARPS * 32), 0, stream, a);
 }
 HE_API int he_latent_dec_args_size() { return (int)sizeof(LatentDecArgs); }
 

@@ -227,9 +227,9 @@ class MilutarExecutor(ListedExecutor):
         if self.exact:
             LA.latent_exact(*args, o_lat, rank, a.scale, a.window, L.sink)
         else:
-            split_len, n_splits = LA.decode_split(min(ctx, a.window) if a.window else ctx, R, H, a.row_cols)
-            part = self.scratch.get("attn_part", (LA.decode_scratch_floats(R, H, n_splits, rank),), torch.float32)
-            LA.latent_decode(*args, part, o_lat, rank, a.scale, split_len, n_splits, a.window, L.sink)
+            plan = LA.decode_plan(min(ctx, a.window) if a.window else ctx, R, H, a.row_cols)
+            part = self.scratch.get("attn_part", (plan.scratch_floats(R, H, rank),), torch.float32)
+            LA.latent_decode(*args, part, o_lat, rank, a.scale, plan, a.window, L.sink)
         mul(o_lat, L.uv.data.view(H, L.dv, rank), out[r0:r1].view(R, H, L.dv))
 
     def _expanded(self, a: LatentAttentionSpec, L: _Layer, kv: torch.Tensor, q: torch.Tensor, b: BatchDesc, s: int, e: int,

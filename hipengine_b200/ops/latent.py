@@ -6,6 +6,7 @@ part, zero-padded.
 from __future__ import annotations
 
 import ctypes as C
+from dataclasses import dataclass
 from typing import Optional, Sequence, Tuple
 
 import torch
@@ -26,9 +27,9 @@ class _PostArgs(C.Structure):
 
 class _DecArgs(C.Structure):
     _fields_ = [("q", c_vp), ("cache", c_vp), ("block_table", c_vp), ("slot", c_vp), ("ctx_len", c_vp),
-                ("partial", c_vp), ("out", c_vp), ("sink", c_vp), ("R", c_int), ("H", c_int), ("W", c_int),
-                ("rank_cols", c_int), ("page", c_int), ("max_pages", c_int), ("split_len", c_int), ("max_splits", c_int),
-                ("window", c_int), ("scale", C.c_float)]
+                ("partial", c_vp), ("out", c_vp), ("sink", c_vp), ("R", c_int), ("H", c_int),
+                ("W", c_int), ("rank_cols", c_int), ("page", c_int), ("max_pages", c_int), ("window", c_int),
+                ("spans", c_int), ("cluster", c_int), ("tile", c_int), ("scale", C.c_float), ("status", c_vp)]
 
 
 class _GatherArgs(C.Structure):
@@ -83,23 +84,34 @@ def latent_post(down: torch.Tensor, q: torch.Tensor, norm_w: torch.Tensor, freq:
     N.check(_lib().he_latent_post(C.byref(a), _stream()), "he_latent_post")
 
 
-def decode_split(span: int, rows: int, heads: int, W: int) -> Tuple[int, int]:
-    """(split_len, max_splits): the spans of all rows and head chunks fill the SMs about once (wide rows: one CTA per SM) or
-    a few times (narrow rows), without a last round of a few stragglers.  Spans are whole tiles of 64 keys, or single tiles
-    of 32 where even those leave SMs idle."""
+@dataclass(frozen=True)
+class DecodePlan:
+    """How a latent-space launch cuts the keys of a row: ``spans`` CTAs, ``cluster`` of them merging on chip, key tiles of
+    ``tile``."""
+    spans: int
+    cluster: int
+    tile: int
+
+    @property
+    def clusters(self) -> int:
+        return self.spans // self.cluster
+
+    def scratch_floats(self, rows: int, heads: int, rank_cols: int) -> int:
+        """Cluster sums and their (maximum, sum) pairs; none when one cluster covers a row."""
+        return rows * heads * self.clusters * (rank_cols + 2) if self.clusters > 1 else 0
+
+
+def decode_plan(span: int, rows: int, heads: int, W: int) -> DecodePlan:
+    """Plan for ``rows`` rows of up to ``span`` visible keys: about one round of CTAs over the GPU, no more spans than
+    tiles, tiles of 32 keys where tiles of 64 would leave SMs idle.  Clusters of four pack the SMs; wider ones do not."""
     chunks, tile_rows = (-(-heads // 32), 32) if heads > 16 else (1, 16)
     per_sm = max(1, min(4, int(227e3 // ((tile_rows + 128) * (2 * W + 16) + tile_rows * 1300))))
-    slots, jobs = 148 * per_sm, max(rows, 1) * chunks
-    if span * jobs <= 32 * slots:
-        return 32, max(1, -(-span // 32))
-    spans = max(1, slots // jobs)                    # whole rounds: every job gets the same number of spans
-    split = max(64, -(-(-(-span // spans)) // 64) * 64)
-    return split, max(1, -(-span // split))
-
-
-def decode_scratch_floats(rows: int, heads: int, max_splits: int, rank_cols: int) -> int:
-    """Span sums, then their (maximum, sum) pairs."""
-    return rows * heads * max_splits * (rank_cols + 2)
+    want = max(1, 128 * per_sm // (max(rows, 1) * chunks))
+    tile = 64 if -(-span // 64) >= min(want, 64) else 32
+    spans = min(want, -(-span // tile))
+    if spans > 4:
+        return DecodePlan(min(512, spans // 4 * 4), 4, tile)
+    return DecodePlan(spans, spans, tile)
 
 
 def _dec_args(q, cache, block_table, slot, ctx_len, out, rank_cols, scale, window, sink) -> _DecArgs:
@@ -111,17 +123,18 @@ def _dec_args(q, cache, block_table, slot, ctx_len, out, rank_cols, scale, windo
     a.q, a.cache, a.block_table, a.slot, a.ctx_len = (t.data_ptr() for t in (q, cache, block_table, slot, ctx_len))
     a.out, a.sink, a.R, a.H, a.W, a.rank_cols = out.data_ptr(), _p(sink), R, H, W, rank_cols
     a.page, a.max_pages, a.window, a.scale = cache.shape[1], block_table.shape[1], window, scale
+    a.status = status_tensor(q.device).data_ptr()
     return a
 
 
 def latent_decode(q: torch.Tensor, cache: torch.Tensor, block_table: torch.Tensor, slot: torch.Tensor,
                   ctx_len: torch.Tensor, partial: torch.Tensor, out: torch.Tensor, rank_cols: int, scale: float,
-                  split_len: int, max_splits: int, window: int = 0, sink: Optional[torch.Tensor] = None) -> None:
+                  plan: DecodePlan, window: int = 0, sink: Optional[torch.Tensor] = None) -> None:
     """Every row of ``q`` [R, H, W] (latent-space queries) against its request's cache rows; ``out`` [R, H, rank_cols] is
-    the weighted sum of latents."""
+    the weighted sum of latents.  ``partial`` holds ``plan.scratch_floats``."""
     a = _dec_args(q, cache, block_table, slot, ctx_len, out, rank_cols, scale, window, sink)
-    a.partial, a.split_len, a.max_splits = partial.data_ptr(), split_len, max_splits
-    assert q.dtype == torch.bfloat16 and partial.numel() >= decode_scratch_floats(a.R, a.H, max_splits, rank_cols)
+    a.partial, a.spans, a.cluster, a.tile = partial.data_ptr(), plan.spans, plan.cluster, plan.tile
+    assert q.dtype == torch.bfloat16 and partial.numel() >= plan.scratch_floats(a.R, a.H, rank_cols)
     N.check(_lib().he_latent_decode(C.byref(a), _stream()), "he_latent_decode")
 
 

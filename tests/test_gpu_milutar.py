@@ -238,11 +238,11 @@ def test_latent_space_attention(heads, rank, rd, window, sink, exact):
         _close(out[:, :, :rank], want, 1e-4)
         assert not out[:, :, rank:].any()
         return
-    span = min(300, window) if window else 300
-    for split in (32, 64, 96, 128, 192, 1024):
-        ns = -(-span // split)
-        part = torch.full((LA.decode_scratch_floats(n, heads, ns, rc),), float("nan"), device="cuda")
-        LA.latent_decode(ql, cache, bt, slot, ctx, part, out, rc, scale, split, ns, window, skc)
+    for spans, cluster, tile in ((1, 1, 64), (1, 1, 32), (3, 3, 64), (8, 8, 32), (5, 1, 64), (6, 2, 32), (16, 8, 32)):
+        plan = LA.DecodePlan(spans, cluster, tile)
+        part = torch.full((max(1, plan.scratch_floats(n, heads, rc)),), float("nan"), device="cuda")
+        out.fill_(7.0)
+        LA.latent_decode(ql, cache, bt, slot, ctx, part, out, rc, scale, plan, window, skc)
         K.check_status()
         _close(out[:, :, :rank], want, 0.02)
         assert not out[:, :, rank:].any()
