@@ -714,7 +714,10 @@ HE_API int he_latent_decode(const LatentDecArgs* args, cudaStream_t stream) {
   const int nb = (a.rank_cols / 16 + DEC_WARPS - 1) / DEC_WARPS;
   const int rc = nb <= 1 ? pick_decode<1>(a, stream) : nb <= 2 ? pick_decode<2>(a, stream) : launch_decode<1, 4, 32>(a, stream);
   if (rc != 0 || a.spans == a.cluster) return rc;
-  return (int)launch_pdl(latent_reduce_kernel, dim3(a.H, a.R, (a.rank_cols + 127) / 128), dim3(RED_WARPS * 32), 0, stream, a);
+  // in plain stream order: started early beside CTAs that fill their SMs, this small grid costs a decode step up to 40 us a layer
+  latent_reduce_kernel<<<dim3(a.H, a.R, (a.rank_cols + 127) / 128), dim3(RED_WARPS * 32), 0, stream>>>(a);
+  HE_LAUNCH_CHECK();
+  return 0;
 }
 HE_API int he_latent_dec_args_size() { return (int)sizeof(LatentDecArgs); }
 
