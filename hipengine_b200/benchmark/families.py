@@ -301,7 +301,7 @@ def main(argv: Optional[List[str]] = None) -> int:
     with NvmlSampler(device_index=torch.cuda.current_device(), interval_s=0.02) as clocks:
         def emit_clocked(r: Dict) -> None:
             """The row with the clocks and throttle reasons sampled since the last one."""
-            seen, clocks.samples = clocks.samples, []
+            seen, clocks.samples = clocks.samples, clocks.samples[-1:]      # a short row falls back on the last sample
             mhz = sorted(s.sm_mhz for s in seen if s.sm_mhz is not None)
             reasons = sorted({n for s in seen for n in decode_reasons(s.reasons)})
             emit({**r, "sm_mhz": mhz[len(mhz) // 2] if mhz else None, "clock_reasons": reasons})
