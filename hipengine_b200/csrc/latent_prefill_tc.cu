@@ -1,4 +1,4 @@
-// Prefill form of latent attention on the 5th-generation tensor cores (same contract as latent_prefill.cu, head widths of 64
+// Prefill form of latent attention on the 5th-generation tensor cores (same arguments as latent_prefill.cu, head widths of 64
 // or 128): a CTA owns 256 query rows of one head as two tiles of 128.
 //
 //   warps 0-3, 4-7 : softmax of one tile each; a thread owns a row (= a TMEM lane), so maxima and sums need no shuffles

@@ -17,6 +17,8 @@ def kv_capability(cfg, kv_cfg) -> Dict[str, Any]:
     compare each path with fp32 PyTorch).  The reference ships such a record per storage mode
     (``hipengine/kvcache/capabilities.py``)."""
     hd = int(getattr(cfg, "head_dim", 0) or 0)
+    mixers = [l.mixer for l in getattr(cfg, "layer_specs", ())]
+    latent = [m for m in mixers if hasattr(m, "row_cols")]
     return {
         "storage": {"bf16": {"supported": True, "evidence": "tests/test_gpu_kernels.py (paged write + decode), "
                                                              "tests/test_gpu_executor.py (end to end vs fp32)"},
@@ -26,14 +28,17 @@ def kv_capability(cfg, kv_cfg) -> Dict[str, Any]:
                                        "backend only"}},
         "selected_storage": getattr(kv_cfg, "storage", "bf16"),
         "page_tokens": int(getattr(kv_cfg, "page_tokens", 16)),
-        "layout": "[pages][k|v][kv_heads][page_tokens][head_dim] bf16, block table per slot",
+        "layout": "[pages][page_tokens][latent | rotated key part] bf16, one row per token for all heads, block table per "
+                  "slot" if latent else "[pages][k|v][kv_heads][page_tokens][head_dim] bf16, block table per slot",
         "head_dim": hd,
-        "decode_kernel": "tensor-core split-K (mma.sync over the query heads of a KV group)" if hd >= 128
+        "decode_kernel": "latent space, split-K (mma.sync over the heads)" if latent else
+                         "tensor-core split-K (mma.sync over the query heads of a KV group)" if hd >= 128
                          else "CUDA-core split-K",
-        "prefill_kernel": "flash (mma.sync)" if hd in (64, 128, 256) else "row-wise decode kernel",
+        "prefill_kernel": "expanded keys and values: tcgen05, or mma.sync by head shape" if latent else
+                          "flash (mma.sync)" if hd in (64, 128, 256) else "row-wise decode kernel",
         "prefix_cache": getattr(kv_cfg, "prefix_cache", "off"),
         "recurrent_state_snapshots": bool(getattr(cfg, "has_recurrent_state", False)),
-        "sliding_window": bool(getattr(cfg, "sliding_window", 0)),
+        "sliding_window": bool(getattr(cfg, "sliding_window", 0)) or any(getattr(m, "window", 0) for m in mixers),
         "cold_tier": True,
     }
 

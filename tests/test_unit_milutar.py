@@ -96,6 +96,16 @@ def test_registry_entries():
     assert all(c in NAMED_CONFIGS for c in ("tiny-milutar", "milutar-8b"))
 
 
+def test_readiness_describes_the_latent_cache():
+    from hipengine_b200.config import EngineConfig
+    from hipengine_b200.server.readiness import kv_capability
+    d = kv_capability(TINY_MILUTAR, EngineConfig().kv)
+    assert "latent" in d["layout"] and "latent" in d["decode_kernel"] and "expanded" in d["prefill_kernel"]
+    assert d["sliding_window"] and d["recurrent_state_snapshots"]
+    plain = kv_capability(NAMED_CONFIGS["tiny-sisisun"], EngineConfig().kv)
+    assert "[k|v]" in plain["layout"] and not plain["sliding_window"]
+
+
 @pytest.mark.parametrize("dims,base,y", [(2, 100.0, None), (12, 3000.0, (6.0, 256.0, 16.0, 1.0)), (64, 1e6, (32.0, 8192.0, 32.0, 1.0)),
                                          (4, 500.0, (3.0, 64.0, 8.0, 2.0)), (16, 10000.0, (1.0, 4096.0, 32.0, 1.0)),
                                          (8, 50.0, (4.0, 2.0, 32.0, 30.0))])
