@@ -28,7 +28,7 @@ def full(heads, dim, rot, vdim, rank, scale, q_rank, base=10000.0):
                                   "q_rank": q_rank, "rot": {"dims": rot, "base": base}}
 
 
-def model(width, vocab, layers, loop=None, eps=1e-5, mult=0.8):
+def model(width, vocab, layers, loop=None, eps=3e-5, mult=0.8):
     return {"architecture": "Milutar", "width": width, "vocab": vocab, "norm": {"eps": eps}, "residual_mult": mult,
             "loop": {"start": loop[0], "stop": loop[1], "times": loop[2]} if loop else None,
             "layers": [{"type": t, "mixer": m, "mlp": {"kind": "dense", "ff": ff} if ff else None} for (t, m), ff in layers]}
@@ -43,9 +43,9 @@ ODD = model(132, 301, [
     (full(4, 8, 10, 12, 50, 0.6, 40, 400.0), 72),
 ], loop=(1, 3, 2), eps=1e-4, mult=0.55)
 # many heads (more than one chunk of the decode kernel), no loop
-HEADS = model(256, 512, [
+HEADS = model(248, 520, [
     (full(40, 24, 20, 16, 136, 0.15, 96), 192),
-    (windowed(17, 64, 32, 48, 72, 0.11, 33, 20000.0, yarn(2.0, 128.0, 4.0, 0.5)), 256),
+    (windowed(17, 64, 32, 48, 72, 0.11, 33, 15000.0, yarn(2.0, 128.0, 4.0, 0.5)), 256),
 ])
 # wide latents and heads: every size class of the kernels, one layer whose heads the prefill kernel does not take
 WIDE = model(160, 200, [
@@ -57,7 +57,7 @@ WIDE = model(160, 200, [
 LOOPED = model(96, 160, [
     (windowed(4, 24, 8, 40, 32, 0.2, 48, 2000.0, yarn(4.0, 128.0, 8.0, 1.0)), 128),
     (full(4, 24, 8, 40, 32, 0.2, 64), 112),
-], loop=(0, 2, 4), mult=0.7)
+], loop=(0, 2, 4), mult=0.75)
 # sizes of one: one head, one pair, windows of one and two tokens, one pass, no residual factor, a scaling that scales by one
 ONES = model(64, 96, [
     (windowed(1, 8, 2, 8, 8, 0.4, 1, 100.0, yarn(1.0, 32.0, 2.0, 1.0)), 16),
