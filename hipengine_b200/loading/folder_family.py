@@ -5,12 +5,13 @@ its shape, in file order); the registry names the module.
 """
 from __future__ import annotations
 
+from dataclasses import asdict
 from importlib import import_module
 from typing import Any, Callable, Dict, Mapping, Optional, Sequence, Tuple
 
 import torch
 
-from ..models.config import LoopSpec, ModelConfig
+from ..models.config import BandSpec, LoopSpec, ModelConfig, RotarySpec, YarnSpec
 from ..quant.ggml import GGMLType
 from .weights import ModelWeights, QTensor
 
@@ -30,6 +31,27 @@ def loop_from_json(c: Mapping[str, Any]) -> Optional[LoopSpec]:
 
 def loop_to_json(loop: Optional[LoopSpec]) -> Optional[Dict[str, int]]:
     return {"start": loop.start, "stop": loop.stop, "times": loop.times} if loop else None
+
+
+# keys of a rotation's scaling -> what it is
+_SCALINGS = (BandSpec, ("factor", "low", "high", "original")), (YarnSpec, ("factor", "original", "fast", "slow"))
+
+
+def rotary_from_json(r: Mapping[str, Any], halves: bool = False) -> RotarySpec:
+    s, scaling = r.get("scaling"), None
+    if s:
+        found = [c(*(float(s[k]) for k in keys)) for c, keys in _SCALINGS if set(keys) == set(s)]
+        if not found:
+            raise ValueError(f"unknown scaling of a rotation: {sorted(s)}")
+        scaling = found[0]
+    return RotarySpec(int(r["dims"]), float(r["base"]), scaling, halves)
+
+
+def rotary_to_json(rot: RotarySpec) -> Dict[str, Any]:
+    out: Dict[str, Any] = {"dims": rot.dims, "base": rot.base}
+    if rot.scaling is not None:
+        out["scaling"] = asdict(rot.scaling)
+    return out
 
 
 def check_tensors(cfg: ModelConfig, have: Shapes) -> None:

@@ -11,9 +11,8 @@ from typing import Any, Dict, List, Mapping, Optional, Tuple
 
 import torch
 
-from ..models.config import (DenseMlpSpec, LatentAttentionSpec, LayerSpec, ModelConfig, RotarySpec, YarnSpec,
-                             milutar_config)
-from .folder_family import build_random_folder, loop_from_json, loop_to_json
+from ..models.config import DenseMlpSpec, LatentAttentionSpec, LayerSpec, ModelConfig, milutar_config
+from .folder_family import build_random_folder, loop_from_json, loop_to_json, rotary_from_json, rotary_to_json
 from .weights import ModelWeights
 
 # mixer name -> (queries go through a latent, the softmax has a sink)
@@ -21,12 +20,6 @@ MIXERS = {"latent_attention": (False, False), "latent_attention_2": (True, True)
 
 
 # ----------------------------------------------------------------------------- configuration
-def _rotary(r: Mapping[str, Any]) -> RotarySpec:
-    y = r.get("scaling")
-    yarn = YarnSpec(*(float(y[k]) for k in ("factor", "original", "fast", "slow"))) if y else None
-    return RotarySpec(int(r["dims"]), float(r["base"]), yarn)
-
-
 def _layer(i: int, l: Mapping[str, Any]) -> LayerSpec:
     if l["type"] not in MIXERS:
         raise ValueError(f"layer {i}: unknown mixer {l['type']!r}")
@@ -35,7 +28,7 @@ def _layer(i: int, l: Mapping[str, Any]) -> LayerSpec:
     if mlp is not None and mlp["kind"] != "dense":
         raise ValueError(f"layer {i}: unknown feed-forward kind {mlp['kind']!r}")
     a = LatentAttentionSpec(heads=int(m["heads"]), dim=int(m["dim"]), rot_dim=int(m["rot_dim"]), vdim=int(m["vdim"]),
-                            kv_rank=int(m["kv_rank"]), scale=float(m["scale"]), rot=_rotary(m["rot"]),
+                            kv_rank=int(m["kv_rank"]), scale=float(m["scale"]), rot=rotary_from_json(m["rot"]),
                             q_rank=int(m["q_rank"]) if q_latent else 0, window=int((m.get("mask") or {}).get("size", 0)),
                             sink=sink)
     return LayerSpec(a, DenseMlpSpec(int(mlp["ff"]), "relu2") if mlp is not None else None, parallel=True, token_shift=True)
@@ -49,12 +42,9 @@ def config_from_json(c: Mapping[str, Any]) -> ModelConfig:
 def config_to_json(cfg: ModelConfig) -> Dict[str, Any]:
     layers: List[Dict[str, Any]] = []
     for l in cfg.layer_specs:
-        a, y = l.mixer, l.mixer.rot.yarn
-        rot: Dict[str, Any] = {"dims": a.rot.dims, "base": a.rot.base}
-        if y is not None:
-            rot["scaling"] = {"factor": y.factor, "original": y.original, "fast": y.fast, "slow": y.slow}
+        a = l.mixer
         m: Dict[str, Any] = {"heads": a.heads, "dim": a.dim, "rot_dim": a.rot_dim, "vdim": a.vdim, "kv_rank": a.kv_rank,
-                             "scale": a.scale, "rot": rot}
+                             "scale": a.scale, "rot": rotary_to_json(a.rot)}
         if a.q_rank:
             m["q_rank"] = a.q_rank
         if a.window:

@@ -25,28 +25,6 @@ def padded_head_width(d: int) -> int:
 
 
 @dataclass(frozen=True)
-class AttentionSpec:
-    """Softmax attention of one layer, for designs whose layers are listed one by one."""
-    heads: int
-    kv_heads: int
-    dim: int                             # query / key width per head
-    vdim: int                            # value width per head
-    scale: float
-    softcap: float = 0.0                 # > 0: score <- softcap * tanh(score / softcap)
-
-    @property
-    def width(self) -> int:
-        """Width a head takes in the KV pages (both planes)."""
-        return padded_head_width(max(self.dim, self.vdim))
-
-
-    @property
-    def cache_elems(self) -> int:
-        """Elements a token takes in the layer's cache plane."""
-        return 2 * self.kv_heads * self.width
-
-
-@dataclass(frozen=True)
 class YarnSpec:
     """Context extension of a rotary table: slow pairs are slowed down by ``factor``, fast ones are kept."""
     factor: float
@@ -56,24 +34,97 @@ class YarnSpec:
 
 
 @dataclass(frozen=True)
+class BandSpec:
+    """Context extension by wave length (Llama 3.1): waves that fit ``high`` times into the original context are kept, those
+    that fit less than ``low`` times are slowed down by ``factor``, those between are mixed."""
+    factor: float
+    low: float
+    high: float
+    original: float
+
+    def scaled(self, freq: float) -> float:
+        turns = self.original * freq / (2 * math.pi)
+        if turns >= self.high:
+            return freq
+        if turns <= self.low:
+            return freq / self.factor
+        keep = (turns - self.low) / (self.high - self.low)
+        return (1.0 - keep) * freq / self.factor + keep * freq
+
+
+@dataclass(frozen=True)
 class RotarySpec:
-    """Rotation of neighbouring pairs (2i, 2i + 1) by position * base^(-2i / dims)."""
+    """Rotation of pairs by position * base^(-2i / dims): of neighbours (2i, 2i + 1), or with ``halves`` of (i, i + dims / 2)."""
     dims: int
     base: float
-    yarn: Optional[YarnSpec] = None
+    scaling: Optional[Union[YarnSpec, BandSpec]] = None
+    halves: bool = False
 
     def table(self) -> Tuple[Tuple[float, ...], float]:
         """(angular frequency per pair, amplitude of sine and cosine)."""
         freq = [self.base ** (-2.0 * i / self.dims) for i in range(self.dims // 2)]
-        y = self.yarn
+        y = self.scaling
         if y is None:
             return tuple(freq), 1.0
+        if isinstance(y, BandSpec):
+            return tuple(y.scaled(f) for f in freq), 1.0
         at = lambda turns: self.dims * math.log(y.original / (2 * math.pi * turns)) / (2 * math.log(self.base))
         lo, hi = max(math.floor(at(y.fast)), 0), min(math.ceil(at(y.slow)), self.dims - 1)
         for i, f in enumerate(freq):
             slow = min(max((i - lo) / max(hi - lo, 0.001), 0.0), 1.0)
             freq[i] = f * (slow / y.factor + 1.0 - slow)
         return tuple(freq), 0.1 * math.log(y.factor) + 1.0
+
+
+# how queries and keys are normalised
+QK_NORM_NONE = "none"
+QK_NORM_HEAD = "head"                    # every head over its own width, gains per dimension, before the rotation
+QK_NORM_ROWS = "rows"                    # the whole projection at once, gains per column, before the rotation
+QK_NORM_UNIT = "unit"                    # every head over its own width, no gains, after the rotation
+
+
+@dataclass(frozen=True)
+class AttentionSpec:
+    """Softmax attention of one layer, for designs whose layers are listed one by one."""
+    heads: int
+    kv_heads: int
+    dim: int                             # query / key width per head
+    vdim: int                            # value width per head
+    scale: float
+    softcap: float = 0.0                 # > 0: score <- softcap * tanh(score / softcap)
+    rot: Optional[RotarySpec] = None     # of the first ``rot.dims`` dimensions of queries and keys
+    window: int = 0                      # > 0: only the last ``window`` positions are visible
+    sink_score: Optional[float] = None   # score of a term in the softmax denominator that has no value
+    qk_norm: str = QK_NORM_HEAD
+    bias: bool = False                   # of the query, key and value projections
+    keys_as_values: bool = False         # the values are the projected keys, before norm and rotation
+    head_gate: bool = False              # sigmoid(w_g . h) per head on the output
+    kv_from: Optional[int] = None        # attends to the keys and values of this earlier layer and has none of its own
+
+    @property
+    def width(self) -> int:
+        """Width a head takes in the KV pages (both planes)."""
+        return padded_head_width(max(self.dim, self.vdim))
+
+    @property
+    def cache_elems(self) -> int:
+        """Elements a token takes in the layer's cache plane."""
+        return 0 if self.kv_from is not None else 2 * self.kv_heads * self.width
+
+    @property
+    def state_elems(self) -> int:
+        return 0
+
+    def check(self) -> None:
+        if min(self.heads, self.kv_heads, self.dim, self.vdim) < 1 or self.heads % self.kv_heads:
+            raise ValueError(f"{self.heads} query heads over {self.kv_heads} key/value heads, {self.dim} / {self.vdim} wide")
+        if self.rot is not None and not (self.rot.dims % 2 == 0 and 2 <= self.rot.dims <= self.dim):
+            raise ValueError(f"rotation of {self.rot.dims} of {self.dim} dimensions")
+        if self.keys_as_values and self.vdim != self.dim:
+            raise ValueError(f"keys of {self.dim} dimensions as values of {self.vdim}")
+        if self.window < 0:
+            raise ValueError(f"window of {self.window}")
+        padded_head_width(max(self.dim, self.vdim))
 
 
 # bounds of the latent attention kernels: padded latent columns, and those plus the padded rotated part
@@ -114,6 +165,10 @@ class LatentAttentionSpec:
     def cache_elems(self) -> int:
         return self.row_cols
 
+    @property
+    def state_elems(self) -> int:
+        return 0
+
     def check(self) -> None:
         if min(self.heads, self.dim, self.vdim, self.kv_rank) < 1 or self.rot_dim < 2 or self.rot_dim % 2:
             raise ValueError(f"latent attention of {self.heads} heads, {self.dim} + {self.rot_dim} / {self.vdim} wide, "
@@ -123,6 +178,57 @@ class LatentAttentionSpec:
         if self.rank_cols > LATENT_MAX_RANK or self.row_cols > LATENT_MAX_ROW:
             raise ValueError(f"latent of {self.kv_rank} + {self.rot_dim} columns is above the widest supported one "
                              f"({LATENT_MAX_RANK}, {LATENT_MAX_ROW} with the rotated part)")
+
+
+@dataclass(frozen=True)
+class RecurrentSpec:
+    """Real-gated linear recurrence (RG-LRU) over a short causal convolution, gated by a GELU branch of the same width."""
+    width: int
+    blocks: int                          # the gates are block-diagonal maps of the convolution's output
+    taps: int                            # of the convolution
+
+    @property
+    def block_cols(self) -> int:
+        """Channels of a block, zero-padded."""
+        return round_up(self.width // self.blocks, 8)
+
+    @property
+    def cols(self) -> int:
+        return self.blocks * self.block_cols
+
+    @property
+    def state_elems(self) -> int:
+        """fp32 numbers a request carries: one per channel, and the convolution's last inputs."""
+        return self.cols * self.taps
+
+    def check(self) -> None:
+        if min(self.width, self.blocks, self.taps) < 1 or self.width % self.blocks:
+            raise ValueError(f"recurrence of {self.width} channels in {self.blocks} blocks, {self.taps} taps")
+
+
+@dataclass(frozen=True)
+class SideBySideSpec:
+    """Attention and a recurrence reading the same row; their outputs are added with a factor each."""
+    left: AttentionSpec
+    right: RecurrentSpec
+    left_scale: float = 1.0
+    right_scale: float = 1.0
+
+    @property
+    def window(self) -> int:
+        return self.left.window
+
+    @property
+    def cache_elems(self) -> int:
+        return self.left.cache_elems
+
+    @property
+    def state_elems(self) -> int:
+        return self.right.state_elems
+
+    def check(self) -> None:
+        self.left.check()
+        self.right.check()
 
 
 @dataclass(frozen=True)
@@ -145,10 +251,19 @@ class MoeMlpSpec:
 
 @dataclass(frozen=True)
 class LayerSpec:
-    mixer: Union[AttentionSpec, LatentAttentionSpec]
+    mixer: Union[AttentionSpec, LatentAttentionSpec, SideBySideSpec]
     mlp: Optional[Union[DenseMlpSpec, MoeMlpSpec]] = None
     parallel: bool = False               # both sublayers read one norm and are added together
     token_shift: bool = False            # the mixer reads a mix of this token's and the previous token's normalised row
+
+    @property
+    def attention(self) -> Union[AttentionSpec, LatentAttentionSpec]:
+        """The part of the mixer that keeps a cache."""
+        return self.mixer.left if isinstance(self.mixer, SideBySideSpec) else self.mixer
+
+    def state_elems(self, hidden: int) -> int:
+        """fp32 numbers a request carries for one run of this layer besides its cache rows."""
+        return self.mixer.state_elems + (round_up(hidden, 8) if self.token_shift else 0)
 
 
 @dataclass(frozen=True)
@@ -230,7 +345,7 @@ class ModelConfig:
     @property
     def has_recurrent_state(self) -> bool:
         """Does a request carry state besides its cache pages (prefix reuse then needs snapshots of it)?"""
-        return self.is_hybrid or any(l.token_shift for l in self.layer_specs)
+        return self.is_hybrid or any(l.state_elems(self.hidden) for l in self.layer_specs)
 
     @property
     def is_moe(self) -> bool:
@@ -293,7 +408,7 @@ class ModelConfig:
 
     def recurrent_state_bytes(self) -> int:
         if self.layer_specs:
-            return sum(4 * round_up(self.hidden, 8) for i, _ in self.layer_runs() if self.layer_specs[i].token_shift)
+            return sum(4 * self.layer_specs[i].state_elems(self.hidden) for i, _ in self.layer_runs())
         gdn = self.n_linear_layers * self.ssm_v_heads * self.ssm_state * self.ssm_state * 4
         conv = self.n_linear_layers * self.linear_qkv_width * self.conv_kernel * 4
         return gdn + conv
@@ -465,6 +580,67 @@ MILUTAR_8B = milutar_config(4096, 128256, tuple(_milutar_layer(_MILUTAR_8B_F if 
                                                 for i in range(28)), loop=LoopSpec(8, 16, 2), residual_mult=0.5)
 
 
+def banelix_config(hidden: int, vocab: int, layers: Tuple[LayerSpec, ...], rms_eps: float = 1e-6, residual_mult: float = 1.0,
+                   embed_scale: float = 1.0, max_context: int = 262144) -> ModelConfig:
+    """``ModelConfig`` of a Banelix model: windowed attention layers (some on an earlier layer's keys and values) and layers
+    of attention beside a gated linear recurrence, dense SiLU feed-forwards."""
+    if not layers:
+        raise ValueError("a model needs layers")
+    for i, l in enumerate(layers):
+        a = l.attention
+        try:
+            l.mixer.check()
+            if a.kv_from is not None:
+                if not 0 <= a.kv_from < i:
+                    raise ValueError(f"keys and values of layer {a.kv_from}")
+                src = layers[a.kv_from].mixer
+                if not isinstance(src, AttentionSpec) or src.kv_from is not None:
+                    raise ValueError(f"layer {a.kv_from} has no keys and values to share")
+                if (src.kv_heads, src.dim, src.vdim) != (a.kv_heads, a.dim, a.vdim):
+                    raise ValueError(f"layer {a.kv_from} has other key/value heads")
+        except ValueError as e:
+            raise ValueError(f"layer {i}: {e}") from None
+    a = layers[0].attention
+    return ModelConfig(
+        arch="banelix", n_layers=len(layers), hidden=hidden, vocab=vocab, n_heads=a.heads, n_kv_heads=a.kv_heads,
+        head_dim=a.dim, ffn=max([l.mlp.ff for l in layers if l.mlp is not None], default=0), rms_eps=rms_eps,
+        rope_theta=a.rot.base, rope_dim=a.rot.dims, attn_scale=a.scale, embed_scale=embed_scale, layer_specs=tuple(layers),
+        residual_mult=residual_mult, max_context=max_context)
+
+
+def _banelix_attention(heads: int, kv_heads: int, dim: int, vdim: int, scale: float, window: int, rot: RotarySpec,
+                       kv_from: Optional[int] = None) -> AttentionSpec:
+    return AttentionSpec(heads, kv_heads, dim, vdim, scale, rot=rot, window=window, sink_score=0.0, qk_norm=QK_NORM_ROWS,
+                         bias=True, kv_from=kv_from)
+
+
+def _banelix_side_by_side(heads: int, kv_heads: int, dim: int, scale: float, rot: RotarySpec, right: RecurrentSpec,
+                          left_scale: float, right_scale: float) -> SideBySideSpec:
+    left = AttentionSpec(heads, kv_heads, dim, dim, scale, rot=rot, qk_norm=QK_NORM_UNIT, bias=True, keys_as_values=True,
+                         head_gate=True)
+    return SideBySideSpec(left, right, left_scale, right_scale)
+
+
+# Small Banelix geometry of the tests and the command line: unequal widths, a layer without a feed-forward, a layer on the
+# keys and values of an earlier one with a window of its own.
+_BANELIX_ROT = RotarySpec(40, 8000.0, YarnSpec(4.0, 512.0, 20.0, 1.5), halves=True)
+_BANELIX_P = _banelix_side_by_side(6, 2, 40, 0.15, RotarySpec(24, 90000.0, BandSpec(6.0, 1.0, 3.0, 400.0), halves=True),
+                                   RecurrentSpec(120, 3, 4), 0.9, 0.7)
+TINY_BANELIX = banelix_config(
+    216, 1024, (LayerSpec(_banelix_attention(4, 2, 48, 56, 0.14, 50, _BANELIX_ROT), DenseMlpSpec(232)),
+                LayerSpec(_BANELIX_P, DenseMlpSpec(184)), LayerSpec(_BANELIX_P, None),
+                LayerSpec(_banelix_attention(4, 2, 48, 56, 0.12, 33, _BANELIX_ROT, kv_from=0), DenseMlpSpec(184))),
+    residual_mult=0.8, embed_scale=6.0, max_context=8192)
+
+# Geometry at the layer sizes of a deployed model, for throughput: an 8B-class width, one windowed layer in four.
+_BANELIX_8B_ROT = RotarySpec(128, 50000.0, YarnSpec(16.0, 8192.0, 32.0, 1.0), halves=True)
+_BANELIX_8B_P = _banelix_side_by_side(32, 8, 128, 128 ** -0.5, RotarySpec(64, 500000.0, BandSpec(8.0, 1.0, 4.0, 8192.0), halves=True),
+                                      RecurrentSpec(4096, 16, 4), 1.0, 1.0)
+BANELIX_8B = banelix_config(4096, 128256, tuple(
+    LayerSpec(_banelix_attention(32, 8, 128, 128, 128 ** -0.5, 4096, _BANELIX_8B_ROT, kv_from=i - 4 if i % 8 == 7 else None)
+              if i % 4 == 3 else _BANELIX_8B_P, DenseMlpSpec(14336)) for i in range(24)), residual_mult=0.5, embed_scale=64.0)
+
+
 @dataclass(frozen=True)
 class AssistantConfig:
     """Gemma 4 assistant (MTP) head: a separate four-block draft model with no K/V projections of its own.  Every
@@ -534,4 +710,6 @@ NAMED_CONFIGS: Dict[str, ModelConfig] = {
     "sisisun-30b-moe": SISISUN_30B_MOE,
     "tiny-milutar": TINY_MILUTAR,
     "milutar-8b": MILUTAR_8B,
+    "tiny-banelix": TINY_BANELIX,
+    "banelix-8b": BANELIX_8B,
 }

@@ -10,7 +10,7 @@ from __future__ import annotations
 from dataclasses import dataclass
 from typing import Any, Dict, List, Optional, Tuple
 
-from .config import ModelConfig, MoeMlpSpec
+from .config import ModelConfig, MoeMlpSpec, SideBySideSpec
 
 
 @dataclass(frozen=True)
@@ -34,11 +34,14 @@ class ModelPlugin:
     notes: str = ""
 
     def layer_sequence(self, cfg: ModelConfig) -> List[str]:
-        """One word per layer of ``cfg``: ``linear`` (Gated-DeltaNet), ``full``, ``sliding`` or ``global``."""
+        """One word per layer of ``cfg``: ``linear`` (Gated-DeltaNet), ``full``, ``sliding`` or ``global``; with
+        ``+recurrent`` where a recurrence runs beside the attention."""
         out = []
         for i in range(cfg.n_layers):
             if cfg.layer_specs:
-                out.append("sliding" if getattr(cfg.layer_specs[i].mixer, "window", 0) else "full")
+                m = cfg.layer_specs[i].mixer
+                word = "sliding" if getattr(m, "window", 0) else "full"
+                out.append(word + "+recurrent" if isinstance(m, SideBySideSpec) else word)
             elif cfg.arch == "gemma4":
                 out.append("global" if cfg.is_global_layer(i) else "sliding")
             elif cfg.is_hybrid:
@@ -106,6 +109,17 @@ PLUGINS: Tuple[ModelPlugin, ...] = (
                 notes="layers listed one by one: latent attention (windowed, or causal with a softmax sink and a query "
                       "latent) beside a squared-ReLU feed-forward on one norm, token shift, layer scale; a range of layers "
                       "may run several times; checkpoints are folders with config.json and model.safetensors"),
+    ModelPlugin("banelix", ("banelix",), "hipengine_b200.models.banelix.BanelixExecutor", default_quant="bf16",
+                native_block_types=("BF16",), widened_block_types=(), kv_storage=("bf16", "f32"),
+                tensor_parallel=False, compute_dtypes=("bfloat16", "float32"),
+                native_sources=("attn_decode.cu", "attn_prefill.cu", "exact_f32.cu", "gemm_sm100.cu", "gemv_float.cu",
+                                "layers.cu", "mixer_post.cu", "quant_util.cu", "rglru.cu", "runtime.cpp", "sampling.cu"),
+                folder_architecture="Banelix", folder_reader="hipengine_b200.loading.banelix",
+                reference="hipengine_b200.ref.banelix.BanelixRef",
+                notes="layers listed one by one: windowed attention with one more unit in the softmax denominator (a layer may "
+                      "attend to an earlier layer's keys and values), or attention over unit keys whose values are the plain "
+                      "keys beside a real-gated linear recurrence; dense SiLU feed-forward or none; checkpoints are folders "
+                      "with config.json and model.safetensors"),
 )
 
 
