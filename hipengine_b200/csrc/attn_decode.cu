@@ -2,7 +2,7 @@
 //
 // One CTA owns (row, kv head, key span) and serves all G = H/Hkv query heads of that kv head from one
 // read of the K/V pages, writing un-normalised partial outputs plus (max, sum) to a scratch buffer;
-// a second small kernel merges the spans, applies sigmoid(gate) and stores bf16.
+// a second small kernel merges the spans (and a sink), applies sigmoid(gate) and stores bf16.
 // Behavioural reference: the split-K producers/reducers in
 // hipengine/kernels/hip_gfx1100/attention/paged_attn_decode.hip (chunk = KV block, reduce_threads = head_dim,
 // gate fused in the reducer) and the live-span oracle hipengine/kernels/cpu_reference/ops.py:2895-2997.
@@ -29,6 +29,10 @@ struct AttnDecArgs {
   float scale;
   int* status;                // optional status word: a bounded wait that gave up records its code here
   float softcap;              // > 0: score <- softcap * tanh(score / softcap), after the scale
+  const float* sink;          // [H] or null: score of one more term in the softmax denominator, which has no value
+  const void* head_gate;      // [R][head_gate_stride] or null: head h's output is multiplied by sigmoid(head_gate[r][h])
+  long long head_gate_stride;
+  int head_gate_dtype;        // 0 f32, 1 bf16
 };
 
 namespace {
@@ -485,6 +489,8 @@ __global__ void attn_decode_reduce_kernel(const AttnDecArgs a) {
     m = fmaxf(m, ms);
   }
   m = block_max(m, red);
+  const float sink = a.sink != nullptr ? a.sink[h] : -INFINITY;
+  m = fmaxf(m, sink);
   float den = 0.f;
   for (int s = d; s < ns; s += blockDim.x) {
     const float w = __expf(wsm[s] - m);
@@ -492,6 +498,7 @@ __global__ void attn_decode_reduce_kernel(const AttnDecArgs a) {
     den += w * pb[(size_t)s * (D + 2) + D + 1];
   }
   den = block_sum(den, red);      // barriers inside also publish wsm[]
+  if (a.sink != nullptr) den += __expf(sink - m);
   float n4[4] = {0.f, 0.f, 0.f, 0.f};
   int s = 0;
   for (; s + 4 <= ns; s += 4) {
@@ -504,6 +511,11 @@ __global__ void attn_decode_reduce_kernel(const AttnDecArgs a) {
   if (a.gate != nullptr) {
     // the reference rounds the attention output to bf16 before the gate multiply (cpu_reference/ops.py:2250)
     o = bf16_to_f32(f32_to_bf16(o)) * sigmoid_f(bf16_to_f32(a.gate[((size_t)r * a.H + h) * D + d]));
+  }
+  if (a.head_gate != nullptr) {
+    const size_t i = (size_t)r * a.head_gate_stride + h;
+    o *= sigmoid_f(a.head_gate_dtype == 0 ? reinterpret_cast<const float*>(a.head_gate)[i]
+                                          : bf16_to_f32(reinterpret_cast<const __nv_bfloat16*>(a.head_gate)[i]));
   }
   a.out[(size_t)r * a.H * D + (size_t)h * D + d] = f32_to_bf16(o);
 }

@@ -34,6 +34,10 @@ struct PrefillArgs {
   const int* pos;
   int n_seg, max_pages;
   float cap_in, cap_log2;      // soft cap: score * log2(e) = cap_log2 * tanh(q.k * cap_in)
+  const float* sink;           // [H] or null: score of one more term in the softmax denominator, which has no value
+  const void* head_gate;       // [T][head_gate_stride] or null: head h's output is multiplied by sigmoid(head_gate[t][h])
+  long long head_gate_stride;
+  int head_gate_dtype;         // 0 f32, 1 bf16
 };
 
 __device__ __forceinline__ void cp_async16(void* smem, const void* gmem, bool valid) {
@@ -90,6 +94,8 @@ __global__ void __launch_bounds__(NTHR) flash_prefill_kernel(const PrefillArgs a
     a.q += (size_t)row0 * a.H * D;
     a.out += (size_t)row0 * a.H * D;
     if (a.gate != nullptr) a.gate += (size_t)row0 * a.H * D;
+    if (a.head_gate != nullptr)
+      a.head_gate = reinterpret_cast<const char*>(a.head_gate) + (size_t)row0 * a.head_gate_stride * (a.head_gate_dtype == 0 ? 4 : 2);
   }
   const int h = blockIdx.y, hk = h / (a.H / a.Hkv);
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
@@ -260,7 +266,13 @@ __global__ void __launch_bounds__(NTHR) flash_prefill_kernel(const PrefillArgs a
     const int row = warp * 16 + g + r * 8;
     if (row >= rows) continue;
     const int t = t0 + row;
-    const float inv = l_run[r] > 0.f ? 1.f / l_run[r] : 0.f;
+    if (a.sink != nullptr) l_run[r] += exp2f(a.sink[h] * 1.4426950408889634f - m_run[r]);
+    float inv = l_run[r] > 0.f ? 1.f / l_run[r] : 0.f;
+    if (a.head_gate != nullptr) {
+      const size_t i = (size_t)t * a.head_gate_stride + h;
+      inv *= sigmoid_f(a.head_gate_dtype == 0 ? reinterpret_cast<const float*>(a.head_gate)[i]
+                                              : bf16_to_f32(reinterpret_cast<const __nv_bfloat16*>(a.head_gate)[i]));
+    }
 #pragma unroll
     for (int i = 0; i < D / 8; ++i) {
       const int d = i * 8 + 2 * c;
@@ -315,7 +327,8 @@ HE_API int he_flash_prefill(const void* q, const void* gate, const void* kv_cach
 HE_API int he_flash_prefill_segs(const void* q, const void* gate, const void* kv_cache, const void* block_table,
                                  int max_pages, const int* seg_start, const int* seg_slot, const int* pos, int n_seg,
                                  int tiles, void* out, int H, int Hkv, int D, int page, float scale, int window,
-                                 float softcap, cudaStream_t stream) {
+                                 float softcap, const float* sink, const void* head_gate, long long head_gate_stride,
+                                 int head_gate_dtype, cudaStream_t stream) {
   if (n_seg <= 0 || tiles <= 0) return 0;
   if (H % Hkv != 0 || seg_start == nullptr || seg_slot == nullptr || pos == nullptr) return -HE_ERR_BAD_ARG;
   PrefillArgs a = {};
@@ -323,6 +336,7 @@ HE_API int he_flash_prefill_segs(const void* q, const void* gate, const void* kv
   a.block_table = (const int*)block_table; a.out = (__nv_bfloat16*)out;
   a.H = H; a.Hkv = Hkv; a.page = page; a.window = window;
   a.seg_start = seg_start; a.seg_slot = seg_slot; a.pos = pos; a.n_seg = n_seg; a.max_pages = max_pages;
+  a.sink = sink; a.head_gate = head_gate; a.head_gate_stride = head_gate_stride; a.head_gate_dtype = head_gate_dtype;
   a.scale_log2 = scale * 1.4426950408889634f;
   if (softcap > 0.f) {
     a.cap_in = scale / softcap;

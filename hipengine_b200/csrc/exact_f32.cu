@@ -14,6 +14,10 @@ struct ExactAttnArgs {
   float* out;                // [R][H*D]
   int R, H, Hkv, D, page, max_pages;
   float scale, softcap;      // softcap 0: none
+  int window;                // > 0: only the last `window` keys are visible
+  const float* sink;         // [H] or null: score of one more term in the softmax denominator
+  const float* head_gate;    // [R][head_gate_stride] or null: outputs times sigmoid(head_gate[r][h])
+  long long head_gate_stride;
 };
 
 struct ExactMoeArgs {
@@ -54,7 +58,7 @@ __global__ void __launch_bounds__(AW * 32) attn_exact_kernel(const ExactAttnArgs
     o[i] = 0.f;
   }
   float m = -INFINITY, l = 0.f;
-  for (int p = warp; p < ctx; p += AW) {
+  for (int p = (a.window > 0 && ctx > a.window ? ctx - a.window : 0) + warp; p < ctx; p += AW) {
     const int pg = bt[HE_INDEX_OK(p / a.page, a.max_pages, HE_SITE_ATTN_DECODE_PAGE) ? p / a.page : 0];
     const float* kr = a.kv_cache + (((size_t)pg * 2 * a.Hkv + hk) * a.page + p % a.page) * D;
     const float* vr = kr + (size_t)a.Hkv * a.page * D;
@@ -79,13 +83,18 @@ __global__ void __launch_bounds__(AW * 32) attn_exact_kernel(const ExactAttnArgs
   float mt = -INFINITY, lt = 0.f;
 #pragma unroll
   for (int w = 0; w < AW; ++w) mt = fmaxf(mt, m_s[w]);
+  if (a.sink != nullptr) {
+    mt = fmaxf(mt, a.sink[h]);
+    lt = expf(a.sink[h] - mt);
+  }
 #pragma unroll
   for (int w = 0; w < AW; ++w) lt += l_s[w] > 0.f ? l_s[w] * expf(m_s[w] - mt) : 0.f;
+  const float gate = a.head_gate != nullptr ? 1.f / (1.f + expf(-a.head_gate[(size_t)r * a.head_gate_stride + h])) : 1.f;
   for (int d = threadIdx.x; d < D; d += AW * 32) {
     float v = 0.f;
 #pragma unroll
     for (int w = 0; w < AW; ++w) v += l_s[w] > 0.f ? o_s[w][d] * expf(m_s[w] - mt) : 0.f;
-    a.out[((size_t)r * a.H + h) * D + d] = lt > 0.f ? v / lt : 0.f;
+    a.out[((size_t)r * a.H + h) * D + d] = lt > 0.f ? v / lt * gate : 0.f;
   }
 }
 

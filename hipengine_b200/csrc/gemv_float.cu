@@ -12,10 +12,13 @@
 //   batches   : grid.y repeats the product with other weights and rows (one small matrix per attention head)
 //   sums      : the two output projections of a layer whose sublayers run side by side are one launch: each has its own
 //               rows and columns, both accumulators get their per-column factors and meet in the residual add
+//   recurrence: one token of a gated linear recurrence per row; both gate products of 16 channels end in the CTA that then
+//               steps these channels' state and multiplies the output gate in
 // The expert forms add an indirection: grid.y is a (token, expert) pair or a token, the weight base comes from the
 // routed expert id, and the down projection walks the concatenated columns of all selected experts (and the shared
 // one), which adds the k expert outputs in a fixed order inside the accumulator.
 #include "common.cuh"
+#include "rglru.cuh"
 
 using namespace he;
 
@@ -424,6 +427,43 @@ __global__ void __launch_bounds__(NW * 32, 2) moe_down_float_kernel(const __grid
   if (threadIdx.x < 16 && n < a.N) a.h[(size_t)t * a.ldh + n] += sum_partials<1, 1>(sm, threadIdx.x, 0);
 }
 
+// One token of every segment through the gated linear recurrence: segment r is row r.  grid (ceil(block_cols / 16), blocks)
+template <int NT>
+__global__ void __launch_bounds__(NW * 32, 2) rglru_step_kernel(const __grid_constant__ RglruArgs a) {
+  __shared__ Tile<2, NT> sm;
+  pdl_launch();
+  const int lane = threadIdx.x & 31, g = lane >> 2, c = lane & 3, bc = a.block_cols, b = blockIdx.y, row0 = blockIdx.x * 16;
+  const __nv_bfloat16* wrow[2][2];
+#pragma unroll
+  for (int hf = 0; hf < 2; ++hf) {
+    const int n = min(row0 + g + 8 * hf, bc - 1);
+    wrow[0][hf] = a.gw + ((size_t)b * 2 * bc + n) * bc + 8 * c;
+    wrow[1][hf] = wrow[0][hf] + (size_t)bc * bc;
+  }
+  const __nv_bfloat16* u = reinterpret_cast<const __nv_bfloat16*>(a.u) + (size_t)b * a.u_bs;
+  float acc[2][NT][4] = {};
+  float ss[NT] = {};
+  product<2, NT, false, true>(wrow, bc, u, a.u_ts, a.n_seg, nullptr, acc, ss);
+  store_partials<2, NT>(sm, acc, ss);
+  __syncthreads();
+  for (int o = threadIdx.x; o < 16 * NT * 8; o += NW * 32) {
+    const int row = o & 15, r = o >> 4, n = row0 + row;
+    if (r >= a.n_seg || n >= bc) continue;
+    const int ch = b * bc + n, slot = a.seg_slot[r];
+    if (!HE_INDEX_OK(slot, a.n_slots, HE_SITE_STATE_SLOT)) continue;
+    float* S = a.S + (size_t)slot * a.C + ch;
+    const float* gb = a.gb + (size_t)b * 2 * bc + n;
+    const float y = rg_load(a.y, a.row_dtype == 0, (size_t)r * a.row_stride + ch) + a.yb[ch];
+    float av, dv;
+    rg_gates(sum_partials<2, NT>(sm, row, r) + gb[0], sum_partials<2, NT>(sm, 16 + row, r) + gb[bc], a.decay[ch],
+             bf16_to_f32(u[(size_t)r * a.u_ts + n]), av, dv);
+    const float s = av * *S + dv;
+    *S = s;
+    reinterpret_cast<__nv_bfloat16*>(a.out)[(size_t)r * a.out_stride + ch] = f32_to_bf16(s * gelu_tanh_f(y));
+    rg_conv_state(a, slot, ch, r, 1);
+  }
+}
+
 template <int MT>
 int launch_rows(const FloatGemvArgs& a, int items, cudaStream_t stream) {
   cudaError_t e;
@@ -479,6 +519,17 @@ HE_API int he_gemv_sum(const FloatSumArgs* args, cudaStream_t stream) {
                         : launch_pdl(gemv_sum_kernel<2>, grid, block, 0, stream, a));
 }
 HE_API int he_gemv_sum_args_size() { return (int)sizeof(FloatSumArgs); }
+
+HE_API int he_rglru_step(const RglruArgs* args, cudaStream_t stream) {
+  const RglruArgs& a = *args;
+  if (a.n_seg <= 0) return 0;
+  if (a.n_seg > 16 || a.block_cols <= 0 || a.block_cols % 8 != 0 || a.C % a.block_cols != 0 || a.taps < 1 || a.act_f32 != 0 ||
+      a.gw == nullptr || a.journal != nullptr || a.u_ts % 8 != 0 || a.u_bs % 8 != 0 || a.C / a.block_cols > 65535)
+    return -HE_ERR_BAD_ARG;
+  const dim3 grid((a.block_cols + 15) / 16, a.C / a.block_cols), block(NW * 32);
+  return (int)(a.n_seg <= 8 ? launch_pdl(rglru_step_kernel<1>, grid, block, 0, stream, a)
+                            : launch_pdl(rglru_step_kernel<2>, grid, block, 0, stream, a));
+}
 
 static int check_moe(const FloatMoeArgs& a) {
   if (a.k <= 0 || a.k > 32 || a.E < a.k || a.F <= 0 || a.F % 8 != 0 || (a.w1s != nullptr && (a.Fs <= 0 || a.Fs % 8 != 0)))

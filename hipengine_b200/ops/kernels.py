@@ -77,7 +77,8 @@ class _AttnDecArgs(C.Structure):
                 ("ctx_len", c_vp), ("partial", c_vp), ("out", c_vp),
                 ("R", C.c_int), ("H", C.c_int), ("Hkv", C.c_int), ("D", C.c_int), ("page", C.c_int),
                 ("max_pages", C.c_int), ("split_len", C.c_int), ("max_splits", C.c_int), ("window", C.c_int),
-                ("scale", C.c_float), ("status", c_vp), ("softcap", C.c_float)]
+                ("scale", C.c_float), ("status", c_vp), ("softcap", C.c_float), ("sink", c_vp), ("head_gate", c_vp),
+                ("head_gate_stride", c_ll), ("head_gate_dtype", C.c_int)]
 
 
 class _GdnDecodeArgs(C.Structure):
@@ -135,7 +136,8 @@ class _FloatMoeArgs(C.Structure):
 class _ExactAttnArgs(C.Structure):
     _fields_ = [("q", c_vp), ("kv_cache", c_vp), ("block_table", c_vp), ("slot", c_vp), ("ctx_len", c_vp),
                 ("out", c_vp), ("R", C.c_int), ("H", C.c_int), ("Hkv", C.c_int), ("D", C.c_int), ("page", C.c_int),
-                ("max_pages", C.c_int), ("scale", C.c_float), ("softcap", C.c_float)]
+                ("max_pages", C.c_int), ("scale", C.c_float), ("softcap", C.c_float), ("window", C.c_int), ("sink", c_vp),
+                ("head_gate", c_vp), ("head_gate_stride", c_ll)]
 
 
 class _ExactMoeArgs(C.Structure):
@@ -554,7 +556,9 @@ def attn_decode_scratch_floats(R: int, H: int, max_splits: int, D: int) -> int:
 def attn_decode(q: torch.Tensor, gate: Optional[torch.Tensor], kv_cache: torch.Tensor, block_table: torch.Tensor,
                 slot: torch.Tensor, ctx_len: torch.Tensor, partial: torch.Tensor, out: torch.Tensor, H: int, Hkv: int,
                 D: int, page: int, split_len: int, max_splits: int, scale: float, window: int = 0,
-                softcap: float = 0.0) -> None:
+                softcap: float = 0.0, sink: Optional[torch.Tensor] = None, head_gate: Optional[torch.Tensor] = None) -> None:
+    """``sink`` (fp32 [H]): scores of a term in the softmax denominator; ``head_gate`` ([R, H], fp32 or bf16): logits of a
+    gate per head on the output."""
     _check_abi()
     a = _AttnDecArgs()
     a.q, a.gate, a.kv_cache = q.data_ptr(), _p(gate), kv_cache.data_ptr()
@@ -564,7 +568,9 @@ def attn_decode(q: torch.Tensor, gate: Optional[torch.Tensor], kv_cache: torch.T
     a.max_pages = block_table.shape[1]
     a.split_len, a.max_splits, a.window, a.scale = split_len, max_splits, window, scale
     a.status = status_tensor(q.device).data_ptr()
-    a.softcap = softcap
+    a.softcap, a.sink = softcap, _p(sink)
+    if head_gate is not None:
+        a.head_gate, a.head_gate_stride, a.head_gate_dtype = head_gate.data_ptr(), head_gate.stride(0), _dt(head_gate)
     assert partial.numel() >= attn_decode_scratch_floats(a.R, H, max_splits, D)
     N.check(N.lib().he_attn_decode(C.byref(a), _stream()), "he_attn_decode")
 
@@ -810,15 +816,18 @@ def moe_down_float(rows: torch.Tensor, ids: torch.Tensor, w_down: torch.Tensor, 
 
 def attn_exact(q: torch.Tensor, kv_cache: torch.Tensor, block_table: torch.Tensor, slot: torch.Tensor,
                ctx_len: torch.Tensor, out: torch.Tensor, H: int, Hkv: int, D: int, page: int, scale: float,
-               softcap: float = 0.0) -> None:
-    """Causal attention of any rows over fp32 pages, fp32 throughout."""
+               softcap: float = 0.0, window: int = 0, sink: Optional[torch.Tensor] = None,
+               head_gate: Optional[torch.Tensor] = None) -> None:
+    """Causal attention of any rows over fp32 pages, fp32 throughout; the options are those of ``attn_decode``."""
     _check_abi()
-    assert q.dtype == kv_cache.dtype == out.dtype == torch.float32
+    assert q.dtype == kv_cache.dtype == out.dtype == torch.float32 and (head_gate is None or head_gate.dtype == torch.float32)
     a = _ExactAttnArgs()
     a.q, a.kv_cache, a.block_table = q.data_ptr(), kv_cache.data_ptr(), block_table.data_ptr()
     a.slot, a.ctx_len, a.out = slot.data_ptr(), ctx_len.data_ptr(), out.data_ptr()
     a.R, a.H, a.Hkv, a.D, a.page, a.max_pages = q.shape[0], H, Hkv, D, page, block_table.shape[1]
-    a.scale, a.softcap = scale, softcap
+    a.scale, a.softcap, a.window, a.sink = scale, softcap, window, _p(sink)
+    if head_gate is not None:
+        a.head_gate, a.head_gate_stride = head_gate.data_ptr(), head_gate.stride(0)
     N.check(N.lib().he_attn_exact(C.byref(a), _stream()), "he_attn_exact")
 
 
