@@ -4,13 +4,15 @@ On top of the hybrid executor (scratch, paged pool, block tables, decode and pre
 families share:
   * bfloat16 weights; widths that are no multiple of eight are zero-padded at load (norms average over the real width);
   * one cache plane per layer RUN: every pass of a looped range attends only to what the same pass wrote;
-  * per-slot recurrent rows (token shift) per layer run, kept where the hybrid executor keeps its convolution windows, so
-    admission, snapshots, the cold tier, graph warm-up and speculative commits treat them alike;
-  * three kernel routes by row count: fp32, up to 16 rows (streaming GEMV), more (tcgen05 GEMM, split over K up to 128 rows).
+  * per-slot recurrent rows per layer run (token shift, the state of a recurrence and of its convolution), kept where the
+    hybrid executor keeps its convolution windows and states, so admission, snapshots, the cold tier, graph warm-up and
+    speculative commits treat them alike;
+  * three kernel routes by row count: fp32, up to 16 rows (streaming GEMV), more (tcgen05 GEMM, split over K up to 128 rows);
+  * grouped-query attention of packed segments, gated feed-forwards and scaled residual adds on these routes.
 """
 from __future__ import annotations
 
-from typing import Callable, Optional
+from typing import Callable, Optional, Sequence, Tuple
 
 import torch
 
@@ -18,6 +20,7 @@ from ..loading.weights import ModelWeights
 from ..ops import kernels as K
 from ..ops.kernels import DeviceWeight
 from ..quant.ggml import GGMLType
+from .config import AttentionSpec, DenseMlpSpec, SideBySideSpec
 from .executor import PAGE, BatchDesc, HybridExecutor
 
 # segments of up to this many rows attend through the split-K decode kernel, longer ones through the flash kernel
@@ -77,6 +80,16 @@ class ListedExecutor(HybridExecutor):
             return t.raw.to(self.device).reshape(-1).view(torch.bfloat16).reshape(t.shape)
         return t.dequant(self.device).to(torch.bfloat16)
 
+    def _out_mat(self, name: str, heads: int, real: int, padded: int) -> torch.Tensor:
+        """Output map [hp, heads * padded] of a matrix over heads (or blocks) of ``real`` columns."""
+        out = torch.zeros(self.hp, heads, padded, dtype=torch.bfloat16, device=self.device)
+        out[:self.cfg.hidden, :, :real] = self._mat(name).reshape(self.cfg.hidden, heads, real)
+        return out.reshape(self.hp, -1)
+
+    def _gate_up(self, p: str, ff: int) -> torch.Tensor:
+        """[gate | up] rows of a gated feed-forward, each zero-padded to a multiple of eight."""
+        return torch.cat([pad2(self._mat(p + n), up8(ff), self.hp) for n in ("gate", "up")], 0)
+
     def _put(self, name: str, t: torch.Tensor) -> DeviceWeight:
         w = self.dw[name] = DeviceWeight(int(GGMLType.BF16), t.shape[0], t.shape[1], t.contiguous())
         return w
@@ -93,11 +106,22 @@ class ListedExecutor(HybridExecutor):
     def _alloc_state(self) -> None:
         dev = self.device
         self.conv_state, self.gdn_state, self.kv = {}, {}, {}
+        self.kv_run = {}                       # run -> run whose plane it attends to
+        latest = {}                            # layer -> its latest run
         for run, (i, _) in enumerate(self.runs):
             spec = self.cfg.layer_specs[i]
-            self.kv[run] = torch.zeros(*self._plane_shape(spec.mixer), dtype=self.act_dtype, device=dev)
+            src = getattr(spec.attention, "kv_from", None)
+            self.kv_run[run] = run if src is None else latest[src]
+            latest[i] = run
+            if src is None:
+                self.kv[run] = torch.zeros(*self._plane_shape(spec.attention), dtype=self.act_dtype, device=dev)
             if spec.token_shift:
                 self.conv_state[run] = torch.zeros(self.max_slots, self.hp, 1, dtype=torch.float32, device=dev)
+            if isinstance(spec.mixer, SideBySideSpec):
+                r = spec.mixer.right
+                self.gdn_state[run] = torch.zeros(self.max_slots, r.cols, dtype=torch.float32, device=dev)
+                if r.taps > 1:
+                    self.conv_state[run] = torch.zeros(self.max_slots, r.taps - 1, r.cols, dtype=torch.float32, device=dev)
         self._alloc_tables()
 
     def _plane_shape(self, mixer):
@@ -113,6 +137,97 @@ class ListedExecutor(HybridExecutor):
 
     def _route(self, T: int) -> str:
         return EXACT if self.exact else FEW if T <= K.FLOAT_GEMV_MAX_ROWS else MANY
+
+    # ------------------------------------------------------------------ projections
+    def _in_proj(self, h: torch.Tensor, norm_w: torch.Tensor, w: DeviceWeight, name: str, route: str,
+                 xn: Optional[torch.Tensor] = None) -> torch.Tensor:
+        """norm(h) @ W^T (fp32, or bf16 rows for large batches); ``xn``: the normalised rows when they exist already."""
+        T, cfg = h.shape[0], self.cfg
+        if route == FEW:
+            out = self.scratch.get(name + "_f32", (T, w.n_rows), torch.float32)
+            K.gemv_float(h, [(w.data, None, out, K.EPI_F32)], norm_w=norm_w, eps=cfg.rms_eps, norm_n=cfg.hidden)
+            return out
+        if xn is None:
+            with self._stage("norm"):
+                xn = self._norm_rows(h, norm_w)
+        if route == EXACT:
+            return K.small_gemm_f32(xn, w.data, self.scratch.get(name + "_f32", (T, w.n_rows), torch.float32))
+        return self._proj(xn, w, name, name)
+
+    def _add_products(self, h: torch.Tensor, parts: Sequence[Tuple[torch.Tensor, DeviceWeight, Optional[torch.Tensor]]],
+                      route: str) -> None:
+        """h += sum of s * (x @ W^T) over one or two (x, W, s); ``s``: fp32 factor per column or None."""
+        from ..ops import gemm as GM
+        if route == FEW:
+            K.gemv_sum(h, [(x, w.data, s) for x, w, s in parts])
+            return
+        for x, w, s in parts:
+            if route == EXACT:
+                K.small_gemm_f32(x, w.data, h, add=True, col_scale=s)
+            elif h.shape[0] <= self.SPLITK_MAX_ROWS:
+                GM.gemm_bf16_splitk_det(x, w.data, h, self.scratch, add=True, col_scale=s)
+            else:
+                GM.gemm_bf16(x, w.data, h, epi=GM.EPI_ADD, col_scale=s)
+
+    # ------------------------------------------------------------------ attention
+    def _attend_run(self, run: int, a: AttentionSpec, q: torch.Tensor, b: BatchDesc, out: torch.Tensor,
+                    sink: Optional[torch.Tensor] = None, head_gate: Optional[torch.Tensor] = None) -> None:
+        """Rows of a packed batch over the pages of run ``run``; ``sink`` fp32 [heads], ``head_gate`` [T, heads] logits."""
+        D, kv = a.width, self.kv[self.kv_run[run]]
+        if self.exact:
+            K.attn_exact(q, kv, self.block_table, b.slot, b.ctx_len, out, a.heads, a.kv_heads, D, PAGE, a.scale,
+                         a.softcap, a.window, sink, head_gate)
+            return
+        from ..ops import attention as A
+
+        def decode(r0: int, r1: int, ctx: int) -> None:
+            span = min(ctx, a.window) if a.window else ctx
+            split_len, max_splits = K.attn_decode_split(span, r1 - r0, a.kv_heads)
+            part = self.scratch.get("attn_part", (K.attn_decode_scratch_floats(r1 - r0, a.heads, max_splits, D),),
+                                    torch.float32)
+            K.attn_decode(q[r0:r1], None, kv, self.block_table, b.slot[r0:r1], b.ctx_len[r0:r1], part, out[r0:r1],
+                          a.heads, a.kv_heads, D, PAGE, split_len, max_splits, a.scale, a.window, a.softcap, sink,
+                          None if head_gate is None else head_gate[r0:r1])
+
+        if b.segs_host is None:
+            decode(0, b.T, b.max_ctx)
+            return
+        # neighbouring segments of the same kind share a launch: prompt portions the flash kernel, single tokens and
+        # short portions the split-K kernel
+        flash = A.flash_prefill_available(D)
+        s, r0 = 0, 0
+        while s < len(b.segs_host):
+            long = flash and b.segs_host[s][2] > DECODE_SEG_ROWS
+            e, r1, ctx = s, r0, 1
+            while e < len(b.segs_host) and (flash and b.segs_host[e][2] > DECODE_SEG_ROWS) == long:
+                _, p0, n = b.segs_host[e]
+                ctx, r1, e = max(ctx, p0 + n), r1 + n, e + 1
+            if long:
+                A.flash_prefill_segs(q, None, kv, self.block_table, b.seg_start[s:], b.seg_slot[s:], b.pos,
+                                     [n for _, _, n in b.segs_host[s:e]], out, a.heads, a.kv_heads, D, PAGE, a.scale,
+                                     a.window, a.softcap, sink, head_gate)
+            else:
+                for c0 in range(r0, r1, 512):       # bounds the split-K scratch of long segments of very wide heads
+                    decode(c0, min(r1, c0 + 512), ctx)
+            s, r0 = e, r1
+
+    # ------------------------------------------------------------------ feed-forward
+    def _dense(self, norm_w: torch.Tensor, gate_up: DeviceWeight, down: DeviceWeight, m: DenseMlpSpec, h: torch.Tensor,
+               route: str, scale: Optional[torch.Tensor] = None) -> None:
+        """h += scale * (Wd act(Wg norm(h), Wu norm(h)))."""
+        T, F = h.shape[0], down.n_cols
+        act = self.scratch.get("ffn_act", (T, F), self.act_dtype)
+        if route == FEW:
+            gu = gate_up.data
+            K.gemv_float(h, [(gu[:F], gu[F:], act, K.EPI_OF_ACT[m.act])], norm_w=norm_w, eps=self.cfg.rms_eps,
+                         norm_n=self.cfg.hidden, limit=m.limit)
+        else:
+            with self._stage("ffn_gateup_gemm"):
+                gu = self._in_proj(h, norm_w, gate_up, "ffn_gu", route)
+            with self._stage("act_mul"):
+                K.act_mul(gu, act, m.act, m.limit)
+        with self._stage("ffn_down_gemm"):
+            self._add_products(h, [(act, down, scale)], route)
 
     # ------------------------------------------------------------------ whole model
     def _embed(self, b: BatchDesc, h: torch.Tensor, copy: Optional[torch.Tensor]) -> None:

@@ -90,8 +90,6 @@ class MilutarExecutor(ListedExecutor):
             down = pad2(mat(p + "mix.dkv"), up8(a.kv_rank + a.rot_dim), hp)
             uk = self._pad_heads(mat(p + "mix.uk"), a.heads, ((a.dim, dn),), a.rank_cols)
             uv = self._pad_heads(mat(p + "mix.uv"), a.heads, ((a.vdim, dv),), a.rank_cols)
-            o = torch.zeros(hp, a.heads, dv, dtype=torch.bfloat16, device=self.device)
-            o[:cfg.hidden, :, :a.vdim] = mat(p + "mix.o").reshape(cfg.hidden, a.heads, a.vdim)
             freq, amp = a.rot.table()
             uk_t = uk.transpose(1, 2).contiguous()
             self.dw[p + "uk_t"] = DeviceWeight(30, a.heads * a.rank_cols, dn, uk_t)
@@ -99,7 +97,8 @@ class MilutarExecutor(ListedExecutor):
                        put(p + "in", torch.cat([first, down], 0)), first.shape[0],
                        self._vec(p + "mix.dkv.norm", a.rank_cols),
                        put(p + "uk", uk.reshape(-1, a.rank_cols)), put(p + "uv", uv.reshape(-1, a.rank_cols)), uk_t,
-                       torch.tensor(freq, dtype=torch.float64, device=self.device), amp, put(p + "o", o.reshape(hp, -1)),
+                       torch.tensor(freq, dtype=torch.float64, device=self.device), amp,
+                       put(p + "o", self._out_mat(p + "mix.o", a.heads, a.vdim, dv)),
                        self._vec(p + "ls1", hp, cfg.residual_mult))
             if a.q_rank:
                 L.q_norm, L.uq = self._vec(p + "mix.dq.norm", qr), put(p + "uq", q)
@@ -162,21 +161,6 @@ class MilutarExecutor(ListedExecutor):
                     qf = GM.gemm_bf16(cq, L.uq.data, sc.get("lat_q_bf", (T, n), torch.bfloat16))
             q = qf
         return q, down, act
-
-    def _add_outputs(self, L: _Layer, attn: torch.Tensor, act: Optional[torch.Tensor], h: torch.Tensor, route: str) -> None:
-        """h += s1 * (attn @ Wo^T) + s2 * (act @ Wdown^T)."""
-        from ..ops import gemm as GM
-        parts = [(attn, L.o.data, L.s1)] + ([] if act is None else [(act, L.down.data, L.s2)])
-        if route == FEW:
-            K.gemv_sum(h, parts)
-            return
-        for x, w, s in parts:
-            if route == EXACT:
-                K.small_gemm_f32(x, w, h, add=True, col_scale=s)
-            elif h.shape[0] <= self.SPLITK_MAX_ROWS:
-                GM.gemm_bf16_splitk_det(x, w, h, self.scratch, add=True, col_scale=s)
-            else:
-                GM.gemm_bf16(x, w, h, epi=GM.EPI_ADD, col_scale=s)
 
     # ------------------------------------------------------------------ attention
     def _segment_groups(self, L: _Layer, b: BatchDesc, route: str):
@@ -266,4 +250,4 @@ class MilutarExecutor(ListedExecutor):
             q, down, act = self._in_projections(L, a, xn, xs, route)
         attn = self._attend(run, a, L, q, down, b, route)
         with self._stage("out_gemm"):
-            self._add_outputs(L, attn, act, h, route)
+            self._add_products(h, [(attn, L.o, L.s1)] + ([] if act is None else [(act, L.down, L.s2)]), route)

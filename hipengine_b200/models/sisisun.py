@@ -19,9 +19,10 @@ import torch
 
 from ..ops import kernels as K
 from ..ops.kernels import DeviceWeight
-from .config import AttentionSpec, DenseMlpSpec, MoeMlpSpec
+from .config import DenseMlpSpec, MoeMlpSpec
 from .executor import PAGE, BatchDesc
-from .listed import DECODE_SEG_ROWS, EXACT, FEW, MANY, ListedExecutor, pad2, up8
+from .listed import EXACT, FEW, MANY, ListedExecutor, pad2, up8
+
 
 @dataclass
 class _Layer:
@@ -52,10 +53,7 @@ class SisisunExecutor(ListedExecutor):
 
     def _load_layers(self) -> None:
         cfg, dev, hp, mat, put, norm = self.cfg, self.device, self.hp, self._mat, self._put, self._norm_weight
-
-        def gate_up(p: str, ff: int) -> torch.Tensor:
-            fp = up8(ff)
-            return torch.cat([pad2(mat(p + "gate"), fp, hp), pad2(mat(p + "up"), fp, hp)], 0)
+        gate_up = self._gate_up
 
         def glu(name: str, p: str, ff: int) -> Tuple[DeviceWeight, DeviceWeight]:
             return put(name + "gate_up", gate_up(p, ff)), put(name + "down", pad2(mat(p + "down"), hp, up8(ff)))
@@ -64,13 +62,11 @@ class SisisunExecutor(ListedExecutor):
         for i, spec in enumerate(cfg.layer_specs):
             a, m, p = spec.mixer, spec.mlp, f"l{i}."
             qkv = torch.cat([mat(p + "mix.q"), mat(p + "mix.k"), mat(p + "mix.v")], 0)
-            o = torch.zeros(hp, a.heads, a.width, dtype=torch.bfloat16, device=dev)
-            o[:cfg.hidden, :, :a.vdim] = mat(p + "mix.o").reshape(cfg.hidden, a.heads, a.vdim)
             for s in ("q.norm", "k.norm"):
                 self.f32[p + "mix." + s] = mat(p + "mix." + s).float().contiguous()
             L = _Layer(norm(p + "norm1"), norm(p + "norm2") if m is not None else None,
                        put(p + "qkv", pad2(qkv, up8(qkv.shape[0]), hp)), self.f32[p + "mix.q.norm"],
-                       self.f32[p + "mix.k.norm"], put(p + "o", o.reshape(hp, -1)))
+                       self.f32[p + "mix.k.norm"], put(p + "o", self._out_mat(p + "mix.o", a.heads, a.vdim, a.width)))
             if isinstance(m, DenseMlpSpec):
                 L.gate_up, L.down = glu(p, p + "mlp.", m.ff)
             elif isinstance(m, MoeMlpSpec):
@@ -91,31 +87,6 @@ class SisisunExecutor(ListedExecutor):
         i = torch.arange((cfg.hidden + 1) // 2, dtype=torch.float64)
         self.pos_freq = torch.pow(torch.tensor(10000.0, dtype=torch.float64), -2.0 * i / cfg.hidden).to(dev)
 
-    # ------------------------------------------------------------------ dispatch
-    def _in_proj(self, h: torch.Tensor, norm_w: torch.Tensor, w: DeviceWeight, name: str, route: str,
-                 xn: Optional[torch.Tensor] = None) -> torch.Tensor:
-        """norm(h) @ W^T (fp32, or bf16 rows for large batches); ``xn``: the normalised rows when they exist already."""
-        T, cfg = h.shape[0], self.cfg
-        if route == FEW:
-            out = self.scratch.get(name + "_f32", (T, w.n_rows), torch.float32)
-            K.gemv_float(h, [(w.data, None, out, K.EPI_F32)], norm_w=norm_w, eps=cfg.rms_eps, norm_n=cfg.hidden)
-            return out
-        if xn is None:
-            with self._stage("norm"):
-                xn = self._norm_rows(h, norm_w)
-        if route == EXACT:
-            return K.small_gemm_f32(xn, w.data, self.scratch.get(name + "_f32", (T, w.n_rows), torch.float32))
-        return self._proj(xn, w, name, name)
-
-    def _add_proj(self, x: torch.Tensor, w: DeviceWeight, h: torch.Tensor, route: str) -> None:
-        """h += x @ W^T."""
-        if route == EXACT:
-            K.small_gemm_f32(x, w.data, h, add=True)
-        elif route == FEW:
-            K.gemv_float(x, [(w.data, None, h, K.EPI_ADD_F32)])
-        else:
-            self._out_big(x, w, h, "o")
-
     # ------------------------------------------------------------------ layers
     def _attention(self, run: int, i: int, h: torch.Tensor, b: BatchDesc, route: str) -> None:
         cfg, sc, L = self.cfg, self.scratch, self.layers[i]
@@ -131,59 +102,7 @@ class SisisunExecutor(ListedExecutor):
         with self._stage("attn_core"):
             self._attend_run(run, a, q_out, b, out)
         with self._stage("out_gemm"):
-            self._add_proj(out, L.o, h, route)
-
-    def _attend_run(self, run: int, a: AttentionSpec, q: torch.Tensor, b: BatchDesc, out: torch.Tensor) -> None:
-        D, kv = a.width, self.kv[run]
-        if self.exact:
-            K.attn_exact(q, kv, self.block_table, b.slot, b.ctx_len, out, a.heads, a.kv_heads, D, PAGE, a.scale,
-                         a.softcap)
-            return
-        from ..ops import attention as A
-
-        def decode(r0: int, r1: int, ctx: int) -> None:
-            split_len, max_splits = K.attn_decode_split(ctx, r1 - r0, a.kv_heads)
-            part = self.scratch.get("attn_part", (K.attn_decode_scratch_floats(r1 - r0, a.heads, max_splits, D),),
-                                    torch.float32)
-            K.attn_decode(q[r0:r1], None, kv, self.block_table, b.slot[r0:r1], b.ctx_len[r0:r1], part, out[r0:r1],
-                          a.heads, a.kv_heads, D, PAGE, split_len, max_splits, a.scale, softcap=a.softcap)
-
-        if b.segs_host is None:
-            decode(0, b.T, b.max_ctx)
-            return
-        # neighbouring segments of the same kind share a launch: prompt portions the flash kernel, single tokens and
-        # short portions the split-K kernel
-        flash = A.flash_prefill_available(D)
-        s, r0 = 0, 0
-        while s < len(b.segs_host):
-            long = flash and b.segs_host[s][2] > DECODE_SEG_ROWS
-            e, r1, ctx = s, r0, 1
-            while e < len(b.segs_host) and (flash and b.segs_host[e][2] > DECODE_SEG_ROWS) == long:
-                _, p0, n = b.segs_host[e]
-                ctx, r1, e = max(ctx, p0 + n), r1 + n, e + 1
-            if long:
-                A.flash_prefill_segs(q, None, kv, self.block_table, b.seg_start[s:], b.seg_slot[s:], b.pos,
-                                     [n for _, _, n in b.segs_host[s:e]], out, a.heads, a.kv_heads, D, PAGE, a.scale,
-                                     softcap=a.softcap)
-            else:
-                for c0 in range(r0, r1, 512):       # bounds the split-K scratch of long segments of very wide heads
-                    decode(c0, min(r1, c0 + 512), ctx)
-            s, r0 = e, r1
-
-    def _dense(self, L: _Layer, m: DenseMlpSpec, h: torch.Tensor, route: str) -> None:
-        T, F = h.shape[0], L.down.n_cols
-        act = self.scratch.get("ffn_act", (T, F), self.act_dtype)
-        if route == FEW:
-            gu = L.gate_up.data
-            K.gemv_float(h, [(gu[:F], gu[F:], act, K.EPI_OF_ACT[m.act])], norm_w=L.norm2, eps=self.cfg.rms_eps,
-                         norm_n=self.cfg.hidden, limit=m.limit)
-        else:
-            with self._stage("ffn_gateup_gemm"):
-                gu = self._in_proj(h, L.norm2, L.gate_up, "ffn_gu", route)
-            with self._stage("act_mul"):
-                K.act_mul(gu, act, m.act, m.limit)
-        with self._stage("ffn_down_gemm"):
-            self._add_proj(act, L.down, h, route)
+            self._add_products(h, [(out, L.o, None)], route)
 
     def _experts(self, L: _Layer, m: MoeMlpSpec, h: torch.Tensor, route: str) -> None:
         from ..ops import gemm as GM
@@ -241,6 +160,7 @@ class SisisunExecutor(ListedExecutor):
         self._attention(run, i, h, b, route)
         m = self.cfg.layer_specs[i].mlp
         if isinstance(m, DenseMlpSpec):
-            self._dense(self.layers[i], m, h, route)
+            L = self.layers[i]
+            self._dense(L.norm2, L.gate_up, L.down, m, h, route)
         elif isinstance(m, MoeMlpSpec):
             self._experts(self.layers[i], m, h, route)
