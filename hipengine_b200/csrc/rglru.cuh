@@ -35,10 +35,12 @@ namespace he {
 
 __device__ __forceinline__ float rg_sigmoid(float x) { return 1.f / (1.f + expf(-x)); }
 
-// decay and drive of one token and channel
+// decay and drive of one token and channel.  Memories of thousands of tokens hang on 1 - a, so it is what is computed: expf
+// next to zero is off by an ulp of one to the same side token after token.
 __device__ __forceinline__ void rg_gates(float gr, float gi, float decay, float u, float& a, float& d) {
-  a = expf(decay * rg_sigmoid(gr));
-  d = sqrtf(1.f - __fmul_rn(a, a)) * rg_sigmoid(gi) * u;
+  const float m = expm1f(decay * rg_sigmoid(gr));                 // a - 1
+  a = 1.f + m;
+  d = sqrtf(-m * (2.f + m)) * rg_sigmoid(gi) * u;
 }
 
 __device__ __forceinline__ float rg_load(const void* p, bool f32, size_t i) {

@@ -210,7 +210,7 @@ class GpuRunner(BaseRunner):
                 loaded.append(got[0])
             sid, state = None, None
             if hybrid:
-                if loaded and end == b0 + n and any(k.startswith("conv.") for k in loaded[-1]):
+                if loaded and end == b0 + n and any(k.startswith(("conv.", "gdn.")) for k in loaded[-1]):
                     state = loaded[-1]
                 else:
                     got = self.cold.get(keys[end - 1] + ".s")
