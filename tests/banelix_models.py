@@ -69,7 +69,7 @@ WIDE = model(160, 200, [
 ])
 # sizes of one: one head, one pair, windows of one and two tokens, blocks of one channel, no convolution, factors of one
 ONES = model(64, 96, [
-    (both(1, 1, 2, 1.0, rotation(2, 100.0, bands(1.0, 1.0, 4.0, 32.0)), 16, 16, 1, 1.0, 1.0), 16),
+    (both(1, 1, 7, 1.0, rotation(2, 100.0, bands(1.0, 1.0, 4.0, 32.0)), 16, 16, 1, 1.0, 1.0), 16),
     (windowed(1, 1, 8, 3, 0.5, 1, rotation(2, 100.0, yarn(1.0, 32.0, 2.0, 1.0))), 8),
     (windowed(2, 2, 16, 16, 0.3, 2, rotation(16, 50.0)), 24),
     (both(3, 3, 8, 0.5, rotation(4, 10.0), 8, 1, 2, 1.0, 1.0), 8),
