@@ -167,11 +167,15 @@ __device__ __forceinline__ float inv_rms_of(const Tile<MT, NT>& sm, int col, int
 }
 
 // acc += W[16 MT rows][K] x[K][8 NT]: this warp's units (every STEP-th one).  wrow[m][half] points at column 8c of row (g + 8 half) of tile m.
-// EARLY: the weights do not depend on earlier kernels, so the first batch is requested before griddepcontrol.wait.
-template <int MT, int NT, bool XF32, bool EARLY, int STEP = NW>
+// EARLY: the weights do not depend on earlier kernels, so the first batch is requested before griddepcontrol.wait; ``after``
+// runs right behind the wait (loads for the epilogue).
+struct Nothing {
+  __device__ void operator()() const {}
+};
+template <int MT, int NT, bool XF32, bool EARLY, int STEP = NW, typename After = Nothing>
 __device__ __forceinline__ void product(const __nv_bfloat16* const (&wrow)[MT][2], int K, const void* x,
                                         long long x_stride, int R, const float* norm_w, float (&acc)[MT][NT][4],
-                                        float (&ss)[NT]) {
+                                        float (&ss)[NT], After after = After()) {
   constexpr int UN = MT == 1 ? 4 : 2;                    // units in flight per warp: 16 x 16 bytes per lane
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, g = lane >> 2, c = lane & 3;
   const int units = (K + UK - 1) / UK, first = STEP == NW ? warp : 0;
@@ -193,6 +197,7 @@ __device__ __forceinline__ void product(const __nv_bfloat16* const (&wrow)[MT][2
   if (EARLY) {
     load_a(first);
     pdl_wait();
+    after();
   }
   for (int u0 = first; u0 < units; u0 += UN * STEP) {
     if (!EARLY || u0 != first) load_a(u0);
@@ -443,25 +448,49 @@ __global__ void __launch_bounds__(NW * 32, 2) rglru_step_kernel(const __grid_con
   const __nv_bfloat16* u = reinterpret_cast<const __nv_bfloat16*>(a.u) + (size_t)b * a.u_bs;
   float acc[2][NT][4] = {};
   float ss[NT] = {};
-  product<2, NT, false, true>(wrow, bc, u, a.u_ts, a.n_seg, nullptr, acc, ss);
+  // what the epilogue of this thread's channel and token needs, requested ahead of the product
+  static_assert(16 * NT * 8 <= NW * 32, "one output per thread");
+  constexpr int PAST = 3;                                  // convolution inputs kept in registers
+  const int row = threadIdx.x & 15, r = threadIdx.x >> 4, n = row0 + row, ch = b * bc + n, past = a.taps - 1;
+  int slot = 0;
+  bool live = r < NT * 8 && r < a.n_seg && n < bc;
+  float S = 0.f, y = 0.f, un = 0.f, dec = 0.f, g0 = 0.f, g1 = 0.f, x = 0.f, hist[PAST] = {};
+  const auto ahead = [&]() {
+    if (!live) return;
+    slot = a.seg_slot[r];
+    if (!HE_INDEX_OK(slot, a.n_slots, HE_SITE_STATE_SLOT)) {
+      live = false;
+      return;
+    }
+    S = a.S[(size_t)slot * a.C + ch];
+    y = rg_load(a.y, a.row_dtype == 0, (size_t)r * a.row_stride + ch) + a.yb[ch];
+    un = bf16_to_f32(u[(size_t)r * a.u_ts + n]);
+    dec = a.decay[ch];
+    g0 = a.gb[(size_t)b * 2 * bc + n];
+    g1 = a.gb[(size_t)b * 2 * bc + bc + n];
+    if (past >= 1 && past <= PAST) {
+      x = rg_load(a.x, a.row_dtype == 0, (size_t)r * a.row_stride + ch) + a.xb[ch];
+#pragma unroll
+      for (int j = 1; j < PAST; ++j)
+        if (j < past) hist[j] = a.cstate[((size_t)slot * past + j) * a.C + ch];
+    }
+  };
+  product<2, NT, false, true, NW>(wrow, bc, u, a.u_ts, a.n_seg, nullptr, acc, ss, ahead);
   store_partials<2, NT>(sm, acc, ss);
   __syncthreads();
-  for (int o = threadIdx.x; o < 16 * NT * 8; o += NW * 32) {
-    const int row = o & 15, r = o >> 4, n = row0 + row;
-    if (r >= a.n_seg || n >= bc) continue;
-    const int ch = b * bc + n, slot = a.seg_slot[r];
-    if (!HE_INDEX_OK(slot, a.n_slots, HE_SITE_STATE_SLOT)) continue;
-    float* S = a.S + (size_t)slot * a.C + ch;
-    const float* gb = a.gb + (size_t)b * 2 * bc + n;
-    const float y = rg_load(a.y, a.row_dtype == 0, (size_t)r * a.row_stride + ch) + a.yb[ch];
-    float av, dv;
-    rg_gates(sum_partials<2, NT>(sm, row, r) + gb[0], sum_partials<2, NT>(sm, 16 + row, r) + gb[bc], a.decay[ch],
-             bf16_to_f32(u[(size_t)r * a.u_ts + n]), av, dv);
-    const float s = av * *S + dv;
-    *S = s;
-    reinterpret_cast<__nv_bfloat16*>(a.out)[(size_t)r * a.out_stride + ch] = f32_to_bf16(s * gelu_tanh_f(y));
+  if (!live) return;
+  float av, dv;
+  rg_gates(sum_partials<2, NT>(sm, row, r) + g0, sum_partials<2, NT>(sm, 16 + row, r) + g1, dec, un, av, dv);
+  S = av * S + dv;
+  a.S[(size_t)slot * a.C + ch] = S;
+  reinterpret_cast<__nv_bfloat16*>(a.out)[(size_t)r * a.out_stride + ch] = f32_to_bf16(S * rg_gelu(y));
+  if (past > PAST) {
     rg_conv_state(a, slot, ch, r, 1);
+    return;
   }
+#pragma unroll
+  for (int j = 1; j <= PAST; ++j)
+    if (j <= past) a.cstate[((size_t)slot * past + j - 1) * a.C + ch] = j == past ? x : hist[j < PAST ? j : 0];
 }
 
 template <int MT>

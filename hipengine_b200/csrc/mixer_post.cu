@@ -2,8 +2,9 @@
 // biases, norm and rotation and go to the query buffer and the pages; the inputs of a recurrence go through its short causal
 // convolution.
 //
-// grid (T, query parts + key parts + value parts + convolution parts): a CTA takes one token and a range of heads (staged in
-// shared memory, a warp per head) or 1024 channels.  Norms: per head or over the whole projection before the rotation (with
+// grid: T * (query parts + key parts + value parts) CTAs of one token and a range of heads (staged in shared memory, a warp per
+// head; a lane keeps the sines and cosines of its dimensions over the heads), then the convolution's CTAs of 1024 channels
+// and one or several tokens.  Norms: per head or over the whole projection before the rotation (with
 // gains), or per head after it (without).  The rotation turns (i, i + n/2) or (2i, 2i + 1) by table frequencies; angles
 // are reduced to one turn in double.  The convolution's state is only read here: the recurrence, which runs later in stream
 // order, replaces it.
@@ -44,7 +45,7 @@ struct MixerPostArgs {
   int T, in_dtype, out_f32;  // 0 f32, 1 bf16; q_out, kv_cache and u in fp32
   int norm;                  // 0 none, 1 per head, 2 whole projection, 3 per head after the rotation
   int rot_dims, halves;
-  int D, page, max_pages, heads_per_cta;
+  int D, page, max_pages, heads_per_cta, conv_tokens;
   float eps, amp;
 };
 
@@ -52,6 +53,7 @@ namespace {
 
 constexpr int NTHR = 256;
 constexpr int CONV_CHANNELS = NTHR * 4;
+constexpr int CONV_TOKENS = 8;     // of a convolution CTA in long batches
 constexpr int MAX_PAIRS = 8;       // head widths up to 512: a lane owns up to eight neighbouring pairs
 
 __device__ __forceinline__ float4 load4(const void* p, int dtype, size_t i) {
@@ -86,39 +88,80 @@ __device__ __forceinline__ float sq_upto(float4 v, int i, int n) {
   return s;
 }
 
-template <typename OutT>
-__device__ __forceinline__ void conv_part(const MixerPostArgs& a, int t, int chunk) {
-  const int c = chunk * CONV_CHANNELS + threadIdx.x * 4;
+// 1024 channels of `a.conv_tokens` tokens.  TAPS > 0: filter and window in registers.
+template <typename OutT, int TAPS>
+__device__ __forceinline__ void conv_part(const MixerPostArgs& a, int index) {
+  const int chunks = (a.C + CONV_CHANNELS - 1) / CONV_CHANNELS;
+  const int c = (index % chunks) * CONV_CHANNELS + threadIdx.x * 4, t0 = (index / chunks) * a.conv_tokens;
   if (c >= a.C) return;
-  const int sg = a.tok_seg[t], s0 = a.seg_start[sg], slot = a.seg_slot[sg], local = t - s0, past = a.taps - 1;
-  if (!HE_INDEX_OK(slot, a.n_slots, HE_SITE_STATE_SLOT)) return;
-  const float4 xb = *reinterpret_cast<const float4*>(a.cx_bias + c);
-  float4 acc = *reinterpret_cast<const float4*>(a.cb + c);
-  for (int j = 0; j < a.taps; ++j) {
-    const int idx = local + j;                   // of [state ++ segment]
-    const float4 w = *reinterpret_cast<const float4*>(a.cw + (size_t)j * a.C + c);
-    const float4 x = idx < past ? *reinterpret_cast<const float4*>(a.cstate + ((size_t)slot * past + idx) * a.C + c)
-                                : add4(load4(a.cx, a.in_dtype, (size_t)(s0 + idx - past) * a.cx_stride + c), xb);
-    acc.x += w.x * x.x; acc.y += w.y * x.y; acc.z += w.z * x.z; acc.w += w.w * x.w;
-    if (a.cjournal != nullptr && j > 0) *reinterpret_cast<float4*>(a.cjournal + ((size_t)t * past + j - 1) * a.C + c) = x;
+  const int taps = TAPS > 0 ? TAPS : a.taps, past = taps - 1, t1 = min(a.T, t0 + a.conv_tokens);
+  const float4 xb = *reinterpret_cast<const float4*>(a.cx_bias + c), bias = *reinterpret_cast<const float4*>(a.cb + c);
+  OutT* out = reinterpret_cast<OutT*>(a.u) + (size_t)(c / a.block_cols) * a.u_bs + c % a.block_cols;
+  float4 w[TAPS > 0 ? TAPS : 1], win[TAPS > 0 ? TAPS : 1];
+  if constexpr (TAPS > 0)
+#pragma unroll
+    for (int j = 0; j < TAPS; ++j) w[j] = *reinterpret_cast<const float4*>(a.cw + (size_t)j * a.C + c);
+  int seg = -1, s0 = 0, slot = 0;
+  for (int t = t0; t < t1; ++t) {
+    const int sg = a.tok_seg[t];
+    const bool first = sg != seg;
+    if (first) {
+      seg = sg;
+      s0 = a.seg_start[sg];
+      slot = a.seg_slot[sg];
+    }
+    if (!HE_INDEX_OK(slot, a.n_slots, HE_SITE_STATE_SLOT)) continue;
+    // input `idx` of [state ++ segment], counted from the oldest one that this token needs
+    const auto input = [&](int j) -> float4 {
+      const int idx = t - s0 + j;
+      return idx < past ? *reinterpret_cast<const float4*>(a.cstate + ((size_t)slot * past + idx) * a.C + c)
+                        : add4(load4(a.cx, a.in_dtype, (size_t)(s0 + idx - past) * a.cx_stride + c), xb);
+    };
+    const auto journal = [&](int j, float4 x) {
+      if (a.cjournal != nullptr && j > 0) *reinterpret_cast<float4*>(a.cjournal + ((size_t)t * past + j - 1) * a.C + c) = x;
+    };
+    float4 acc = bias;
+    const auto tap = [&](float4 f, float4 x) {
+      acc.x += f.x * x.x; acc.y += f.y * x.y; acc.z += f.z * x.z; acc.w += f.w * x.w;
+    };
+    if constexpr (TAPS > 0) {
+#pragma unroll
+      for (int j = 0; j < TAPS; ++j) win[j] = first || j == TAPS - 1 ? input(j) : win[j + 1];
+#pragma unroll
+      for (int j = 0; j < TAPS; ++j) {
+        tap(w[j], win[j]);
+        journal(j, win[j]);
+      }
+    } else {
+      for (int j = 0; j < taps; ++j) {
+        const float4 x = input(j);
+        tap(*reinterpret_cast<const float4*>(a.cw + (size_t)j * a.C + c), x);
+        journal(j, x);
+      }
+    }
+    store4(out + (size_t)t * a.u_ts, acc);
   }
-  store4(reinterpret_cast<OutT*>(a.u) + (size_t)(c / a.block_cols) * a.u_bs + (size_t)t * a.u_ts + c % a.block_cols, acc);
 }
 
-template <typename OutT>
+template <typename OutT, int NP>
 __global__ void __launch_bounds__(NTHR) mixer_post_kernel(const __grid_constant__ MixerPostArgs a) {
   extern __shared__ __align__(16) float sm[];    // [rot_dims] (cos, sin) pairs, then the staged columns
   __shared__ float red[33];
   pdl_wait();
   pdl_launch();
-  const int t = blockIdx.x, lane = threadIdx.x & 31, warp = threadIdx.x >> 5, D = a.D;
-  int y = blockIdx.y, kind = 0;                  // 0 query, 1 key, 2 value
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, D = a.D;
   const auto parts = [&](const HeadRows& r) { return r.x == nullptr ? 0 : (r.heads + a.heads_per_cta - 1) / a.heads_per_cta; };
-  const int nq = parts(a.q), nk = parts(a.k), nv = parts(a.v);
-  if (y >= nq + nk + nv) {
-    conv_part<OutT>(a, t, y - nq - nk - nv);
+  const int nq = parts(a.q), nk = parts(a.k), np = nq + nk + parts(a.v);
+  if ((int)blockIdx.x >= a.T * np) {
+    const int i = blockIdx.x - a.T * np;
+    if (a.taps == 4) conv_part<OutT, 4>(a, i);
+    else if (a.taps == 3) conv_part<OutT, 3>(a, i);
+    else if (a.taps == 2) conv_part<OutT, 2>(a, i);
+    else conv_part<OutT, 0>(a, i);
     return;
   }
+  const int t = blockIdx.x / np;
+  int y = blockIdx.x - t * np, kind = 0;         // 0 query, 1 key, 2 value
   if (y >= nq + nk) { kind = 2; y -= nq + nk; }
   else if (y >= nq) { kind = 1; y -= nq; }
   const HeadRows& r = kind == 0 ? a.q : kind == 1 ? a.k : a.v;
@@ -135,83 +178,118 @@ __global__ void __launch_bounds__(NTHR) mixer_post_kernel(const __grid_constant_
   }
   float* cols = sm + ((a.rot_dims + 3) & ~3);
   const size_t in0 = (size_t)t * r.stride;
-  float ss = 0.f;
-  for (int i = threadIdx.x * 4; i < n; i += NTHR * 4) {
-    float4 v = load4(r.x, a.in_dtype, in0 + c0 + i);
-    if (r.bias != nullptr) v = add4(v, *reinterpret_cast<const float4*>(r.bias + c0 + i));
-    *reinterpret_cast<float4*>(cols + i) = v;
-    ss += sq_upto(v, i, n);
+  // columns [lo, hi) are read (the whole projection where its norm needs it), [c0, c0 + n) are kept; the first 4096 are
+  // requested before the angles are computed
+  const int lo = norm == 2 ? 0 : c0, hi = norm == 2 ? all : c0 + n;
+  constexpr int PRE = 4;
+  float4 pre[PRE];
+  const auto biased = [&](int i) -> float4 {
+    const float4 v = load4(r.x, a.in_dtype, in0 + i);
+    return r.bias != nullptr ? add4(v, *reinterpret_cast<const float4*>(r.bias + i)) : v;
+  };
+#pragma unroll
+  for (int k = 0; k < PRE; ++k) {
+    const int i = lo + (threadIdx.x + k * NTHR) * 4;
+    if (i < hi) pre[k] = biased(i);
   }
   if (turned)
     for (int i = threadIdx.x; i < half; i += NTHR) {
-      const double two_pi = 6.283185307179586476925286766559;
+      const double two_pi = 6.283185307179586476925286766559, per_turn = 0.15915494309189533576888376337251;
       const double ang = (double)p * a.freq[i];
       float sn, c;
-      sincosf((float)(ang - two_pi * rint(ang / two_pi)), &sn, &c);
+      sincosf((float)(ang - two_pi * rint(ang * per_turn)), &sn, &c);
       sm[2 * i] = c * a.amp;
       sm[2 * i + 1] = sn * a.amp;
     }
-  if (norm == 2) {
-    if (n < all) {                               // a part of the heads: the squares of the whole projection again
-      ss = 0.f;
-      for (int i = threadIdx.x * 4; i < all; i += NTHR * 4) {
-        float4 v = load4(r.x, a.in_dtype, in0 + i);
-        if (r.bias != nullptr) v = add4(v, *reinterpret_cast<const float4*>(r.bias + i));
-        ss += sq_upto(v, i, all);
-      }
-    }
-    const float inv = rsqrtf(block_sum(ss, red) / (float)all + a.eps);
-    for (int i = threadIdx.x * 4; i < n; i += NTHR * 4) {                   // the columns this thread staged
-      float4 v = *reinterpret_cast<float4*>(cols + i);
-      const float4 g = *reinterpret_cast<const float4*>(r.gain + c0 + i);
-      *reinterpret_cast<float4*>(cols + i) = make_float4(v.x * inv * g.x, v.y * inv * g.y, v.z * inv * g.z, v.w * inv * g.w);
-    }
+  float ss = 0.f;
+  const auto keep = [&](int i, float4 v) {
+    if (i >= c0 && i < c0 + n) *reinterpret_cast<float4*>(cols + i - c0) = v;
+    ss += sq_upto(v, i, hi);
+  };
+#pragma unroll
+  for (int k = 0; k < PRE; ++k) {
+    const int i = lo + (threadIdx.x + k * NTHR) * 4;
+    if (i < hi) keep(i, pre[k]);
   }
+  for (int i = lo + (threadIdx.x + PRE * NTHR) * 4; i < hi; i += NTHR * 4) keep(i, biased(i));
+  float inv_all = 1.f;
+  if (norm == 2) inv_all = rsqrtf(block_sum(ss, red) / (float)all + a.eps);
   __syncthreads();
 
+  // value of dimension d = c * x[d] + s * x[partner]; both of a lane's neighbouring dimensions are turned or none is
+  float2 cs[NP][2];
+#pragma unroll
+  for (int j = 0; j < NP; ++j) {
+    const int d = lane * 2 + 64 * j;
+    cs[j][0] = cs[j][1] = make_float2(1.f, 0.f);
+    if (turned && d < a.rot_dims) {
+#pragma unroll
+      for (int e = 0; e < 2; ++e) {
+        const int i = a.halves ? (d + e < half ? d + e : d + e - half) : (d >> 1);
+        const bool lower = a.halves ? d + e < half : e == 0;
+        cs[j][e] = make_float2(sm[2 * i], lower ? -sm[2 * i + 1] : sm[2 * i + 1]);
+      }
+    }
+  }
+  const bool pairs = (dim & 1) == 0 && (!turned || !a.halves || (half & 1) == 0);   // two dimensions and their partners are neighbours
+  const size_t plane = (size_t)r.heads * a.page * D;                         // from a key row to its value row
   for (int h = warp; h < nh; h += NTHR / 32) {
     float* x = cols + h * dim;
     const size_t out0 = kind == 0 ? ((size_t)t * r.heads + h0 + h) * D : row0 + (size_t)h * a.page * D;
-    const size_t plane = (size_t)r.heads * a.page * D;                       // from a key row to its value row
     if (kind == 1 && a.v.x == nullptr)
       for (int d = lane * 2; d < D; d += 64)
         store2(reinterpret_cast<OutT*>(a.kv_cache) + out0 + plane + d, d < dim ? x[d] : 0.f, d + 1 < dim ? x[d + 1] : 0.f);
     __syncwarp();
-    if (norm == 1) {
-      float s = 0.f;
-      for (int d = lane; d < dim; d += 32) s += x[d] * x[d];
-      const float inv = rsqrtf(warp_sum(s) / (float)dim + a.eps);
-      for (int d = lane; d < dim; d += 32) x[d] *= inv * r.gain[d];
+    if (norm == 1 || norm == 2) {
+      float inv = inv_all;
+      const float* gain = norm == 1 ? r.gain : r.gain + c0 + h * dim;
+      if (norm == 1) {
+        float s = 0.f;
+        for (int d = lane; d < dim; d += 32) s += x[d] * x[d];
+        inv = rsqrtf(warp_sum(s) / (float)dim + a.eps);
+      }
+      for (int d = lane; d < dim; d += 32) x[d] *= inv * gain[d];
+      __syncwarp();
     }
-    __syncwarp();
-    const auto value = [&](int d) -> float {
-      if (d >= dim) return 0.f;
-      const float v = x[d];
-      if (!turned || d >= a.rot_dims) return v;
-      if (a.halves) {
-        const int i = d < half ? d : d - half;
-        const float c = sm[2 * i], s = sm[2 * i + 1];
-        return d < half ? v * c - x[d + half] * s : v * c + x[i] * s;
-      }
-      const float c = sm[d & ~1], s = sm[d | 1];
-      return (d & 1) == 0 ? v * c - x[d + 1] * s : v * c + x[d - 1] * s;
-    };
-    float v[MAX_PAIRS][2], s = 0.f;
+    float v[NP][2], s = 0.f;
 #pragma unroll
-    for (int j = 0; j < MAX_PAIRS; ++j) {
+    for (int j = 0; j < NP; ++j) {
       const int d = lane * 2 + 64 * j;
-      if (64 * j < D) {
-        v[j][0] = value(d);
-        v[j][1] = value(d + 1);
-        s += v[j][0] * v[j][0] + v[j][1] * v[j][1];
+      v[j][0] = v[j][1] = 0.f;
+      if (d >= dim) continue;
+      const bool mine = turned && d < a.rot_dims;
+      if (pairs) {
+        const float2 own = *reinterpret_cast<const float2*>(x + d);
+        float2 other = own;
+        if (mine) {
+          other = *reinterpret_cast<const float2*>(x + (!a.halves ? d : d < half ? d + half : d - half));
+          if (!a.halves) other = make_float2(own.y, own.x);
+        }
+        v[j][0] = cs[j][0].x * own.x + cs[j][0].y * other.x;
+        v[j][1] = cs[j][1].x * own.y + cs[j][1].y * other.y;
+      } else {
+#pragma unroll
+        for (int e = 0; e < 2; ++e) {
+          if (d + e >= dim) continue;
+          float other = 0.f;
+          if (mine) other = x[!a.halves ? d + (e ^ 1) : d + e < half ? d + e + half : d + e - half];
+          v[j][e] = cs[j][e].x * x[d + e] + cs[j][e].y * other;
+        }
       }
+      s += v[j][0] * v[j][0] + v[j][1] * v[j][1];
     }
     const float inv = norm == 3 ? rsqrtf(warp_sum(s) / (float)dim + a.eps) : 1.f;
     OutT* out = reinterpret_cast<OutT*>(kind == 0 ? a.q_out : a.kv_cache) + out0 + (kind == 2 ? plane : 0);
 #pragma unroll
-    for (int j = 0; j < MAX_PAIRS; ++j)
+    for (int j = 0; j < NP; ++j)
       if (64 * j < D) store2(out + lane * 2 + 64 * j, v[j][0] * inv, v[j][1] * inv);
   }
+}
+
+template <int NP>
+int launch(const MixerPostArgs& a, dim3 grid, dim3 block, size_t smem, cudaStream_t stream) {
+  return (int)(a.out_f32 ? launch_pdl(mixer_post_kernel<float, NP>, grid, block, smem, stream, a)
+                         : launch_pdl(mixer_post_kernel<__nv_bfloat16, NP>, grid, block, smem, stream, a));
 }
 
 }  // namespace
@@ -246,10 +324,18 @@ HE_API int he_mixer_post(const MixerPostArgs* args, cudaStream_t stream) {
   if (per > most) per = most;
   if (per < 1) return -HE_ERR_BAD_ARG;
   a.heads_per_cta = per;
+  a.conv_tokens = a.T < 148 ? 1 : CONV_TOKENS;
   const auto parts = [&](const HeadRows& r) { return r.x == nullptr ? 0 : (r.heads + per - 1) / per; };
   const size_t smem = (size_t)(((a.rot_dims + 3) & ~3) + per * widest + 8) * sizeof(float);
-  const dim3 grid(a.T, parts(a.q) + parts(a.k) + parts(a.v) + conv), block(NTHR);
-  return (int)(a.out_f32 ? launch_pdl(mixer_post_kernel<float>, grid, block, smem, stream, a)
-                         : launch_pdl(mixer_post_kernel<__nv_bfloat16>, grid, block, smem, stream, a));
+  const long long ctas = (long long)a.T * (parts(a.q) + parts(a.k) + parts(a.v)) +
+                         (long long)conv * ((a.T + a.conv_tokens - 1) / a.conv_tokens);
+  if (ctas > 0x7fffffffLL) return -HE_ERR_BAD_ARG;
+  const dim3 grid((unsigned)ctas), block(NTHR);
+  switch (a.D / 64) {
+    case 1: return launch<1>(a, grid, block, smem, stream);
+    case 2: return launch<2>(a, grid, block, smem, stream);
+    case 3: case 4: return launch<4>(a, grid, block, smem, stream);
+    default: return launch<8>(a, grid, block, smem, stream);
+  }
 }
 HE_API int he_mixer_post_args_size() { return (int)sizeof(MixerPostArgs); }

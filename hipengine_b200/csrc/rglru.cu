@@ -31,22 +31,34 @@ __global__ void __launch_bounds__(NTHR, 2) rglru_scan_kernel(const __grid_consta
   const float decay = a.decay[cc], yb = a.yb[cc];
   float S0 = cw < a.C ? a.S[(size_t)slot * a.C + cw] : 0.f;                  // of channel cw, before the tile
   for (int tile = s0; tile < s1; tile += TILE) {
-    const int t0 = tile + grp * LEN;
-    float A[LEN], d[LEN], y[LEN];
+    const int t0 = tile + grp * LEN, last = s1 - 1 - t0;                      // tokens behind the last one repeat it
+    float A[LEN], d[LEN], u[LEN];
+    if (last >= LEN - 1) {
+      const float* gp = g + (size_t)t0 * a.g_ts;
+      size_t ui = u0 + (size_t)t0 * a.u_ts;
 #pragma unroll
-    for (int k = 0; k < LEN; ++k) {
-      const int t = min(t0 + k, s1 - 1);
-      A[k] = g[(size_t)t * a.g_ts];
-      d[k] = g[(size_t)t * a.g_ts + a.block_cols];
-      y[k] = rg_load(a.y, ROW_F32, (size_t)t * a.row_stride + cc);
+      for (int k = 0; k < LEN; ++k) {
+        A[k] = gp[0];
+        d[k] = gp[a.block_cols];
+        u[k] = rg_load(a.u, ACT_F32, ui);
+        gp += a.g_ts;
+        ui += a.u_ts;
+      }
+    } else {
+#pragma unroll
+      for (int k = 0; k < LEN; ++k) {
+        const int t = min(t0 + k, s1 - 1);
+        A[k] = g[(size_t)t * a.g_ts];
+        d[k] = g[(size_t)t * a.g_ts + a.block_cols];
+        u[k] = rg_load(a.u, ACT_F32, u0 + (size_t)t * a.u_ts);
+      }
     }
     float pa = 1.f, pb = 0.f;
 #pragma unroll
     for (int k = 0; k < LEN; ++k) {
-      const float u = rg_load(a.u, ACT_F32, u0 + (size_t)min(t0 + k, s1 - 1) * a.u_ts);
       float ak, dk;
-      rg_gates(A[k] + gb0, d[k] + gb1, decay, u, ak, dk);
-      if (t0 + k >= s1) {
+      rg_gates(A[k] + gb0, d[k] + gb1, decay, u[k], ak, dk);
+      if (k > last) {
         ak = 1.f;
         dk = 0.f;
       }
@@ -57,6 +69,9 @@ __global__ void __launch_bounds__(NTHR, 2) rglru_scan_kernel(const __grid_consta
     }
     sA[grp][ch] = pa;
     sB[grp][ch] = pb;
+    float y[LEN];                                        // on their way while the groups are composed
+#pragma unroll
+    for (int k = 0; k < LEN; ++k) y[k] = rg_load(a.y, ROW_F32, (size_t)min(t0 + k, s1 - 1) * a.row_stride + cc);
     __syncthreads();
     pa = sA[lane][warp];
     pb = sB[lane][warp];
@@ -81,8 +96,8 @@ __global__ void __launch_bounds__(NTHR, 2) rglru_scan_kernel(const __grid_consta
     for (int k = 0; k < LEN; ++k) {
       S = A[k] * S + d[k];
       const int t = t0 + k;
-      if (live && t < s1) {
-        const float v = S * gelu_tanh_f(y[k] + yb);
+      if (live && k <= last) {
+        const float v = S * rg_gelu(y[k] + yb);
         const size_t o = (size_t)t * a.out_stride + c;
         if constexpr (ACT_F32) reinterpret_cast<float*>(a.out)[o] = v;
         else reinterpret_cast<__nv_bfloat16*>(a.out)[o] = f32_to_bf16(v);
@@ -110,7 +125,7 @@ __global__ void __launch_bounds__(256) rglru_rows_kernel(const __grid_constant__
   rg_gates(g[0] + gb[0], g[a.block_cols] + gb[a.block_cols], a.decay[c],
            rg_load(a.u, ACT_F32, (size_t)b * a.u_bs + (size_t)t * a.u_ts + cb), ak, dk);
   const float S = ak * a.S[(size_t)slot * a.C + c] + dk;
-  const float v = S * gelu_tanh_f(rg_load(a.y, ROW_F32, (size_t)t * a.row_stride + c) + a.yb[c]);
+  const float v = S * rg_gelu(rg_load(a.y, ROW_F32, (size_t)t * a.row_stride + c) + a.yb[c]);
   const size_t o = (size_t)t * a.out_stride + c;
   if constexpr (ACT_F32) reinterpret_cast<float*>(a.out)[o] = v;
   else reinterpret_cast<__nv_bfloat16*>(a.out)[o] = f32_to_bf16(v);

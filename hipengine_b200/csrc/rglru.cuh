@@ -33,14 +33,32 @@ struct RglruArgs {
 
 namespace he {
 
-__device__ __forceinline__ float rg_sigmoid(float x) { return 1.f / (1.f + expf(-x)); }
+__device__ __forceinline__ float rg_sigmoid(float x) { return __fdividef(1.f, 1.f + __expf(fminf(-x, 80.f))); }
 
-// decay and drive of one token and channel.  Memories of thousands of tokens hang on 1 - a, so it is what is computed: expf
-// next to zero is off by an ulp of one to the same side token after token.
+// e^x - 1 for x <= 0 with a small relative error: the power series (nested) near zero, the difference elsewhere
+__device__ __forceinline__ float rg_expm1(float x) {
+  const float s = x * (1.f + x * (1.f / 2.f) * (1.f + x * (1.f / 3.f) * (1.f + x * (1.f / 4.f) * (1.f + x * (1.f / 5.f) *
+                  (1.f + x * (1.f / 6.f))))));
+  return x > -0.25f ? s : __expf(x) - 1.f;
+}
+
+__device__ __forceinline__ float rg_sqrt(float x) {
+  float y;
+  asm("sqrt.approx.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+
+// gelu_tanh(z) = z / 2 (1 + tanh w) = z sigmoid(2 w)
+__device__ __forceinline__ float rg_gelu(float z) {
+  return z * rg_sigmoid(1.5957691216057308f * (z + 0.044715f * z * z * z));
+}
+
+// decay and drive of one token and channel.  Memories of thousands of tokens hang on 1 - a, so it is what is computed: an
+// exponential next to one that is off by an ulp is off to the same side token after token.
 __device__ __forceinline__ void rg_gates(float gr, float gi, float decay, float u, float& a, float& d) {
-  const float m = expm1f(decay * rg_sigmoid(gr));                 // a - 1
+  const float m = rg_expm1(decay * rg_sigmoid(gr));               // a - 1
   a = 1.f + m;
-  d = sqrtf(-m * (2.f + m)) * rg_sigmoid(gi) * u;
+  d = rg_sqrt(-m * (2.f + m)) * rg_sigmoid(gi) * u;
 }
 
 __device__ __forceinline__ float rg_load(const void* p, bool f32, size_t i) {

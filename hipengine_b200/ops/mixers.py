@@ -26,7 +26,7 @@ class _PostArgs(C.Structure):
                 ("tok_seg", c_vp), ("u", c_vp), ("u_ts", c_ll), ("u_bs", c_ll), ("C", c_int), ("block_cols", c_int),
                 ("taps", c_int), ("n_slots", c_int), ("T", c_int), ("in_dtype", c_int), ("out_f32", c_int), ("norm", c_int),
                 ("rot_dims", c_int), ("halves", c_int), ("D", c_int), ("page", c_int), ("max_pages", c_int),
-                ("heads_per_cta", c_int), ("eps", C.c_float), ("amp", C.c_float)]
+                ("heads_per_cta", c_int), ("conv_tokens", c_int), ("eps", C.c_float), ("amp", C.c_float)]
 
 
 class _RglruArgs(C.Structure):
