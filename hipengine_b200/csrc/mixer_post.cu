@@ -144,16 +144,16 @@ __device__ __forceinline__ void conv_part(const MixerPostArgs& a, int index) {
 }
 
 template <typename OutT, int NP>
-__global__ void __launch_bounds__(NTHR) mixer_post_kernel(const __grid_constant__ MixerPostArgs a) {
+__global__ void __launch_bounds__(NTHR, NP <= 2 ? 4 : 2) mixer_post_kernel(const __grid_constant__ MixerPostArgs a) {
   extern __shared__ __align__(16) float sm[];    // [rot_dims] (cos, sin) pairs, then the staged columns
   __shared__ float red[33];
-  pdl_wait();
   pdl_launch();
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, D = a.D;
   const auto parts = [&](const HeadRows& r) { return r.x == nullptr ? 0 : (r.heads + a.heads_per_cta - 1) / a.heads_per_cta; };
   const int nq = parts(a.q), nk = parts(a.k), np = nq + nk + parts(a.v);
   if ((int)blockIdx.x >= a.T * np) {
     const int i = blockIdx.x - a.T * np;
+    pdl_wait();
     if (a.taps == 4) conv_part<OutT, 4>(a, i);
     else if (a.taps == 3) conv_part<OutT, 3>(a, i);
     else if (a.taps == 2) conv_part<OutT, 2>(a, i);
@@ -168,7 +168,21 @@ __global__ void __launch_bounds__(NTHR) mixer_post_kernel(const __grid_constant_
   const int h0 = y * a.heads_per_cta, nh = min(a.heads_per_cta, r.heads - h0), dim = r.dim;
   const int c0 = h0 * dim, n = nh * dim, all = r.heads * dim;
   const bool turned = kind < 2 && a.rot_dims > 0;
-  const int norm = kind < 2 ? a.norm : 0, p = a.pos[t], half = a.rot_dims >> 1;
+  const int norm = kind < 2 ? a.norm : 0, half = a.rot_dims >> 1;
+  // columns [lo, hi) are read (the whole projection where its norm needs it), [c0, c0 + n) are kept; the first 4096 are
+  // requested before the angles are computed, and what does not depend on earlier kernels before these end
+  const int lo = norm == 2 ? 0 : c0, hi = norm == 2 ? all : c0 + n;
+  constexpr int PRE = 4;
+  float4 pre[PRE], pre_b[PRE];
+  const auto bias = [&](int i) { return r.bias != nullptr ? *reinterpret_cast<const float4*>(r.bias + i) : make_float4(0.f, 0.f, 0.f, 0.f); };
+#pragma unroll
+  for (int k = 0; k < PRE; ++k) {
+    const int i = lo + (threadIdx.x + k * NTHR) * 4;
+    if (i < hi) pre_b[k] = bias(i);
+  }
+  const double freq0 = turned && (int)threadIdx.x < half ? a.freq[threadIdx.x] : 0.0;
+  pdl_wait();
+  const int p = a.pos[t];
   size_t row0 = 0;                               // of the key or value rows in the pages
   if (kind > 0) {
     const int pi = p / a.page;
@@ -178,24 +192,15 @@ __global__ void __launch_bounds__(NTHR) mixer_post_kernel(const __grid_constant_
   }
   float* cols = sm + ((a.rot_dims + 3) & ~3);
   const size_t in0 = (size_t)t * r.stride;
-  // columns [lo, hi) are read (the whole projection where its norm needs it), [c0, c0 + n) are kept; the first 4096 are
-  // requested before the angles are computed
-  const int lo = norm == 2 ? 0 : c0, hi = norm == 2 ? all : c0 + n;
-  constexpr int PRE = 4;
-  float4 pre[PRE];
-  const auto biased = [&](int i) -> float4 {
-    const float4 v = load4(r.x, a.in_dtype, in0 + i);
-    return r.bias != nullptr ? add4(v, *reinterpret_cast<const float4*>(r.bias + i)) : v;
-  };
 #pragma unroll
   for (int k = 0; k < PRE; ++k) {
     const int i = lo + (threadIdx.x + k * NTHR) * 4;
-    if (i < hi) pre[k] = biased(i);
+    if (i < hi) pre[k] = load4(r.x, a.in_dtype, in0 + i);
   }
   if (turned)
     for (int i = threadIdx.x; i < half; i += NTHR) {
       const double two_pi = 6.283185307179586476925286766559, per_turn = 0.15915494309189533576888376337251;
-      const double ang = (double)p * a.freq[i];
+      const double ang = (double)p * (i < NTHR ? freq0 : a.freq[i]);
       float sn, c;
       sincosf((float)(ang - two_pi * rint(ang * per_turn)), &sn, &c);
       sm[2 * i] = c * a.amp;
@@ -209,9 +214,10 @@ __global__ void __launch_bounds__(NTHR) mixer_post_kernel(const __grid_constant_
 #pragma unroll
   for (int k = 0; k < PRE; ++k) {
     const int i = lo + (threadIdx.x + k * NTHR) * 4;
-    if (i < hi) keep(i, pre[k]);
+    if (i < hi) keep(i, add4(pre[k], pre_b[k]));
   }
-  for (int i = lo + (threadIdx.x + PRE * NTHR) * 4; i < hi; i += NTHR * 4) keep(i, biased(i));
+  for (int i = lo + (threadIdx.x + PRE * NTHR) * 4; i < hi; i += NTHR * 4)
+    keep(i, add4(load4(r.x, a.in_dtype, in0 + i), bias(i)));
   float inv_all = 1.f;
   if (norm == 2) inv_all = rsqrtf(block_sum(ss, red) / (float)all + a.eps);
   __syncthreads();
