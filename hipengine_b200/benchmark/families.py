@@ -4,9 +4,10 @@
     python -m hipengine_b200.benchmark.families [family] [--kernels-only | --models-only]
 
 Each kernel row gives the new design's kernel and the like kernel of the closest model (Sisisun beside the Qwen3-shaped
-dense / MoE decoder on the hybrid executor, Milutar and Banelix beside Sisisun, ``latent_rows.py`` and ``recurrent_rows.py``), their device times and the fraction of the measured peak that bounds them: HBM for the
-weight or KV streams (every format counts its own bytes), the bf16 tensor peak for the large products.  Operands are
-rotated through more than the L2 holds.  Weights are random.
+dense / MoE decoder on the hybrid executor, Milutar and Banelix beside Sisisun, ``latent_rows.py`` and
+``recurrent_rows.py``), their device times and the fraction of the measured peak that bounds them: HBM for the weight or KV
+streams (every format counts its own bytes), the bf16 tensor peak for the large products.  Operands are rotated through more
+than the L2 holds.  Weights are random.
 """
 from __future__ import annotations
 

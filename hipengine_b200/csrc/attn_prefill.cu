@@ -1,4 +1,4 @@
-// Causal paged GQA prefill attention (append-then-attend) with the fused sigmoid output gate.
+// Causal paged GQA prefill attention (append-then-attend) with the fused sigmoid output gate (per element, or per head) and sink.
 //
 // Flash-style single pass: a CTA owns 64 query rows of one head (4 warps x 16 rows), streams 32-key tiles of
 // K and V out of the paged cache with cp.async (double buffered), keeps running max / sum per row and the

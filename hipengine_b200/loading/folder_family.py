@@ -40,7 +40,7 @@ _SCALINGS = (BandSpec, ("factor", "low", "high", "original")), (YarnSpec, ("fact
 def rotary_from_json(r: Mapping[str, Any], halves: bool = False) -> RotarySpec:
     s, scaling = r.get("scaling"), None
     if s:
-        found = [c(*(float(s[k]) for k in keys)) for c, keys in _SCALINGS if set(keys) == set(s)]
+        found = [c(*(float(s[k]) for k in keys)) for c, keys in _SCALINGS if set(keys) <= set(s)]
         if not found:
             raise ValueError(f"unknown scaling of a rotation: {sorted(s)}")
         scaling = found[0]
