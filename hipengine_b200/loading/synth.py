@@ -98,6 +98,9 @@ def build_random_model(cfg: ModelConfig, seed: int = 0, device="cpu", recipe: st
     if cfg.arch == "banelix":
         from .banelix import build_random_banelix
         return build_random_banelix(cfg, seed=seed, device=device, std=std)
+    if cfg.arch == "mepatar":
+        from .mepatar import build_random_mepatar
+        return build_random_mepatar(cfg, seed=seed, device=device, std=std)
     b = _Builder(cfg, seed, device, recipe, std)
     base, hi = b.base_type(), b.hi_type()
     H = cfg.hidden

@@ -93,13 +93,16 @@ class AttentionSpec:
     scale: float
     softcap: float = 0.0                 # > 0: score <- softcap * tanh(score / softcap)
     rot: Optional[RotarySpec] = None     # of the first ``rot.dims`` dimensions of queries and keys
-    window: int = 0                      # > 0: only the last ``window`` positions are visible
+    window: int = 0                      # > 0: only the last ``window`` positions are visible ...
+    keep_first: int = 0                  # ... and the sequence's first ``keep_first`` ones
     sink_score: Optional[float] = None   # score of a term in the softmax denominator that has no value
     qk_norm: str = QK_NORM_HEAD
     bias: bool = False                   # of the query, key and value projections
     keys_as_values: bool = False         # the values are the projected keys, before norm and rotation
     head_gate: bool = False              # sigmoid(w_g . h) per head on the output
     kv_from: Optional[int] = None        # attends to the keys and values of this earlier layer and has none of its own
+    head_scale: bool = False             # a learned factor per head on the scores
+    out_bias: bool = False               # of the output projection
 
     @property
     def width(self) -> int:
@@ -122,8 +125,8 @@ class AttentionSpec:
             raise ValueError(f"rotation of {self.rot.dims} of {self.dim} dimensions")
         if self.keys_as_values and self.vdim != self.dim:
             raise ValueError(f"keys of {self.dim} dimensions as values of {self.vdim}")
-        if self.window < 0:
-            raise ValueError(f"window of {self.window}")
+        if self.window < 0 or self.keep_first < 0:
+            raise ValueError(f"window of {self.window}, {self.keep_first} first tokens kept")
         padded_head_width(max(self.dim, self.vdim))
 
 
@@ -231,6 +234,64 @@ class SideBySideSpec:
         self.right.check()
 
 
+# bounds of the linear attention kernels: key and value columns per head, taps of a convolution
+LINEAR_MAX_DIM = 512
+CONV_MAX_TAPS = 16
+
+
+@dataclass(frozen=True)
+class LinearAttentionSpec:
+    """Linear attention with a matrix state per head: S <- g S + k w^T, o = S^T q, o normalised per head and gated by silu.
+
+    ``decay`` given (retention): g is that constant per head, w the value, queries and keys are rotated.  Without it (gated
+    delta rule): g and a step size b come from the row, w = b (v - g S^T k), queries, keys and values pass a short causal
+    convolution and silu, queries and keys are unit vectors, the norm has gains."""
+    heads: int
+    kv_heads: int                        # query and key heads; head h uses number h // (heads / kv_heads)
+    dim: int
+    vdim: int
+    decay: Optional[Tuple[float, ...]] = None
+    rot: Optional[RotarySpec] = None
+    taps: int = 1                        # of the convolution
+
+    window = 0
+
+    @property
+    def delta(self) -> bool:
+        return self.decay is None
+
+    @property
+    def vcols(self) -> int:
+        """Value columns of a head, zero-padded."""
+        return round_up(self.vdim, 8)
+
+    @property
+    def conv_cols(self) -> int:
+        """Columns of the convolution: query, key and value rows, each zero-padded."""
+        return 2 * round_up(self.kv_heads * self.dim, 8) + round_up(self.heads * self.vdim, 8)
+
+    @property
+    def cache_elems(self) -> int:
+        return 0
+
+    @property
+    def state_elems(self) -> int:
+        """fp32 numbers a request carries: the matrices, and a ring of the convolution's last inputs."""
+        return self.heads * self.dim * self.vcols + (self.conv_cols * self.taps if self.delta and self.taps > 1 else 0)
+
+    def check(self) -> None:
+        if min(self.heads, self.kv_heads, self.dim, self.vdim) < 1 or self.heads % self.kv_heads:
+            raise ValueError(f"{self.heads} heads over {self.kv_heads} query/key heads, {self.dim} / {self.vdim} wide")
+        if max(self.dim, self.vdim) > LINEAR_MAX_DIM:
+            raise ValueError(f"heads of {self.dim} / {self.vdim} columns are above the widest supported one ({LINEAR_MAX_DIM})")
+        if not 1 <= self.taps <= CONV_MAX_TAPS:
+            raise ValueError(f"convolution of {self.taps} taps")
+        if self.decay is not None and (len(self.decay) != self.heads or min(self.decay) <= 0 or max(self.decay) > 1):
+            raise ValueError(f"decays {self.decay} of {self.heads} heads")
+        if self.rot is not None and not (self.rot.dims % 2 == 0 and 2 <= self.rot.dims <= self.dim):
+            raise ValueError(f"rotation of {self.rot.dims} of {self.dim} dimensions")
+
+
 @dataclass(frozen=True)
 class DenseMlpSpec:
     ff: int
@@ -247,23 +308,33 @@ class MoeMlpSpec:
     groups_kept: int = 1                 # ... of which only the best ones may be chosen from
     scale: float = 1.0                   # factor on the normalised routing weights
     shared_ff: int = 0                   # > 0: shared expert, scaled per token by sigmoid(w_sg . h)
+    score: str = "sigmoid"               # "sigmoid", normalised over the chosen experts | "softmax" over all, as it is
+    act: str = "silu"                    # of the experts, as in DenseMlpSpec
+    limit: float = 0.0
+
+    def check(self) -> None:
+        if min(self.experts, self.top, self.ff) < 1 or self.top > min(self.experts, 32) or self.experts > 512:
+            raise ValueError(f"top {self.top} of {self.experts} experts of {self.ff} columns (up to 32 of 512 are supported)")
 
 
 @dataclass(frozen=True)
 class LayerSpec:
-    mixer: Union[AttentionSpec, LatentAttentionSpec, SideBySideSpec]
+    mixer: Union[AttentionSpec, LatentAttentionSpec, SideBySideSpec, LinearAttentionSpec]
     mlp: Optional[Union[DenseMlpSpec, MoeMlpSpec]] = None
     parallel: bool = False               # both sublayers read one norm and are added together
     token_shift: bool = False            # the mixer reads a mix of this token's and the previous token's normalised row
+    input_taps: int = 1                  # > 1: a causal convolution of the normalised rows is added to what the mixer reads
 
     @property
-    def attention(self) -> Union[AttentionSpec, LatentAttentionSpec]:
-        """The part of the mixer that keeps a cache."""
+    def attention(self) -> Optional[Union[AttentionSpec, LatentAttentionSpec]]:
+        """The part of the mixer that keeps a cache, if there is one."""
+        if isinstance(self.mixer, LinearAttentionSpec):
+            return None
         return self.mixer.left if isinstance(self.mixer, SideBySideSpec) else self.mixer
 
     def state_elems(self, hidden: int) -> int:
         """fp32 numbers a request carries for one run of this layer besides its cache rows."""
-        return self.mixer.state_elems + (round_up(hidden, 8) if self.token_shift else 0)
+        return self.mixer.state_elems + round_up(hidden, 8) * (int(self.token_shift) + self.input_taps - 1)
 
 
 @dataclass(frozen=True)
@@ -323,6 +394,7 @@ class ModelConfig:
     layer_specs: Tuple[LayerSpec, ...] = ()
     loop: Optional[LoopSpec] = None
     residual_mult: float = 1.0           # factor on what a layer adds to the residual
+    norm_groups: int = 1                 # equal runs of channels that the norms of the residual are taken over
 
     # ---- derived
     def is_global_layer(self, i: int) -> bool:
@@ -641,6 +713,77 @@ BANELIX_8B = banelix_config(4096, 128256, tuple(
               if i % 4 == 3 else _BANELIX_8B_P, DenseMlpSpec(14336)) for i in range(24)), residual_mult=0.5, embed_scale=64.0)
 
 
+def mepatar_config(hidden: int, vocab: int, layers: Tuple[LayerSpec, ...], rms_eps: float = 1e-6, norm_groups: int = 1,
+                   embed_scale: float = 1.0, max_context: int = 262144) -> ModelConfig:
+    """``ModelConfig`` of a Mepatar model: parallel layers of two norms over groups of channels with an input convolution;
+    mixers are attention over a window and the first tokens, retention, or the gated delta rule."""
+    if not layers:
+        raise ValueError("a model needs layers")
+    if norm_groups < 1 or hidden % norm_groups:
+        raise ValueError(f"norm over {norm_groups} groups of {hidden} channels")
+    for i, l in enumerate(layers):
+        try:
+            l.mixer.check()
+            if not 1 <= l.input_taps <= CONV_MAX_TAPS:
+                raise ValueError(f"input convolution of {l.input_taps} taps")
+            if isinstance(l.mlp, MoeMlpSpec):
+                l.mlp.check()
+        except ValueError as e:
+            raise ValueError(f"layer {i}: {e}") from None
+    att = next((l.attention for l in layers if l.attention is not None), None)
+    m, rot = att or layers[0].mixer, next((l.mixer.rot for l in layers if l.mixer.rot is not None), None)
+    moe = [l.mlp for l in layers if isinstance(l.mlp, MoeMlpSpec)]
+    return ModelConfig(
+        arch="mepatar", n_layers=len(layers), hidden=hidden, vocab=vocab, n_heads=m.heads, n_kv_heads=m.kv_heads,
+        head_dim=m.dim, ffn=max([l.mlp.ff for l in layers if isinstance(l.mlp, DenseMlpSpec)], default=0), rms_eps=rms_eps,
+        rope_theta=rot.base if rot else 0.0, rope_dim=rot.dims if rot else 0, attn_scale=att.scale if att else None,
+        n_experts=max([e.experts for e in moe], default=0), n_experts_used=max([e.top for e in moe], default=0),
+        expert_ffn=max([e.ff for e in moe], default=0), embed_scale=embed_scale, layer_specs=tuple(layers),
+        norm_groups=norm_groups, max_context=max_context)
+
+
+def mepatar_attention(heads: int, kv_heads: int, dim: int, vdim: int, scale: float, window: int, keep_first: int,
+                      rot: RotarySpec) -> AttentionSpec:
+    return AttentionSpec(heads, kv_heads, dim, vdim, scale, rot=rot, window=window, keep_first=keep_first, bias=True,
+                         head_scale=True, out_bias=True)
+
+
+def mepatar_layer(mixer: Union[AttentionSpec, LinearAttentionSpec], mlp: Optional[Union[DenseMlpSpec, MoeMlpSpec]],
+                  taps: int) -> LayerSpec:
+    return LayerSpec(mixer, mlp, parallel=True, input_taps=taps)
+
+
+def mepatar_experts(experts: int, top: int, ff: int, limit: float) -> MoeMlpSpec:
+    return MoeMlpSpec(experts, top, ff, score="softmax", act="clamped_glu", limit=limit)
+
+
+# Small Mepatar geometry of the tests and the command line: every kind of layer, unequal widths, a layer without a
+# feed-forward.
+TINY_MEPATAR = mepatar_config(
+    208, 1024, (mepatar_layer(LinearAttentionSpec(4, 2, 40, 48, taps=4), DenseMlpSpec(232, "gelu_tanh"), 3),
+                mepatar_layer(mepatar_attention(6, 2, 48, 56, 0.14, 50, 6, RotarySpec(32, 20000.0)), mepatar_experts(12, 3, 72, 2.0), 3),
+                mepatar_layer(LinearAttentionSpec(3, 3, 56, 40, (0.97, 0.99, 0.998), RotarySpec(24, 5000.0, halves=True)),
+                              mepatar_experts(12, 3, 72, 2.0), 3),
+                mepatar_layer(LinearAttentionSpec(4, 2, 40, 48, taps=4), None, 3)),
+    rms_eps=1e-5, norm_groups=4, embed_scale=8.0, max_context=8192)
+
+# Geometry at the layer sizes of a deployed model, for throughput: an 8B-class width, a period of three delta, three retention
+# and two attention layers.
+_MEPATAR_8B_D = LinearAttentionSpec(32, 16, 128, 128, taps=4)
+_MEPATAR_8B_R = LinearAttentionSpec(32, 32, 128, 128, tuple(1.0 - 2.0 ** (-5 - 5 * h / 31) for h in range(32)),
+                                    RotarySpec(128, 1e6, halves=True))
+_MEPATAR_8B_A = mepatar_attention(32, 8, 128, 128, 128 ** -0.5, 4096, 128, RotarySpec(64, 50000.0))
+_MEPATAR_8B_PERIOD = (_MEPATAR_8B_D, _MEPATAR_8B_R, _MEPATAR_8B_D, _MEPATAR_8B_A, _MEPATAR_8B_D, _MEPATAR_8B_R, _MEPATAR_8B_R,
+                      _MEPATAR_8B_A)
+MEPATAR_8B = mepatar_config(4096, 128256, tuple(mepatar_layer(m, DenseMlpSpec(14336, "gelu_tanh"), 4)
+                                                for m in _MEPATAR_8B_PERIOD * 3), norm_groups=8, embed_scale=64.0)
+# ... and a 30B-A3B-class mixture
+MEPATAR_30B_MOE = mepatar_config(2048, 151936, tuple(
+    mepatar_layer(m, mepatar_experts(128, 8, 768, 7.0), 4) for m in (
+        LinearAttentionSpec(32, 16, 128, 128, taps=4), _MEPATAR_8B_R, LinearAttentionSpec(32, 16, 128, 128, taps=4),
+        mepatar_attention(32, 4, 128, 128, 128 ** -0.5, 4096, 128, RotarySpec(64, 50000.0))) * 12), norm_groups=4, embed_scale=45.0)
+
+
 @dataclass(frozen=True)
 class AssistantConfig:
     """Gemma 4 assistant (MTP) head: a separate four-block draft model with no K/V projections of its own.  Every
@@ -712,4 +855,7 @@ NAMED_CONFIGS: Dict[str, ModelConfig] = {
     "milutar-8b": MILUTAR_8B,
     "tiny-banelix": TINY_BANELIX,
     "banelix-8b": BANELIX_8B,
+    "tiny-mepatar": TINY_MEPATAR,
+    "mepatar-8b": MEPATAR_8B,
+    "mepatar-30b-moe": MEPATAR_30B_MOE,
 }

@@ -10,7 +10,7 @@ from __future__ import annotations
 from dataclasses import dataclass
 from typing import Any, Dict, List, Optional, Tuple
 
-from .config import ModelConfig, MoeMlpSpec, SideBySideSpec
+from .config import LinearAttentionSpec, ModelConfig, MoeMlpSpec, SideBySideSpec
 
 
 @dataclass(frozen=True)
@@ -34,13 +34,15 @@ class ModelPlugin:
     notes: str = ""
 
     def layer_sequence(self, cfg: ModelConfig) -> List[str]:
-        """One word per layer of ``cfg``: ``linear`` (Gated-DeltaNet), ``full``, ``sliding`` or ``global``; with
+        """One word per layer of ``cfg``: ``linear`` (Gated-DeltaNet), ``retention``, ``full``, ``sliding`` or ``global``; with
         ``+recurrent`` where a recurrence runs beside the attention."""
         out = []
         for i in range(cfg.n_layers):
             if cfg.layer_specs:
                 m = cfg.layer_specs[i].mixer
                 word = "sliding" if getattr(m, "window", 0) else "full"
+                if isinstance(m, LinearAttentionSpec):
+                    word = "linear" if m.delta else "retention"
                 out.append(word + "+recurrent" if isinstance(m, SideBySideSpec) else word)
             elif cfg.arch == "gemma4":
                 out.append("global" if cfg.is_global_layer(i) else "sliding")
@@ -120,6 +122,18 @@ PLUGINS: Tuple[ModelPlugin, ...] = (
                       "attend to an earlier layer's keys and values), or attention over unit keys whose values are the plain "
                       "keys beside a real-gated linear recurrence; dense SiLU feed-forward or none; checkpoints are folders "
                       "with config.json and model.safetensors"),
+    ModelPlugin("mepatar", ("mepatar",), "hipengine_b200.models.mepatar.MepatarExecutor", default_quant="bf16",
+                native_block_types=("BF16",), widened_block_types=(), kv_storage=("bf16", "f32"),
+                tensor_parallel=False, compute_dtypes=("bfloat16", "float32"),
+                native_sources=("attn_decode.cu", "attn_prefill.cu", "exact_f32.cu", "gemm_sm100.cu", "gemv_float.cu",
+                                "layers.cu", "linear_attn.cu", "mixer_post.cu", "moe.cu", "norm_conv.cu",
+                                "quant_util.cu", "runtime.cpp", "sampling.cu"),
+                folder_architecture="Mepatar", folder_reader="hipengine_b200.loading.mepatar",
+                reference="hipengine_b200.ref.mepatar.MepatarRef",
+                notes="layers listed one by one, mixer and feed-forward side by side under grouped norms, a convolution ahead of "
+                      "the mixer; mixers: attention over a window and the sequence's first tokens, retention, gated delta rule; "
+                      "feed-forwards: dense, softmax-routed clamped experts or none; checkpoints are folders with config.json "
+                      "and model.safetensors"),
 )
 
 
