@@ -25,7 +25,7 @@ struct AttnDecArgs {
   __nv_bfloat16* out;         // [R][H*D]
   int R, H, Hkv, D, page, max_pages;
   int split_len, max_splits;
-  int window;                 // > 0: only the last `window` keys are visible
+  int window;                 // > 0: only the last `window` keys are visible ...
   float scale;
   int* status;                // optional status word: a bounded wait that gave up records its code here
   float softcap;              // > 0: score <- softcap * tanh(score / softcap), after the scale
@@ -33,11 +33,24 @@ struct AttnDecArgs {
   const void* head_gate;      // [R][head_gate_stride] or null: head h's output is multiplied by sigmoid(head_gate[r][h])
   long long head_gate_stride;
   int head_gate_dtype;        // 0 f32, 1 bf16
+  int keep_first;             // ... and the first `keep_first` ones of the sequence
 };
 
 namespace {
 
 constexpr int NWARP = 8;
+
+// The visible keys of a row in order: the kept first ones that its window has left behind, then the window.
+struct Visible {
+  int first, skip, n;         // key i of n sits at position i, from `first` on at i + skip
+  __device__ __forceinline__ Visible(const AttnDecArgs& a, int ctx) {
+    const int start = (a.window > 0 && ctx > a.window) ? ctx - a.window : 0;
+    first = min(a.keep_first, start);
+    skip = start - first;
+    n = ctx - skip;
+  }
+  __device__ __forceinline__ int pos(int i) const { return i < first ? i : i + skip; }
+};
 
 template <int D, int G>
 __global__ void __launch_bounds__(256) attn_decode_split_kernel(const AttnDecArgs a) {
@@ -45,11 +58,10 @@ __global__ void __launch_bounds__(256) attn_decode_split_kernel(const AttnDecArg
   const int sp = blockIdx.x, hk = blockIdx.y, r = blockIdx.z;
   pdl_wait();
   pdl_launch();
-  const int ctx = a.ctx_len[r];
-  const int start = (a.window > 0 && ctx > a.window) ? ctx - a.window : 0;
-  const int k0 = start + sp * a.split_len;
-  if (k0 >= ctx) return;
-  const int n = min(a.split_len, ctx - k0);
+  const Visible vis(a, a.ctx_len[r]);
+  const int k0 = sp * a.split_len;
+  if (k0 >= vis.n) return;
+  const int n = min(a.split_len, vis.n - k0);
   float* q_s = smem;                       // [G][D]
   float* sc = q_s + G * D;                 // [G][split_len]
   float* red = sc + G * a.split_len;       // [NWARP][G][D]
@@ -72,7 +84,7 @@ __global__ void __launch_bounds__(256) attn_decode_split_kernel(const AttnDecArg
 #pragma unroll
       for (int g = 0; g < G; ++g) acc[g] = 0.f;
       if (tk < n) {
-        const int pos = k0 + tk;
+        const int pos = vis.pos(k0 + tk);
         const int pg = bt[HE_INDEX_OK(pos / a.page, a.max_pages, HE_SITE_ATTN_DECODE_PAGE) ? pos / a.page : 0];
         const __nv_bfloat16* kr = a.kv_cache + ((((size_t)pg * 2 + 0) * a.Hkv + hk) * a.page + (pos % a.page)) * D;
 #pragma unroll
@@ -143,7 +155,7 @@ __global__ void __launch_bounds__(256) attn_decode_split_kernel(const AttnDecArg
   for (int t0 = warp * TPS; t0 < n; t0 += NWARP * TPS) {
     const int tk = t0 + tgrp;
     if (tk < n) {
-      const int pos = k0 + tk;
+      const int pos = vis.pos(k0 + tk);
       const int pg = bt[HE_INDEX_OK(pos / a.page, a.max_pages, HE_SITE_ATTN_DECODE_PAGE) ? pos / a.page : 0];
       const __nv_bfloat16* vr = a.kv_cache + ((((size_t)pg * 2 + 1) * a.Hkv + hk) * a.page + (pos % a.page)) * D;
       float p[G];
@@ -274,11 +286,10 @@ __global__ void __launch_bounds__(NTHREADS) attn_decode_mma_kernel(const AttnDec
   const int G = GT > 0 ? GT : gc;
   pdl_wait();
   pdl_launch();
-  const int ctx = a.ctx_len[r];
-  const int start = (a.window > 0 && ctx > a.window) ? ctx - a.window : 0;
-  const int k0 = start + sp * a.split_len;
-  if (k0 >= ctx) return;
-  const int n = min(a.split_len, ctx - k0);
+  const Visible vis(a, a.ctx_len[r]);
+  const int k0 = sp * a.split_len;
+  if (k0 >= vis.n) return;
+  const int n = min(a.split_len, vis.n - k0);
   const int ntile = (n + TILE_KEYS - 1) / TILE_KEYS;
   const int NST = stages_for<D>(a.split_len);
   const int PP = a.split_len * 2 + 16;                 // pitch of a P row (bytes)
@@ -315,7 +326,7 @@ __global__ void __launch_bounds__(NTHREADS) attn_decode_mma_kernel(const AttnDec
       for (int h2 = 0; h2 < TILE_KEYS / 32; ++h2) {
         const int row = lane + 32 * h2;
         // rows past the span re-read its last key: finite values that the zero probabilities then ignore
-        const int pos = k0 + min(tile * TILE_KEYS + row, n - 1);
+        const int pos = vis.pos(k0 + min(tile * TILE_KEYS + row, n - 1));
         const int pg = bt[HE_INDEX_OK(pos / a.page, a.max_pages, HE_SITE_ATTN_DECODE_PAGE) ? pos / a.page : 0];
         const __nv_bfloat16* src =
             a.kv_cache + ((((size_t)pg * 2 + kv) * a.Hkv + hk) * a.page + (pos % a.page)) * D;
@@ -476,11 +487,10 @@ __global__ void attn_decode_reduce_kernel(const AttnDecArgs a) {
   const int D = a.D;
   pdl_wait();
   pdl_launch();
-  const int ctx = a.ctx_len[r];
-  const int start = (a.window > 0 && ctx > a.window) ? ctx - a.window : 0;
+  const Visible vis(a, a.ctx_len[r]);
   // never past what the split kernel wrote (its grid is max_splits wide) nor past wsm[]: a context longer than
   // split_len * max_splits is the caller's error and is reduced over the first max_splits splits only
-  const int ns = min((ctx - start + a.split_len - 1) / a.split_len, a.max_splits);
+  const int ns = min((vis.n + a.split_len - 1) / a.split_len, a.max_splits);
   const float* pb = a.partial + ((size_t)r * a.H + h) * a.max_splits * (D + 2);
   float m = -INFINITY;
   for (int s = d; s < ns; s += blockDim.x) {

@@ -5,7 +5,7 @@
 // 16 x D output accumulator in registers.  Tensor-core path: mma.sync m16n8k16 bf16 with fp32 accumulation
 // (the projections, which are >98% of prefill FLOPs, run on tcgen05; this kernel is bounded by the softmax
 // pipeline, not by the MMA rate).  The queries of one segment sit at consecutive positions
-// pos0 .. pos0+T-1 and attend keys 0 .. their own position (optionally only the last `window` keys).
+// pos0 .. pos0+T-1 and attend keys 0 .. their own position (optionally only the last `window` keys and the first `keep` ones).
 // Behavioural reference: hipengine/kernels/hip_gfx1100/attention/paged_attn_decode.hip (prefill_gqa_gate_*
 // kernels) and the oracle hipengine/kernels/cpu_reference/ops.py:2144-2256 (output rounded to bf16 before the
 // gate multiply).
@@ -38,6 +38,7 @@ struct PrefillArgs {
   const void* head_gate;       // [T][head_gate_stride] or null: head h's output is multiplied by sigmoid(head_gate[t][h])
   long long head_gate_stride;
   int head_gate_dtype;         // 0 f32, 1 bf16
+  int keep;                    // with a window: keys [0, keep) stay visible
 };
 
 __device__ __forceinline__ void cp_async16(void* smem, const void* gmem, bool valid) {
@@ -106,10 +107,13 @@ __global__ void __launch_bounds__(NTHR) flash_prefill_kernel(const PrefillArgs a
   const int kv_end = q_pos_last + 1;                                   // keys [0, kv_end)
   int kv_begin = 0;
   if (a.window > 0) kv_begin = max(0, a.pos0 + t0 - a.window + 1) / BN * BN;
-  const int n_tiles = (kv_end - kv_begin + BN - 1) / BN;
+  // kept first keys that lie before the window's first tile come ahead of it, in tiles of their own
+  const int n_kept = (min(a.keep, kv_begin) + BN - 1) / BN;
+  const int n_tiles = n_kept + (kv_end - kv_begin + BN - 1) / BN;
+  const auto first_key = [&](int tile) { return tile < n_kept ? tile * BN : kv_begin + (tile - n_kept) * BN; };
 
   auto load_kv = [&](int tile, int buf) {
-    const int k0 = kv_begin + tile * BN;
+    const int k0 = first_key(tile);
     constexpr int CH = D / 8;                                          // 16-byte chunks per row
     for (int i = tid; i < BN * CH; i += NTHR) {
       const int r = i / CH, ch = i % CH;
@@ -171,7 +175,7 @@ __global__ void __launch_bounds__(NTHR) flash_prefill_kernel(const PrefillArgs a
     }
 
     // ---- mask + online softmax (rows g and g+8 of this warp's 16)
-    const int k0 = kv_begin + tile * BN;
+    const int k0 = first_key(tile);
     float mx[2] = {-INFINITY, -INFINITY};
     if constexpr (CAP) {
       // soft cap: the power series when every score of the warp's tile is small against the cap, else the quotient form
@@ -203,7 +207,7 @@ __global__ void __launch_bounds__(NTHR) flash_prefill_kernel(const PrefillArgs a
         const int key = k0 + j * 8 + 2 * c + (e & 1);
         const int qp = qrow0 + (e >> 1) * 8;
         bool ok = key <= qp && key < kv_end;
-        if (a.window > 0) ok = ok && key > qp - a.window;
+        if (a.window > 0) ok = ok && (key > qp - a.window || key < a.keep);
         const float v = ok ? sacc[j][e] * sc_log2 : -INFINITY;
         sacc[j][e] = v;
         mx[e >> 1] = fmaxf(mx[e >> 1], v);
@@ -328,7 +332,7 @@ HE_API int he_flash_prefill_segs(const void* q, const void* gate, const void* kv
                                  int max_pages, const int* seg_start, const int* seg_slot, const int* pos, int n_seg,
                                  int tiles, void* out, int H, int Hkv, int D, int page, float scale, int window,
                                  float softcap, const float* sink, const void* head_gate, long long head_gate_stride,
-                                 int head_gate_dtype, cudaStream_t stream) {
+                                 int head_gate_dtype, int keep_first, cudaStream_t stream) {
   if (n_seg <= 0 || tiles <= 0) return 0;
   if (H % Hkv != 0 || seg_start == nullptr || seg_slot == nullptr || pos == nullptr) return -HE_ERR_BAD_ARG;
   PrefillArgs a = {};
@@ -337,6 +341,7 @@ HE_API int he_flash_prefill_segs(const void* q, const void* gate, const void* kv
   a.H = H; a.Hkv = Hkv; a.page = page; a.window = window;
   a.seg_start = seg_start; a.seg_slot = seg_slot; a.pos = pos; a.n_seg = n_seg; a.max_pages = max_pages;
   a.sink = sink; a.head_gate = head_gate; a.head_gate_stride = head_gate_stride; a.head_gate_dtype = head_gate_dtype;
+  a.keep = window > 0 ? keep_first : 0;
   a.scale_log2 = scale * 1.4426950408889634f;
   if (softcap > 0.f) {
     a.cap_in = scale / softcap;

@@ -18,6 +18,7 @@ struct ExactAttnArgs {
   const float* sink;         // [H] or null: score of one more term in the softmax denominator
   const float* head_gate;    // [R][head_gate_stride] or null: outputs times sigmoid(head_gate[r][h])
   long long head_gate_stride;
+  int keep_first;            // with a window: the first `keep_first` keys stay visible
 };
 
 struct ExactMoeArgs {
@@ -34,6 +35,8 @@ struct ExactMoeArgs {
   float* rows_s;             // [T][Fs]
   float* h;
   long long ldh;
+  int act;                   // 0 SiLU, 2 clamped GLU
+  float limit;
 };
 
 namespace {
@@ -58,7 +61,9 @@ __global__ void __launch_bounds__(AW * 32) attn_exact_kernel(const ExactAttnArgs
     o[i] = 0.f;
   }
   float m = -INFINITY, l = 0.f;
-  for (int p = (a.window > 0 && ctx > a.window ? ctx - a.window : 0) + warp; p < ctx; p += AW) {
+  const int start = a.window > 0 && ctx > a.window ? ctx - a.window : 0, kept = min(a.keep_first, start);
+  for (int i = warp; i < ctx - start + kept; i += AW) {
+    const int p = i < kept ? i : i - kept + start;
     const int pg = bt[HE_INDEX_OK(p / a.page, a.max_pages, HE_SITE_ATTN_DECODE_PAGE) ? p / a.page : 0];
     const float* kr = a.kv_cache + (((size_t)pg * 2 * a.Hkv + hk) * a.page + p % a.page) * D;
     const float* vr = kr + (size_t)a.Hkv * a.page * D;
@@ -121,7 +126,13 @@ __global__ void __launch_bounds__(256) moe_gateup_exact_kernel(const ExactMoeArg
   const float g = dot_row(base + (size_t)n * a.K, x, a.K, lane), u = dot_row(base + (size_t)(F + n) * a.K, x, a.K, lane);
   if (lane != 0) return;
   const float wt = shared ? (a.sg != nullptr ? sigmoid_exact(a.sg[(size_t)t * a.ld_sg]) : 1.f) : a.wts[p];
-  const float v = g * sigmoid_exact(g) * u * wt;
+  float v;
+  if (a.act == 2) {
+    const float gc = fminf(g, a.limit);
+    v = gc * sigmoid_exact(1.702f * gc) * (fminf(fmaxf(u, -a.limit), a.limit) + 1.f) * wt;
+  } else {
+    v = g * sigmoid_exact(g) * u * wt;
+  }
   if (shared) a.rows_s[(size_t)t * F + n] = v;
   else a.rows[(size_t)p * F + n] = v;
 }
@@ -162,6 +173,7 @@ HE_API int he_exact_attn_args_size() { return (int)sizeof(ExactAttnArgs); }
 HE_API int he_moe_gateup_exact(const ExactMoeArgs* args, cudaStream_t stream) {
   const ExactMoeArgs& a = *args;
   if (a.T <= 0) return 0;
+  if (a.act != 0 && a.act != 2) return -HE_ERR_BAD_ARG;
   const int F = a.w1s != nullptr && a.Fs > a.F ? a.Fs : a.F;
   const dim3 grid(a.T * a.k + (a.w1s != nullptr ? a.T : 0), (F + 7) / 8);
   return (int)launch_pdl(moe_gateup_exact_kernel, grid, dim3(256), 0, stream, a);

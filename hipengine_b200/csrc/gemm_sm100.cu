@@ -49,6 +49,7 @@ struct GemmArgs {
   void* C;
   long long ldc;        // elements
   const float* col_scale;   // epi 2: factor per output column, or null
+  const float* col_bias;    // epi 2: added per output column (not scaled), or null
   int M, N, K;
   int epi;              // 0: bf16 store, 1: fp32 store, 2: fp32 += (C is fp32, in place), 6: bf16 store of relu(v)^2
   int* status;
@@ -493,6 +494,13 @@ __device__ __forceinline__ void store_tile(const GemmArgs& g, uint8_t* stage, ui
           if (left > 2) sc.z = __ldg(g.col_scale + col + 2);
           if (left > 3) sc.w = __ldg(g.col_scale + col + 3);
         }
+        float4 bi = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (g.epi == 2 && g.col_bias != nullptr) {
+          bi.x = __ldg(g.col_bias + col);
+          if (left > 1) bi.y = __ldg(g.col_bias + col + 1);
+          if (left > 2) bi.z = __ldg(g.col_bias + col + 2);
+          if (left > 3) bi.w = __ldg(g.col_bias + col + 3);
+        }
         float4 old[8];
         if (g.epi == 2 && vec) {
 #pragma unroll
@@ -506,7 +514,7 @@ __device__ __forceinline__ void store_tile(const GemmArgs& g, uint8_t* stage, ui
           const int rl = it * 4 + rq, row = row0 + rl;
           if (row >= g.M) break;
           float4 v = *reinterpret_cast<const float4*>(stage + rl * 128 + ((ch ^ (rl & 7)) << 4));
-          v.x *= sc.x; v.y *= sc.y; v.z *= sc.z; v.w *= sc.w;
+          v.x = v.x * sc.x + bi.x; v.y = v.y * sc.y + bi.y; v.z = v.z * sc.z + bi.z; v.w = v.w * sc.w + bi.w;
           float* dst = base + (size_t)row * g.ldc;
           if (g.epi == 3) {
             if (!empty_split) {
@@ -927,10 +935,12 @@ constexpr size_t SMEM_Q = STAGES_Q * STAGE_BYTES + QSTAGES * Q_STAGE_BYTES + siz
 }  // namespace
 
 // C[M][N] = A[M][K] (bf16, row stride lda) * B[N][K]^T (bf16, row stride ldb).
-// epi: 0 bf16 store, 1 fp32 store, 2 fp32 accumulate into C (times col_scale[n] when given), 6 bf16 store of relu(v)^2.
+// epi: 0 bf16 store, 1 fp32 store, 2 fp32 accumulate into C (times col_scale[n], plus col_bias[n] when given), 6 bf16 store of
+// relu(v)^2.
 // `status` (device int, may be null) receives a non-zero code if a bounded wait inside the kernel gave up.
 HE_API int he_gemm_bf16(const void* A, long long lda, const void* B, long long ldb, void* C, long long ldc, int M,
-                        int N, int K, int epi, const void* col_scale, void* status, int num_sms, cudaStream_t stream) {
+                        int N, int K, int epi, const void* col_scale, const void* col_bias, void* status, int num_sms,
+                        cudaStream_t stream) {
   if (M <= 0 || N <= 0 || K <= 0) return 0;
   if (K % 8 != 0 || !(epi == 0 || epi == 1 || epi == 2 || epi == 6)) return -HE_ERR_BAD_ARG;
   CUtensorMap tmA, tmB;
@@ -940,6 +950,7 @@ HE_API int he_gemm_bf16(const void* A, long long lda, const void* B, long long l
   if (rc != 0) return rc;
   GemmArgs g = {};
   g.C = C; g.ldc = ldc; g.col_scale = (const float*)col_scale; g.M = M; g.N = N; g.K = K; g.epi = epi; g.status = (int*)status;
+  g.col_bias = (const float*)col_bias;
   g.tile_group = nullptr;
   g.k_splits = 1;
   g.split_stride = 0;
@@ -1036,10 +1047,10 @@ HE_API int he_gemm_bf16_grouped(const void* A, long long lda, const void* B, lon
 // residual stream).  k_splits <= 0 picks a split that gives about one tile per SM.
 namespace {
 // out[m][n] (+)= sum over splits, in split order (deterministic).  mode 0: fp32 store, 1: fp32 add in place (of the sum
-// times col_scale[n] when given), 2: bf16 store of relu(sum)^2.
+// times col_scale[n], plus col_bias[n] when given), 2: bf16 store of relu(sum)^2.
 __global__ void splitk_reduce_kernel(const float* __restrict__ part, long long split_stride, int k_splits,
                                      void* __restrict__ out_v, long long ldo, int M, int N, int mode,
-                                     const float* __restrict__ col_scale) {
+                                     const float* __restrict__ col_scale, const float* __restrict__ col_bias) {
   const long long i = ((long long)blockIdx.x * blockDim.x + threadIdx.x) * 4;
   if (i >= (long long)M * N) return;
   const int m = (int)(i / N), n = (int)(i % N);
@@ -1061,6 +1072,10 @@ __global__ void splitk_reduce_kernel(const float* __restrict__ part, long long s
       const float4 c = *reinterpret_cast<const float4*>(col_scale + n);
       s.x *= c.x; s.y *= c.y; s.z *= c.z; s.w *= c.w;
     }
+    if (col_bias != nullptr) {
+      const float4 c = *reinterpret_cast<const float4*>(col_bias + n);
+      s.x += c.x; s.y += c.y; s.z += c.z; s.w += c.w;
+    }
     const float4 h = *o;
     s.x += h.x; s.y += h.y; s.z += h.z; s.w += h.w;
   }
@@ -1070,7 +1085,7 @@ __global__ void splitk_reduce_kernel(const float* __restrict__ part, long long s
 
 // Deterministic split-K: partial tiles go to `partials` ([k_splits][M][N] fp32, caller scratch of at least
 // he_gemm_splitk_scratch_floats(M, N, K) floats), then one pass sums them in split order into `out`
-// (mode 0: store, 1: add in place -- the residual add, with an optional factor per column --, 2: bf16 squared ReLU).  Same
+// (mode 0: store, 1: add in place -- the residual add, with an optional factor and bias per column --, 2: bf16 squared ReLU).  Same
 // use as he_gemm_bf16_splitk, bit-reproducible.
 HE_API long long he_gemm_splitk_plan(int M, int N, int K, int num_sms) {
   const int tiles = ((M + BM - 1) / BM) * ((N + BN - 1) / BN);
@@ -1084,7 +1099,7 @@ HE_API long long he_gemm_splitk_plan(int M, int N, int K, int num_sms) {
 
 HE_API int he_gemm_bf16_splitk_det(const void* A, long long lda, const void* B, long long ldb, void* partials,
                                    void* out, long long ldo, int M, int N, int K, int mode, const void* col_scale,
-                                   void* status, int num_sms, cudaStream_t stream) {
+                                   const void* col_bias, void* status, int num_sms, cudaStream_t stream) {
   if (M <= 0 || N <= 0 || K <= 0) return 0;
   if (K % 8 != 0 || N % 4 != 0 || mode < 0 || mode > 2) return -HE_ERR_BAD_ARG;
   CUtensorMap tmA, tmB;
@@ -1108,7 +1123,7 @@ HE_API int he_gemm_bf16_splitk_det(const void* A, long long lda, const void* B, 
   const long long n4 = ((long long)M * N + 3) / 4;
   splitk_reduce_kernel<<<(unsigned)((n4 + 255) / 256), 256, 0, stream>>>((const float*)partials, g.split_stride,
                                                                         k_splits, out, ldo, M, N, mode,
-                                                                        (const float*)col_scale);
+                                                                        (const float*)col_scale, (const float*)col_bias);
   HE_LAUNCH_CHECK();
   return 0;
 }

@@ -49,7 +49,7 @@ struct FloatGemvArgs {
   long long w_bs, x_bs, out_bs;
 };
 
-struct FloatSumArgs {        // out[r][n] += sum over i of scale_i[n] * (x_i[r] . w_i[n]),  bf16 rows and weights
+struct FloatSumArgs {        // out[r][n] += bias[n] + sum over i of scale_i[n] * (x_i[r] . w_i[n]),  bf16 rows and weights
   const __nv_bfloat16* w[2];
   const __nv_bfloat16* x[2];
   const float* scale[2];     // null: 1
@@ -58,10 +58,11 @@ struct FloatSumArgs {        // out[r][n] += sum over i of scale_i[n] * (x_i[r] 
   float* out;
   long long out_stride;
   int n_rows, R;
+  const float* bias;         // [n_rows] added as well, or null
 };
 
 struct FloatMoeArgs {
-  const void* x;             // gate/up: fp32 residual rows [T][ldx]
+  const void* x;             // gate/up: rows [T][ldx], fp32 (with norm_w: residual rows) or bf16
   long long ldx;
   const float* norm_w;
   float eps;
@@ -79,6 +80,7 @@ struct FloatMoeArgs {
   __nv_bfloat16* rows_s;     // [T][Fs] activations of the shared expert, gate folded in
   float* h;                  // down: residual rows, added in place
   long long ldh;
+  int x_dtype;               // 0 f32, 1 bf16
 };
 
 namespace {
@@ -335,11 +337,13 @@ __global__ void __launch_bounds__(NW * 32, 2) gemv_sum_kernel(const __grid_const
   __syncthreads();
   for (int o = threadIdx.x; o < 16 * NT * 8; o += NW * 32) {
     const int row = o & 15, col = o >> 4, n = row0 + row;
-    if (col < a.R && n < a.n_rows) a.out[(size_t)col * a.out_stride + n] += sum_partials<1, NT>(sm, row, col);
+    if (col < a.R && n < a.n_rows)
+      a.out[(size_t)col * a.out_stride + n] += sum_partials<1, NT>(sm, row, col) + (a.bias != nullptr ? a.bias[n] : 0.f);
   }
 }
 
 // grid (ceil(max(F, Fs) / 16), T * k [+ T]): activation rows of the selected experts, then of the shared expert
+template <bool XF32>
 __global__ void __launch_bounds__(NW * 32, 2) moe_gateup_float_kernel(const __grid_constant__ FloatMoeArgs a) {
   __shared__ Tile<2, 1> sm;
   pdl_launch();
@@ -363,8 +367,8 @@ __global__ void __launch_bounds__(NW * 32, 2) moe_gateup_float_kernel(const __gr
   }
   float acc[2][1][4] = {};
   float ss[1] = {};
-  product<2, 1, true, false>(wrow, a.K, reinterpret_cast<const float*>(a.x) + (size_t)t * a.ldx, a.ldx, 1, a.norm_w, acc,
-                             ss);
+  const char* x = reinterpret_cast<const char*>(a.x) + (size_t)t * a.ldx * (XF32 ? 4 : 2);
+  product<2, 1, XF32, false>(wrow, a.K, x, a.ldx, 1, a.norm_w, acc, ss);
   store_partials<2, 1>(sm, acc, ss);
   __syncthreads();
   const int row = threadIdx.x, n = row0 + row;
@@ -569,10 +573,13 @@ static int check_moe(const FloatMoeArgs& a) {
 HE_API int he_moe_gateup_float(const FloatMoeArgs* args, cudaStream_t stream) {
   const FloatMoeArgs& a = *args;
   if (a.T <= 0) return 0;
-  if (check_moe(a) != 0 || a.K % 8 != 0 || a.ldx % 8 != 0 || a.act < 3 || a.act > 5) return -HE_ERR_BAD_ARG;
+  if (check_moe(a) != 0 || a.K % 8 != 0 || a.ldx % 8 != 0 || a.act < 3 || a.act > 5 ||
+      (a.x_dtype != 0 && a.norm_w != nullptr))
+    return -HE_ERR_BAD_ARG;
   const int F = a.w1s != nullptr && a.Fs > a.F ? a.Fs : a.F;
   const dim3 grid((F + 15) / 16, a.T * a.k + (a.w1s != nullptr ? a.T : 0));
-  return (int)launch_pdl(moe_gateup_float_kernel, grid, dim3(NW * 32), 0, stream, a);
+  return (int)(a.x_dtype == 0 ? launch_pdl(moe_gateup_float_kernel<true>, grid, dim3(NW * 32), 0, stream, a)
+                              : launch_pdl(moe_gateup_float_kernel<false>, grid, dim3(NW * 32), 0, stream, a));
 }
 
 HE_API int he_moe_down_float(const FloatMoeArgs* args, cudaStream_t stream) {

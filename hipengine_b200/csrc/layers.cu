@@ -616,7 +616,7 @@ HE_API int he_advance_positions(void* pos, void* ctx_len, const void* active, in
 // ---------------------------------------------------------------- skinny fp32 GEMM: out[T][N] = x[T][K] * W[N][K]^T
 // For the few projections whose weights stay F32 in GGUF files (router, ssm_alpha/beta) at prefill row counts, and every
 // projection of the float32 compute dtype.  grid.z repeats the product at the batch strides (one matrix per head).
-// mode 0: store, 1: add (times col_scale[n] when given), 2: store relu(v)^2.
+// mode 0: store, 1: add (times col_scale[n], or plus col_bias[n], when given), 2: store relu(v)^2.
 namespace {
 constexpr int SG_TM = 64, SG_TN = 64, SG_TK = 16;
 __global__ void __launch_bounds__(256) small_gemm_f32_kernel(const void* __restrict__ x, int x_dtype,
@@ -624,7 +624,8 @@ __global__ void __launch_bounds__(256) small_gemm_f32_kernel(const void* __restr
                                                              int w_dtype, long long w_stride,
                                                              float* __restrict__ out, long long out_stride, int T,
                                                              int N, int K, int mode,
-                                                             const float* __restrict__ col_scale, long long x_bs,
+                                                             const float* __restrict__ col_scale,
+                                                             const float* __restrict__ col_bias, long long x_bs,
                                                              long long w_bs, long long out_bs) {
   __shared__ float xs[SG_TK][SG_TM + 1];
   __shared__ float ws[SG_TK][SG_TN + 1];
@@ -664,7 +665,7 @@ __global__ void __launch_bounds__(256) small_gemm_f32_kernel(const void* __restr
       const int t = t0 + ty * 4 + i, n = n0 + tx * 4 + j;
       if (t < T && n < N) {
         float* o = out + (size_t)t * out_stride + n;
-        const float v = acc[i][j];
+        const float v = acc[i][j] + (mode == 1 && col_scale == nullptr && col_bias != nullptr ? col_bias[n] : 0.f);
         *o = mode == 1 ? *o + (col_scale != nullptr ? v * col_scale[n] : v) : mode == 2 ? relu2_f(v) : v;
       }
     }
@@ -673,13 +674,13 @@ __global__ void __launch_bounds__(256) small_gemm_f32_kernel(const void* __restr
 
 HE_API int he_small_gemm_f32(const void* x, int x_dtype, long long x_stride, const void* w, int w_dtype,
                              long long w_stride, void* out, long long out_stride, int T, int N, int K, int mode,
-                             const void* col_scale, int n_batch, long long x_bs, long long w_bs, long long out_bs,
+                             const void* col_scale, const void* col_bias, int n_batch, long long x_bs, long long w_bs, long long out_bs,
                              cudaStream_t stream) {
   if (T <= 0 || N <= 0) return 0;
-  if (mode < 0 || mode > 2 || n_batch < 1 || n_batch > 65535) return -HE_ERR_BAD_ARG;
+  if (mode < 0 || mode > 2 || n_batch < 1 || n_batch > 65535 || (col_scale != nullptr && col_bias != nullptr)) return -HE_ERR_BAD_ARG;
   dim3 grid((N + SG_TN - 1) / SG_TN, (T + SG_TM - 1) / SG_TM, n_batch);
   small_gemm_f32_kernel<<<grid, 256, 0, stream>>>(x, x_dtype, x_stride, w, w_dtype, w_stride, (float*)out, out_stride, T,
-                                                  N, K, mode, (const float*)col_scale, x_bs, w_bs, out_bs);
+                                                  N, K, mode, (const float*)col_scale, (const float*)col_bias, x_bs, w_bs, out_bs);
   HE_LAUNCH_CHECK();
   return 0;
 }

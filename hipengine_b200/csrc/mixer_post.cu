@@ -16,8 +16,8 @@ struct HeadRows {
   const void* x;             // [T][stride], null: none
   long long stride;          // multiple of 8, as is the column the rows start at; columns are zero-padded to a multiple of 8
   const float* bias;         // [heads * dim, padded] or null
-  const float* gain;         // norm 1: [dim], norm 2: [heads * dim, padded]
-  int heads, dim;
+  const float* gain;         // norm 1: [dim] or, with gain_heads, [heads][dim]; norm 2: [heads * dim, padded]
+  int heads, dim, gain_heads;
 };
 
 struct MixerPostArgs {
@@ -248,7 +248,7 @@ __global__ void __launch_bounds__(NTHR, NP <= 2 ? 4 : 2) mixer_post_kernel(const
     __syncwarp();
     if (norm == 1 || norm == 2) {
       float inv = inv_all;
-      const float* gain = norm == 1 ? r.gain : r.gain + c0 + h * dim;
+      const float* gain = norm == 1 && r.gain_heads == 0 ? r.gain : r.gain + c0 + h * dim;
       if (norm == 1) {
         float s = 0.f;
         for (int d = lane; d < dim; d += 32) s += x[d] * x[d];

@@ -21,7 +21,8 @@ namespace {
 
 // ------------------------------------------------------------------------------------------ router select
 // One warp per token.  mode 0: softmax over all experts, top-k, renormalise (Qwen).  mode 1: top-k on the
-// logits, softmax over the selected k only (Gemma), times per-expert scale if given.
+// logits, softmax over the selected k only (Gemma), times per-expert scale if given.  mode 2: softmax over all experts, top-k, the
+// scores as they are.
 template <int MAXPL>
 __global__ void moe_route_kernel(const float* __restrict__ logits, long long ld, int T, int E, int k, int mode,
                                  const float* __restrict__ expert_scale, int* __restrict__ ids,
@@ -42,7 +43,7 @@ __global__ void moe_route_kernel(const float* __restrict__ logits, long long ld,
   mx = warp_max(mx);
   float den = 0.f;
 #pragma unroll
-  for (int i = 0; i < MAXPL; ++i) den += (i * 32 + lane < E) ? __expf(v[i] - mx) : 0.f;
+  for (int i = 0; i < MAXPL; ++i) den += (i * 32 + lane < E) ? (mode == 2 ? expf(v[i] - mx) : __expf(v[i] - mx)) : 0.f;
   den = warp_sum(den);
   float sel_sum = 0.f;
   float my_w = 0.f;   // lane j keeps the j-th selected weight (k <= 32)
@@ -66,13 +67,13 @@ __global__ void moe_route_kernel(const float* __restrict__ logits, long long ld,
       for (int i = 0; i < MAXPL; ++i)
         if (i == (bi >> 5)) v[i] = -INFINITY;
     }
-    const float p = mode == 0 ? __expf(bv - mx) / den : bv;
+    const float p = mode == 0 ? __expf(bv - mx) / den : mode == 2 ? expf(bv - mx) / den : bv;
     if (lane == j) { my_w = p; my_id = bi; }
     sel_sum += (mode == 0) ? p : 0.f;
   }
   if (mode == 0) {
     my_w = my_w / fmaxf(sel_sum, 6.1e-5f);
-  } else {
+  } else if (mode == 1) {
     float m2 = warp_max(lane < k ? my_w : -INFINITY);
     const float ex = lane < k ? __expf(my_w - m2) : 0.f;
     const float s2 = warp_sum(ex);
@@ -474,7 +475,7 @@ int set_smem(F fn, size_t bytes) {
 HE_API int he_moe_route(const float* logits, long long ld, int T, int E, int k, int mode, const float* expert_scale,
                         int* ids, float* wts, cudaStream_t stream) {
   if (T <= 0) return 0;
-  if (k > 32 || k <= 0 || E > 512 || E < k) return -HE_ERR_BAD_ARG;
+  if (k > 32 || k <= 0 || E > 512 || E < k || mode < 0 || mode > 2) return -HE_ERR_BAD_ARG;
   const int wpb = 4;
   const dim3 grid((T + wpb - 1) / wpb);
   if (E <= 128) (void)launch_pdl(moe_route_kernel<4>, dim3(grid), dim3(wpb * 32), 0, stream, logits, ld, T, E, k, mode, expert_scale, ids, wts);

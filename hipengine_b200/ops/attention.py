@@ -20,10 +20,11 @@ FLASH_TILE_ROWS = 64
 
 
 def flash_prefill_segs(q, gate, kv_cache, block_table, seg_start, seg_slot, pos, seg_rows, out, H, Hkv, D, page, scale,
-                       window: int = 0, softcap: float = 0.0, sink=None, head_gate=None) -> None:
+                       window: int = 0, softcap: float = 0.0, sink=None, head_gate=None, keep_first: int = 0) -> None:
     """``flash_prefill`` for several segments in one launch: ``seg_start`` (device, n + 1 absolute row offsets),
     ``seg_slot`` (device), ``pos`` (device, per row) and ``seg_rows`` (host row counts, sizes the grid).  ``sink`` (fp32 [H]):
-    scores of a term in the softmax denominator; ``head_gate`` ([rows, H], fp32 or bf16): logits of a gate per head."""
+    scores of a term in the softmax denominator; ``head_gate`` ([rows, H], fp32 or bf16): logits of a gate per head; with a
+    ``window`` the sequence's first ``keep_first`` keys stay visible."""
     tiles = sum(-(-n // FLASH_TILE_ROWS) for n in seg_rows)
     N.check(N.lib().he_flash_prefill_segs(
         C.c_void_p(q.data_ptr()), C.c_void_p(None if gate is None else gate.data_ptr()),
@@ -34,6 +35,7 @@ def flash_prefill_segs(q, gate, kv_cache, block_table, seg_start, seg_slot, pos,
         C.c_void_p(None if sink is None else sink.data_ptr()),
         C.c_void_p(None if head_gate is None else head_gate.data_ptr()),
         C.c_longlong(0 if head_gate is None else head_gate.stride(0)), C.c_int(0 if head_gate is None else _dt(head_gate)),
+        C.c_int(keep_first),
         C.c_void_p(torch.cuda.current_stream().cuda_stream)), "he_flash_prefill_segs")
 
 

@@ -21,9 +21,9 @@ EPI_BF16, EPI_F32, EPI_ADD, EPI_RELU2 = 0, 1, 2, 6
 
 
 def gemm_bf16(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, epi: Optional[int] = None,
-              col_scale: Optional[torch.Tensor] = None) -> torch.Tensor:
+              col_scale: Optional[torch.Tensor] = None, col_bias: Optional[torch.Tensor] = None) -> torch.Tensor:
     """out[M, N] = x[M, K] @ w[N, K]^T.  x, w bf16 (row strides allowed); out bf16 or fp32.  ``col_scale`` (fp32 [N])
-    multiplies what ``EPI_ADD`` adds."""
+    multiplies what ``EPI_ADD`` adds, ``col_bias`` (fp32 [N]) is added to it."""
     assert x.dtype == torch.bfloat16 and w.dtype == torch.bfloat16
     _check_device(x)
     M, K = x.shape
@@ -36,6 +36,7 @@ def gemm_bf16(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, epi: Optional
                                  C.c_longlong(w.stride(0)), C.c_void_p(out.data_ptr()), C.c_longlong(out.stride(0)),
                                  C.c_int(M), C.c_int(Nn), C.c_int(K), C.c_int(epi),
                                  C.c_void_p(None if col_scale is None else col_scale.data_ptr()),
+                                 C.c_void_p(None if col_bias is None else col_bias.data_ptr()),
                                  C.c_void_p(st.data_ptr()), C.c_int(N.num_sms()), _stream()), "he_gemm_bf16")
     return out
 
@@ -178,10 +179,11 @@ def gemm_bf16_splitk_add(x: torch.Tensor, w: torch.Tensor, acc: torch.Tensor, k_
 
 
 def gemm_bf16_splitk_det(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, scratch, add: bool = False,
-                         col_scale: Optional[torch.Tensor] = None, relu2: bool = False) -> torch.Tensor:
+                         col_scale: Optional[torch.Tensor] = None, relu2: bool = False,
+                         col_bias: Optional[torch.Tensor] = None) -> torch.Tensor:
     """out[M, N] (fp32) = (or +=) x[M, K] @ w[N, K]^T with K split over CTAs and the partial tiles summed in a
     fixed order: the bit-reproducible form of ``gemm_bf16_splitk_add`` (``out`` may be a strided row view).  ``col_scale``
-    multiplies what is added; ``relu2`` stores the squared ReLU as bf16."""
+    multiplies what is added, ``col_bias`` is added to it; ``relu2`` stores the squared ReLU as bf16."""
     assert x.dtype == torch.bfloat16 and w.dtype == torch.bfloat16 and not (relu2 and add)
     assert out.dtype == (torch.bfloat16 if relu2 else torch.float32)
     _check_device(x)
@@ -197,6 +199,7 @@ def gemm_bf16_splitk_det(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, sc
                                       C.c_void_p(out.data_ptr()), C.c_longlong(out.stride(0)), C.c_int(M), C.c_int(Nn),
                                       C.c_int(K), C.c_int(1 if add else 2 if relu2 else 0),
                                       C.c_void_p(None if col_scale is None else col_scale.data_ptr()),
+                                      C.c_void_p(None if col_bias is None else col_bias.data_ptr()),
                                       C.c_void_p(st.data_ptr()), C.c_int(N.num_sms()), _stream()),
             "he_gemm_bf16_splitk_det")
     return out

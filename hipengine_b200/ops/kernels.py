@@ -78,7 +78,7 @@ class _AttnDecArgs(C.Structure):
                 ("R", C.c_int), ("H", C.c_int), ("Hkv", C.c_int), ("D", C.c_int), ("page", C.c_int),
                 ("max_pages", C.c_int), ("split_len", C.c_int), ("max_splits", C.c_int), ("window", C.c_int),
                 ("scale", C.c_float), ("status", c_vp), ("softcap", C.c_float), ("sink", c_vp), ("head_gate", c_vp),
-                ("head_gate_stride", c_ll), ("head_gate_dtype", C.c_int)]
+                ("head_gate_stride", c_ll), ("head_gate_dtype", C.c_int), ("keep_first", C.c_int)]
 
 
 class _GdnDecodeArgs(C.Structure):
@@ -117,7 +117,7 @@ class _FloatGemvArgs(C.Structure):
 
 class _FloatSumArgs(C.Structure):
     _fields_ = [("w", c_vp * 2), ("x", c_vp * 2), ("scale", c_vp * 2), ("ldw", c_ll * 2), ("x_stride", c_ll * 2),
-                ("K", C.c_int * 2), ("out", c_vp), ("out_stride", c_ll), ("n_rows", C.c_int), ("R", C.c_int)]
+                ("K", C.c_int * 2), ("out", c_vp), ("out_stride", c_ll), ("n_rows", C.c_int), ("R", C.c_int), ("bias", c_vp)]
 
 
 class _NormShiftArgs(C.Structure):
@@ -130,21 +130,22 @@ class _FloatMoeArgs(C.Structure):
     _fields_ = [("x", c_vp), ("ldx", c_ll), ("norm_w", c_vp), ("eps", C.c_float), ("norm_n", C.c_int), ("ids", c_vp),
                 ("wts", c_vp), ("sg", c_vp), ("ld_sg", c_ll), ("w1", c_vp), ("w1s", c_vp), ("E", C.c_int),
                 ("T", C.c_int), ("k", C.c_int), ("K", C.c_int), ("F", C.c_int), ("Fs", C.c_int), ("N", C.c_int),
-                ("act", C.c_int), ("limit", C.c_float), ("rows", c_vp), ("rows_s", c_vp), ("h", c_vp), ("ldh", c_ll)]
+                ("act", C.c_int), ("limit", C.c_float), ("rows", c_vp), ("rows_s", c_vp), ("h", c_vp), ("ldh", c_ll),
+                ("x_dtype", C.c_int)]
 
 
 class _ExactAttnArgs(C.Structure):
     _fields_ = [("q", c_vp), ("kv_cache", c_vp), ("block_table", c_vp), ("slot", c_vp), ("ctx_len", c_vp),
                 ("out", c_vp), ("R", C.c_int), ("H", C.c_int), ("Hkv", C.c_int), ("D", C.c_int), ("page", C.c_int),
                 ("max_pages", C.c_int), ("scale", C.c_float), ("softcap", C.c_float), ("window", C.c_int), ("sink", c_vp),
-                ("head_gate", c_vp), ("head_gate_stride", c_ll)]
+                ("head_gate", c_vp), ("head_gate_stride", c_ll), ("keep_first", C.c_int)]
 
 
 class _ExactMoeArgs(C.Structure):
     _fields_ = [("x", c_vp), ("ldx", c_ll), ("ids", c_vp), ("wts", c_vp), ("sg", c_vp), ("ld_sg", c_ll),
                 ("w1", c_vp), ("w1s", c_vp), ("E", C.c_int), ("T", C.c_int), ("k", C.c_int), ("K", C.c_int),
                 ("F", C.c_int), ("Fs", C.c_int), ("N", C.c_int), ("rows", c_vp), ("rows_s", c_vp), ("h", c_vp),
-                ("ldh", c_ll)]
+                ("ldh", c_ll), ("act", C.c_int), ("limit", C.c_float)]
 
 
 _CHECKED = False
@@ -556,8 +557,9 @@ def attn_decode_scratch_floats(R: int, H: int, max_splits: int, D: int) -> int:
 def attn_decode(q: torch.Tensor, gate: Optional[torch.Tensor], kv_cache: torch.Tensor, block_table: torch.Tensor,
                 slot: torch.Tensor, ctx_len: torch.Tensor, partial: torch.Tensor, out: torch.Tensor, H: int, Hkv: int,
                 D: int, page: int, split_len: int, max_splits: int, scale: float, window: int = 0,
-                softcap: float = 0.0, sink: Optional[torch.Tensor] = None, head_gate: Optional[torch.Tensor] = None) -> None:
-    """``sink`` (fp32 [H]): scores of a term in the softmax denominator; ``head_gate`` ([R, H], fp32 or bf16): logits of a
+                softcap: float = 0.0, sink: Optional[torch.Tensor] = None, head_gate: Optional[torch.Tensor] = None,
+                keep_first: int = 0) -> None:
+    """With a ``window`` the sequence's first ``keep_first`` keys stay visible (``max_splits`` covers both).  ``sink`` (fp32 [H]): scores of a term in the softmax denominator; ``head_gate`` ([R, H], fp32 or bf16): logits of a
     gate per head on the output."""
     _check_abi()
     a = _AttnDecArgs()
@@ -568,7 +570,7 @@ def attn_decode(q: torch.Tensor, gate: Optional[torch.Tensor], kv_cache: torch.T
     a.max_pages = block_table.shape[1]
     a.split_len, a.max_splits, a.window, a.scale = split_len, max_splits, window, scale
     a.status = status_tensor(q.device).data_ptr()
-    a.softcap, a.sink = softcap, _p(sink)
+    a.softcap, a.sink, a.keep_first = softcap, _p(sink), keep_first if window > 0 else 0
     if head_gate is not None:
         a.head_gate, a.head_gate_stride, a.head_gate_dtype = head_gate.data_ptr(), head_gate.stride(0), _dt(head_gate)
     assert partial.numel() >= attn_decode_scratch_floats(a.R, H, max_splits, D)
@@ -605,7 +607,8 @@ def ffn_combine(h: torch.Tensor, dense: torch.Tensor, expert: torch.Tensor, w1: 
 
 def moe_route(logits: torch.Tensor, k: int, ids: torch.Tensor, wts: torch.Tensor, n_experts: Optional[int] = None,
               mode: int = 0, expert_scale: Optional[torch.Tensor] = None) -> None:
-    """logits fp32 [T, >=E] (row stride allowed) -> ids int32 [T, k], wts fp32 [T, k]."""
+    """logits fp32 [T, >=E] (row stride allowed) -> ids int32 [T, k], wts fp32 [T, k].  mode 0: softmax over all, chosen ones
+    normalised; 1: softmax over the chosen ones; 2: softmax over all, as it is."""
     T = logits.shape[0]
     E = logits.shape[1] if n_experts is None else n_experts
     N.check(N.lib().he_moe_route(c_vp(logits.data_ptr()), c_ll(logits.stride(0)), C.c_int(T), C.c_int(E), C.c_int(k),
@@ -748,8 +751,9 @@ def gemv_float_batched(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor) -> N
         N.check(N.lib().he_gemv_float(C.byref(a), _stream()), "he_gemv_float")
 
 
-def gemv_sum(h: torch.Tensor, parts: Sequence[Tuple[torch.Tensor, torch.Tensor, Optional[torch.Tensor]]]) -> None:
-    """h[r, n] += sum over one or two (x, w, scale) of scale[n] * (x[r] . w[n]); bf16 rows and weights, 1..16 rows."""
+def gemv_sum(h: torch.Tensor, parts: Sequence[Tuple[torch.Tensor, torch.Tensor, Optional[torch.Tensor]]],
+             bias: Optional[torch.Tensor] = None) -> None:
+    """h[r, n] += bias[n] + sum over one or two (x, w, scale) of scale[n] * (x[r] . w[n]); bf16 rows and weights, 1..16 rows."""
     _check_abi()
     _check_device(h)
     assert 1 <= len(parts) <= 2 and h.dtype == torch.float32
@@ -758,7 +762,7 @@ def gemv_sum(h: torch.Tensor, parts: Sequence[Tuple[torch.Tensor, torch.Tensor, 
         assert x.dtype == w.dtype == torch.bfloat16 and x.shape == (h.shape[0], w.shape[1]) and w.shape[0] == parts[0][1].shape[0]
         a.w[i], a.x[i], a.scale[i] = w.data_ptr(), x.data_ptr(), _p(scale)
         a.ldw[i], a.x_stride[i], a.K[i] = w.stride(0), x.stride(0), w.shape[1]
-    a.out, a.out_stride, a.n_rows, a.R = h.data_ptr(), h.stride(0), parts[0][1].shape[0], h.shape[0]
+    a.out, a.out_stride, a.n_rows, a.R, a.bias = h.data_ptr(), h.stride(0), parts[0][1].shape[0], h.shape[0], _p(bias)
     N.check(N.lib().he_gemv_sum(C.byref(a), _stream()), "he_gemv_sum")
 
 
@@ -781,15 +785,16 @@ def norm_shift(x: torch.Tensor, w: torch.Tensor, shift: torch.Tensor, state: tor
     N.check(N.lib().he_norm_shift(C.byref(a), _stream()), "he_norm_shift")
 
 
-def moe_gateup_float(h: torch.Tensor, norm_w: torch.Tensor, eps: float, norm_n: int, ids: torch.Tensor,
+def moe_gateup_float(h: torch.Tensor, norm_w: Optional[torch.Tensor], eps: float, norm_n: int, ids: torch.Tensor,
                      wts: torch.Tensor, w_gu: torch.Tensor, n_experts: int, rows: torch.Tensor,
                      sg: Optional[torch.Tensor] = None, w_gu_shared: Optional[torch.Tensor] = None,
                      rows_shared: Optional[torch.Tensor] = None, act: str = "silu", limit: float = 0.0) -> None:
     """Selected experts, few tokens: ``rows`` [T*k, F] = weight * act(Wg xn) * (Wu xn) in bf16, and ``rows_shared``
-    [T, Fs] the same for the shared expert with weight sigmoid(sg).  ``w_gu`` stacks [gate | up] rows per expert."""
+    [T, Fs] the same for the shared expert with weight sigmoid(sg).  ``w_gu`` stacks [gate | up] rows per expert; without
+    ``norm_w`` the rows (fp32 or bf16) are taken as they are."""
     _check_abi()
     a = _FloatMoeArgs()
-    a.x, a.ldx, a.norm_w, a.eps, a.norm_n = h.data_ptr(), h.stride(0), norm_w.data_ptr(), eps, norm_n
+    a.x, a.ldx, a.norm_w, a.eps, a.norm_n, a.x_dtype = h.data_ptr(), h.stride(0), _p(norm_w), eps, norm_n, _dt(h)
     a.ids, a.wts, a.sg, a.ld_sg = ids.data_ptr(), wts.data_ptr(), _p(sg), sg.stride(0) if sg is not None else 0
     a.w1, a.w1s = w_gu.data_ptr(), _p(w_gu_shared)
     a.E, a.T, a.k, a.K = n_experts, ids.shape[0], ids.shape[1], w_gu.shape[1]
@@ -817,7 +822,7 @@ def moe_down_float(rows: torch.Tensor, ids: torch.Tensor, w_down: torch.Tensor, 
 def attn_exact(q: torch.Tensor, kv_cache: torch.Tensor, block_table: torch.Tensor, slot: torch.Tensor,
                ctx_len: torch.Tensor, out: torch.Tensor, H: int, Hkv: int, D: int, page: int, scale: float,
                softcap: float = 0.0, window: int = 0, sink: Optional[torch.Tensor] = None,
-               head_gate: Optional[torch.Tensor] = None) -> None:
+               head_gate: Optional[torch.Tensor] = None, keep_first: int = 0) -> None:
     """Causal attention of any rows over fp32 pages, fp32 throughout; the options are those of ``attn_decode``."""
     _check_abi()
     assert q.dtype == kv_cache.dtype == out.dtype == torch.float32 and (head_gate is None or head_gate.dtype == torch.float32)
@@ -825,7 +830,7 @@ def attn_exact(q: torch.Tensor, kv_cache: torch.Tensor, block_table: torch.Tenso
     a.q, a.kv_cache, a.block_table = q.data_ptr(), kv_cache.data_ptr(), block_table.data_ptr()
     a.slot, a.ctx_len, a.out = slot.data_ptr(), ctx_len.data_ptr(), out.data_ptr()
     a.R, a.H, a.Hkv, a.D, a.page, a.max_pages = q.shape[0], H, Hkv, D, page, block_table.shape[1]
-    a.scale, a.softcap, a.window, a.sink = scale, softcap, window, _p(sink)
+    a.scale, a.softcap, a.window, a.sink, a.keep_first = scale, softcap, window, _p(sink), keep_first if window > 0 else 0
     if head_gate is not None:
         a.head_gate, a.head_gate_stride = head_gate.data_ptr(), head_gate.stride(0)
     N.check(N.lib().he_attn_exact(C.byref(a), _stream()), "he_attn_exact")
@@ -834,8 +839,8 @@ def attn_exact(q: torch.Tensor, kv_cache: torch.Tensor, block_table: torch.Tenso
 def moe_exact(xn: torch.Tensor, ids: torch.Tensor, wts: torch.Tensor, w_gu: torch.Tensor, w_down: torch.Tensor,
               n_experts: int, rows: torch.Tensor, h: torch.Tensor, sg: Optional[torch.Tensor] = None,
               w_gu_shared: Optional[torch.Tensor] = None, w_down_shared: Optional[torch.Tensor] = None,
-              rows_shared: Optional[torch.Tensor] = None) -> None:
-    """Selected SiLU experts (and the shared one) of normalised fp32 rows, added to ``h``; fp32 throughout."""
+              rows_shared: Optional[torch.Tensor] = None, act: str = "silu", limit: float = 0.0) -> None:
+    """Selected experts (and the shared one) of normalised fp32 rows, added to ``h``; fp32 throughout."""
     _check_abi()
     a = _ExactMoeArgs()
     a.x, a.ldx, a.ids, a.wts = xn.data_ptr(), xn.stride(0), ids.data_ptr(), wts.data_ptr()
@@ -844,6 +849,7 @@ def moe_exact(xn: torch.Tensor, ids: torch.Tensor, wts: torch.Tensor, w_gu: torc
     a.E, a.T, a.k, a.K, a.N = n_experts, ids.shape[0], ids.shape[1], w_gu.shape[1], w_down.shape[0] // n_experts
     a.F, a.Fs = rows.shape[1], rows_shared.shape[1] if rows_shared is not None else 0
     a.rows, a.rows_s, a.h, a.ldh = rows.data_ptr(), _p(rows_shared), h.data_ptr(), h.stride(0)
+    a.act, a.limit = ACT_CODES[act], limit
     N.check(N.lib().he_moe_gateup_exact(C.byref(a), _stream()), "he_moe_gateup_exact")
     a.w1, a.w1s = w_down.data_ptr(), _p(w_down_shared)
     N.check(N.lib().he_moe_down_exact(C.byref(a), _stream()), "he_moe_down_exact")
@@ -972,10 +978,10 @@ GEMM_STORE, GEMM_ADD, GEMM_RELU2 = 0, 1, 2
 
 
 def small_gemm_f32(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, add: bool = False, mode: int = GEMM_STORE,
-                   col_scale: Optional[torch.Tensor] = None) -> torch.Tensor:
+                   col_scale: Optional[torch.Tensor] = None, col_bias: Optional[torch.Tensor] = None) -> torch.Tensor:
     """out[T, N] (fp32) = (or +=, or relu(.)^2 of) x[T, K] @ w[N, K]^T in fp32 arithmetic; w fp32 (router / ssm_alpha /
-    ssm_beta at prefill) or bf16 (the float32 compute dtype).  ``col_scale`` [N] multiplies what is added.  Three-dimensional
-    operands x [T, B, K], w [B, N, K], out [T, B, N] are B products."""
+    ssm_beta at prefill) or bf16 (the float32 compute dtype).  ``col_scale`` [N] multiplies what is added, or ``col_bias`` [N]
+    is added to it.  Three-dimensional operands x [T, B, K], w [B, N, K], out [T, B, N] are B products."""
     mode = GEMM_ADD if add else mode
     assert out.dtype == torch.float32 and w.shape[-1] == x.shape[-1] and (col_scale is None or mode == GEMM_ADD)
     B = x.shape[1] if x.dim() == 3 else 1
@@ -983,6 +989,6 @@ def small_gemm_f32(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, add: boo
     N.check(N.lib().he_small_gemm_f32(c_vp(x.data_ptr()), C.c_int(_dt(x)), c_ll(x.stride(0)), c_vp(w.data_ptr()),
                                       C.c_int(_dt(w)), c_ll(w.stride(-2)), c_vp(out.data_ptr()), c_ll(out.stride(0)),
                                       C.c_int(x.shape[0]), C.c_int(w.shape[-2]), C.c_int(x.shape[-1]), C.c_int(mode),
-                                      c_vp(_p(col_scale)), C.c_int(B), c_ll(bs[0]), c_ll(bs[1]), c_ll(bs[2]), _stream()),
+                                      c_vp(_p(col_scale)), c_vp(_p(col_bias)), C.c_int(B), c_ll(bs[0]), c_ll(bs[1]), c_ll(bs[2]), _stream()),
             "he_small_gemm_f32")
     return out

@@ -16,7 +16,8 @@ NORM_CODES = {"none": 0, "head": 1, "rows": 2, "unit": 3}
 
 
 class _HeadRows(C.Structure):
-    _fields_ = [("x", c_vp), ("stride", c_ll), ("bias", c_vp), ("gain", c_vp), ("heads", c_int), ("dim", c_int)]
+    _fields_ = [("x", c_vp), ("stride", c_ll), ("bias", c_vp), ("gain", c_vp), ("heads", c_int), ("dim", c_int),
+                ("gain_heads", c_int)]
 
 
 class _PostArgs(C.Structure):
@@ -58,7 +59,7 @@ class HeadRows:
     heads: int
     dim: int
     bias: Optional[torch.Tensor] = None     # fp32, padded like x
-    gain: Optional[torch.Tensor] = None     # fp32: [dim] (norm "head") or padded like x (norm "rows")
+    gain: Optional[torch.Tensor] = None     # fp32: [dim] or [heads, dim] (norm "head"), or padded like x (norm "rows")
 
 
 @dataclass
@@ -88,6 +89,8 @@ def mixer_post(q: HeadRows, k: Optional[HeadRows], v: Optional[HeadRows], norm: 
         assert (r.bias is None or r.bias.numel() == r.x.shape[1]) and (norm != "rows" or r is v or r.gain.numel() == r.x.shape[1])
         dst.x, dst.stride, dst.bias, dst.gain, dst.heads, dst.dim = (r.x.data_ptr(), r.x.stride(0), _p(r.bias), _p(r.gain),
                                                                      r.heads, r.dim)
+        dst.gain_heads = int(r.gain is not None and r.gain.dim() == 2)
+        assert not dst.gain_heads or (norm == "head" and r.gain.shape == (r.heads, r.dim) and r.gain.is_contiguous())
     T, D = q.x.shape[0], q_out.shape[2]
     assert q_out.is_contiguous() and q_out.shape == (T, q.heads, D)
     assert k is None or (kv_cache.dtype == q_out.dtype and kv_cache.shape[1:] == (2, k.heads, page, D))
