@@ -13,7 +13,7 @@ In both modes residual, norms, scores, softmax, router and positions are fp32.  
 from __future__ import annotations
 
 from dataclasses import dataclass
-from typing import List, Optional, Tuple
+from typing import List, Optional
 
 import torch
 
@@ -21,7 +21,7 @@ from ..ops import kernels as K
 from ..ops.kernels import DeviceWeight
 from .config import DenseMlpSpec, MoeMlpSpec
 from .executor import PAGE, BatchDesc
-from .listed import EXACT, FEW, MANY, ListedExecutor, pad2, up8
+from .listed import ExpertWeights, ListedExecutor, pad2, up8
 
 
 @dataclass
@@ -34,11 +34,7 @@ class _Layer:
     o: DeviceWeight                              # [Hp, heads * D]
     gate_up: Optional[DeviceWeight] = None       # dense: [gate | up rows, Hp]
     down: Optional[DeviceWeight] = None          # dense: [Hp, F]
-    router: Optional[DeviceWeight] = None        # [experts (+ shared gate), Hp], rows padded to eight
-    e_gate_up: Optional[DeviceWeight] = None     # [experts * (gate | up), Hp]
-    e_down: Optional[DeviceWeight] = None        # [experts * Hp, F]
-    s_gate_up: Optional[DeviceWeight] = None
-    s_down: Optional[DeviceWeight] = None
+    experts: Optional[ExpertWeights] = None
 
 
 class SisisunExecutor(ListedExecutor):
@@ -53,11 +49,6 @@ class SisisunExecutor(ListedExecutor):
 
     def _load_layers(self) -> None:
         cfg, dev, hp, mat, put, norm = self.cfg, self.device, self.hp, self._mat, self._put, self._norm_weight
-        gate_up = self._gate_up
-
-        def glu(name: str, p: str, ff: int) -> Tuple[DeviceWeight, DeviceWeight]:
-            return put(name + "gate_up", gate_up(p, ff)), put(name + "down", pad2(mat(p + "down"), hp, up8(ff)))
-
         self.layers: List[_Layer] = []
         for i, spec in enumerate(cfg.layer_specs):
             a, m, p = spec.mixer, spec.mlp, f"l{i}."
@@ -68,21 +59,10 @@ class SisisunExecutor(ListedExecutor):
                        put(p + "qkv", pad2(qkv, up8(qkv.shape[0]), hp)), self.f32[p + "mix.q.norm"],
                        self.f32[p + "mix.k.norm"], put(p + "o", self._out_mat(p + "mix.o", a.heads, a.vdim, a.width)))
             if isinstance(m, DenseMlpSpec):
-                L.gate_up, L.down = glu(p, p + "mlp.", m.ff)
+                L.gate_up = put(p + "gate_up", self._gate_up(p + "mlp.", m.ff))
+                L.down = put(p + "down", pad2(mat(p + "mlp.down"), hp, up8(m.ff)))
             elif isinstance(m, MoeMlpSpec):
-                fp = up8(m.ff)
-                gu = torch.empty(m.experts * 2 * fp, hp, dtype=torch.bfloat16, device=dev)
-                dn = torch.empty(m.experts * hp, fp, dtype=torch.bfloat16, device=dev)
-                for e in range(m.experts):
-                    gu[e * 2 * fp:(e + 1) * 2 * fp] = gate_up(p + f"mlp.e{e}.", m.ff)
-                    dn[e * hp:(e + 1) * hp] = pad2(mat(p + f"mlp.e{e}.down"), hp, fp)
-                L.e_gate_up, L.e_down = put(p + "experts.gate_up", gu), put(p + "experts.down", dn)
-                rows = [mat(p + "mlp.router")]
-                if m.shared_ff:
-                    L.s_gate_up, L.s_down = glu(p + "shared.", p + "mlp.shared.", m.shared_ff)
-                    rows.append(mat(p + "mlp.shared.sg"))
-                r = torch.cat(rows, 0)
-                L.router = put(p + "router", pad2(r, up8(r.shape[0]), hp))
+                L.experts = self._load_experts(p, m)
             self.layers.append(L)
         i = torch.arange((cfg.hidden + 1) // 2, dtype=torch.float64)
         self.pos_freq = torch.pow(torch.tensor(10000.0, dtype=torch.float64), -2.0 * i / cfg.hidden).to(dev)
@@ -104,54 +84,6 @@ class SisisunExecutor(ListedExecutor):
         with self._stage("out_gemm"):
             self._add_products(h, [(out, L.o, None)], route)
 
-    def _experts(self, L: _Layer, m: MoeMlpSpec, h: torch.Tensor, route: str) -> None:
-        from ..ops import gemm as GM
-        sc, cfg, T, E, k = self.scratch, self.cfg, h.shape[0], m.experts, m.top
-        F = L.e_down.n_cols
-        xn = None
-        if route != FEW:
-            with self._stage("norm"):
-                xn = self._norm_rows(h, L.norm2)
-        if route == MANY:
-            logits = GM.gemm_bf16(xn, L.router.data, sc.get("moe_logits_f32", (T, L.router.n_rows), torch.float32))
-        else:
-            logits = self._in_proj(h, L.norm2, L.router, "moe_logits", route, xn=xn)
-        ids = sc.get("moe_ids", (T, k), torch.int32)
-        wts = sc.get("moe_wts", (T, k), torch.float32)
-        K.moe_route_grouped(logits, k, ids, wts, E, m.groups, m.groups_kept, m.scale)
-        sg = logits[:, E:E + 1] if m.shared_ff else None
-        s_gu = L.s_gate_up.data if m.shared_ff else None
-        s_dn = L.s_down.data if m.shared_ff else None
-        if route != MANY:
-            rows = sc.get("moe_act", (T * k, F), self.act_dtype)
-            rows_s = sc.get("moe_act_sh", (T, L.s_down.n_cols), self.act_dtype) if m.shared_ff else None
-            if route == EXACT:
-                K.moe_exact(xn, ids, wts, L.e_gate_up.data, L.e_down.data, E, rows, h, sg, s_gu, s_dn, rows_s)
-                return
-            K.moe_gateup_float(h, L.norm2, cfg.rms_eps, cfg.hidden, ids, wts, L.e_gate_up.data, E, rows, sg, s_gu, rows_s)
-            K.moe_down_float(rows, ids, L.e_down.data, E, h, rows_s, s_dn)
-            return
-        P = T * k
-        bound = K.moe_sorted_rows_bound(P, E)
-        pos = sc.get("moe_pos", (P,), torch.int32)
-        tiles = sc.get("moe_tiles", (bound // 128,), torch.int32)
-        K.moe_group(ids, E, pos, tiles, sc.get("moe_meta", (4,), torch.int32))
-        xs = sc.get("moe_xs", (bound, self.hp), torch.bfloat16)
-        K.moe_gather(xn, pos, k, xs)
-        gu = sc.get("moe_gu", (bound, 2 * F), torch.bfloat16)
-        GM.gemm_bf16_grouped(xs, L.e_gate_up.data, gu, E, tiles)
-        act = sc.get("moe_act_g", (bound, F), torch.bfloat16)
-        K.act_mul(gu, act, "silu")
-        ys = sc.get("moe_ys", (bound, self.hp), torch.bfloat16)
-        GM.gemm_bf16_grouped(act, L.e_down.data, ys, E, tiles)
-        ysh = None
-        if m.shared_ff:
-            gus = self._proj(xn, L.s_gate_up, "moe_gus", "g")
-            acts = sc.get("moe_acts", (T, L.s_down.n_cols), torch.bfloat16)
-            K.act_mul(gus, acts, "silu")
-            ysh = self._gemm(acts, L.s_down, sc.get("y_bf", (T, self.hp), torch.bfloat16), tag="d")
-        K.moe_combine(h, ys, pos, wts, k, ysh, sg)
-
     # ------------------------------------------------------------------ whole model
     def _embed(self, b: BatchDesc, h: torch.Tensor, copy: Optional[torch.Tensor]) -> None:
         K.embed_sinusoid(self.embed_w, b.tokens, b.pos, self.pos_freq, h, copy)
@@ -163,4 +95,5 @@ class SisisunExecutor(ListedExecutor):
             L = self.layers[i]
             self._dense(L.norm2, L.gate_up, L.down, m, h, route)
         elif isinstance(m, MoeMlpSpec):
-            self._experts(self.layers[i], m, h, route)
+            L = self.layers[i]
+            self._experts(L.experts, L.norm2, m, h, route)
