@@ -126,7 +126,7 @@ PLUGINS: Tuple[ModelPlugin, ...] = (
                 native_block_types=("BF16",), widened_block_types=(), kv_storage=("bf16", "f32"),
                 tensor_parallel=False, compute_dtypes=("bfloat16", "float32"),
                 native_sources=("attn_decode.cu", "attn_prefill.cu", "exact_f32.cu", "gemm_sm100.cu", "gemv_float.cu",
-                                "layers.cu", "linear_attn.cu", "mixer_post.cu", "moe.cu", "norm_conv.cu",
+                                "layers.cu", "linear_attn.cu", "linear_chunk.cu", "mixer_post.cu", "moe.cu", "norm_conv.cu",
                                 "quant_util.cu", "runtime.cpp", "sampling.cu"),
                 folder_architecture="Mepatar", folder_reader="hipengine_b200.loading.mepatar",
                 reference="hipengine_b200.ref.mepatar.MepatarRef",
