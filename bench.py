@@ -122,7 +122,7 @@ def main() -> int:
                          "packed step per token (continuous-batching steady state)")
     ap.add_argument("--no-mtp", action="store_true", help="N = 1: skip the speculative (NextN depth 3) cycle figures")
     ap.add_argument("--mtp-depth", type=int, default=3)
-    ap.add_argument("--beside", default=None, choices=["sisisun", "milutar", "banelix"],
+    ap.add_argument("--beside", default=None, choices=["sisisun", "milutar", "banelix", "mepatar"],
                     help="instead of the workload above: kernels and models of this family beside the closest other "
                          "family at equal size (one JSON line per row)")
     args = ap.parse_args()

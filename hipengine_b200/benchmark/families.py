@@ -1,11 +1,11 @@
 """A family beside its closest existing one at equal size: kernel by kernel against the roofline, then whole models.
 
-    python bench.py --beside sisisun|milutar|banelix    # what this module prints, as one JSON line per row
+    python bench.py --beside sisisun|milutar|banelix|mepatar    # what this module prints, as one JSON line per row
     python -m hipengine_b200.benchmark.families [family] [--kernels-only | --models-only]
 
 Each kernel row gives the new design's kernel and the like kernel of the closest model (Sisisun beside the Qwen3-shaped
-dense / MoE decoder on the hybrid executor, Milutar and Banelix beside Sisisun, ``latent_rows.py`` and
-``recurrent_rows.py``), their device times and the fraction of the measured peak that bounds them: HBM for the weight or KV
+dense / MoE decoder on the hybrid executor, Milutar, Banelix and Mepatar beside Sisisun, ``latent_rows.py``,
+``recurrent_rows.py`` and ``linear_rows.py``), their device times and the fraction of the measured peak that bounds them: HBM for the weight or KV
 streams (every format counts its own bytes), the bf16 tensor peak for the large products.  Operands are rotated through more
 than the L2 holds.  Weights are random.
 """
@@ -288,7 +288,7 @@ def model_rows(emit: Callable[[Dict], None]) -> None:
 
 def main(argv: Optional[List[str]] = None) -> int:
     ap = argparse.ArgumentParser(prog="families")
-    ap.add_argument("family", nargs="?", default="sisisun", choices=["sisisun", "milutar", "banelix"])
+    ap.add_argument("family", nargs="?", default="sisisun", choices=["sisisun", "milutar", "banelix", "mepatar"])
     ap.add_argument("--kernels-only", action="store_true")
     ap.add_argument("--models-only", action="store_true")
     a = ap.parse_args(argv)
@@ -299,6 +299,8 @@ def main(argv: Optional[List[str]] = None) -> int:
         from . import latent_rows as rows
     elif a.family == "banelix":
         from . import recurrent_rows as rows
+    elif a.family == "mepatar":
+        from . import linear_rows as rows
     else:
         rows = sys.modules[__name__]
     with NvmlSampler(device_index=torch.cuda.current_device(), interval_s=0.02) as clocks:

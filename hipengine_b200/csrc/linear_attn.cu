@@ -148,6 +148,19 @@ __global__ void __launch_bounds__(256) linear_out_kernel(const __grid_constant__
   const int t = (int)(w / a.H), h = (int)(w % a.H);
   const float* o = a.o + (size_t)w * a.vcols;
   float ss = 0.f;
+  if (a.vdim == 128 && a.row_dtype == 1 && sizeof(OutT) == 2 && a.stride % 4 == 0 && a.cz % 4 == 0) {        // four columns per lane
+    const float4 x = *reinterpret_cast<const float4*>(o + lane * 4);
+    const uint2 zr = *reinterpret_cast<const uint2*>(reinterpret_cast<const __nv_bfloat16*>(a.rows) + (size_t)t * a.stride + a.cz + h * 128 + lane * 4);
+    float4 g = make_float4(1.f, 1.f, 1.f, 1.f);
+    if (a.gain != nullptr) g = make_float4(a.gain[lane * 4], a.gain[lane * 4 + 1], a.gain[lane * 4 + 2], a.gain[lane * 4 + 3]);
+    const float inv = rsqrtf(warp_sum(x.x * x.x + x.y * x.y + x.z * x.z + x.w * x.w) / 128.f + a.eps);
+    const float2 z0 = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&zr.x)),
+                 z1 = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&zr.y));
+    __align__(8) __nv_bfloat162 r2[2] = {__floats2bfloat162_rn(x.x * inv * g.x * silu_f(z0.x), x.y * inv * g.y * silu_f(z0.y)),
+                                         __floats2bfloat162_rn(x.z * inv * g.z * silu_f(z1.x), x.w * inv * g.w * silu_f(z1.y))};
+    *reinterpret_cast<uint2*>(reinterpret_cast<__nv_bfloat16*>(a.out) + (size_t)w * 128 + lane * 4) = *reinterpret_cast<const uint2*>(r2);
+    return;
+  }
   for (int i = lane; i < a.vdim; i += 32) ss += o[i] * o[i];
   const float inv = rsqrtf(warp_sum(ss) / (float)a.vdim + a.eps);
   OutT* out = reinterpret_cast<OutT*>(a.out) + (size_t)w * a.vcols;
@@ -161,15 +174,17 @@ __global__ void __launch_bounds__(256) linear_out_kernel(const __grid_constant__
 }
 
 // ---------------------------------------------------------------- one token per segment
-constexpr int STEP_THREADS = 512;
+constexpr int STEP_WARPS = 16, STEP_THREADS = STEP_WARPS * 32, STEP_COLS = 128;
 
-// grid (H, T); lanes per column: 4 up to 128 rows, 16 above
-template <int DK, bool DELTA, typename OutT>
-__global__ void __launch_bounds__(STEP_THREADS) linear_step_kernel(const __grid_constant__ LinearArgs a) {
-  constexpr int L = DK <= 128 ? 4 : 16, RPL = DK / L, COLS = STEP_THREADS / L, KPAD = DK + 4 * L;
+// grid (H, T).  A warp owns rows of the state, a lane four of 128 columns: whole lines in and out; sums over the rows meet in shared
+// memory.  NB > 1: more rows than the registers hold (NB blocks), read once for S^T k and once for the update.
+template <int RW, int NB, bool DELTA, typename OutT>
+__global__ void __launch_bounds__(STEP_THREADS, 2) linear_step_kernel(const __grid_constant__ LinearArgs a) {
+  constexpr int DK = RW * STEP_WARPS * NB;
   extern __shared__ __align__(16) float dyn[];                 // values, outputs: vcols each
-  __shared__ __align__(16) float sq[KPAD], sk[KPAD];
-  __shared__ float raw[2][DK], red[33], gate[2];
+  __shared__ __align__(16) float part[STEP_WARPS][STEP_COLS];
+  __shared__ __align__(16) float su[STEP_COLS];
+  __shared__ float sq[DK], sk[DK], red[33], gate[2], unit[2];
   pdl_launch();
   const int h = blockIdx.x, t = blockIdx.y, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
   const int grp = a.H / a.G, kh = h / grp;
@@ -178,81 +193,135 @@ __global__ void __launch_bounds__(STEP_THREADS) linear_step_kernel(const __grid_
   if (!HE_INDEX_OK(slot, a.n_slots, HE_SITE_STATE_SLOT)) return;
   float* sv = dyn;
   float* so = dyn + a.vcols;
-  // the state's rows are on their way while the token's rows are prepared
-  const int cw = tid / L, ks = tid % L;
   float* Sg = a.S + ((size_t)slot * a.H + h) * a.dim * a.vcols;
-  float S[RPL];
-  const auto load = [&](int col) {
+  float4 S[RW];
+  const auto load = [&](int block, int col) {
 #pragma unroll
-    for (int i = 0; i < RPL; ++i) {
-      const int d = ks * RPL + i;
-      S[i] = col < a.vcols && d < a.dim ? Sg[(size_t)d * a.vcols + col] : 0.f;
+    for (int i = 0; i < RW; ++i) {
+      const int d = (block * STEP_WARPS + warp) * RW + i;
+      S[i] = col < a.vcols && d < a.dim ? *reinterpret_cast<const float4*>(Sg + (size_t)d * a.vcols + col) : make_float4(0.f, 0.f, 0.f, 0.f);
     }
   };
-  load(cw);
-  if (warp < 2) {
-    la_prepare_head(a, t, t, slot, p, (warp == 0 ? 0 : a.ck) + kh * a.dim, warp == 0 ? a.qscale : a.kscale, raw[warp], lane);
-    __syncwarp();
-    float* dst = warp == 0 ? sq : sk;
-    for (int d = lane; d < DK; d += 32) dst[d + (d / RPL) * 4] = d < a.dim ? raw[warp][d] : 0.f;
-  } else {
-    for (int d = tid - 64; d < a.vcols; d += STEP_THREADS - 64) {
-      const int c = a.cv + h * a.vdim + d;
-      sv[d] = d >= a.vdim ? 0.f : DELTA ? la_conv(a, t, t, slot, p, c) : la_row(a, (size_t)t * a.stride + c);
+  // the state's rows are on their way while the token's rows are prepared
+  if constexpr (NB == 1) load(0, lane * 4);
+  const size_t row0 = (size_t)t * a.stride;
+  if constexpr (DELTA) {
+    // a channel of query, key or value per thread; the ring's entry of `back` tokens ago lies at (p - back) % taps
+    const int e0 = p % a.taps, total = 2 * a.dim + a.vcols;
+    const float* ring = a.taps > 1 ? a.ring + (size_t)slot * a.taps * a.C : nullptr;
+    for (int i = tid; i < total; i += STEP_THREADS) {
+      const int d = i < a.dim ? i : i < 2 * a.dim ? i - a.dim : i - 2 * a.dim;
+      float v = 0.f;
+      if (i < 2 * a.dim || d < a.vdim) {
+        const int c = (i < a.dim ? kh * a.dim : i < 2 * a.dim ? a.ck + kh * a.dim : a.cv + h * a.vdim) + d;
+        float acc = 0.f;
+#pragma unroll 4
+        for (int back = a.taps - 1; back > 0; --back)
+          if (p >= back) acc += a.cw[(size_t)(a.taps - 1 - back) * a.C + c] * ring[(size_t)(e0 >= back ? e0 - back : e0 - back + a.taps) * a.C + c];
+        v = la_silu(acc + a.cw[(size_t)(a.taps - 1) * a.C + c] * la_row(a, row0 + c));
+      }
+      if (i < a.dim) sq[d] = v;
+      else if (i < 2 * a.dim) sk[d] = v;
+      else sv[d] = v;
     }
-    if (DELTA && tid == STEP_THREADS - 1) {
+    if (tid == STEP_THREADS - 1) {
       gate[0] = expm1f(la_log_decay(a, t, h));
       gate[1] = la_beta(a, t, h);
     }
+  } else {
+    const int half = a.rot_dims >> 1;
+    for (int i = tid; i < 2 * half; i += STEP_THREADS) {       // pairs of the query, then of the key
+      const bool key = i >= half;
+      const int j = key ? i - half : i;
+      const size_t c0 = row0 + (key ? a.ck : 0) + kh * a.dim + j;
+      const float u = la_row(a, c0), v = la_row(a, c0 + half);
+      float c, s;
+      la_angle(a.freq[j], p, c, s);
+      float* dst = key ? sk : sq;
+      dst[j] = u * c - v * s;
+      dst[half + j] = v * c + u * s;
+    }
+    for (int d = a.rot_dims + tid; d < a.dim; d += STEP_THREADS) {
+      sq[d] = la_row(a, row0 + kh * a.dim + d);
+      sk[d] = la_row(a, row0 + a.ck + kh * a.dim + d);
+    }
+    for (int d = STEP_THREADS - 1 - tid; d < a.vcols; d += STEP_THREADS)
+      sv[d] = d < a.vdim ? la_row(a, row0 + a.cv + h * a.vdim + d) : 0.f;
   }
+  for (int d = a.dim + tid; d < DK; d += STEP_THREADS) sq[d] = sk[d] = 0.f;
   __syncthreads();
-  const float g1 = DELTA ? gate[0] : a.gm[h];
-  const float* kp = sk + ks * (RPL + 4);
-  const float* qp = sq + ks * (RPL + 4);
+  if (DELTA && warp < 2) {                                     // unit length: factors of query and key
+    const float* x = warp == 0 ? sq : sk;
+    float ss = 0.f;
+    for (int d = lane; d < a.dim; d += 32) ss += x[d] * x[d];
+    ss = warp_sum(ss);
+    if (lane == 0) unit[warp] = (warp == 0 ? a.qscale : a.kscale) / sqrtf(ss + 1e-6f);
+  }
+  if (DELTA) __syncthreads();
+  const float qs = DELTA ? unit[0] : a.qscale, ks = DELTA ? unit[1] : a.kscale, g1 = DELTA ? gate[0] : a.gm[h];
   float ss = 0.f;
-  for (int c0 = 0; c0 < a.vcols; c0 += COLS) {
-    const int col = c0 + cw;
-    const bool live = col < a.vcols;
-    if (c0 > 0) load(col);
-    float u = live ? sv[col] : 0.f;
+  for (int c0 = 0; c0 < a.vcols; c0 += STEP_COLS) {
+    const int col = c0 + lane * 4, mine = c0 + tid;            // columns of the lane; column summed up by the thread
     if constexpr (DELTA) {
-      float p4[4] = {0.f, 0.f, 0.f, 0.f};
+      float4 acc = make_float4(0.f, 0.f, 0.f, 0.f);
+      for (int nb = 0; nb < NB; ++nb) {
+        if (NB > 1 || c0 > 0) load(nb, col);
 #pragma unroll
-      for (int i = 0; i < RPL; ++i) {
-        S[i] = fmaf(g1, S[i], S[i]);
-        p4[i & 3] += kp[i] * S[i];
+        for (int i = 0; i < RW; ++i) {
+          S[i].x = fmaf(g1, S[i].x, S[i].x); S[i].y = fmaf(g1, S[i].y, S[i].y);
+          S[i].z = fmaf(g1, S[i].z, S[i].z); S[i].w = fmaf(g1, S[i].w, S[i].w);
+          const float k = sk[(nb * STEP_WARPS + warp) * RW + i];
+          acc.x += k * S[i].x; acc.y += k * S[i].y; acc.z += k * S[i].z; acc.w += k * S[i].w;
+        }
       }
-      float kv = (p4[0] + p4[1]) + (p4[2] + p4[3]);
+      *reinterpret_cast<float4*>(&part[warp][lane * 4]) = acc;
+      __syncthreads();
+      if (tid < STEP_COLS) {
+        float kv = 0.f;
 #pragma unroll
-      for (int o = 1; o < L; o <<= 1) kv += __shfl_xor_sync(0xffffffffu, kv, o);
-      u = (u - kv) * gate[1];
+        for (int w = 0; w < STEP_WARPS; ++w) kv += part[w][tid];
+        su[tid] = mine < a.vcols ? (sv[mine] - ks * kv) * gate[1] * ks : 0.f;
+      }
+    } else {
+      if (tid < STEP_COLS) su[tid] = mine < a.vcols ? sv[mine] * ks : 0.f;
     }
-    float o4[4] = {0.f, 0.f, 0.f, 0.f};
+    __syncthreads();
+    const float4 u = *reinterpret_cast<const float4*>(su + lane * 4);
+    float4 acc = make_float4(0.f, 0.f, 0.f, 0.f);
+    for (int nb = 0; nb < NB; ++nb) {
+      const bool fresh = NB > 1 || (!DELTA && c0 > 0);
+      if (fresh) load(nb, col);
 #pragma unroll
-    for (int i = 0; i < RPL; ++i) {
-      if (!DELTA) S[i] = fmaf(g1, S[i], S[i]);
-      S[i] += kp[i] * u;
-      o4[i & 3] += qp[i] * S[i];
-    }
-    float o = (o4[0] + o4[1]) + (o4[2] + o4[3]);
-#pragma unroll
-    for (int of = 1; of < L; of <<= 1) o += __shfl_xor_sync(0xffffffffu, o, of);
-    if (live) {
-#pragma unroll
-      for (int i = 0; i < RPL; ++i)
-        if (ks * RPL + i < a.dim) Sg[(size_t)(ks * RPL + i) * a.vcols + col] = S[i];
-      if (ks == 0) {
-        so[col] = o;
-        if (col < a.vdim) ss += o * o;
+      for (int i = 0; i < RW; ++i) {
+        const int d = (nb * STEP_WARPS + warp) * RW + i;
+        if (fresh || !DELTA) {
+          S[i].x = fmaf(g1, S[i].x, S[i].x); S[i].y = fmaf(g1, S[i].y, S[i].y);
+          S[i].z = fmaf(g1, S[i].z, S[i].z); S[i].w = fmaf(g1, S[i].w, S[i].w);
+        }
+        const float k = sk[d], q = sq[d];
+        S[i].x += k * u.x; S[i].y += k * u.y; S[i].z += k * u.z; S[i].w += k * u.w;
+        acc.x += q * S[i].x; acc.y += q * S[i].y; acc.z += q * S[i].z; acc.w += q * S[i].w;
+        if (col < a.vcols && d < a.dim) *reinterpret_cast<float4*>(Sg + (size_t)d * a.vcols + col) = S[i];
       }
     }
+    *reinterpret_cast<float4*>(&part[warp][lane * 4]) = acc;
+    __syncthreads();
+    if (tid < STEP_COLS && mine < a.vcols) {
+      float o = 0.f;
+#pragma unroll
+      for (int w = 0; w < STEP_WARPS; ++w) o += part[w][tid];
+      o *= qs;
+      so[mine] = o;
+      if (mine < a.vdim) ss += o * o;
+    }
+    if (c0 + STEP_COLS < a.vcols) __syncthreads();             // part and su are written again
   }
   const float inv = rsqrtf(block_sum(ss, red) / (float)a.vdim + a.eps);      // its barriers publish so[]
   OutT* out = reinterpret_cast<OutT*>(a.out) + ((size_t)t * a.H + h) * a.vcols;
   for (int i = tid; i < a.vcols; i += STEP_THREADS) {
     float v = 0.f;
     if (i < a.vdim)
-      v = so[i] * inv * (a.gain != nullptr ? a.gain[i] : 1.f) * la_silu(la_row(a, (size_t)t * a.stride + a.cz + h * a.vdim + i));
+      v = so[i] * inv * (a.gain != nullptr ? a.gain[i] : 1.f) * la_silu(la_row(a, row0 + a.cz + h * a.vdim + i));
     if constexpr (sizeof(OutT) == 2) out[i] = f32_to_bf16(v);
     else out[i] = v;
   }
@@ -260,10 +329,8 @@ __global__ void __launch_bounds__(STEP_THREADS) linear_step_kernel(const __grid_
     // own value columns, and the query and key columns for the first head that shares them
     for (int i = tid; i < a.vdim; i += STEP_THREADS) la_ring_update(a, slot, t, t + 1, a.cv + h * a.vdim + i);
     if (h % grp == 0)
-      for (int i = tid; i < a.dim; i += STEP_THREADS) {
-        la_ring_update(a, slot, t, t + 1, kh * a.dim + i);
-        la_ring_update(a, slot, t, t + 1, a.ck + kh * a.dim + i);
-      }
+      for (int i = tid; i < 2 * a.dim; i += STEP_THREADS)
+        la_ring_update(a, slot, t, t + 1, (i < a.dim ? i : a.ck + i - a.dim) + kh * a.dim);
   }
 }
 
@@ -284,21 +351,21 @@ int launch_scan(const LinearArgs& a, cudaStream_t stream) {
                        : launch_pdl(linear_scan_kernel<DK, false>, grid, block, 0, stream, a));
 }
 
-template <int DK, typename OutT>
+template <int RW, int NB, typename OutT>
 int launch_step(const LinearArgs& a, cudaStream_t stream) {
   const dim3 grid(a.H, a.T), block(STEP_THREADS);
   const size_t smem = 2 * (size_t)a.vcols * sizeof(float);
-  return (int)(a.delta ? launch_pdl(linear_step_kernel<DK, true, OutT>, grid, block, smem, stream, a)
-                       : launch_pdl(linear_step_kernel<DK, false, OutT>, grid, block, smem, stream, a));
+  return (int)(a.delta ? launch_pdl(linear_step_kernel<RW, NB, true, OutT>, grid, block, smem, stream, a)
+                       : launch_pdl(linear_step_kernel<RW, NB, false, OutT>, grid, block, smem, stream, a));
 }
 
 template <typename OutT>
 int dispatch_step(const LinearArgs& a, cudaStream_t stream) {
   switch (dk_of(a.dim)) {
-    case 64: return launch_step<64, OutT>(a, stream);
-    case 128: return launch_step<128, OutT>(a, stream);
-    case 256: return launch_step<256, OutT>(a, stream);
-    default: return launch_step<512, OutT>(a, stream);
+    case 64: return launch_step<4, 1, OutT>(a, stream);
+    case 128: return launch_step<8, 1, OutT>(a, stream);
+    case 256: return launch_step<8, 2, OutT>(a, stream);
+    default: return launch_step<8, 4, OutT>(a, stream);
   }
 }
 

@@ -79,17 +79,109 @@ template <int DK>
 struct PrepSmem {
   static constexpr int LD = DK + 8;
   __nv_bfloat16 q[2][CK * LD], k[2][CK * LD];      // value, remainder
-  float raw[NTHR / 32][DK];
-  float A[CK][CK + 4];
+  union {
+    float tile[(CK + 15) * DK];                    // rows of a projection, those the convolution needs ahead of them first
+    float A[CK][CK + 4];
+  };
   float b[CK], beta[CK];
 };
+
+// dst[past + 64][DK] <- columns [col, col + width) of tokens t0 - past .. t0 + 63 (zero behind n tokens and behind width; ahead of
+// the segment from the ring)
+template <int DK>
+__device__ __forceinline__ void stage_tile(const LinearArgs& a, float* dst, int t0, int n, int s0, int slot, int past, int col, int width) {
+  const bool vec = (col & 7) == 0 && (width & 7) == 0 && (a.stride & 7) == 0;
+  const int p0 = a.pos[s0];
+  for (int i = threadIdx.x; i < (past + CK) * (DK / 8); i += NTHR) {
+    const int r = i / (DK / 8), d = i % (DK / 8) * 8, t = t0 - past + r;
+    float v[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
+    if (r < past + n && d < width) {
+      if (t >= s0) {
+        const size_t o = (size_t)t * a.stride + col + d;
+        if (vec && a.row_dtype == 1) {
+          const uint4 u = *reinterpret_cast<const uint4*>(reinterpret_cast<const __nv_bfloat16*>(a.rows) + o);
+          const __nv_bfloat162* h2 = reinterpret_cast<const __nv_bfloat162*>(&u);
+#pragma unroll
+          for (int e = 0; e < 4; ++e) {
+            const float2 f2 = __bfloat1622float2(h2[e]);
+            v[2 * e] = f2.x;
+            v[2 * e + 1] = f2.y;
+          }
+        } else {
+#pragma unroll
+          for (int e = 0; e < 8; ++e)
+            if (d + e < width) v[e] = la_row(a, o + e);
+        }
+      } else if (p0 - (s0 - t) >= 0) {
+        const float* src = a.ring + ((size_t)slot * a.taps + (p0 - (s0 - t)) % a.taps) * a.C + col + d;
+#pragma unroll
+        for (int e = 0; e < 8; ++e)
+          if (d + e < width) v[e] = src[e];
+      }
+    }
+    *reinterpret_cast<float4*>(dst + r * DK + d) = make_float4(v[0], v[1], v[2], v[3]);
+    *reinterpret_cast<float4*>(dst + r * DK + d + 4) = make_float4(v[4], v[5], v[6], v[7]);
+  }
+}
+
+__device__ __forceinline__ float silu_fast(float x) { return __fdividef(x, 1.f + __expf(fminf(-x, 80.f))); }
+
+// Convolution and silu of eight tokens (from row r0 of the tile on) for NC columns at d: each(token, values).  TAPS 0: any number
+template <int DK, int TAPS, typename Each>
+__device__ __forceinline__ void conv_tokens(const LinearArgs& a, const float* tile, int r0, int d, int col, int width, Each each) {
+  constexpr int NC = DK / 32;
+  const int taps = TAPS > 0 ? TAPS : a.taps;
+  constexpr int WN = TAPS > 0 ? TAPS : 1;
+  float w[WN][NC], x[WN][NC];
+  const auto weight = [&](int j, int e) { return d + e < width ? a.cw[(size_t)j * a.C + col + d + e] : 0.f; };
+  if constexpr (TAPS > 0) {
+#pragma unroll
+    for (int j = 0; j < TAPS; ++j)
+#pragma unroll
+      for (int e = 0; e < NC; ++e) {
+        w[j][e] = weight(j, e);
+        x[j][e] = j > 0 ? tile[(r0 + j - 1) * DK + d + e] : 0.f;
+      }
+  }
+#pragma unroll
+  for (int r = 0; r < CK / 8; ++r) {
+    float v[NC];
+    if constexpr (TAPS > 0) {
+#pragma unroll
+      for (int e = 0; e < NC; ++e) {
+#pragma unroll
+        for (int j = 0; j + 1 < TAPS; ++j) x[j][e] = x[j + 1][e];
+        x[TAPS - 1][e] = tile[(r0 + r + TAPS - 1) * DK + d + e];
+        v[e] = 0.f;
+#pragma unroll
+        for (int j = 0; j < TAPS; ++j) v[e] += w[j][e] * x[j][e];
+        v[e] = silu_fast(v[e]);
+      }
+    } else {
+#pragma unroll
+      for (int e = 0; e < NC; ++e) {
+        v[e] = 0.f;
+        for (int j = 0; j < taps; ++j) v[e] += weight(j, e) * tile[(r0 + r + j) * DK + d + e];
+        v[e] = silu_fast(v[e]);
+      }
+    }
+    each(r0 + r, v);
+  }
+}
+template <int DK, typename Each>
+__device__ __forceinline__ void conv_dispatch(const LinearArgs& a, const float* tile, int r0, int d, int col, int width, Each each) {
+  if (a.taps == 4) conv_tokens<DK, 4>(a, tile, r0, d, col, width, each);
+  else if (a.taps == 3) conv_tokens<DK, 3>(a, tile, r0, d, col, width, each);
+  else if (a.taps == 2) conv_tokens<DK, 2>(a, tile, r0, d, col, width, each);
+  else conv_tokens<DK, 0>(a, tile, r0, d, col, width, each);
+}
 
 // grid (chunks, H)
 template <int DK, bool DELTA>
 __global__ void __launch_bounds__(NTHR, 2) linear_chunk_prepare_kernel(const __grid_constant__ LinearArgs a) {
   extern __shared__ __align__(16) uint8_t smem_raw[];
   PrepSmem<DK>& sm = *reinterpret_cast<PrepSmem<DK>*>(smem_raw);
-  constexpr int LD = PrepSmem<DK>::LD;
+  constexpr int LD = PrepSmem<DK>::LD, NC = DK / 32;
   pdl_wait();
   pdl_launch();
   const int chunk = blockIdx.x, h = blockIdx.y, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
@@ -99,37 +191,107 @@ __global__ void __launch_bounds__(NTHR, 2) linear_chunk_prepare_kernel(const __g
   if (!HE_INDEX_OK(slot, a.n_slots, HE_SITE_STATE_SLOT)) return;
   const int grp = a.H / a.G, kh = h / grp;
   const bool own = h % grp == 0;                   // writes the query and key rows its group shares
+  const size_t qk_plane = (size_t)a.T * a.G * DK;
 
-  for (int r = warp; r < CK; r += NTHR / 32) {
-    const int t = t0 + r;
+  if constexpr (DELTA) {
+    const int past = a.taps - 1, r0 = warp * (CK / 8), d = lane * NC;
 #pragma unroll
     for (int which = 0; which < 2; ++which) {
-      if (r < n) {
-        la_prepare_head(a, t, s0, slot, a.pos[t], (which ? a.ck : 0) + kh * a.dim, which ? a.kscale : a.qscale, sm.raw[warp], lane);
-        __syncwarp();
-      }
-      __nv_bfloat16* p0 = (which ? sm.k[0] : sm.q[0]) + r * LD;
-      __nv_bfloat16* p1 = (which ? sm.k[1] : sm.q[1]) + r * LD;
-      for (int d = lane * 2; d < DK; d += 64) {
-        __align__(4) __nv_bfloat16 hi[2], lo[2];
-        split(r < n && d < a.dim ? sm.raw[warp][d] : 0.f, hi[0], lo[0]);
-        split(r < n && d + 1 < a.dim ? sm.raw[warp][d + 1] : 0.f, hi[1], lo[1]);
-        const uint32_t wh = *reinterpret_cast<uint32_t*>(hi), wl = *reinterpret_cast<uint32_t*>(lo);
-        *reinterpret_cast<uint32_t*>(p0 + d) = wh;
-        *reinterpret_cast<uint32_t*>(p1 + d) = wl;
-        if (own && r < n) {
-          const size_t plane = (size_t)a.T * a.G * DK, o = ((size_t)t * a.G + kh) * DK + d;
-          *reinterpret_cast<uint32_t*>(a.qk + (size_t)(2 * which) * plane + o) = wh;
-          *reinterpret_cast<uint32_t*>(a.qk + (size_t)(2 * which + 1) * plane + o) = wl;
+      const int col = (which ? a.ck : 0) + kh * a.dim;
+      if (which) __syncthreads();
+      stage_tile<DK>(a, sm.tile, t0, n, s0, slot, past, col, a.dim);
+      __syncthreads();
+      const float scale = which ? a.kscale : a.qscale;
+      __nv_bfloat16* p0 = which ? sm.k[0] : sm.q[0];
+      __nv_bfloat16* p1 = which ? sm.k[1] : sm.q[1];
+      conv_dispatch<DK>(a, sm.tile, r0, d, col, a.dim, [&](int r, float (&v)[NC]) {
+        float ss = 0.f;
+#pragma unroll
+        for (int e = 0; e < NC; ++e) ss += v[e] * v[e];
+        const float inv = r < n ? scale * rsqrtf(warp_sum(ss) + 1e-6f) : 0.f;
+        __align__(8) __nv_bfloat16 hi[NC], lo[NC];
+#pragma unroll
+        for (int e = 0; e < NC; ++e) split(v[e] * inv, hi[e], lo[e]);
+        __nv_bfloat16* g0 = a.qk + (size_t)(2 * which) * qk_plane + ((size_t)(t0 + r) * a.G + kh) * DK + d;
+        if constexpr (NC == 4) {
+          const uint2 wh = *reinterpret_cast<const uint2*>(hi), wl = *reinterpret_cast<const uint2*>(lo);
+          *reinterpret_cast<uint2*>(p0 + r * LD + d) = wh;
+          *reinterpret_cast<uint2*>(p1 + r * LD + d) = wl;
+          if (own && r < n) {
+            *reinterpret_cast<uint2*>(g0) = wh;
+            *reinterpret_cast<uint2*>(g0 + qk_plane) = wl;
+          }
+        } else {
+          const uint32_t wh = *reinterpret_cast<const uint32_t*>(hi), wl = *reinterpret_cast<const uint32_t*>(lo);
+          *reinterpret_cast<uint32_t*>(p0 + r * LD + d) = wh;
+          *reinterpret_cast<uint32_t*>(p1 + r * LD + d) = wl;
+          if (own && r < n) {
+            *reinterpret_cast<uint32_t*>(g0) = wh;
+            *reinterpret_cast<uint32_t*>(g0 + qk_plane) = wl;
+          }
         }
-      }
-      __syncwarp();
+      });
     }
-    if (r < n)
-      for (int d = lane; d < a.vcols; d += 32) {
-        const int c = a.cv + h * a.vdim + d;
-        const float v = d >= a.vdim ? 0.f : DELTA ? la_conv(a, t, s0, slot, a.pos[t], c) : la_row(a, (size_t)t * a.stride + c);
-        a.vb[((size_t)t * a.H + h) * a.vcols + d] = f32_to_bf16(v);
+    for (int v0 = 0; v0 < a.vcols; v0 += DK) {
+      const int col = a.cv + h * a.vdim + v0, width = max(0, min(DK, a.vdim - v0));
+      __syncthreads();
+      stage_tile<DK>(a, sm.tile, t0, n, s0, slot, past, col, width);
+      __syncthreads();
+      conv_dispatch<DK>(a, sm.tile, r0, d, col, width, [&](int r, float (&v)[NC]) {
+        if (r >= n || v0 + d >= a.vcols) return;               // silu(0) = 0 in padded columns
+        __align__(8) __nv_bfloat16 o[NC];
+#pragma unroll
+        for (int e = 0; e < NC; ++e) o[e] = f32_to_bf16(v[e]);
+        __nv_bfloat16* dst = a.vb + ((size_t)(t0 + r) * a.H + h) * a.vcols + v0 + d;
+        if constexpr (NC == 4) *reinterpret_cast<uint2*>(dst) = *reinterpret_cast<const uint2*>(o);
+        else *reinterpret_cast<uint32_t*>(dst) = *reinterpret_cast<const uint32_t*>(o);
+      });
+    }
+    __syncthreads();
+  } else {
+    // a warp turns the queries and keys of a token; a lane has pairs (i, i + half) of both
+    const int half = a.rot_dims >> 1;
+    const auto put = [&](int which, int r, int dd, float x) {
+      __nv_bfloat16 hi, lo;
+      split(x, hi, lo);
+      (which ? sm.k[0] : sm.q[0])[r * LD + dd] = hi;
+      (which ? sm.k[1] : sm.q[1])[r * LD + dd] = lo;
+    };
+    for (int r = warp; r < CK; r += NTHR / 32) {
+      const size_t q0 = (size_t)(t0 + r) * a.stride + kh * a.dim, k0 = q0 + a.ck;
+      const bool live = r < n;
+      const int p = live ? a.pos[t0 + r] : 0;
+      for (int i = lane; i < half; i += 32) {
+        float c = 1.f, s = 0.f, qu = 0.f, qv = 0.f, ku = 0.f, kv = 0.f;
+        if (live) {
+          qu = la_row(a, q0 + i);
+          qv = la_row(a, q0 + half + i);
+          ku = la_row(a, k0 + i) * a.kscale;
+          kv = la_row(a, k0 + half + i) * a.kscale;
+          la_angle(a.freq[i], p, c, s);
+        }
+        put(0, r, i, qu * c - qv * s);
+        put(0, r, half + i, qv * c + qu * s);
+        put(1, r, i, ku * c - kv * s);
+        put(1, r, half + i, kv * c + ku * s);
+      }
+      for (int dd = a.rot_dims + lane; dd < DK; dd += 32) {
+        const bool in = live && dd < a.dim;
+        put(0, r, dd, in ? la_row(a, q0 + dd) * a.qscale : 0.f);
+        put(1, r, dd, in ? la_row(a, k0 + dd) * a.kscale : 0.f);
+      }
+      if (live)
+        for (int dd = lane; dd < a.vcols; dd += 32)
+          a.vb[((size_t)(t0 + r) * a.H + h) * a.vcols + dd] =
+              f32_to_bf16(dd < a.vdim ? la_row(a, (size_t)(t0 + r) * a.stride + a.cv + h * a.vdim + dd) : 0.f);
+    }
+    __syncthreads();
+    if (own)
+      for (int i = tid; i < 4 * n * (DK / 8); i += NTHR) {
+        const int pl = i / (n * (DK / 8)), r = i / (DK / 8) % n, dd = i % (DK / 8) * 8;
+        const __nv_bfloat16* src = pl < 2 ? sm.q[pl] : sm.k[pl - 2];
+        *reinterpret_cast<uint4*>(a.qk + pl * qk_plane + ((size_t)(t0 + r) * a.G + kh) * DK + dd) =
+            *reinterpret_cast<const uint4*>(src + r * LD + dd);
       }
   }
   if (DELTA && warp == 0) {                        // log decays summed over the chunk, two tokens per lane

@@ -237,6 +237,7 @@ class SideBySideSpec:
 # bounds of the linear attention kernels: key and value columns per head, taps of a convolution
 LINEAR_MAX_DIM = 512
 CONV_MAX_TAPS = 16
+NORM_CONV_MAX_ROWS = 50 * 1024           # channels of a norm group times rows that its kernel keeps in shared memory
 
 
 @dataclass(frozen=True)
@@ -726,6 +727,8 @@ def mepatar_config(hidden: int, vocab: int, layers: Tuple[LayerSpec, ...], rms_e
             l.mixer.check()
             if not 1 <= l.input_taps <= CONV_MAX_TAPS:
                 raise ValueError(f"input convolution of {l.input_taps} taps")
+            if hidden // norm_groups * max(1, 2 * (l.input_taps - 1)) > NORM_CONV_MAX_ROWS:
+                raise ValueError(f"norms over {hidden // norm_groups} channels with an input convolution of {l.input_taps} taps")
             if isinstance(l.mlp, MoeMlpSpec):
                 l.mlp.check()
         except ValueError as e:

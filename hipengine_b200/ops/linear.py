@@ -4,7 +4,7 @@ from __future__ import annotations
 
 import ctypes as C
 from dataclasses import dataclass
-from typing import Optional
+from typing import Optional, Tuple
 
 import torch
 
@@ -113,6 +113,19 @@ def linear_attention(p: LinearParams, rows: torch.Tensor, ab: Optional[torch.Ten
     """out [T, H * vcols] = the gated output of a layer's linear attention; ``S`` and ``ring`` (the states of all slots) advance,
     or with journals stay while the state after every token is recorded.  ``ab`` (delta rule): fp32 rows with the step size's
     logits at column 0 and the decay's inputs at column ``ca``."""
+    a, steps = plan(p, rows, ab, ca, S, ring, batch, out, eps, scratch, jS, jring)
+    for name in steps:
+        launch(name, a)
+
+
+def launch(name: str, a: _LinearArgs) -> None:
+    N.check(getattr(_lib(), name)(C.byref(a), _stream()), name)
+
+
+def plan(p: LinearParams, rows: torch.Tensor, ab: Optional[torch.Tensor], ca: int, S: torch.Tensor, ring: Optional[torch.Tensor],
+         batch, out: torch.Tensor, eps: float, scratch, jS: Optional[torch.Tensor] = None,
+         jring: Optional[torch.Tensor] = None) -> Tuple[_LinearArgs, Tuple[str, ...]]:
+    """(arguments, kernels in order) of ``linear_attention``."""
     s, T = p.spec, rows.shape[0]
     _check_device(rows)
     a = _LinearArgs()
@@ -133,10 +146,8 @@ def linear_attention(p: LinearParams, rows: torch.Tensor, ab: Optional[torch.Ten
     a.seg_start, a.seg_slot, a.tok_seg, a.pos = (t.data_ptr() for t in (batch.seg_start, batch.seg_slot, batch.tok_seg, batch.pos))
     a.T, a.n_seg, a.n_slots, a.H, a.G = T, batch.n_seg, S.shape[0], s.heads, s.kv_heads
     a.dim, a.vdim, a.vcols, a.ck, a.cv, a.cz, a.delta = s.dim, s.vdim, s.vcols, p.ck, p.cv, p.cz, int(s.delta)
-    L = _lib()
     if batch.n_seg == T and jS is None:
-        N.check(L.he_linear_step(C.byref(a), _stream()), "he_linear_step")
-        return
+        return a, ("he_linear_step",)
     get = lambda name, n, dtype=torch.float32: scratch.get("lin_" + name, (n,), dtype).data_ptr()
     a.o = get("o", T * s.heads * s.vcols)
     if use_chunks(s, batch, f32 or jS is not None):
@@ -145,16 +156,12 @@ def linear_attention(p: LinearParams, rows: torch.Tensor, ab: Optional[torch.Ten
         a.qk, a.vb = get("qk", 4 * T * s.kv_heads * dk, torch.bfloat16), get("vb", T * s.heads * s.vcols, torch.bfloat16)
         a.mats = get("mats", 4 * a.chunks * s.heads * CHUNK * CHUNK, torch.bfloat16)
         a.lg, a.beta = get("lg", T * s.heads), get("beta", T * s.heads)
-        N.check(L.he_linear_chunk_prepare(C.byref(a), _stream()), "he_linear_chunk_prepare")
-        N.check(L.he_linear_chunk_scan(C.byref(a), _stream()), "he_linear_chunk_scan")
-    else:
-        a.qf, a.kf = get("q", T * s.kv_heads * s.dim), get("k", T * s.kv_heads * s.dim)
-        a.vf, a.g1, a.beta = get("v", T * s.heads * s.vcols), get("g1", T * s.heads), get("beta", T * s.heads)
-        N.check(L.he_linear_prepare(C.byref(a), _stream()), "he_linear_prepare")
-        N.check(L.he_linear_scan(C.byref(a), _stream()), "he_linear_scan")
-    N.check(L.he_linear_out(C.byref(a), _stream()), "he_linear_out")
+        return a, ("he_linear_chunk_prepare", "he_linear_chunk_scan", "he_linear_out")
+    a.qf, a.kf = get("q", T * s.kv_heads * s.dim), get("k", T * s.kv_heads * s.dim)
+    a.vf, a.g1, a.beta = get("v", T * s.heads * s.vcols), get("g1", T * s.heads), get("beta", T * s.heads)
+    return a, ("he_linear_prepare", "he_linear_scan", "he_linear_out")
 
 
 def use_chunks(s, batch, serial: bool) -> bool:
     """Prompt portions take the chunked form; fp32, journals, wider heads and batches of short portions the serial one."""
-    return not serial and s.dim <= CHUNK_MAX_DIM and batch.T >= 16 * batch.n_seg and hasattr(N.lib(), "he_linear_chunk_scan")
+    return not serial and s.dim <= CHUNK_MAX_DIM and batch.T >= 16 * batch.n_seg

@@ -167,7 +167,7 @@ def _specs():
     return {
         "delta-20": L(6, 3, 20, 28, taps=3), "delta-128": L(4, 2, 128, 128, taps=4), "delta-64": L(2, 2, 64, 64, taps=2),
         "delta-1": L(1, 1, 1, 1, taps=1), "delta-wide": L(3, 1, 136, 264, taps=6), "delta-100": L(8, 1, 100, 40, taps=5),
-        "delta-512": L(2, 1, 512, 512, taps=3),
+        "delta-512": L(2, 1, 512, 512, taps=3), "delta-40": L(2, 1, 40, 200, taps=4), "delta-16": L(4, 4, 16, 36, taps=9),
         "ret-33": L(3, 3, 33, 18, dec(3), rot(14)), "ret-128": L(4, 4, 128, 128, dec(4), rot(128)),
         "ret-64": L(9, 9, 64, 64, dec(9), rot(64, 1e6)), "ret-2": L(1, 1, 2, 1, (1.0,), rot(2)),
         "ret-wide": L(2, 2, 300, 72, dec(2), rot(200)), "ret-100": L(5, 5, 100, 200, dec(5), rot(32)),
@@ -179,8 +179,8 @@ CUTS = {"steps": [1] * 40, "mixed": [5, 1, 1, 30, 2, 64, 1, 7], "chunks": [64, 6
 
 @pytest.mark.parametrize("dtype", [F32, BF])
 @pytest.mark.parametrize("cut", list(CUTS))
-@pytest.mark.parametrize("name", ["delta-20", "delta-128", "delta-64", "delta-1", "delta-wide", "delta-100", "delta-512", "ret-33",
-                                  "ret-128", "ret-64", "ret-2", "ret-wide", "ret-100"])
+@pytest.mark.parametrize("name", ["delta-20", "delta-128", "delta-64", "delta-1", "delta-wide", "delta-100", "delta-512", "delta-40",
+                                  "delta-16", "ret-33", "ret-128", "ret-64", "ret-2", "ret-wide", "ret-100"])
 def test_linear_attention(name, cut, dtype):
     """Two sequences, cut differently, in the same batches as a third one that waits between; every form (one-token steps, serial
     scans, chunks) from the states the others left; outputs, states, the convolution's past, states of other slots."""

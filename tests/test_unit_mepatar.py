@@ -58,6 +58,7 @@ def _change(i, part="mixer", **kw):
     {"norm": {"eps": 1e-5, "groups": 5}},
     {"canon": {"taps": 0}},
     {"canon": {"taps": 40}},
+    {"width": 13200, "norm": {"eps": 1e-5, "groups": 1}},
     {"layers": [{"type": "recurrent", "mixer": {"heads": 1, "dim": 8, "vdim": 8}, "mlp": None}]},
     {"layers": [{**ODD["layers"][0], "mlp": {"kind": "sparse"}}]},
     _change(0, kv_heads=4), _change(0, dim=600), _change(0, vdim=513), _change(0, conv=0),
