@@ -249,41 +249,57 @@ __global__ void __launch_bounds__(NTHR, 2) linear_chunk_prepare_kernel(const __g
     }
     __syncthreads();
   } else {
-    // a warp turns the queries and keys of a token; a lane has pairs (i, i + half) of both
-    const int half = a.rot_dims >> 1;
-    const auto put = [&](int which, int r, int dd, float x) {
-      __nv_bfloat16 hi, lo;
-      split(x, hi, lo);
-      (which ? sm.k[0] : sm.q[0])[r * LD + dd] = hi;
-      (which ? sm.k[1] : sm.q[1])[r * LD + dd] = lo;
-    };
-    for (int r = warp; r < CK; r += NTHR / 32) {
-      const size_t q0 = (size_t)(t0 + r) * a.stride + kh * a.dim, k0 = q0 + a.ck;
-      const bool live = r < n;
-      const int p = live ? a.pos[t0 + r] : 0;
-      for (int i = lane; i < half; i += 32) {
-        float c = 1.f, s = 0.f, qu = 0.f, qv = 0.f, ku = 0.f, kv = 0.f;
-        if (live) {
-          qu = la_row(a, q0 + i);
-          qv = la_row(a, q0 + half + i);
-          ku = la_row(a, k0 + i) * a.kscale;
-          kv = la_row(a, k0 + half + i) * a.kscale;
-          la_angle(a.freq[i], p, c, s);
+    // rows as they are into the planes (bf16 rows have no remainder), values on their way out; then a warp turns the queries and
+    // keys of a token in place, a lane has pairs (i, i + half) of both
+    const bool plain = a.row_dtype == 1 && ((a.stride | a.ck | a.cv | a.dim | a.vdim) & 7) == 0;
+    const __nv_bfloat16* rows = reinterpret_cast<const __nv_bfloat16*>(a.rows);
+    for (int i = tid; i < 2 * CK * (DK / 8); i += NTHR) {
+      const int which = i / (CK * (DK / 8)), r = i / (DK / 8) % CK, dd = i % (DK / 8) * 8;
+      const size_t o = (size_t)(t0 + r) * a.stride + (which ? a.ck : 0) + kh * a.dim + dd;
+      __align__(16) __nv_bfloat16 hi[8], lo[8];
+      uint4 wh = make_uint4(0u, 0u, 0u, 0u), wl = wh;
+      if (r < n && dd < a.dim) {
+        if (plain) {
+          wh = *reinterpret_cast<const uint4*>(rows + o);
+        } else {
+#pragma unroll
+          for (int e = 0; e < 8; ++e) split(dd + e < a.dim ? la_row(a, o + e) : 0.f, hi[e], lo[e]);
+          wh = *reinterpret_cast<const uint4*>(hi);
+          wl = *reinterpret_cast<const uint4*>(lo);
         }
-        put(0, r, i, qu * c - qv * s);
-        put(0, r, half + i, qv * c + qu * s);
-        put(1, r, i, ku * c - kv * s);
-        put(1, r, half + i, kv * c + ku * s);
       }
-      for (int dd = a.rot_dims + lane; dd < DK; dd += 32) {
-        const bool in = live && dd < a.dim;
-        put(0, r, dd, in ? la_row(a, q0 + dd) * a.qscale : 0.f);
-        put(1, r, dd, in ? la_row(a, k0 + dd) * a.kscale : 0.f);
+      *reinterpret_cast<uint4*>((which ? sm.k[0] : sm.q[0]) + r * LD + dd) = wh;
+      *reinterpret_cast<uint4*>((which ? sm.k[1] : sm.q[1]) + r * LD + dd) = wl;
+    }
+    for (int i = tid; i < n * (a.vcols / 8); i += NTHR) {
+      const int r = i / (a.vcols / 8), dd = i % (a.vcols / 8) * 8;
+      const size_t o = (size_t)(t0 + r) * a.stride + a.cv + h * a.vdim + dd;
+      uint4 w;
+      if (plain) {
+        w = *reinterpret_cast<const uint4*>(rows + o);
+      } else {
+        __align__(16) __nv_bfloat16 v[8];
+#pragma unroll
+        for (int e = 0; e < 8; ++e) v[e] = f32_to_bf16(dd + e < a.vdim ? la_row(a, o + e) : 0.f);
+        w = *reinterpret_cast<const uint4*>(v);
       }
-      if (live)
-        for (int dd = lane; dd < a.vcols; dd += 32)
-          a.vb[((size_t)(t0 + r) * a.H + h) * a.vcols + dd] =
-              f32_to_bf16(dd < a.vdim ? la_row(a, (size_t)(t0 + r) * a.stride + a.cv + h * a.vdim + dd) : 0.f);
+      *reinterpret_cast<uint4*>(a.vb + ((size_t)(t0 + r) * a.H + h) * a.vcols + dd) = w;
+    }
+    __syncthreads();
+    const int half = a.rot_dims >> 1;
+    for (int r = warp; r < n; r += NTHR / 32) {
+      const int p = a.pos[t0 + r];
+      const auto get = [&](const __nv_bfloat16 (&x)[2][CK * LD], int dd) { return bf16_to_f32(x[0][r * LD + dd]) + bf16_to_f32(x[1][r * LD + dd]); };
+      for (int i = lane; i < half; i += 32) {
+        float c, s;
+        la_angle(a.freq[i], p, c, s);
+        const float qu = get(sm.q, i), qv = get(sm.q, half + i), ku = get(sm.k, i) * a.kscale, kv = get(sm.k, half + i) * a.kscale;
+        split(qu * c - qv * s, sm.q[0][r * LD + i], sm.q[1][r * LD + i]);
+        split(qv * c + qu * s, sm.q[0][r * LD + half + i], sm.q[1][r * LD + half + i]);
+        split(ku * c - kv * s, sm.k[0][r * LD + i], sm.k[1][r * LD + i]);
+        split(kv * c + ku * s, sm.k[0][r * LD + half + i], sm.k[1][r * LD + half + i]);
+      }
+      for (int dd = a.rot_dims + lane; dd < a.dim; dd += 32) split(get(sm.k, dd) * a.kscale, sm.k[0][r * LD + dd], sm.k[1][r * LD + dd]);
     }
     __syncthreads();
     if (own)

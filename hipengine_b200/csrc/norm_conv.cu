@@ -32,7 +32,7 @@ namespace {
 
 constexpr int NW = 8, NTHR = NW * 32;
 constexpr int MAX_TILE = 32;
-constexpr size_t SMEM_SOFT = 64 * 1024, SMEM_HARD = 200 * 1024;
+constexpr size_t SMEM_SOFT = 36 * 1024, SMEM_HARD = 200 * 1024;
 
 template <int V> struct Vec;
 template <> struct Vec<1> { float v[1]; };
