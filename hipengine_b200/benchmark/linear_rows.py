@@ -224,7 +224,7 @@ def products(M: int) -> List[Dict]:
         elif "gate" in what:
             if few:
                 continue                                     # they ride in the input product
-            ms = time_launches(lambda i: GM.gemm_bf16(x, ws[i], h), n)
+            ms = time_launches(lambda i: GM.gemm_bf16_splitk_det(x, ws[i], h, sc), n)
             r = _bf(128, Kc)
             lo = torch.empty(M, 128, device="cuda")
             lms, lk, like = time_launches(lambda i: GM.gemm_bf16(x, r, lo), n), 128, "router rows, 128 columns"

@@ -126,7 +126,7 @@ class MepatarExecutor(ListedExecutor):
         ab = rows[:, c0:]
         if rows.dtype != torch.float32:                    # what the decays are made of is not rounded
             from ..ops import gemm as GM
-            ab = GM.gemm_bf16(xs, w.data[c0:], self.scratch.get("lin_ab", (T, w.n_rows - c0), torch.float32))
+            ab = GM.gemm_bf16_splitk_det(xs, w.data[c0:], self.scratch.get("lin_ab", (T, w.n_rows - c0), torch.float32), self.scratch)
         return rows, ab, logits
 
     def _attention(self, run: int, i: int, rows: torch.Tensor, b: BatchDesc) -> torch.Tensor:
